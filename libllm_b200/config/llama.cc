@@ -193,6 +193,8 @@ void register_builtin_architectures() {
   register_sobezen_architecture();
   extern void register_tazizen_architecture();     // config/tazizen.cc
   register_tazizen_architecture();
+  extern void register_rarelorn_architecture();    // config/rarelorn.cc
+  register_rarelorn_architecture();
 }
 
 }  // namespace llm

@@ -59,7 +59,14 @@ __device__ __forceinline__ float dot_row(const float *q, const __nv_bfloat16 *k,
   return acc;
 }
 
-template <typename T, int MAX_D>
+// Weights that stand for themselves instead of a softmax's (SIG): a visible key's weight is sigmoid(cap tanh(temp s / cap) + bias)
+// with a temperature and a bias per head (cap 0: no bound); the result is multiplied by out_scale.
+struct SigmoidWeights {
+  const float *temp, *bias;
+  float cap, out_scale;
+};
+
+template <typename T, int MAX_D, bool SIG>
 __global__ void __launch_bounds__(WARPS * 32)
 attention_generic_kernel(const T *__restrict__ q, long long q_stride, T *__restrict__ out,
                          long long out_stride, const T *__restrict__ kcache,
@@ -67,7 +74,7 @@ attention_generic_kernel(const T *__restrict__ q, long long q_stride, T *__restr
                          const int *__restrict__ tok_pos, const int *__restrict__ page_table,
                          int pt_stride, int n_tokens, int n_heads, int n_kv, int d, int dv, int page_size,
                          int window, int block, int sink, float scale, const float *__restrict__ gate,
-                         long long gate_stride, int vec, int v_ld, float null_score) {
+                         long long gate_stride, int vec, int v_ld, float null_score, SigmoidWeights sig) {
   __shared__ __align__(16) float q_s[WARPS][MAX_D];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const long long w = (long long)blockIdx.x * WARPS + warp;
@@ -83,6 +90,7 @@ attention_generic_kernel(const T *__restrict__ q, long long q_stride, T *__restr
   int kstart = window > 0 ? max(0, p - window + 1) : 0;
   if (block > 0) kstart = max(kstart, p / block * block);
   float m = -INFINITY, l = 0.f;
+  const float temp = SIG ? sig.temp[h] : 0.f, bias = SIG ? sig.bias[h] : 0.f;
   float acc[MAX_D / 32];
 #pragma unroll
   for (int i = 0; i < MAX_D / 32; ++i) acc[i] = 0.f;
@@ -100,12 +108,20 @@ attention_generic_kernel(const T *__restrict__ q, long long q_stride, T *__restr
         const T *krow = kcache + (((size_t)page * n_kv + kvh) * page_size + (j % page_size)) * d;
         s = dot_row(q_s[warp], krow, d, vec != 0) * scale;
       }
-      const float m_new = fmaxf(m, warp_max(s));          // finite: lane 0 always holds a key
-      const float pj = valid ? expf(s - m_new) : 0.f;
-      const float alpha = expf(m - m_new);                // 0 on the first block (m = -inf)
-      l = l * alpha + warp_sum(pj);
+      float pj;
+      if (SIG) {
+        s *= temp;
+        if (sig.cap > 0.f) s = sig.cap * tanhf(s / sig.cap);
+        pj = valid ? 1.f / (1.f + expf(-(s + bias))) : 0.f;
+      } else {
+        const float m_new = fmaxf(m, warp_max(s));          // finite: lane 0 always holds a key
+        pj = valid ? expf(s - m_new) : 0.f;
+        const float alpha = expf(m - m_new);                // 0 on the first block (m = -inf)
+        l = l * alpha + warp_sum(pj);
 #pragma unroll
-      for (int i = 0; i < MAX_D / 32; ++i) acc[i] *= alpha;
+        for (int i = 0; i < MAX_D / 32; ++i) acc[i] *= alpha;
+        m = m_new;
+      }
       const int nvalid = min(32, k1 - kb);
       for (int jj = 0; jj < nvalid; ++jj) {
         const float pv = __shfl_sync(0xffffffffu, pj, jj);
@@ -118,17 +134,16 @@ attention_generic_kernel(const T *__restrict__ q, long long q_stride, T *__restr
           if (c < dv) acc[i] = fmaf(pv, to_float(vrow[c]), acc[i]);
         }
       }
-      m = m_new;
     }
   }
   T *orow = out + (size_t)token * out_stride + (size_t)h * dv;
-  if (null_score > -INFINITY) {     // one more key whose score is null_score and whose value is nought
+  if (!SIG && null_score > -INFINITY) {     // one more key whose score is null_score and whose value is nought
     const float m_new = fmaxf(m, null_score), alpha = expf(m - m_new);
     l = l * alpha + expf(null_score - m_new);
 #pragma unroll
     for (int i = 0; i < MAX_D / 32; ++i) acc[i] *= alpha;
   }
-  float inv = 1.f / l;
+  float inv = SIG ? sig.out_scale : 1.f / l;
   if (gate) inv *= 1.f / (1.f + expf(-gate[(size_t)token * gate_stride + h]));
 #pragma unroll
   for (int i = 0; i < MAX_D / 32; ++i) {
@@ -139,12 +154,12 @@ attention_generic_kernel(const T *__restrict__ q, long long q_stride, T *__restr
 
 // v_ld: channels between two value rows of the value storage (dv for a storage of its own; the key rows' width
 // when the values are the first dv channels of the keys and vcache is kcache).
-LLM_EXPORT int llm_attention_generic_ld(int dtype, const void *q, long long q_stride, void *out,
-                                        long long out_stride, const void *kcache, const void *vcache,
-                                        const int *tok_seq, const int *tok_pos, const int *page_table,
-                                        int pt_stride, int n_tokens, int n_heads, int n_kv, int d, int dv, int v_ld,
-                                        int page_size, int window, int block, int sink, float scale, const float *gate,
-                                        long long gate_stride, float null_score, cudaStream_t stream) {
+static int launch_generic(int dtype, const void *q, long long q_stride, void *out,
+                          long long out_stride, const void *kcache, const void *vcache,
+                          const int *tok_seq, const int *tok_pos, const int *page_table,
+                          int pt_stride, int n_tokens, int n_heads, int n_kv, int d, int dv, int v_ld,
+                          int page_size, int window, int block, int sink, float scale, const float *gate,
+                          long long gate_stride, float null_score, const SigmoidWeights *sig, cudaStream_t stream) {
   if (n_tokens == 0) return LLM_OK;
   LLM_REQUIRE(n_tokens > 0 && n_heads > 0 && n_kv > 0 && n_heads % n_kv == 0, "attention: bad head counts %d/%d", n_heads, n_kv);
   LLM_REQUIRE(d > 0 && d <= MAX_D_LARGE && dv > 0 && dv <= MAX_D_LARGE, "attention: head sizes %d / %d are not supported (up to %d)", d, dv,
@@ -158,18 +173,45 @@ LLM_EXPORT int llm_attention_generic_ld(int dtype, const void *q, long long q_st
   const long long blocks = (warps + WARPS - 1) / WARPS;
   LLM_REQUIRE(blocks < 2147483647LL, "attention: too many tokens for one launch");
   const bool small = d <= MAX_D_SMALL && dv <= MAX_D_SMALL;
+  const SigmoidWeights sw = sig ? *sig : SigmoidWeights{};
 #define GENERIC_GO(T, MAXD)                                                                                              \
-  attention_generic_kernel<T, MAXD><<<(unsigned)blocks, WARPS * 32, 0, stream>>>(                                          \
+  if (sig) GENERIC_RUN(T, MAXD, true);                                                                                   \
+  else GENERIC_RUN(T, MAXD, false)
+#define GENERIC_RUN(T, MAXD, SIG)                                                                                        \
+  attention_generic_kernel<T, MAXD, SIG><<<(unsigned)blocks, WARPS * 32, 0, stream>>>(                                          \
       (const T *)q, q_stride, (T *)out, out_stride, (const T *)kcache, (const T *)vcache, tok_seq, tok_pos, page_table, pt_stride, \
-      n_tokens, n_heads, n_kv, d, dv, page_size, window, block, sink, scale, gate, gate_stride, vec, v_ld, null_score)
-  if (dtype == LLM_F32 && small) GENERIC_GO(float, MAX_D_SMALL);
-  else if (dtype == LLM_F32) GENERIC_GO(float, MAX_D_LARGE);
-  else if (dtype == LLM_BF16 && small) GENERIC_GO(__nv_bfloat16, MAX_D_SMALL);
-  else if (dtype == LLM_BF16) GENERIC_GO(__nv_bfloat16, MAX_D_LARGE);
+      n_tokens, n_heads, n_kv, d, dv, page_size, window, block, sink, scale, gate, gate_stride, vec, v_ld, null_score, sw)
+  if (dtype == LLM_F32 && small) { GENERIC_GO(float, MAX_D_SMALL); }
+  else if (dtype == LLM_F32) { GENERIC_GO(float, MAX_D_LARGE); }
+  else if (dtype == LLM_BF16 && small) { GENERIC_GO(__nv_bfloat16, MAX_D_SMALL); }
+  else if (dtype == LLM_BF16) { GENERIC_GO(__nv_bfloat16, MAX_D_LARGE); }
   else LLM_FAIL("attention: unknown dtype %d", dtype);
+#undef GENERIC_RUN
 #undef GENERIC_GO
   LLM_CHECK_LAUNCH("attention_generic");
   return LLM_OK;
+}
+
+LLM_EXPORT int llm_attention_generic_ld(int dtype, const void *q, long long q_stride, void *out,
+                                        long long out_stride, const void *kcache, const void *vcache,
+                                        const int *tok_seq, const int *tok_pos, const int *page_table,
+                                        int pt_stride, int n_tokens, int n_heads, int n_kv, int d, int dv, int v_ld,
+                                        int page_size, int window, int block, int sink, float scale, const float *gate,
+                                        long long gate_stride, float null_score, cudaStream_t stream) {
+  return launch_generic(dtype, q, q_stride, out, out_stride, kcache, vcache, tok_seq, tok_pos, page_table, pt_stride, n_tokens, n_heads,
+                        n_kv, d, dv, v_ld, page_size, window, block, sink, scale, gate, gate_stride, null_score, nullptr, stream);
+}
+
+// The weights of SigmoidWeights instead of a softmax's.
+LLM_EXPORT int llm_attention_generic_sigmoid(int dtype, const void *q, long long q_stride, void *out, long long out_stride,
+                                             const void *kcache, const void *vcache, const int *tok_seq, const int *tok_pos,
+                                             const int *page_table, int pt_stride, int n_tokens, int n_heads, int n_kv, int d, int dv,
+                                             int page_size, int window, float scale, const float *temp, const float *bias, float cap,
+                                             float out_scale, cudaStream_t stream) {
+  LLM_REQUIRE(temp && bias && cap >= 0.f, "attention: sigmoid weights need a temperature and a bias per head");
+  const SigmoidWeights sig{temp, bias, cap, out_scale};
+  return launch_generic(dtype, q, q_stride, out, out_stride, kcache, vcache, tok_seq, tok_pos, page_table, pt_stride, n_tokens, n_heads,
+                        n_kv, d, dv, dv, page_size, window, 0, 0, scale, nullptr, 0, -INFINITY, &sig, stream);
 }
 
 LLM_EXPORT int llm_attention_generic(int dtype, const void *q, long long q_stride, void *out,

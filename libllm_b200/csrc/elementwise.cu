@@ -1229,3 +1229,38 @@ LLM_EXPORT int llm_add_scalar(float *x, long long n, float value, cudaStream_t s
   LLM_CHECK_LAUNCH("add_scalar");
   return LLM_OK;
 }
+
+// ---------------------------------------------------------------- additions at the start of a pass over looped layers
+// resid[r, c] = resid[r, c] + (sum of delta's parts + col_bias) * col_scale + other[r, c] + vec[c]; delta, other and vec may be
+// null.  32-bit, parts in order.  A CTA a row.
+__global__ void __launch_bounds__(256)
+stream_add_kernel(float *__restrict__ resid, const float *__restrict__ delta, int n_parts, long long part_stride,
+                  const float *__restrict__ col_scale, const float *__restrict__ col_bias, const float *__restrict__ other,
+                  const float *__restrict__ vec, int hidden) {
+  grid_dependents_launch();
+  grid_dependency_wait();
+  const size_t row = (size_t)blockIdx.x * hidden;
+  for (int c = threadIdx.x; c < hidden; c += 256) {
+    float v = resid[row + c];
+    if (n_parts > 0) {
+      float d = 0.f;
+      for (int p = 0; p < n_parts; ++p) d += delta[(size_t)p * part_stride + row + c];
+      if (col_bias) d += col_bias[c];
+      if (col_scale) d *= col_scale[c];
+      v += d;
+    }
+    if (other) v += other[row + c];
+    if (vec) v += vec[c];
+    resid[row + c] = v;
+  }
+}
+
+LLM_EXPORT int llm_stream_add(float *resid, const float *delta, int n_parts, long long part_stride, const float *col_scale,
+                              const float *col_bias, const float *other, const float *vec, int n_rows, int hidden, cudaStream_t stream) {
+  if (n_rows == 0) return LLM_OK;
+  LLM_REQUIRE(n_rows > 0 && hidden > 0 && resid && n_parts >= 0 && (n_parts == 0 || delta), "stream_add: bad arguments");
+  llm_launch(stream_add_kernel, dim3(n_rows), dim3(256), 0, stream, resid, delta, n_parts, part_stride, col_scale, col_bias, other, vec,
+             hidden);
+  LLM_CHECK_LAUNCH("stream_add");
+  return LLM_OK;
+}

@@ -227,6 +227,14 @@ void concat_stream(const float *resid, const Act *delta, const float *other, con
 void swiglu(const Act &gu, void *out, DType out_dtype, cudaStream_t s) {
   LLM_CALL("elementwise", llm_swiglu, code(gu.dtype), code(out_dtype), gu.data, out, (int)gu.rows, (int)(gu.cols / 2), s);
 }
+LLM_KERNEL("elementwise", llm_stream_add, float *, const float *, int, long long, const float *, const float *, const float *, const float *,
+           int, int, cudaStream_t)
+void stream_add(float *resid, const Act *delta, const float *other, const float *vec, int n_rows, int hidden, cudaStream_t s) {
+  if (delta && (delta->dtype != DType::F32 || delta->ld != hidden)) LLM_THROW(InvalidArg, "stream_add: the addition must be dense 32-bit rows");
+  LLM_CALL("elementwise", llm_stream_add, resid, delta ? (const float *)delta->data : nullptr, delta ? delta->parts : 0,
+           delta ? (long long)delta->part_stride : 0, delta ? delta->col_scale : nullptr, delta ? delta->col_bias : nullptr, other, vec,
+           n_rows, hidden, s);
+}
 void scale_rows(float *x, long long n, float scale, cudaStream_t s) { LLM_CALL("elementwise", llm_scale_rows, x, n, scale, s); }
 void logit_transform(float *logits, long long n, float scale, float softcap, cudaStream_t s) {
   LLM_CALL("elementwise", llm_logit_transform, logits, n, scale, softcap, s);
@@ -504,6 +512,29 @@ void attention_prefill_tc(const Act &q, const Act &out, const void *kc, const vo
            page_size, window, block, sink, scale, null_score, 0, status, s);
 }
 
+LLM_KERNEL("attention_generic", llm_attention_generic_sigmoid, int, const void *, long long, void *, long long, const void *, const void *,
+           const int *, const int *, const int *, int, int, int, int, int, int, int, int, float, const float *, const float *, float, float,
+           cudaStream_t)
+void attention_generic_sigmoid(const Act &q, const Act &out, const void *kc, const void *vc, const int *tok_seq, const int *tok_pos,
+                               const int *page_table, int pt_stride, int n_heads, int n_kv, int d, int dv, int page_size, int window,
+                               float scale, const float *temp, const float *bias, float cap, float out_scale, cudaStream_t s) {
+  LLM_CALL("attention_generic", llm_attention_generic_sigmoid, code(q.dtype), q.data, (long long)q.ld, out.data, (long long)out.ld, kc, vc,
+           tok_seq, tok_pos, page_table, pt_stride, (int)q.rows, n_heads, n_kv, d, dv, page_size, window, scale, temp, bias, cap, out_scale,
+           s);
+}
+LLM_KERNEL("rope", llm_conv_rope_place, int, const float *, long long, const float *, const float *, int, float *, void *, long long, int,
+           int, int, int, int, int, const float *, int, int, const int *, const int *, const int *, const int *, const int *, const int *,
+           int, void *, void *, int, int, int, cudaStream_t)
+void conv_rope_place(const Act &qkv, const float *bias, const float *conv, int taps, float *state, const Act &q_out, int n_heads, int n_kv,
+                     int d, int dv, const float *table, int table_rows, int rot_dim, const int *tok_seq, const int *tok_pos,
+                     const int *seq_start, const int *seq_past, const int *seq_slot, int n_seqs, const int *page_table, int pt_stride,
+                     void *kcache, void *vcache, int page_size, bool write_cache, bool single_tokens, cudaStream_t s) {
+  if (qkv.dtype != DType::F32) LLM_THROW(InvalidArg, "conv_rope_place: projections are 32-bit");
+  LLM_CALL("rope", llm_conv_rope_place, code(q_out.dtype), (const float *)qkv.data, (long long)qkv.ld, bias, conv, taps, state, q_out.data,
+           (long long)q_out.ld, (int)qkv.rows, n_seqs, n_heads, n_kv, d, dv, table, table_rows, rot_dim, tok_seq, tok_pos, seq_start, seq_past,
+           seq_slot, page_table, pt_stride, kcache, vcache, page_size, write_cache ? 1 : 0, single_tokens ? 1 : 0, s);
+}
+
 // ---------------------------------------------------------------- routed feed-forward
 LLM_KERNEL("moe", llm_activation, int, int, const void *, void *, long long, int, cudaStream_t)
 LLM_KERNEL("moe", llm_moe_route, const float *, long long, int, int, int, int, int, int *, float *, cudaStream_t)
@@ -632,6 +663,94 @@ void head_norm_gate(const Act &x, const float *weight, const float *gate, long l
   if (x.dtype != DType::F32) LLM_THROW(InvalidArg, "head_norm_gate: the heads' results are 32-bit");
   LLM_CALL("recurrent", llm_head_norm_gate, (const float *)x.data, (long long)x.ld, weight, gate, gate_stride, eps, (int)x.rows,
            n_heads, dv, out.data, code(out.dtype), (long long)out.ld, s);
+}
+
+// ---------------------------------------------------------------- linear recurrences over a matrix of state per head
+LLM_KERNEL("state_scan", llm_state_scan, int, const float *, const float *, const float *, long long, float *, float *, long long, float *,
+           const int *, const int *, int, int, int, int, int, int, cudaStream_t)
+LLM_KERNEL("state_scan", llm_delta_pack, const float *, long long, const float *, long long, int, int, const float *, const float *, float,
+           float, float *, float *, int, int, int, int, cudaStream_t)
+LLM_KERNEL("state_scan", llm_bonus_pack, const float *, long long, const float *, long long, const float *, long long, int, const float *,
+           const float *, const float *, float *, float *, int, int, int, cudaStream_t)
+LLM_KERNEL("state_scan", llm_memory_pack, const float *, long long, int, int, int, int, const float *, const float *, float, float, float *,
+           float *, float *, const int *, const int *, int, int, int, int, cudaStream_t)
+LLM_KERNEL("state_scan", llm_head_finish, const float *, long long, const float *, const float *, const float *, int, const float *,
+           long long, int, float, float, int, int, int, void *, int, long long, cudaStream_t)
+LLM_KERNEL("state_scan", llm_token_shift, int, const void *, long long, const float *, int, void *, long long, void *, const int *,
+           const int *, const int *, const int *, const int *, int, int, int, int, cudaStream_t)
+LLM_KERNEL("state_scan", llm_delta_gated_step, const float *, long long, int, int, int, int, int, int, const float *, float *, int,
+           const float *, const float *, float, float, float *, const float *, int, int, float, float, void *, int, long long, const int *,
+           int, int, int, int, int, cudaStream_t)
+LLM_KERNEL("state_scan", llm_bonus_step, const float *, long long, const float *, long long, const float *, long long, const float *,
+           long long, const float *, long long, int, const float *, const float *, const float *, float *, const float *, int, float, float,
+           void *, int, long long, const int *, int, int, int, int, cudaStream_t)
+LLM_KERNEL("state_scan", llm_memory_step, const float *, long long, int, int, int, int, int, int, const float *, const float *, float, float,
+           float *, float *, const float *, int, float, float, void *, int, long long, const int *, int, int, int, int, cudaStream_t)
+void state_scan(ScanRule rule, const float *rec, const float *scal, const float *v, long long ldv, float *state, const Act &out, float *den,
+                const int *seq_start, const int *seq_slot, int n_seqs, int n_heads, int n_kv, int d, int dv, cudaStream_t s) {
+  if (out.dtype != DType::F32) LLM_THROW(InvalidArg, "state_scan: results are 32-bit");
+  LLM_CALL("state_scan", llm_state_scan, (int)rule, rec, scal, v, ldv, state, (float *)out.data, (long long)out.ld, den, seq_start, seq_slot,
+           (int)out.rows, n_seqs, n_heads, n_kv, d, dv, s);
+}
+void delta_pack(const Act &cv, const Act &proj, int off_b, int off_a, const float *dt_bias, const float *a_log, float key_eps, float q_scale,
+                float *rec, float *scal, int n_heads, int n_kv, int d, cudaStream_t s) {
+  if (cv.dtype != DType::F32 || proj.dtype != DType::F32) LLM_THROW(InvalidArg, "delta_pack: projections are 32-bit");
+  LLM_CALL("state_scan", llm_delta_pack, (const float *)cv.data, (long long)cv.ld, (const float *)proj.data, (long long)proj.ld, off_b, off_a,
+           dt_bias, a_log, key_eps, q_scale, rec, scal, (int)proj.rows, n_heads, n_kv, d, s);
+}
+void bonus_pack(const Act &r, const Act &k, const Act &x1, int rank, const float *w2, const float *w0, const float *u, float *rec,
+                float *scal, int n_heads, int d, cudaStream_t s) {
+  if (r.dtype != DType::F32 || k.dtype != DType::F32 || x1.dtype != DType::F32) LLM_THROW(InvalidArg, "bonus_pack: projections are 32-bit");
+  LLM_CALL("state_scan", llm_bonus_pack, (const float *)r.data, (long long)r.ld, (const float *)k.data, (long long)k.ld,
+           (const float *)x1.data, (long long)x1.ld, rank, w2, w0, u, rec, scal, (int)r.rows, n_heads, d, s);
+}
+void memory_pack(const Act &proj, int off_q, int off_k, int off_i, int off_f, const float *bias_i, const float *bias_f, float cap,
+                 float q_scale, float *state_m, float *rec, float *scal, const int *seq_start, const int *seq_slot, int n_seqs, int n_heads,
+                 int d, cudaStream_t s) {
+  if (proj.dtype != DType::F32) LLM_THROW(InvalidArg, "memory_pack: projections are 32-bit");
+  LLM_CALL("state_scan", llm_memory_pack, (const float *)proj.data, (long long)proj.ld, off_q, off_k, off_i, off_f, bias_i, bias_f, cap,
+           q_scale, state_m, rec, scal, seq_start, seq_slot, (int)proj.rows, n_seqs, n_heads, d, s);
+}
+void head_finish(const Act &x, const float *den, const float *scal, const float *weight, bool shared_weight, const float *gate,
+                 long long gate_stride, GateAct act, float eps, float out_scale, int n_heads, int dv, const Act &out, cudaStream_t s) {
+  if (x.dtype != DType::F32) LLM_THROW(InvalidArg, "head_finish: the heads' results are 32-bit");
+  LLM_CALL("state_scan", llm_head_finish, (const float *)x.data, (long long)x.ld, den, scal, weight, shared_weight ? 1 : 0, gate, gate_stride,
+           (int)act, eps, out_scale, (int)x.rows, n_heads, dv, out.data, code(out.dtype), (long long)out.ld, s);
+}
+void token_shift(const Act &h, const float *mu, int n_mix, const Act &out, void *state, const int *tok_seq, const int *tok_pos,
+                 const int *seq_start, const int *seq_past, const int *seq_slot, int n_seqs, bool single_tokens, cudaStream_t s) {
+  if (h.dtype != out.dtype) LLM_THROW(InvalidArg, "token_shift: input and output have one type");
+  LLM_CALL("state_scan", llm_token_shift, code(h.dtype), h.data, (long long)h.ld, mu, n_mix, out.data, (long long)(h.rows * h.cols), state,
+           tok_seq, tok_pos, seq_start, seq_past, seq_slot, (int)h.rows, n_seqs, (int)h.cols, single_tokens ? 1 : 0, s);
+}
+bool state_step_supported(int d, int dv, int group, int rank) {
+  static auto f = resolve<int (*)(int, int, int, int)>("state_scan", "llm_state_step_supports");
+  return f(d, dv, group, rank) != 0;
+}
+void delta_gated_step(const Act &proj, int off_q, int off_k, int off_v, int off_g, int off_b, int off_a, const float *conv, float *conv_state,
+                      int taps, const float *dt_bias, const float *a_log, float key_eps, float q_scale, float *state, const float *weight,
+                      bool shared_weight, GateAct act, float eps, float out_scale, const Act &out, const int *seq_slot, int n_heads, int n_kv,
+                      int d, int dv, cudaStream_t s) {
+  if (proj.dtype != DType::F32) LLM_THROW(InvalidArg, "delta_gated_step: projections are 32-bit");
+  LLM_CALL("state_scan", llm_delta_gated_step, (const float *)proj.data, (long long)proj.ld, off_q, off_k, off_v, off_g, off_b, off_a, conv,
+           conv_state, taps, dt_bias, a_log, key_eps, q_scale, state, weight, shared_weight ? 1 : 0, (int)act, eps, out_scale, out.data,
+           code(out.dtype), (long long)out.ld, seq_slot, (int)proj.rows, n_heads, n_kv, d, dv, s);
+}
+void bonus_step(const Act &r, const Act &k, const Act &v, const Act &g, const Act &x1, int rank, const float *w2, const float *w0,
+                const float *u, float *state, const float *weight, GateAct act, float eps, float out_scale, const Act &out, const int *seq_slot,
+                int n_heads, int d, int dv, cudaStream_t s) {
+  if (r.dtype != DType::F32 || x1.dtype != DType::F32) LLM_THROW(InvalidArg, "bonus_step: projections are 32-bit");
+  LLM_CALL("state_scan", llm_bonus_step, (const float *)r.data, (long long)r.ld, (const float *)k.data, (long long)k.ld, (const float *)v.data,
+           (long long)v.ld, (const float *)g.data, (long long)g.ld, (const float *)x1.data, (long long)x1.ld, rank, w2, w0, u, state, weight,
+           (int)act, eps, out_scale, out.data, code(out.dtype), (long long)out.ld, seq_slot, (int)r.rows, n_heads, d, dv, s);
+}
+void memory_step(const Act &proj, int off_q, int off_k, int off_v, int off_g, int off_i, int off_f, const float *bias_i, const float *bias_f,
+                 float cap, float q_scale, float *state_m, float *state, const float *weight, GateAct act, float eps, float out_scale,
+                 const Act &out, const int *seq_slot, int n_heads, int d, int dv, cudaStream_t s) {
+  if (proj.dtype != DType::F32) LLM_THROW(InvalidArg, "memory_step: projections are 32-bit");
+  LLM_CALL("state_scan", llm_memory_step, (const float *)proj.data, (long long)proj.ld, off_q, off_k, off_v, off_g, off_i, off_f, bias_i,
+           bias_f, cap, q_scale, state_m, state, weight, (int)act, eps, out_scale, out.data, code(out.dtype), (long long)out.ld, seq_slot,
+           (int)proj.rows, n_heads, d, dv, s);
 }
 
 // ---------------------------------------------------------------- sampling

@@ -53,6 +53,8 @@ void swiglu(const Act &gu, void *out, DType out_dtype, cudaStream_t s);
 void clamped_glu(const Act &gu, const float *bias, const Act &out, float limit, float slope, float up_shift, cudaStream_t s);
 // out[t] = [resid[t] + delta's parts at t | other[t]] in out's type, [rows, 2 * hidden]
 void concat_stream(const float *resid, const Act *delta, const float *other, const Act &out, int hidden, cudaStream_t s);
+// resid += delta's parts (with its column bias and scale) + other's rows + vec; delta, other and vec may be null
+void stream_add(float *resid, const Act *delta, const float *other, const float *vec, int n_rows, int hidden, cudaStream_t s);
 void scale_rows(float *x, long long n, float scale, cudaStream_t s);
 void logit_transform(float *logits, long long n, float scale, float softcap, cudaStream_t s);
 void random_fill(void *out, DType dtype, long long n, unsigned long long seed, int law, float a, float b, cudaStream_t s);
@@ -116,6 +118,12 @@ void rope_pairs_place(const Act &qkv, const Act &q_out, int n_heads, int n_kv, i
 void kv_place(const Act &qkv, const Act &q_out, int n_heads, int n_kv, int d, int dv, const float *bias, float v_eps,
               const int *tok_seq, const int *tok_pos, const int *page_table, int pt_stride, void *kcache, void *vcache,
               int page_size, bool write_cache, cudaStream_t s);
+// 32-bit rows [q | k | v] + bias, a causal convolution over time per channel (conv [taps, channels]; state [slots, taps - 1,
+// channels] of biased inputs), rotation of q and k (pairs i, i + rot_dim/2), q -> q_out, k and v to the cache: one pass.
+void conv_rope_place(const Act &qkv, const float *bias, const float *conv, int taps, float *state, const Act &q_out, int n_heads, int n_kv,
+                     int d, int dv, const float *table, int table_rows, int rot_dim, const int *tok_seq, const int *tok_pos,
+                     const int *seq_start, const int *seq_past, const int *seq_slot, int n_seqs, const int *page_table, int pt_stride,
+                     void *kcache, void *vcache, int page_size, bool write_cache, bool single_tokens, cudaStream_t s);
 // ---- attention
 constexpr float NO_NULL_KEY = -__builtin_huge_valf();
 // Masks: `window` > 0, a query sees the last `window` keys; `block` > 0, only keys of its own block
@@ -128,6 +136,11 @@ void attention_generic(const Act &q, const Act &out, const void *kc, const void 
 // v_ld > 0: value rows lie v_ld channels apart (the values are the first dv channels of the key rows when vc is kc).
 // null_score: every query also sees one key of that score that has no value (exp(null_score) joins the softmax's
 // denominator); NO_NULL_KEY: none.
+// Weights that stand for themselves: sigmoid(cap tanh(temp[h] s / cap) + bias[h]) (cap 0: no bound), not normalised; the result
+// times out_scale.
+void attention_generic_sigmoid(const Act &q, const Act &out, const void *kc, const void *vc, const int *tok_seq, const int *tok_pos,
+                               const int *page_table, int pt_stride, int n_heads, int n_kv, int d, int dv, int page_size, int window,
+                               float scale, const float *temp, const float *bias, float cap, float out_scale, cudaStream_t s);
 // ---- latent attention (csrc/latent.cu): attention over one cached row [c | k_r] per position that every head reads
 // proj rows (32-bit) hold the query latent at off_q and, with off_kv >= 0, the key/value latent and the shared key part;
 // cq_out = rms(query latent) * q_weight; the token's cache row = [rms(first kv_rank) * kv_weight | rotated last rot].
@@ -235,6 +248,37 @@ void delta_step(const Act &proj, int off_r, int off_k, int off_v, int off_g, int
 // out[t, h, :] = x / rms(x over the head; eps < 0: no norm) * weight (null: none) * sigmoid(gate) (null: none)
 void head_norm_gate(const Act &x, const float *weight, const float *gate, long long gate_stride, float eps, int n_heads, int dv,
                     const Act &out, cudaStream_t s);
+// ---- linear recurrences over a matrix of state per head (csrc/state_scan.cu)
+enum ScanRule { ScanDelta = 0, ScanBonus = 1, ScanMemory = 2 };
+enum GateAct { GateSigmoid = 0, GateSilu = 1 };
+// rec [tokens, kv_heads, 2 (bonus: 3), d padded to 4], scal [tokens, heads, 4], v rows; state [slots, heads, dv (memory: + 1), d]
+void state_scan(ScanRule rule, const float *rec, const float *scal, const float *v, long long ldv, float *state, const Act &out, float *den,
+                const int *seq_start, const int *seq_slot, int n_seqs, int n_heads, int n_kv, int d, int dv, cudaStream_t s);
+void delta_pack(const Act &cv, const Act &proj, int off_b, int off_a, const float *dt_bias, const float *a_log, float key_eps, float q_scale,
+                float *rec, float *scal, int n_heads, int n_kv, int d, cudaStream_t s);
+void bonus_pack(const Act &r, const Act &k, const Act &x1, int rank, const float *w2, const float *w0, const float *u, float *rec,
+                float *scal, int n_heads, int d, cudaStream_t s);
+void memory_pack(const Act &proj, int off_q, int off_k, int off_i, int off_f, const float *bias_i, const float *bias_f, float cap,
+                 float q_scale, float *state_m, float *rec, float *scal, const int *seq_start, const int *seq_slot, int n_seqs, int n_heads,
+                 int d, cudaStream_t s);
+// norm per head (of x / (max(|den|, floor) + 1e-6) where den is given), weight, gate, out_scale
+void head_finish(const Act &x, const float *den, const float *scal, const float *weight, bool shared_weight, const float *gate,
+                 long long gate_stride, GateAct act, float eps, float out_scale, int n_heads, int dv, const Act &out, cudaStream_t s);
+// out [n_mix * tokens, width]: h + (the token before's h - h) mu; state [slots, width] in h's type, a sequence's last row
+void token_shift(const Act &h, const float *mu, int n_mix, const Act &out, void *state, const int *tok_seq, const int *tok_pos,
+                 const int *seq_start, const int *seq_past, const int *seq_slot, int n_seqs, bool single_tokens, cudaStream_t s);
+// A step of single tokens (row b = sequence b): everything between the products and the output projection in one launch.
+bool state_step_supported(int d, int dv, int group, int rank);
+void delta_gated_step(const Act &proj, int off_q, int off_k, int off_v, int off_g, int off_b, int off_a, const float *conv, float *conv_state,
+                      int taps, const float *dt_bias, const float *a_log, float key_eps, float q_scale, float *state, const float *weight,
+                      bool shared_weight, GateAct act, float eps, float out_scale, const Act &out, const int *seq_slot, int n_heads, int n_kv,
+                      int d, int dv, cudaStream_t s);
+void bonus_step(const Act &r, const Act &k, const Act &v, const Act &g, const Act &x1, int rank, const float *w2, const float *w0,
+                const float *u, float *state, const float *weight, GateAct act, float eps, float out_scale, const Act &out, const int *seq_slot,
+                int n_heads, int d, int dv, cudaStream_t s);
+void memory_step(const Act &proj, int off_q, int off_k, int off_v, int off_g, int off_i, int off_f, const float *bias_i, const float *bias_f,
+                 float cap, float q_scale, float *state_m, float *state, const float *weight, GateAct act, float eps, float out_scale,
+                 const Act &out, const int *seq_slot, int n_heads, int d, int dv, cudaStream_t s);
 // ---- sampling
 void argmax(const float *logits, long long stride, int n_rows, int vocab, int *out, cudaStream_t s);
 void sample(const float *logits, long long stride, int n_rows, int vocab, float temperature, int top_k, float top_p,

@@ -726,3 +726,232 @@ LLM_EXPORT int llm_rope_headnorm_place(int in_dtype, int dtype, const void *qkv,
   LLM_CHECK_LAUNCH("rope_headnorm_place");
   return LLM_OK;
 }
+
+// ---------------------------------------------------------------- convolution, rotation, placement in one pass
+// 32-bit rows [q (heads x d) | k (kv_heads x d) | v (kv_heads x dv)] of a stacked product; u = row + bias.  Every channel goes
+// through a causal convolution over time, y_t = sum_j w[j] u_(t - taps + 1 + j) (w [taps][channels]; nought before the sequence's
+// start); then q and k are rotated as above (pairs i, i + rot_dim/2 of each head), q goes to q_out, k and v to the cache.
+// The last taps - 1 rows of u are the sequence's state, state[slot][i] for the position length - (taps - 1) + i, 32-bit.
+// A thread owns a unit of two groups of V channels, the two halves of V pairs, or one group that is not rotated, and walks
+// CP_ROWS rows with the last taps values of its channels in registers.  Rows whose window lies inside the step belong to CTAs
+// of a run of rows (blockIdx.x < n_chunks), the first taps - 1 rows of every sequence, and its state, to a CTA of that
+// sequence, whose threads read the old state of their channels before they write the new one: nobody else reads it.
+// The order of operations is the same wherever a row is computed.
+constexpr int CP_THREADS = 128, CP_ROWS = 16, CP_MAX_TAPS = 8;
+
+template <int V>
+__device__ __forceinline__ void cp_load(const float *p, float (&x)[V]) {
+  if constexpr (V == 4) {
+    const float4 v = ld4(p);
+    x[0] = v.x, x[1] = v.y, x[2] = v.z, x[3] = v.w;
+  } else {
+    x[0] = p[0];
+  }
+}
+template <typename T, int V>
+__device__ __forceinline__ void cp_store(T *p, const float (&x)[V]) {
+  if constexpr (V == 4) st4(p, make_float4(x[0], x[1], x[2], x[3]));
+  else p[0] = from_float<T>(x[0]);
+}
+
+template <typename T, int V, int TAPS>
+__global__ void __launch_bounds__(CP_THREADS)
+conv_rope_place_kernel(const float *__restrict__ qkv, long long ld, const float *__restrict__ bias, const float *__restrict__ conv,
+                       int taps, float *__restrict__ state, T *__restrict__ q_out, long long q_stride, int n_heads, int n_kv, int d, int dv,
+                       const float *__restrict__ table, int table_rows, int rot_dim, const int *__restrict__ tok_seq,
+                       const int *__restrict__ tok_pos, const int *__restrict__ seq_start, const int *__restrict__ seq_past,
+                       const int *__restrict__ seq_slot, const int *__restrict__ page_table, int pt_stride, T *__restrict__ kcache,
+                       T *__restrict__ vcache, int page_size, int write_cache, int n_tokens, int n_chunks) {
+  grid_dependents_launch();
+  const int half = rot_dim / 2, rot_units = half / V, head_units = rot_units + (d - rot_dim) / V;
+  const int qk_units = (n_heads + n_kv) * head_units, n_units = qk_units + n_kv * (dv / V);
+  const int unit = blockIdx.y * CP_THREADS + threadIdx.x;
+  const int channels = (n_heads + n_kv) * d + n_kv * dv;
+  // the unit's channels: c0 and, where it is rotated, c1 = c0 + half
+  int head = 0, ch = 0, c0 = 0;
+  bool rotated = false, is_v = false;
+  if (unit < qk_units) {
+    head = unit / head_units;
+    const int i = unit - head * head_units;
+    rotated = i < rot_units;
+    ch = rotated ? i * V : rot_dim + (i - rot_units) * V;
+    c0 = head * d + ch;
+  } else if (unit < n_units) {
+    is_v = true;
+    head = (unit - qk_units) / (dv / V);
+    ch = (unit - qk_units - head * (dv / V)) * V;
+    c0 = (n_heads + n_kv) * d + head * dv + ch;
+  }
+  const int c1 = rotated ? c0 + half : c0;
+  float w[2][TAPS][V], bs[2][V];
+  if (unit < n_units) {                                // weights: nothing of the step is read yet
+#pragma unroll
+    for (int s = 0; s < 2; ++s) {
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        if (j < taps && conv) cp_load<V>(conv + (size_t)j * channels + (s ? c1 : c0), w[s][j]);
+        else
+#pragma unroll
+          for (int e = 0; e < V; ++e) w[s][j][e] = j == taps - 1 ? 1.f : 0.f;
+      }
+      if (bias) cp_load<V>(bias + (s ? c1 : c0), bs[s]);
+      else
+#pragma unroll
+        for (int e = 0; e < V; ++e) bs[s][e] = 0.f;
+    }
+  }
+  grid_dependency_wait();
+  if (unit >= n_units) return;
+  const int keep = taps - 1;
+  float win[2][TAPS][V];                               // win[.][j]: u at the row's position - taps + 1 + j
+  auto take = [&](int row, float (&x0)[V], float (&x1)[V]) {
+    cp_load<V>(qkv + (size_t)row * ld + c0, x0);
+    if (rotated) cp_load<V>(qkv + (size_t)row * ld + c1, x1);
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      x0[e] += bs[0][e];
+      if (rotated) x1[e] += bs[1][e];
+    }
+  };
+  auto shift = [&](const float (&x0)[V], const float (&x1)[V]) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        if (j < taps - 1 && j + 1 < TAPS) {
+          win[0][j][e] = win[0][j + 1 < TAPS ? j + 1 : j][e];
+          win[1][j][e] = win[1][j + 1 < TAPS ? j + 1 : j][e];
+        } else if (j == taps - 1) {
+          win[0][j][e] = x0[e];
+          win[1][j][e] = x1[e];
+        }
+      }
+  };
+  auto place = [&](int row) {
+    float y0[V], y1[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      y0[e] = y1[e] = 0.f;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j)
+        if (j < taps) {
+          y0[e] = fmaf(w[0][j][e], win[0][j][e], y0[e]);
+          if (rotated) y1[e] = fmaf(w[1][j][e], win[1][j][e], y1[e]);
+        }
+    }
+    const int pos = tok_pos[row];
+    if (rotated) {
+      const float *cs = table + (size_t)(pos < table_rows ? pos : table_rows - 1) * rot_dim + ch;
+      float co[V], si[V];
+      cp_load<V>(cs, co);
+      cp_load<V>(cs + half, si);
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        const float a = y0[e], b = y1[e];
+        y0[e] = a * co[e] - b * si[e];
+        y1[e] = b * co[e] + a * si[e];
+      }
+    }
+    T *dst;
+    if (!is_v && head < n_heads) {
+      dst = q_out + (size_t)row * q_stride + c0;
+    } else {
+      if (!write_cache) return;
+      const int page = page_table[(size_t)tok_seq[row] * pt_stride + pos / page_size];
+      const int kvh = is_v ? head : head - n_heads, width = is_v ? dv : d;
+      dst = (is_v ? vcache : kcache) + (((size_t)page * n_kv + kvh) * page_size + pos % page_size) * (size_t)width + ch;
+    }
+    cp_store<T, V>(dst, y0);
+    if (rotated) cp_store<T, V>(dst + half, y1);
+  };
+  float x0[V], x1[V];
+#pragma unroll
+  for (int e = 0; e < V; ++e) x0[e] = x1[e] = 0.f;
+  if ((int)blockIdx.x < n_chunks) {
+    const int r0 = blockIdx.x * CP_ROWS, r1 = min(n_tokens, r0 + CP_ROWS);
+    int filled = -1;                                   // the last row in the window; -1: none
+    for (int row = r0; row < r1; ++row) {
+      if (tok_pos[row] - seq_past[tok_seq[row]] < keep) {          // the sequence's own CTA computes it
+        filled = -1;
+        continue;
+      }
+      if (filled != row - 1 || filled < 0)
+        for (int k = keep; k > 0; --k) {
+          take(row - k, x0, x1);
+          shift(x0, x1);
+        }
+      take(row, x0, x1);
+      shift(x0, x1);
+      filled = row;
+      place(row);
+    }
+    return;
+  }
+  const int b = blockIdx.x - n_chunks, start = seq_start[b], n = seq_start[b + 1] - start;
+  float *st = state ? state + (size_t)seq_slot[b] * keep * channels : nullptr;
+  for (int i = 0; i < keep; ++i) {
+    cp_load<V>(st + (size_t)i * channels + c0, x0);
+    if (rotated) cp_load<V>(st + (size_t)i * channels + c1, x1);
+    shift(x0, x1);
+  }
+  // the first rows through the window, then what the state holds next: the last `keep` inputs
+  for (int i = 0; i < min(n, keep > 0 ? keep : 0); ++i) {
+    take(start + i, x0, x1);
+    shift(x0, x1);
+    place(start + i);
+  }
+  if (n > keep)
+    for (int k = keep; k > 0; --k) {
+      take(start + n - k, x0, x1);
+      shift(x0, x1);
+    }
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j)
+    if (j >= 1 && j < taps) {
+      cp_store<float, V>(st + (size_t)(j - 1) * channels + c0, win[0][j]);
+      if (rotated) cp_store<float, V>(st + (size_t)(j - 1) * channels + c1, win[1][j]);
+    }
+}
+
+// `conv` null with taps 1: no convolution.  single_tokens: every sequence brings one token.
+LLM_EXPORT int llm_conv_rope_place(int dtype, const float *qkv, long long ld, const float *bias, const float *conv, int taps, float *state,
+                                   void *q_out, long long q_stride, int n_tokens, int n_seqs, int n_heads, int n_kv, int d, int dv,
+                                   const float *table, int table_rows, int rot_dim, const int *tok_seq, const int *tok_pos,
+                                   const int *seq_start, const int *seq_past, const int *seq_slot, const int *page_table, int pt_stride,
+                                   void *kcache, void *vcache, int page_size, int write_cache, int single_tokens, cudaStream_t stream) {
+  if (n_tokens == 0) return LLM_OK;
+  LLM_REQUIRE(n_tokens > 0 && n_seqs > 0 && n_heads > 0 && n_kv > 0 && d > 0 && dv > 0, "conv_rope_place: bad sizes");
+  LLM_REQUIRE(taps >= 1 && taps <= CP_MAX_TAPS && (taps == 1 || (conv && state)), "conv_rope_place: a convolution of %d taps (1 to %d) needs its weight and state",
+              taps, CP_MAX_TAPS);
+  LLM_REQUIRE(rot_dim % 2 == 0 && rot_dim <= d && rot_dim >= 0 && (rot_dim == 0 || (table && table_rows > 0)),
+              "conv_rope_place: rotated width %d does not fit head size %d", rot_dim, d);
+  const long long channels = (long long)(n_heads + n_kv) * d + (long long)n_kv * dv;
+  LLM_REQUIRE(ld >= channels, "conv_rope_place: the stacked rows are too short");
+  const int n_chunks = single_tokens && taps > 1 ? 0 : (n_tokens + CP_ROWS - 1) / CP_ROWS, n_own = taps > 1 ? n_seqs : 0;
+  const int esz = dtype == LLM_F32 ? 4 : 2;
+  const bool vec = d % 4 == 0 && dv % 4 == 0 && rot_dim % 8 == 0 && ld % 4 == 0 && q_stride % 4 == 0 && (uintptr_t)qkv % 16 == 0 &&
+                   (uintptr_t)bias % 16 == 0 && (uintptr_t)conv % 16 == 0 && (uintptr_t)state % 16 == 0 && (uintptr_t)table % 16 == 0 &&
+                   (uintptr_t)q_out % (4 * esz) == 0 && (uintptr_t)kcache % (4 * esz) == 0 && (uintptr_t)vcache % (4 * esz) == 0;
+  const int v = vec ? 4 : 1;
+  const long long units = (long long)(n_heads + n_kv) * (rot_dim / 2 / v + (d - rot_dim) / v) + (long long)n_kv * (dv / v);
+  const dim3 grid(n_chunks + n_own, (unsigned)((units + CP_THREADS - 1) / CP_THREADS));
+  LLM_REQUIRE(grid.y <= 65535, "conv_rope_place: too many channels");
+#define CP_GO(T, V, TAPS)                                                                                                    \
+  llm_launch(conv_rope_place_kernel<T, V, TAPS>, grid, dim3(CP_THREADS), 0, stream, qkv, ld, bias, conv, taps, state, (T *)q_out, q_stride, \
+             n_heads, n_kv, d, dv, table, table_rows, rot_dim, tok_seq, tok_pos, seq_start, seq_past, seq_slot, page_table, pt_stride, \
+             (T *)kcache, (T *)vcache, page_size, write_cache, n_tokens, n_chunks)
+#define CP_TAPS(T, V)                  \
+  do {                                 \
+    if (taps <= 4) CP_GO(T, V, 4);     \
+    else CP_GO(T, V, CP_MAX_TAPS);     \
+  } while (0)
+  if (dtype == LLM_F32 && vec) CP_TAPS(float, 4);
+  else if (dtype == LLM_F32) CP_TAPS(float, 1);
+  else if (dtype == LLM_BF16 && vec) CP_TAPS(__nv_bfloat16, 4);
+  else if (dtype == LLM_BF16) CP_TAPS(__nv_bfloat16, 1);
+  else LLM_FAIL("conv_rope_place: unsupported dtype %d", dtype);
+#undef CP_TAPS
+#undef CP_GO
+  LLM_CHECK_LAUNCH("conv_rope_place");
+  return LLM_OK;
+}

@@ -83,7 +83,18 @@ Model::Model(ModelSpec spec, Json config, DType dtype, int64_t max_positions, in
       LLM_THROW(Config, "schedule entry %zu reads the cache of entry %d, which does not run before it", i, e.cache_from);
     if (!e.input_mix.empty() && spec_.streams > 1) LLM_THROW(Unsupported, "an input mix goes with one residual stream");
     if (!e.input_mix.empty()) input_mixes_[e.input_mix];
+    if ((e.add_tokens || !e.add_vector.empty()) && spec_.streams > 1) LLM_THROW(Unsupported, "additions before a run go with one residual stream");
+    if (!e.add_vector.empty()) {
+      int64_t &rows = added_vectors_[e.add_vector].rows;
+      rows = std::max<int64_t>(rows, e.add_row + 1);
+    }
+    needs_tokens_ = needs_tokens_ || e.add_tokens || !e.input_mix.empty();
   }
+}
+
+// drawn, not read: a step vector no larger than the stream it is added to
+TensorNeed Model::added_need(const std::string &name, int64_t rows) const {
+  return {name, {rows, spec_.hidden}, TensorRole::Vector, false, 0.1f};
 }
 
 std::vector<TensorNeed> Model::tensor_needs() const {
@@ -94,6 +105,7 @@ std::vector<TensorNeed> Model::tensor_needs() const {
     for (auto &n : l->tensor_needs()) needs.push_back(n);
   for (auto &n : final_norm_->tensor_needs()) needs.push_back(n);
   for (const auto &kv : input_mixes_) needs.push_back({kv.first, {spec_.hidden, 2 * spec_.hidden}});
+  for (const auto &kv : added_vectors_) needs.push_back(added_need(kv.first, kv.second.rows));
   if (!spec_.head.empty()) needs.push_back({spec_.head, {spec_.vocab_size, spec_.hidden}});
   return needs;
 }
@@ -120,6 +132,7 @@ void Model::load_with(const Loader &loader) {
   for (auto &l : layers_) l->load(loader);
   final_norm_->load(loader);
   for (auto &kv : input_mixes_) kv.second = loader.fetch({kv.first, {spec_.hidden, 2 * spec_.hidden}});
+  for (auto &kv : added_vectors_) kv.second = loader.fetch(added_need(kv.first, kv.second.rows));
   if (spec_.head.empty()) {
     head_ = &embedding_;
   } else {
@@ -178,6 +191,18 @@ void Model::mix_input(StepContext &ctx, ResidualStream &stream, const float *x0,
   LLM_CUDA(cudaMemcpyAsync(stream.resid, y.data, sizeof(float) * (size_t)(T * H), cudaMemcpyDeviceToDevice, ctx.stream));
 }
 
+// x <- x (+ what is pending) + x0 + a vector: what a run of looped layers has added to its input.
+void Model::add_to_input(StepContext &ctx, ResidualStream &stream, const float *x0, const float *vec) {
+  flush_chain(ctx);
+  const int64_t T = stream.rows, H = stream.hidden;
+  if (stream.pending.data && stream.pending.dtype != DType::F32) {
+    kernels::add_rmsnorm(stream.resid, &stream.pending, nullptr, 0.f, nullptr, ctx.dtype, nullptr, (int)T, (int)H, ctx.stream);
+    stream.pending = Act();
+  }
+  kernels::stream_add(stream.resid, stream.pending.data ? &stream.pending : nullptr, x0, vec, (int)T, (int)H, ctx.stream);
+  stream.pending = Act();
+}
+
 Act Model::forward(StepContext &ctx, KVCache &cache, const std::vector<const int *> &tables, int table_width,
                    const int *fed_tokens, const int *fed_rows) {
   if (!loaded_) LLM_THROW(InvalidArg, "the model has no weights yet");
@@ -188,7 +213,7 @@ Act Model::forward(StepContext &ctx, KVCache &cache, const std::vector<const int
                      (int)spec_.vocab_size, ctx.stream, positions_.data(), (int)positions_.rows, ctx.tok_pos);
   if (spec_.embedding_scale != 1.0) kernels::scale_rows(resid, T * H, (float)spec_.embedding_scale, ctx.stream);
   float *x0 = nullptr;                       // the token rows, kept for the runs that mix them in again
-  if (!input_mixes_.empty()) {
+  if (needs_tokens_) {
     x0 = ctx.arena->alloc_n<float>((size_t)(T * H));
     LLM_CUDA(cudaMemcpyAsync(x0, resid, sizeof(float) * (size_t)(T * H), cudaMemcpyDeviceToDevice, ctx.stream));
   }
@@ -207,6 +232,9 @@ Act Model::forward(StepContext &ctx, KVCache &cache, const std::vector<const int
       ctx.arena->reset();
     }
     if (!e.input_mix.empty()) mix_input(ctx, stream, x0, input_mixes_.at(e.input_mix));
+    if (e.add_tokens || !e.add_vector.empty())
+      add_to_input(ctx, stream, e.add_tokens ? x0 : nullptr,
+                   e.add_vector.empty() ? nullptr : added_vectors_.at(e.add_vector).buf.as<float>() + (size_t)e.add_row * (size_t)H);
     const bool last = i + 1 == spec_.schedule.size();
     ctx.rows_read_after = last && ctx.n_want > 0 && ctx.n_want < ctx.n_tokens ? ctx.want_rows : nullptr;
     ctx.n_rows_read_after = ctx.rows_read_after ? ctx.n_want : 0;

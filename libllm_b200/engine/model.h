@@ -68,7 +68,11 @@ class Model {
   std::unique_ptr<Norm> final_norm_;
   Weight embedding_, head_own_, positions_;        // positions_: ModelSpec::position_table, in the token table's type
   std::map<std::string, Weight> input_mixes_;      // ScheduleEntry::input_mix -> [hidden, 2 * hidden]
+  std::map<std::string, Weight> added_vectors_;    // ScheduleEntry::add_vector -> [rows, hidden], 32-bit
+  bool needs_tokens_ = false;                      // some run mixes or adds the token rows in again
   void mix_input(StepContext &ctx, ResidualStream &stream, const float *x0, const Weight &w);
+  void add_to_input(StepContext &ctx, ResidualStream &stream, const float *x0, const float *vec);
+  TensorNeed added_need(const std::string &name, int64_t rows) const;
   const Weight *head_ = nullptr;
   bool loaded_ = false;
 };

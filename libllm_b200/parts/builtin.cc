@@ -17,7 +17,8 @@ ConfigReader reader_of(const Json &spec, const char *what) { return ConfigReader
 
 // ---------------------------------------------------------------- RMSNorm
 // y = x * w / sqrt(mean(x^2) + eps), sums and scaling in 32-bit (src/flint/cpu/normalizations.cc:52-64,
-// src/flint/cuda/rms_norm.cu:59-75).  With `weight_offset` c the stored weight is applied as (c + w).  Before the norm the stream's pending addition is applied in
+// src/flint/cuda/rms_norm.cu:59-75).  With `weight_offset` c the stored weight is applied as (c + w); with `one_gain` it is a
+// single number for all channels (a tensor without dimensions).  Before the norm the stream's pending addition is applied in
 // 32-bit: the reference's separate residual add (src/libllm/llama.cc:252-266).
 class RMSNorm : public Norm {
  public:
@@ -27,10 +28,21 @@ class RMSNorm : public Norm {
     eps_ = r.number("eps");
     name_ = r.string("weight");
     offset_ = r.number_or("weight_offset", 0.0, false);
+    one_gain_ = r.boolean_or("one_gain", false);
   }
-  std::vector<TensorNeed> tensor_needs() const override { return {{name_, {size_}, TensorRole::Vector, false}}; }
+  std::vector<TensorNeed> tensor_needs() const override {
+    return {{name_, one_gain_ ? std::vector<int64_t>{} : std::vector<int64_t>{size_}, TensorRole::Vector, false}};
+  }
   void load(const Loader &l) override {
     weight_ = l.fetch(tensor_needs()[0]);
+    if (one_gain_) {                        // one copy per channel, as the norm kernels read it
+      float gain = 0.f;
+      LLM_CUDA(cudaMemcpy(&gain, weight_.buf.get(), sizeof(float), cudaMemcpyDeviceToHost));
+      const std::vector<float> row((size_t)size_, gain);
+      weight_.cols = size_;
+      weight_.buf.allocate(row.size() * sizeof(float));
+      LLM_CUDA(cudaMemcpy(weight_.buf.get(), row.data(), row.size() * sizeof(float), cudaMemcpyHostToDevice));
+    }
     // a weight stored around nought and applied as (offset + w): added once, in 32-bit, to the 32-bit copy
     if (offset_ != 0.0) kernels::add_scalar(weight_.buf.as<float>(), size_, (float)offset_, nullptr);
   }
@@ -61,6 +73,7 @@ class RMSNorm : public Norm {
  private:
   int64_t size_;
   double eps_, offset_ = 0.0;
+  bool one_gain_ = false;
   std::string name_;
   Weight weight_;
 };
@@ -1086,12 +1099,16 @@ void register_part_raw(const std::string &category, const std::string &kind, Par
 void register_feed_forward_parts();   // parts/feed_forward.cc
 void register_recurrent_parts();      // parts/recurrent.cc
 void register_latent_parts();         // parts/latent.cc
+void register_state_parts();          // parts/state_mixers.cc
+void register_sigmoid_parts();        // parts/sigmoid_attention.cc
 
 void register_builtin_parts() {
   register_part_raw("block", "parallel", factory_of<ParallelBlock>());
   register_feed_forward_parts();
   register_recurrent_parts();
   register_latent_parts();
+  register_state_parts();
+  register_sigmoid_parts();
   register_part_raw("norm", "rmsnorm", factory_of<RMSNorm>());
   register_part_raw("norm", "layernorm", factory_of<LayerNorm>());
   register_part_raw("position", "rope", factory_of<RotaryEmbedding>());

@@ -20,6 +20,11 @@ Json ModelSpec::to_json() const {
     o.set("layer", e.layer);
     o.set("cache_from", e.cache_from < 0 ? Json() : Json(e.cache_from));
     o.set("input_mix", e.input_mix.empty() ? Json() : Json(e.input_mix));
+    if (e.add_tokens) o.set("add_tokens", true);
+    if (!e.add_vector.empty()) {
+      o.set("add_vector", e.add_vector);
+      o.set("add_row", e.add_row);
+    }
     sch.push(o);
   }
   j.set("schedule", sch);
@@ -64,6 +69,9 @@ ModelSpec ModelSpec::from_json(const Json &j) {
         se.layer = (int)er.integer("layer", 0);
         se.cache_from = (int)er.integer_or("cache_from", -1, 0);
         se.input_mix = er.string_or("input_mix", "");
+        se.add_tokens = er.boolean_or("add_tokens", false);
+        se.add_vector = er.string_or("add_vector", "");
+        se.add_row = (int)er.integer_or("add_row", 0, 0);
       } else {
         r.fail("a schedule entry is a layer number or {layer, cache_from}");
       }

@@ -9,9 +9,11 @@
 // builds its one architecture in code (src/libllm/llama.cc:111-141, 231-249, 273-292); the keys
 // here are the arguments of those build functions.
 //
-//   norm "rmsnorm":        size, eps, weight (tensor name)
+//   norm "rmsnorm":        size, eps, weight (tensor name); one_gain: the weight is a single number for all channels
 //   norm "layernorm":      size, eps, weight, bias (tensor names; bias optional)
 //   mixer "general_delta": hidden, n_heads, head_dim, eps, decay_rank, decay_scale, key_eps, tensor names (parts/recurrent.cc)
+//   mixers "gated_delta", "time_mixing", "matrix_memory": a matrix of state per head (parts/state_mixers.cc)
+//   mixer "sigmoid_attention": attention without a softmax; mixer "sum": mixers side by side (parts/sigmoid_attention.cc)
 //   position "rope":       head_dim, rotary_dim, theta, scaling (null or the llama3 parameters)
 //   mixer "attention":     hidden, n_heads, n_kv_heads, head_dim, v_head_dim (default head_dim),
 //                          position (a position description or null), window (null: all keys),
@@ -36,11 +38,16 @@ namespace llm {
 // names an earlier entry whose cache this run reads instead of keeping one: it appends nothing.
 // `input_mix` names a matrix [hidden, 2 * hidden]: right before this run the residual stream x
 // becomes W [x; x0], x0 being the token rows as they entered the first layer (a model that runs some
-// of its layers several times feeds the tokens to every pass this way).
+// of its layers several times feeds the tokens to every pass this way).  `add_tokens`: right before this run the token
+// rows x0 are added to the stream; `add_vector`: so is row `add_row` of the table [rows, hidden] of that name (as many
+// rows as the entries that name it ask for).
 struct ScheduleEntry {
   int layer = 0;
   int cache_from = -1;
   std::string input_mix;
+  bool add_tokens = false;
+  std::string add_vector;
+  int add_row = 0;
 };
 
 struct ModelSpec {
