@@ -673,6 +673,102 @@ def run_compare_tazizen(args):
     return 0
 
 
+def rarelorn_config(hidden, runs, heads, kv, dim, ff, vocab, window=1024, experts=32, top=4, taps=4):
+    """A Rarelorn model of `runs` layer runs: [parallel, mlstm, delta, delta] as often as the runs ask for (a loop over the
+    four layers), every layer with `experts` experts of ff / 4 of which `top` are chosen in the better half of four groups (a
+    token uses as many feed-forward values as a dense one of ff).  Recurrent heads: hidden / dim of `dim` channels each."""
+    mlp = dict(kind="moe", expert=dict(ff=ff // 4), router=dict(experts=experts, top=top, scale=2.0, groups=dict(count=4, keep=2)))
+    left = dict(heads=heads, kv_heads=kv, dim=dim, vdim=dim, conv=taps, scale=dim ** -0.5, softcap=20.0, rot=dict(dims=dim // 2, base=5e4),
+                mask=dict(size=window))
+    n = hidden // dim
+    layers = [dict(type="parallel", mixer=dict(left=left, left_scale=0.9, right=dict(heads=n, dim=dim), right_scale=1.1)),
+              dict(type="mlstm", mixer=dict(heads=n, dim=dim, vdim=dim, gate_cap=15.0))]
+    layers += [dict(type="delta", mixer=dict(heads=n, kv_heads=n, dim=dim, vdim=dim, conv=taps))] * 2
+    return dict(architecture="Rarelorn", vocab=vocab, width=hidden, norm=dict(eps=1e-5), layers=[dict(L, mlp=mlp) for L in layers],
+                loop=dict(start=0, stop=4, times=max(1, runs // 4)))
+
+
+def rarelorn_numbers(c, batch, rank=16):
+    """(bytes a decode step of `batch` sequences reads apart from cache and state, cache bytes of a sequence as a function of
+    its length, bytes of state a step reads and writes per sequence, prefill flops of T tokens with one wanted row)."""
+    H, V = c["width"], c["vocab"]
+    loop = c["loop"]
+    runs = list(range(loop["start"])) + list(range(loop["start"], loop["stop"])) * loop["times"] + list(range(loop["stop"], len(c["layers"])))
+    used = touched = state = rec = 0
+    att = []                                          # (window, cache bytes a key, flops a key)
+    for i in runs:
+        m, kind = c["layers"][i]["mixer"], c["layers"][i]["type"]
+        if kind == "parallel":
+            l, r = m["left"], m["right"]
+            W = r["heads"] * r["dim"]
+            C = l["heads"] * l["dim"] + l["kv_heads"] * (l["dim"] + l["vdim"])
+            mats = H * C + l["heads"] * l["vdim"] * H + 5 * H * W + rank * (H + 2 * W)
+            att.append((l["mask"]["size"], 2 * l["kv_heads"] * (l["dim"] + l["vdim"]), 2 * l["heads"] * (l["dim"] + l["vdim"])))
+            state += 2 * 4 * (r["heads"] * r["dim"] ** 2 + (l["conv"] - 1) * C)
+            rec += 6 * r["heads"] * r["dim"] ** 2
+        else:
+            G = m.get("kv_heads", m["heads"])
+            W = m["heads"] * m["vdim"]
+            mats = H * (2 * G * m["dim"] + 3 * W + 2 * m["heads"])
+            state += 2 * 4 * m["heads"] * m["dim"] * m["vdim"]
+            if kind == "delta":
+                state += 2 * 4 * (m["conv"] - 1) * (2 * G * m["dim"] + W)
+            rec += (8 if kind == "delta" else 6) * m["heads"] * m["dim"] * m["vdim"]
+        f = c["layers"][i]["mlp"]
+        r, one = f["router"], 3 * H * f["expert"]["ff"]
+        used += mats + r["experts"] * H + r["top"] * one
+        touched += mats + r["experts"] * H + min(r["experts"], batch * r["top"]) * one
+
+    def cache_bytes(n):
+        return sum(b * min(n, w) for w, b, _ in att)
+
+    def prefill_flops(T):
+        return 2 * T * used + T * rec + sum(fl * sum(min(p + 1, w) for p in range(T)) for w, _, fl in att) + 2 * V * H
+    return 2 * (touched + V * H), cache_bytes, state, prefill_flops
+
+
+def run_compare_rarelorn(args):
+    """Prefill and decode of Rarelorn beside Sesuzen (the other design with a recurrent state, windowed attention and routed
+    experts), both with random weights, at equal hidden size, number of layer runs, heads, head size, feed-forward values
+    used per token and vocabulary: one JSON line per size and model."""
+    import torch
+    from libllm_b200 import Model
+    pk = peaks()
+    for name in [n for n in ("2k", "4k") if not args.sizes or n in args.sizes.split(",")]:
+        hidden, runs, heads, kv, dim, ff, vocab, window, keep, _ = SESUZEN_SIZES[name]
+        for label in ("sesuzen", "rarelorn"):
+            if args.model and args.model != label:
+                continue
+            if label == "sesuzen":
+                cfg = sesuzen_config(hidden, runs, heads, kv, dim, ff, vocab, window, keep)
+                wbytes, kv_tok, state, flops_fn = sesuzen_numbers(cfg, args.batch)
+                cache_fn = lambda n: kv_tok * min(n, window + keep)
+            else:
+                cfg = rarelorn_config(hidden, runs, heads, kv, dim, ff, vocab, window)
+                wbytes, cache_fn, state, flops_fn = rarelorn_numbers(cfg, args.batch)
+            flops = flops_fn(PROMPT)
+            model = Model.from_random(cfg, seed=0, dtype="bfloat16", max_tokens=args.batch * CONTEXT, max_seq_len=CONTEXT)
+            sampler = ClockSampler()
+            sampler.start()
+            pre = prefill_rate(model, vocab, lambda T: flops, pk["bf16_tflops"])
+            rate, ms, ctx_len, launches = decode_rate(model, args.batch, args.steps, args.warmup, vocab)
+            clocks = sampler.stop()
+            step_bytes = wbytes + args.batch * (cache_fn(ctx_len) + state)
+            print(json.dumps({"compare": name, "model": label, "batch": args.batch, "prompt": PROMPT,
+                              "config": {"hidden": hidden, "runs": runs, "heads": heads, "kv_heads": kv, "head_dim": dim, "ff": ff,
+                                         "vocab": vocab, "window": window},
+                              "prefill": {"ms": round(pre["ms"], 3), "tok_s": round(pre["value"], 1), "tflop": round(flops / 1e12, 3),
+                                          "frac_of_gemm_peak": round(pre["frac"], 4)},
+                              "decode": {"tok_s": round(rate, 1), "ms_per_step": round(ms, 4), "launches_per_step": launches,
+                                         "step_gb": round(step_bytes / 1e9, 3),
+                                         "hbm_frac": round(step_bytes / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)},
+                              "clocks": clocks, "peaks": pk["source"]}), flush=True)
+            model.engine.close()
+            del model
+            torch.cuda.empty_cache()
+    return 0
+
+
 def run_compare(args):
     """Prefill and decode of Sinezen beside Llama, both with random weights, at equal hidden size, layer
     runs, heads, head size, feed-forward width (with experts: equal matrix values used per token) and
@@ -787,10 +883,10 @@ def main():
                     help="1b: the benchmark line (default); 3b, 8b: the larger workloads, a line of their own")
     ap.add_argument("--only", choices=["decode", "prefill"], default=None,
                     help="run one part only and print a short line (for profiling; not a bench record)")
-    ap.add_argument("--compare", choices=["sinezen", "sesuzen", "sobezen", "tazizen"], default=None,
-                    help="Sinezen, Sesuzen, Sobezen or Tazizen beside Llama at equal sizes: prefill and decode, a line per size and model (not a bench record)")
-    ap.add_argument("--model", choices=["llama", "sesuzen", "sobezen", "tazizen"], default=None,
-                    help="with --compare sesuzen, sobezen or tazizen: one of the two models only")
+    ap.add_argument("--compare", choices=["sinezen", "sesuzen", "sobezen", "tazizen", "rarelorn"], default=None,
+                    help="Sinezen, Sesuzen, Sobezen or Tazizen beside Llama (Rarelorn beside Sesuzen) at equal sizes: prefill and decode, a line per size and model (not a bench record)")
+    ap.add_argument("--model", choices=["llama", "sesuzen", "sobezen", "tazizen", "rarelorn"], default=None,
+                    help="with --compare sesuzen, sobezen, tazizen or rarelorn: one of the two models only")
     ap.add_argument("--sizes", default=None, help="with --compare: which of the sizes (2k, 4k, 2k-routed), with commas")
     ap.add_argument("--prompt-len", type=int, default=None,
                     help="with --only: prompts of this many tokens instead of 2048 (the context grows to fit)")
@@ -814,6 +910,8 @@ def main():
         return run_compare_sobezen(args)
     if args.compare == "tazizen":
         return run_compare_tazizen(args)
+    if args.compare == "rarelorn":
+        return run_compare_rarelorn(args)
     if args.compare:
         return run_compare(args)
     if args.workload != "1b":

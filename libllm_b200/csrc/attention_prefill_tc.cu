@@ -369,7 +369,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       __syncwarp();
       if (lane == 0) mbar_arrive(bar_pfull + 8 * (j & 1));
     }
-    if (ok) ok = __all_sync(0xffffffffu, mbar_wait(bar_ofull, (n_tiles - 1) & 1, abort_flag, status, 20));
+    // the last two products one after the other: a parity alone does not tell the last from the last but two
+    if (ok && n_tiles > 1) ok = mbar_wait(bar_ofull, (n_tiles - 2) & 1, abort_flag, status, 20);
+    if (ok) ok = mbar_wait(bar_ofull, (n_tiles - 1) & 1, abort_flag, status, 20);
+    ok = __all_sync(0xffffffffu, ok);
     // The row's sum is the two threads' sums, first half first.  Every row warp comes here, whatever
     // happened above.
     asm volatile("bar.sync 5, 256;" ::: "memory");          // the last tile's maxima have been read

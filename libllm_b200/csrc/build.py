@@ -49,8 +49,9 @@ FAMILIES: Dict[str, dict] = {
     "gemm_plain": dict(sources=["gemm_plain.cu"], headers=["common.cuh"]),
     "rope": dict(sources=["rope.cu"], headers=["common.cuh"]),
     "recurrent": dict(sources=["recurrent.cu"], headers=["common.cuh"]),
-    "state_scan": dict(sources=["state_scan.cu"], headers=["common.cuh"]),
+    "state_scan": dict(sources=["state_scan.cu"], headers=["common.cuh", "tc_common.cuh"]),
     "attention_generic": dict(sources=["attention_generic.cu"], headers=["common.cuh"]),
+    "attention_sigmoid": dict(sources=["attention_sigmoid.cu"], headers=["common.cuh", "mma_tiles.cuh", "tc_common.cuh"]),
     "latent": dict(sources=["latent.cu"], headers=["common.cuh"]),
     "latent_tc": dict(sources=["latent_tc.cu"], headers=["common.cuh", "mma_tiles.cuh"]),
     "sampling": dict(sources=["sampling.cu"], headers=["common.cuh"]),

@@ -522,6 +522,38 @@ void attention_generic_sigmoid(const Act &q, const Act &out, const void *kc, con
            tok_seq, tok_pos, page_table, pt_stride, (int)q.rows, n_heads, n_kv, d, dv, page_size, window, scale, temp, bias, cap, out_scale,
            s);
 }
+LLM_KERNEL("attention_sigmoid", llm_sigmoid_prefill, const void *, long long, long long, void *, long long, const void *, const void *,
+           long long, const int *, const int *, const int *, int, int, int, int, int, int, int, int, int, float, const float *, const float *,
+           float, float, int *, cudaStream_t)
+LLM_KERNEL("attention_sigmoid", llm_sigmoid_decode, const void *, long long, void *, long long, const void *, const void *, const int *,
+           const int *, int, int, int, int, int, int, int, int, float, const float *, const float *, float, float, int, float *, int *,
+           cudaStream_t)
+bool sigmoid_prefill_supported(int d, int dv, int page_size) {
+  static auto f = resolve<int (*)(int, int, int)>("attention_sigmoid", "llm_sigmoid_prefill_supports");
+  return f(d, dv, page_size) != 0;
+}
+void sigmoid_prefill(const Act &q, const Act &out, const void *kc, const void *vc, long long n_pages, const int *seq_start,
+                     const int *seq_past, const int *page_table, int pt_stride, int n_seqs, int max_q_len, int n_heads, int n_kv, int d,
+                     int dv, int page_size, int window, float scale, const float *temp, const float *bias, float cap, float out_scale,
+                     int *status, cudaStream_t s) {
+  LLM_CALL("attention_sigmoid", llm_sigmoid_prefill, q.data, (long long)q.ld, (long long)q.rows, out.data, (long long)out.ld, kc, vc, n_pages,
+           seq_start, seq_past, page_table, pt_stride, n_seqs, max_q_len, n_heads, n_kv, d, dv, page_size, window, scale, temp, bias, cap,
+           out_scale, status, s);
+}
+bool sigmoid_decode_supported(int d, int dv, int group, int page_size) {
+  static auto f = resolve<int (*)(int, int, int, int)>("attention_sigmoid", "llm_sigmoid_decode_supports");
+  return f(d, dv, group, page_size) != 0;
+}
+int sigmoid_decode_ctas_per_sm(int d, int dv) {
+  static auto f = resolve<int (*)(int, int)>("attention_sigmoid", "llm_sigmoid_decode_ctas_per_sm");
+  return f(d, dv);
+}
+void sigmoid_decode(const Act &q, const Act &out, const void *kc, const void *vc, const int *tok_pos, const int *page_table, int pt_stride,
+                    int n_heads, int n_kv, int d, int dv, int page_size, int window, float scale, const float *temp, const float *bias,
+                    float cap, float out_scale, int n_splits, float *ws, int *counters, cudaStream_t s) {
+  LLM_CALL("attention_sigmoid", llm_sigmoid_decode, q.data, (long long)q.ld, out.data, (long long)out.ld, kc, vc, tok_pos, page_table, pt_stride,
+           (int)q.rows, n_heads, n_kv, d, dv, page_size, window, scale, temp, bias, cap, out_scale, n_splits, ws, counters, s);
+}
 LLM_KERNEL("rope", llm_conv_rope_place, int, const float *, long long, const float *, const float *, int, float *, void *, long long, int,
            int, int, int, int, int, const float *, int, int, const int *, const int *, const int *, const int *, const int *, const int *,
            int, void *, void *, int, int, int, cudaStream_t)
@@ -666,14 +698,15 @@ void head_norm_gate(const Act &x, const float *weight, const float *gate, long l
 }
 
 // ---------------------------------------------------------------- linear recurrences over a matrix of state per head
-LLM_KERNEL("state_scan", llm_state_scan, int, const float *, const float *, const float *, long long, float *, float *, long long, float *,
-           const int *, const int *, int, int, int, int, int, int, cudaStream_t)
-LLM_KERNEL("state_scan", llm_delta_pack, const float *, long long, const float *, long long, int, int, const float *, const float *, float,
-           float, float *, float *, int, int, int, int, cudaStream_t)
-LLM_KERNEL("state_scan", llm_bonus_pack, const float *, long long, const float *, long long, const float *, long long, int, const float *,
-           const float *, const float *, float *, float *, int, int, int, cudaStream_t)
-LLM_KERNEL("state_scan", llm_memory_pack, const float *, long long, int, int, int, int, const float *, const float *, float, float, float *,
-           float *, float *, const int *, const int *, int, int, int, int, cudaStream_t)
+LLM_KERNEL("state_scan", llm_state_scan, int, const float *, const float *, const float *, float *, float *, long long, float *, const int *,
+           const int *, int, int, int, int, int, int, int *, cudaStream_t)
+LLM_KERNEL("state_scan", llm_delta_pack, const float *, long long, int, int, const float *, int, float *, const float *, const float *, float,
+           float, float *, float *, float *, const int *, const int *, const int *, const int *, const int *, int, int, int, int, int, int,
+           int, cudaStream_t)
+LLM_KERNEL("state_scan", llm_bonus_pack, const float *, long long, const float *, long long, const float *, long long, const float *, long long,
+           int, const float *, const float *, const float *, float *, float *, float *, int, int, int, int, cudaStream_t)
+LLM_KERNEL("state_scan", llm_memory_pack, const float *, long long, int, int, int, int, int, const float *, const float *, float, float, float *,
+           float *, float *, float *, const int *, const int *, int, int, int, int, int, cudaStream_t)
 LLM_KERNEL("state_scan", llm_head_finish, const float *, long long, const float *, const float *, const float *, int, const float *,
            long long, int, float, float, int, int, int, void *, int, long long, cudaStream_t)
 LLM_KERNEL("state_scan", llm_token_shift, int, const void *, long long, const float *, int, void *, long long, void *, const int *,
@@ -686,30 +719,41 @@ LLM_KERNEL("state_scan", llm_bonus_step, const float *, long long, const float *
            void *, int, long long, const int *, int, int, int, int, cudaStream_t)
 LLM_KERNEL("state_scan", llm_memory_step, const float *, long long, int, int, int, int, int, int, const float *, const float *, float, float,
            float *, float *, const float *, int, float, float, void *, int, long long, const int *, int, int, int, int, cudaStream_t)
-void state_scan(ScanRule rule, const float *rec, const float *scal, const float *v, long long ldv, float *state, const Act &out, float *den,
-                const int *seq_start, const int *seq_slot, int n_seqs, int n_heads, int n_kv, int d, int dv, cudaStream_t s) {
+int scan_padded(int d) {
+  static auto f = resolve<int (*)(int)>("state_scan", "llm_scan_padded");
+  return f(d);
+}
+int scan_columns(int d) {
+  static auto f = resolve<int (*)(int)>("state_scan", "llm_scan_columns");
+  return f(d);
+}
+void state_scan(ScanRule rule, const ScanPack &pack, float *state, const Act &out, float *den, const int *seq_start, const int *seq_slot,
+                int n_seqs, int n_heads, int n_kv, int d, int dv, int *status, cudaStream_t s) {
   if (out.dtype != DType::F32) LLM_THROW(InvalidArg, "state_scan: results are 32-bit");
-  LLM_CALL("state_scan", llm_state_scan, (int)rule, rec, scal, v, ldv, state, (float *)out.data, (long long)out.ld, den, seq_start, seq_slot,
-           (int)out.rows, n_seqs, n_heads, n_kv, d, dv, s);
+  LLM_CALL("state_scan", llm_state_scan, (int)rule, pack.rec, pack.scal, pack.vals, state, (float *)out.data, (long long)out.ld, den, seq_start,
+           seq_slot, (int)out.rows, n_seqs, n_heads, n_kv, d, dv, status, s);
 }
-void delta_pack(const Act &cv, const Act &proj, int off_b, int off_a, const float *dt_bias, const float *a_log, float key_eps, float q_scale,
-                float *rec, float *scal, int n_heads, int n_kv, int d, cudaStream_t s) {
-  if (cv.dtype != DType::F32 || proj.dtype != DType::F32) LLM_THROW(InvalidArg, "delta_pack: projections are 32-bit");
-  LLM_CALL("state_scan", llm_delta_pack, (const float *)cv.data, (long long)cv.ld, (const float *)proj.data, (long long)proj.ld, off_b, off_a,
-           dt_bias, a_log, key_eps, q_scale, rec, scal, (int)proj.rows, n_heads, n_kv, d, s);
+void delta_pack(const Act &proj, int off_b, int off_a, const float *conv, int taps, float *conv_state, const float *dt_bias, const float *a_log,
+                float key_eps, float q_scale, const ScanPack &pack, const int *tok_seq, const int *tok_pos, const int *seq_start,
+                const int *seq_past, const int *seq_slot, int n_seqs, int n_heads, int n_kv, int d, int dv, bool single_tokens, cudaStream_t s) {
+  if (proj.dtype != DType::F32) LLM_THROW(InvalidArg, "delta_pack: projections are 32-bit");
+  LLM_CALL("state_scan", llm_delta_pack, (const float *)proj.data, (long long)proj.ld, off_b, off_a, conv, taps, conv_state, dt_bias, a_log,
+           key_eps, q_scale, pack.rec, pack.scal, pack.vals, tok_seq, tok_pos, seq_start, seq_past, seq_slot, (int)proj.rows, n_seqs, n_heads,
+           n_kv, d, dv, single_tokens ? 1 : 0, s);
 }
-void bonus_pack(const Act &r, const Act &k, const Act &x1, int rank, const float *w2, const float *w0, const float *u, float *rec,
-                float *scal, int n_heads, int d, cudaStream_t s) {
+void bonus_pack(const Act &r, const Act &k, const Act &v, const Act &x1, int rank, const float *w2, const float *w0, const float *u,
+                const ScanPack &pack, int n_heads, int d, int dv, cudaStream_t s) {
   if (r.dtype != DType::F32 || k.dtype != DType::F32 || x1.dtype != DType::F32) LLM_THROW(InvalidArg, "bonus_pack: projections are 32-bit");
-  LLM_CALL("state_scan", llm_bonus_pack, (const float *)r.data, (long long)r.ld, (const float *)k.data, (long long)k.ld,
-           (const float *)x1.data, (long long)x1.ld, rank, w2, w0, u, rec, scal, (int)r.rows, n_heads, d, s);
+  LLM_CALL("state_scan", llm_bonus_pack, (const float *)r.data, (long long)r.ld, (const float *)k.data, (long long)k.ld, (const float *)v.data,
+           (long long)v.ld, (const float *)x1.data, (long long)x1.ld, rank, w2, w0, u, pack.rec, pack.scal, pack.vals, (int)r.rows, n_heads, d,
+           dv, s);
 }
-void memory_pack(const Act &proj, int off_q, int off_k, int off_i, int off_f, const float *bias_i, const float *bias_f, float cap,
-                 float q_scale, float *state_m, float *rec, float *scal, const int *seq_start, const int *seq_slot, int n_seqs, int n_heads,
-                 int d, cudaStream_t s) {
+void memory_pack(const Act &proj, int off_q, int off_k, int off_v, int off_i, int off_f, const float *bias_i, const float *bias_f, float cap,
+                 float q_scale, float *state_m, const ScanPack &pack, const int *seq_start, const int *seq_slot, int n_seqs, int n_heads,
+                 int d, int dv, cudaStream_t s) {
   if (proj.dtype != DType::F32) LLM_THROW(InvalidArg, "memory_pack: projections are 32-bit");
-  LLM_CALL("state_scan", llm_memory_pack, (const float *)proj.data, (long long)proj.ld, off_q, off_k, off_i, off_f, bias_i, bias_f, cap,
-           q_scale, state_m, rec, scal, seq_start, seq_slot, (int)proj.rows, n_seqs, n_heads, d, s);
+  LLM_CALL("state_scan", llm_memory_pack, (const float *)proj.data, (long long)proj.ld, off_q, off_k, off_v, off_i, off_f, bias_i, bias_f, cap,
+           q_scale, state_m, pack.rec, pack.scal, pack.vals, seq_start, seq_slot, (int)proj.rows, n_seqs, n_heads, d, dv, s);
 }
 void head_finish(const Act &x, const float *den, const float *scal, const float *weight, bool shared_weight, const float *gate,
                  long long gate_stride, GateAct act, float eps, float out_scale, int n_heads, int dv, const Act &out, cudaStream_t s) {

@@ -141,6 +141,18 @@ void attention_generic(const Act &q, const Act &out, const void *kc, const void 
 void attention_generic_sigmoid(const Act &q, const Act &out, const void *kc, const void *vc, const int *tok_seq, const int *tok_pos,
                                const int *page_table, int pt_stride, int n_heads, int n_kv, int d, int dv, int page_size, int window,
                                float scale, const float *temp, const float *bias, float cap, float out_scale, cudaStream_t s);
+// The same for bfloat16 (csrc/attention_sigmoid.cu): prompt steps on tcgen05, and single tokens (ws: sequences * heads * dv *
+// n_splits floats, counters: sequences * kv_heads zeros, both for n_splits > 1).
+bool sigmoid_prefill_supported(int d, int dv, int page_size);
+void sigmoid_prefill(const Act &q, const Act &out, const void *kc, const void *vc, long long n_pages, const int *seq_start,
+                     const int *seq_past, const int *page_table, int pt_stride, int n_seqs, int max_q_len, int n_heads, int n_kv, int d,
+                     int dv, int page_size, int window, float scale, const float *temp, const float *bias, float cap, float out_scale,
+                     int *status, cudaStream_t s);
+bool sigmoid_decode_supported(int d, int dv, int group, int page_size);
+int sigmoid_decode_ctas_per_sm(int d, int dv);
+void sigmoid_decode(const Act &q, const Act &out, const void *kc, const void *vc, const int *tok_pos, const int *page_table, int pt_stride,
+                    int n_heads, int n_kv, int d, int dv, int page_size, int window, float scale, const float *temp, const float *bias,
+                    float cap, float out_scale, int n_splits, float *ws, int *counters, cudaStream_t s);
 // ---- latent attention (csrc/latent.cu): attention over one cached row [c | k_r] per position that every head reads
 // proj rows (32-bit) hold the query latent at off_q and, with off_kv >= 0, the key/value latent and the shared key part;
 // cq_out = rms(query latent) * q_weight; the token's cache row = [rms(first kv_rank) * kv_weight | rotated last rot].
@@ -251,16 +263,24 @@ void head_norm_gate(const Act &x, const float *weight, const float *gate, long l
 // ---- linear recurrences over a matrix of state per head (csrc/state_scan.cu)
 enum ScanRule { ScanDelta = 0, ScanBonus = 1, ScanMemory = 2 };
 enum GateAct { GateSigmoid = 0, GateSilu = 1 };
-// rec [tokens, kv_heads, 2 (bonus: 3), d padded to 4], scal [tokens, heads, 4], v rows; state [slots, heads, dv (memory: + 1), d]
-void state_scan(ScanRule rule, const float *rec, const float *scal, const float *v, long long ldv, float *state, const Act &out, float *den,
-                const int *seq_start, const int *seq_slot, int n_seqs, int n_heads, int n_kv, int d, int dv, cudaStream_t s);
-void delta_pack(const Act &cv, const Act &proj, int off_b, int off_a, const float *dt_bias, const float *a_log, float key_eps, float q_scale,
-                float *rec, float *scal, int n_heads, int n_kv, int d, cudaStream_t s);
-void bonus_pack(const Act &r, const Act &k, const Act &x1, int rank, const float *w2, const float *w0, const float *u, float *rec,
-                float *scal, int n_heads, int d, cudaStream_t s);
-void memory_pack(const Act &proj, int off_q, int off_k, int off_i, int off_f, const float *bias_i, const float *bias_f, float cap,
-                 float q_scale, float *state_m, float *rec, float *scal, const int *seq_start, const int *seq_slot, int n_seqs, int n_heads,
-                 int d, cudaStream_t s);
+// What the tokens bring, packed: rec [kv_heads, tokens, 2 (bonus: 3), scan_padded(d)], scal [heads, tokens, 4], vals [heads,
+// slices, tokens, scan_columns(d)] for dv (memory: + 1) columns; state [slots, heads, dv (memory: + 1), d]
+int scan_padded(int d);
+int scan_columns(int d);
+struct ScanPack {
+  float *rec, *scal, *vals;
+};
+void state_scan(ScanRule rule, const ScanPack &pack, float *state, const Act &out, float *den, const int *seq_start, const int *seq_slot,
+                int n_seqs, int n_heads, int n_kv, int d, int dv, int *status, cudaStream_t s);
+// rows of proj begin with [q | k | v]: convolution over time and silu, unit vectors, gates; state as causal_conv's, 32-bit
+void delta_pack(const Act &proj, int off_b, int off_a, const float *conv, int taps, float *conv_state, const float *dt_bias, const float *a_log,
+                float key_eps, float q_scale, const ScanPack &pack, const int *tok_seq, const int *tok_pos, const int *seq_start,
+                const int *seq_past, const int *seq_slot, int n_seqs, int n_heads, int n_kv, int d, int dv, bool single_tokens, cudaStream_t s);
+void bonus_pack(const Act &r, const Act &k, const Act &v, const Act &x1, int rank, const float *w2, const float *w0, const float *u,
+                const ScanPack &pack, int n_heads, int d, int dv, cudaStream_t s);
+void memory_pack(const Act &proj, int off_q, int off_k, int off_v, int off_i, int off_f, const float *bias_i, const float *bias_f, float cap,
+                 float q_scale, float *state_m, const ScanPack &pack, const int *seq_start, const int *seq_slot, int n_seqs, int n_heads,
+                 int d, int dv, cudaStream_t s);
 // norm per head (of x / (max(|den|, floor) + 1e-6) where den is given), weight, gate, out_scale
 void head_finish(const Act &x, const float *den, const float *scal, const float *weight, bool shared_weight, const float *gate,
                  long long gate_stride, GateAct act, float eps, float out_scale, int n_heads, int dv, const Act &out, cudaStream_t s);

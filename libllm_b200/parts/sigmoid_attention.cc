@@ -112,7 +112,7 @@ class SigmoidAttention : public Mixer {
   std::vector<std::string> kernel_families() const override {
     std::vector<std::string> fams = product_families(env_.dtype);
     fams.push_back("rope");
-    fams.push_back("attention_generic");
+    fams.push_back(tiled(env_.page_size) ? "attention_sigmoid" : "attention_generic");
     return fams;
   }
   bool wants_cache() const override { return true; }
@@ -146,9 +146,7 @@ class SigmoidAttention : public Mixer {
                              rot_dim, ctx.tok_seq, ctx.tok_pos, ctx.seq_start, ctx.seq_past, ctx.seq_slot, ctx.n_seqs, cache->page_table,
                              cache->table_width, cache->k, cache->v, cache->page_size, cache->writes, ctx.decode_only, ctx.stream);
     Act out = ctx.arena->act(ctx.dtype, ctx.n_tokens, (int64_t)n_heads_ * dv_);
-    kernels::attention_generic_sigmoid(q, out, cache->k, cache->v, ctx.tok_seq, ctx.tok_pos, cache->page_table, cache->table_width, n_heads_,
-                                       n_kv_, d_, dv_, cache->page_size, window_, scale_, temp_.buf.as<float>(), score_bias_.buf.as<float>(),
-                                       cap_, out_scale_, ctx.stream);
+    attend(ctx, q, out, *cache);
     if (o_bias_name_.empty()) return linear(ctx, out, w_o_, nullptr, DType::F32, true);
     // with a bias the product cannot add to the stream as it stores: the bias goes with the result
     float *const sink = ctx.residual_sink;
@@ -160,6 +158,31 @@ class SigmoidAttention : public Mixer {
   }
 
  private:
+  // bfloat16 heads that both tensor-core kernels take; all else is the general kernel's
+  bool tiled(int page_size) const {
+    return env_.dtype == DType::BF16 && fast_switches().prefill_attention_tc && page_size == 64 && d_ % 16 == 0 && d_ <= 128 && dv_ % 16 == 0 &&
+           dv_ <= 256 && n_heads_ / n_kv_ <= 16;
+  }
+  void attend(StepContext &ctx, const Act &q, const Act &out, LayerCache &cache) const {
+    const float *temp = temp_.buf.as<float>(), *bias = score_bias_.buf.as<float>();
+    if (!tiled(cache.page_size)) {
+      kernels::attention_generic_sigmoid(q, out, cache.k, cache.v, ctx.tok_seq, ctx.tok_pos, cache.page_table, cache.table_width, n_heads_,
+                                         n_kv_, d_, dv_, cache.page_size, window_, scale_, temp, bias, cap_, out_scale_, ctx.stream);
+    } else if (ctx.decode_only) {
+      // as many runs of pages as fill the GPU once, at the longest length the step's shape allows
+      const int longest = window_ > 0 ? std::min(ctx.max_kv_len, window_ + cache.page_size) : ctx.max_kv_len;
+      const int pages = std::max(1, (longest + cache.page_size - 1) / cache.page_size), pairs = std::max(1, ctx.n_seqs * n_kv_);
+      int n_splits = std::max(1, std::min(ctx.sm_count * kernels::sigmoid_decode_ctas_per_sm(d_, dv_) / pairs, pages));
+      if (pairs > ctx.n_zero_counters) n_splits = 1;
+      float *ws = n_splits > 1 ? ctx.arena->alloc_n<float>((size_t)ctx.n_seqs * n_heads_ * dv_ * n_splits) : nullptr;
+      kernels::sigmoid_decode(q, out, cache.k, cache.v, ctx.tok_pos, cache.page_table, cache.table_width, n_heads_, n_kv_, d_, dv_,
+                              cache.page_size, window_, scale_, temp, bias, cap_, out_scale_, n_splits, ws, ctx.zero_counters, ctx.stream);
+    } else {
+      kernels::sigmoid_prefill(q, out, cache.k, cache.v, cache.n_pages, ctx.seq_start, ctx.seq_past, cache.page_table, cache.table_width,
+                               ctx.n_seqs, ctx.max_q_len, n_heads_, n_kv_, d_, dv_, cache.page_size, window_, scale_, temp, bias, cap_,
+                               out_scale_, ctx.tc_status, ctx.stream);
+    }
+  }
   Weight per_head(const Loader &l, const std::string &name, float fallback) const {
     if (!name.empty()) return l.fetch(vector_need(name, n_heads_));
     Weight w;

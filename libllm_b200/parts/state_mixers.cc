@@ -52,8 +52,6 @@ void *state_of(StateView *state, const std::string &name) {
   return nullptr;
 }
 
-int64_t padded4(int64_t d) { return (d + 3) / 4 * 4; }
-
 class StateMixer : public Mixer {
  public:
   StateMixer(const Json &spec, const BuildEnv &env, const char *what) : Mixer(spec, env) {
@@ -79,6 +77,16 @@ class StateMixer : public Mixer {
   }
 
  protected:
+  // room for what a step's tokens bring to the scan: `vectors` per key head, `columns` of values per head
+  kernels::ScanPack pack_room(StepContext &ctx, int vectors, int columns) const {
+    const size_t T = (size_t)ctx.n_tokens;
+    const int per = kernels::scan_columns(d_), slices = (columns + per - 1) / per;
+    kernels::ScanPack p;
+    p.rec = ctx.arena->alloc_n<float>(T * (size_t)(n_kv_ * vectors * kernels::scan_padded(d_)));
+    p.scal = ctx.arena->alloc_n<float>(T * (size_t)(n_heads_ * 4));
+    p.vals = ctx.arena->alloc_n<float>(T * (size_t)(n_heads_ * slices * per));
+    return p;
+  }
   bool single_step(const StepContext &ctx, int rank) const {
     return ctx.decode_only && ctx.n_tokens == ctx.n_seqs && kernels::state_step_supported(d_, dv_, n_heads_ / n_kv_, rank);
   }
@@ -137,7 +145,6 @@ class GatedDelta : public StateMixer {
   }
   std::vector<std::string> kernel_families() const override {
     std::vector<std::string> fams = StateMixer::kernel_families();
-    fams.push_back("recurrent");
     fams.push_back("elementwise");
     return fams;
   }
@@ -160,19 +167,14 @@ class GatedDelta : public StateMixer {
                                 out_scale_, y, ctx.seq_slot, n_heads_, n_kv_, d_, dv_, ctx.stream);
       return linear(ctx, y, w_o_, nullptr, DType::F32, true);
     }
-    Act cv = ctx.arena->act(DType::F32, T, padded4(conv_width_));
-    Act conv_in = proj, conv_out = cv;
-    conv_in.cols = conv_out.cols = conv_width_;
-    kernels::causal_conv(conv_in, conv_out, conv_.buf.as<float>(), inputs, ctx.tok_seq, ctx.tok_pos, ctx.seq_start, ctx.seq_past,
-                         ctx.seq_slot, ctx.n_seqs, taps_, ctx.decode_only, ctx.stream, true);
-    float *rec = ctx.arena->alloc_n<float>((size_t)T * n_kv_ * 2 * padded4(d_));
-    float *scal = ctx.arena->alloc_n<float>((size_t)T * n_heads_ * 4);
-    kernels::delta_pack(cv, proj, off_b, off_a, dt_bias_.buf.as<float>(), a_log_.buf.as<float>(), key_eps_, q_scale_, rec, scal, n_heads_,
-                        n_kv_, d_, ctx.stream);
+    const kernels::ScanPack pack = pack_room(ctx, 2, dv_);
+    kernels::delta_pack(proj, off_b, off_a, conv_.buf.as<float>(), taps_, inputs, dt_bias_.buf.as<float>(), a_log_.buf.as<float>(), key_eps_,
+                        q_scale_, pack, ctx.tok_seq, ctx.tok_pos, ctx.seq_start, ctx.seq_past, ctx.seq_slot, ctx.n_seqs, n_heads_, n_kv_, d_,
+                        dv_, ctx.decode_only, ctx.stream);
     Act o = ctx.arena->act(DType::F32, T, v_width_);
-    kernels::state_scan(kernels::ScanDelta, rec, scal, (const float *)cv.data + 2 * q_width_, cv.ld, S, o, nullptr, ctx.seq_start,
-                        ctx.seq_slot, ctx.n_seqs, n_heads_, n_kv_, d_, dv_, ctx.stream);
-    kernels::head_finish(o, nullptr, scal, norm_.buf.as<float>(), true, (const float *)proj.data + off_g, proj.ld, kernels::GateSilu, eps_,
+    kernels::state_scan(kernels::ScanDelta, pack, S, o, nullptr, ctx.seq_start, ctx.seq_slot, ctx.n_seqs, n_heads_, n_kv_, d_, dv_,
+                        ctx.tc_status, ctx.stream);
+    kernels::head_finish(o, nullptr, pack.scal, norm_.buf.as<float>(), true, (const float *)proj.data + off_g, proj.ld, kernels::GateSilu, eps_,
                          out_scale_, n_heads_, dv_, y, ctx.stream);
     return linear(ctx, y, w_o_, nullptr, DType::F32, true);
   }
@@ -255,14 +257,13 @@ class TimeMixing : public StateMixer {
                           norm_.buf.as<float>(), kernels::GateSilu, eps_, out_scale_, y, ctx.seq_slot, n_heads_, d_, dv_, ctx.stream);
       return linear(ctx, y, w_o_, nullptr, DType::F32, true);
     }
-    float *rec = ctx.arena->alloc_n<float>((size_t)T * n_heads_ * 3 * padded4(d_));
-    float *scal = ctx.arena->alloc_n<float>((size_t)T * n_heads_ * 4);
-    kernels::bonus_pack(in[0], in[1], in[4], (int)rank_, w2_.buf.as<float>(), w0_.buf.as<float>(), u_.buf.as<float>(), rec, scal, n_heads_,
-                        d_, ctx.stream);
+    const kernels::ScanPack pack = pack_room(ctx, 3, dv_);
+    kernels::bonus_pack(in[0], in[1], in[2], in[4], (int)rank_, w2_.buf.as<float>(), w0_.buf.as<float>(), u_.buf.as<float>(), pack, n_heads_, d_,
+                        dv_, ctx.stream);
     Act o = ctx.arena->act(DType::F32, T, v_width_);
-    kernels::state_scan(kernels::ScanBonus, rec, scal, (const float *)in[2].data, in[2].ld, S, o, nullptr, ctx.seq_start, ctx.seq_slot,
-                        ctx.n_seqs, n_heads_, n_heads_, d_, dv_, ctx.stream);
-    kernels::head_finish(o, nullptr, scal, norm_.buf.as<float>(), false, (const float *)in[3].data, in[3].ld, kernels::GateSilu, eps_,
+    kernels::state_scan(kernels::ScanBonus, pack, S, o, nullptr, ctx.seq_start, ctx.seq_slot, ctx.n_seqs, n_heads_, n_heads_, d_, dv_,
+                        ctx.tc_status, ctx.stream);
+    kernels::head_finish(o, nullptr, pack.scal, norm_.buf.as<float>(), false, (const float *)in[3].data, in[3].ld, kernels::GateSilu, eps_,
                          out_scale_, n_heads_, dv_, y, ctx.stream);
     return linear(ctx, y, w_o_, nullptr, DType::F32, true);
   }
@@ -319,15 +320,14 @@ class MatrixMemory : public StateMixer {
                            norm_.buf.as<float>(), kernels::GateSigmoid, eps_, out_scale_, y, ctx.seq_slot, n_heads_, d_, dv_, ctx.stream);
       return linear(ctx, y, w_o_, nullptr, DType::F32, true);
     }
-    float *rec = ctx.arena->alloc_n<float>((size_t)T * n_heads_ * 2 * padded4(d_));
-    float *scal = ctx.arena->alloc_n<float>((size_t)T * n_heads_ * 4);
+    const kernels::ScanPack pack = pack_room(ctx, 2, dv_ + 1);
     float *den = ctx.arena->alloc_n<float>((size_t)T * n_heads_);
-    kernels::memory_pack(proj, 0, off_k, off_i, off_f, i_bias_.buf.as<float>(), f_bias_.buf.as<float>(), cap_, q_scale_, m, rec, scal,
-                         ctx.seq_start, ctx.seq_slot, ctx.n_seqs, n_heads_, d_, ctx.stream);
+    kernels::memory_pack(proj, 0, off_k, off_v, off_i, off_f, i_bias_.buf.as<float>(), f_bias_.buf.as<float>(), cap_, q_scale_, m, pack,
+                         ctx.seq_start, ctx.seq_slot, ctx.n_seqs, n_heads_, d_, dv_, ctx.stream);
     Act o = ctx.arena->act(DType::F32, T, v_width_);
-    kernels::state_scan(kernels::ScanMemory, rec, scal, (const float *)proj.data + off_v, proj.ld, S, o, den, ctx.seq_start, ctx.seq_slot,
-                        ctx.n_seqs, n_heads_, n_heads_, d_, dv_, ctx.stream);
-    kernels::head_finish(o, den, scal, norm_.buf.as<float>(), false, (const float *)proj.data + off_g, proj.ld, kernels::GateSigmoid, eps_,
+    kernels::state_scan(kernels::ScanMemory, pack, S, o, den, ctx.seq_start, ctx.seq_slot, ctx.n_seqs, n_heads_, n_heads_, d_, dv_,
+                        ctx.tc_status, ctx.stream);
+    kernels::head_finish(o, den, pack.scal, norm_.buf.as<float>(), false, (const float *)proj.data + off_g, proj.ld, kernels::GateSigmoid, eps_,
                          out_scale_, n_heads_, dv_, y, ctx.stream);
     return linear(ctx, y, w_o_, nullptr, DType::F32, true);
   }
