@@ -737,7 +737,7 @@ LLM_EXPORT int llm_rope_headnorm_place(int in_dtype, int dtype, const void *qkv,
 // of a run of rows (blockIdx.x < n_chunks), the first taps - 1 rows of every sequence, and its state, to a CTA of that
 // sequence, whose threads read the old state of their channels before they write the new one: nobody else reads it.
 // The order of operations is the same wherever a row is computed.
-constexpr int CP_THREADS = 128, CP_ROWS = 16, CP_MAX_TAPS = 8;
+constexpr int CP_THREADS = 128, CP_ROWS = 8, CP_MAX_TAPS = 8;
 
 template <int V>
 __device__ __forceinline__ void cp_load(const float *p, float (&x)[V]) {
@@ -801,8 +801,15 @@ conv_rope_place_kernel(const float *__restrict__ qkv, long long ld, const float 
     }
   }
   grid_dependency_wait();
-  if (unit >= n_units) return;
   const int keep = taps - 1;
+  // which rows of a run are its CTA's (a bit per row); the others belong to their sequence's own CTA
+  unsigned mine = 0;
+  if ((int)blockIdx.x < n_chunks) {
+    const int lane = threadIdx.x & 31, row = blockIdx.x * CP_ROWS + lane;
+    const bool in = lane < CP_ROWS && row < n_tokens;
+    mine = __ballot_sync(0xffffffffu, in && tok_pos[in ? row : 0] - seq_past[tok_seq[in ? row : 0]] >= keep);
+  }
+  if (unit >= n_units) return;
   float win[2][TAPS][V];                               // win[.][j]: u at the row's position - taps + 1 + j
   auto take = [&](int row, float (&x0)[V], float (&x1)[V]) {
     cp_load<V>(qkv + (size_t)row * ld + c0, x0);
@@ -810,7 +817,7 @@ conv_rope_place_kernel(const float *__restrict__ qkv, long long ld, const float 
 #pragma unroll
     for (int e = 0; e < V; ++e) {
       x0[e] += bs[0][e];
-      if (rotated) x1[e] += bs[1][e];
+      x1[e] = rotated ? x1[e] + bs[1][e] : 0.f;
     }
   };
   auto shift = [&](const float (&x0)[V], const float (&x1)[V]) {
@@ -869,20 +876,32 @@ conv_rope_place_kernel(const float *__restrict__ qkv, long long ld, const float 
   for (int e = 0; e < V; ++e) x0[e] = x1[e] = 0.f;
   if ((int)blockIdx.x < n_chunks) {
     const int r0 = blockIdx.x * CP_ROWS, r1 = min(n_tokens, r0 + CP_ROWS);
-    int filled = -1;                                   // the last row in the window; -1: none
-    for (int row = r0; row < r1; ++row) {
-      if (tok_pos[row] - seq_past[tok_seq[row]] < keep) {          // the sequence's own CTA computes it
-        filled = -1;
-        continue;
+    if (mine == (1u << CP_ROWS) - 1u) {                // all of them: four rows' loads on their way at once
+      for (int k = keep; k > 0; --k) {
+        take(r0 - k, x0, x1);
+        shift(x0, x1);
       }
-      if (filled != row - 1 || filled < 0)
+      for (int i0 = 0; i0 < CP_ROWS; i0 += 4) {
+        float y0[4][V], y1[4][V];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) take(r0 + i0 + i, y0[i], y1[i]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          shift(y0[i], y1[i]);
+          place(r0 + i0 + i);
+        }
+      }
+      return;
+    }
+    for (int row = r0; row < r1; ++row) {
+      if (!((mine >> (row - r0)) & 1u)) continue;
+      if (row == r0 || !((mine >> (row - r0 - 1)) & 1u))
         for (int k = keep; k > 0; --k) {
           take(row - k, x0, x1);
           shift(x0, x1);
         }
       take(row, x0, x1);
       shift(x0, x1);
-      filled = row;
       place(row);
     }
     return;

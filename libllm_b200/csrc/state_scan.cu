@@ -34,17 +34,22 @@ __device__ __forceinline__ float log_sigmoid32(float x) { return fminf(x, 0.f) -
 __host__ __device__ constexpr int scan_dmax(int d) { return d <= 16 ? 16 : d <= 32 ? 32 : d <= 64 ? 64 : d <= 128 ? 128 : 256; }
 
 // ---------------------------------------------------------------- the scan over a step's tokens
-// CTA (sequence, head, slice of columns): SC_THREADS threads of arithmetic, LANES neighbouring lanes to a column (lane `sub`
+// CTA (sequence, head, slice of columns): SC_THREADS threads of arithmetic, LANES neighbouring lanes to two columns (lane `sub`
 // owns rows 4 (sub + LANES i) .. + 3), and a warp one lane of which brings groups of SC_GROUP tokens into a ring in shared
 // memory by bulk copies, several groups ahead of the arithmetic.  Every wait has a time limit (tc_common.cuh).
 constexpr int SC_THREADS = 64;
 constexpr int SC_GROUP = 8;
 
-__host__ __device__ constexpr int scan_lanes(int dmax) { return dmax <= 32 ? 2 : dmax / 16; }
+__host__ __device__ constexpr int scan_lanes(int dmax) { return dmax <= 64 ? dmax / 8 : dmax / 16; }
 // columns of a slice, and slices of a head (memory: one more column, n)
-__host__ __device__ constexpr int scan_cols(int d) { return SC_THREADS / scan_lanes(scan_dmax(d)); }
+__host__ __device__ constexpr int scan_cols(int d) { return 2 * SC_THREADS / scan_lanes(scan_dmax(d)); }
 __host__ __device__ constexpr int scan_slices(int d, int n_cols) { return (n_cols + scan_cols(d) - 1) / scan_cols(d); }
 
+inline int scan_shift(int d) {
+  int s = 0;
+  while ((1 << s) < scan_cols(d)) ++s;
+  return s;
+}
 // floats of a vector in a record, and of a slice's row of values
 LLM_EXPORT int llm_scan_padded(int d) { return scan_dmax(d); }
 LLM_EXPORT int llm_scan_columns(int d) { return scan_cols(d); }
@@ -100,13 +105,109 @@ __device__ __forceinline__ float scan_token(float2 (&S)[ROWS / 2], const float *
   return fmaf(sc.z, z, RULE == RULE_BONUS ? rs : sc.x * rs);
 }
 
+// Loads that say they read shared memory, in the order they are written: a token's vectors are asked for a token ahead.
+__device__ __forceinline__ float4 shared_ld4(unsigned at) {
+  float4 v;
+  asm volatile("ld.shared.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(at));
+  return v;
+}
+__device__ __forceinline__ float2 shared_ld2(unsigned at) {
+  float2 v;
+  asm volatile("ld.shared.v2.f32 {%0, %1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(at));
+  return v;
+}
+
+// The same for N tokens in a row and two columns of a lane: the read-outs' sums over the lanes wait until the group is through
+// (nothing in it needs them), and a token's vectors are on their way while the token before is worked on.
+template <int RULE, int LANES, int ROWS, int REC, int DMAX, int N>
+__device__ __forceinline__ void scan_group(float2 (&S)[2][ROWS / 2], unsigned rec, unsigned scal, unsigned vals, unsigned v_step,
+                                           float (&out)[2][N]) {
+  constexpr int NV = RULE == RULE_BONUS ? 3 : 2;
+  float4 x[2][NV][ROWS / 4], sc[2];
+  float2 v[2];
+  float rs[2][N], cz[2][N];
+  auto fetch = [&](int e) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k)
+#pragma unroll
+      for (int i = 0; i < ROWS / 4; ++i) x[e & 1][k][i] = shared_ld4(rec + (e * REC + k * DMAX + 4 * LANES * i) * 4);
+    sc[e & 1] = shared_ld4(scal + e * 16);
+    v[e & 1] = shared_ld2(vals + e * v_step);
+  };
+  fetch(0);
+#pragma unroll
+  for (int e = 0; e < N; ++e) {
+    if (e + 1 < N) fetch(e + 1);
+    __syncwarp();                                     // keeps the loads where they are written: ahead of this token's work
+    const float4 (&k4)[ROWS / 4] = x[e & 1][0], (&q4)[ROWS / 4] = x[e & 1][1];
+    const float4 s4 = sc[e & 1];
+    float z[2];
+    if (RULE == RULE_DELTA) {
+      float ps[2];
+#pragma unroll
+      for (int c = 0; c < 2; ++c) {
+        float2 p0 = make_float2(0.f, 0.f), p1 = p0;
+#pragma unroll
+        for (int i = 0; i < ROWS / 4; ++i) {
+          p0 = __ffma2_rn(make_float2(k4[i].x, k4[i].y), S[c][2 * i], p0);
+          p1 = __ffma2_rn(make_float2(k4[i].z, k4[i].w), S[c][2 * i + 1], p1);
+        }
+        p0 = __fadd2_rn(p0, p1);
+        ps[c] = p0.x + p0.y;
+      }
+#pragma unroll
+      for (int o = 1; o < LANES; o <<= 1)
+#pragma unroll
+        for (int c = 0; c < 2; ++c) ps[c] += __shfl_xor_sync(0xffffffffu, ps[c], o);
+      z[0] = s4.y * fmaf(-s4.x, ps[0], v[e & 1].x);
+      z[1] = s4.y * fmaf(-s4.x, ps[1], v[e & 1].y);
+    } else {
+      z[0] = RULE == RULE_BONUS ? v[e & 1].x : s4.y * v[e & 1].x;
+      z[1] = RULE == RULE_BONUS ? v[e & 1].y : s4.y * v[e & 1].y;
+    }
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+      float2 r0 = make_float2(0.f, 0.f), r1 = r0;
+#pragma unroll
+      for (int i = 0; i < ROWS / 4; ++i) {
+        r0 = __ffma2_rn(make_float2(q4[i].x, q4[i].y), S[c][2 * i], r0);
+        r1 = __ffma2_rn(make_float2(q4[i].z, q4[i].w), S[c][2 * i + 1], r1);
+      }
+      r0 = __fadd2_rn(r0, r1);
+      rs[c][e] = RULE == RULE_BONUS ? r0.x + r0.y : s4.x * (r0.x + r0.y);
+      cz[c][e] = s4.z * z[c];
+      const float2 z2 = make_float2(z[c], z[c]);
+      float2 w0 = make_float2(s4.x, s4.x), w1 = w0;
+#pragma unroll
+      for (int i = 0; i < ROWS / 4; ++i) {
+        if constexpr (RULE == RULE_BONUS) {
+          w0 = make_float2(x[e & 1][2][i].x, x[e & 1][2][i].y);
+          w1 = make_float2(x[e & 1][2][i].z, x[e & 1][2][i].w);
+        }
+        S[c][2 * i] = __ffma2_rn(w0, S[c][2 * i], __fmul2_rn(make_float2(k4[i].x, k4[i].y), z2));
+        S[c][2 * i + 1] = __ffma2_rn(w1, S[c][2 * i + 1], __fmul2_rn(make_float2(k4[i].z, k4[i].w), z2));
+      }
+    }
+  }
+#pragma unroll
+  for (int o = 1; o < LANES; o <<= 1)
+#pragma unroll
+    for (int e = 0; e < N; ++e)
+#pragma unroll
+      for (int c = 0; c < 2; ++c) rs[c][e] += __shfl_xor_sync(0xffffffffu, rs[c][e], o);
+#pragma unroll
+  for (int e = 0; e < N; ++e)
+#pragma unroll
+    for (int c = 0; c < 2; ++c) out[c][e] = rs[c][e] + cz[c][e];
+}
+
 template <int RULE, int DMAX>
 __global__ void __launch_bounds__(SC_THREADS + 32)
 state_scan_kernel(const float *__restrict__ rec, const float4 *__restrict__ scal, const float *__restrict__ vals, float *__restrict__ state,
                   float *__restrict__ out, long long ldo, float *__restrict__ den, const int *__restrict__ seq_start,
                   const int *__restrict__ seq_slot, int n_tokens, int n_heads, int n_kv, int d, int dv, int n_groups_ring, int *status) {
   constexpr int NV = RULE == RULE_BONUS ? 3 : 2;
-  constexpr int LANES = scan_lanes(DMAX), ROWS = DMAX / LANES, COLS = SC_THREADS / LANES;
+  constexpr int LANES = scan_lanes(DMAX), ROWS = DMAX / LANES, COLS = 2 * SC_THREADS / LANES;
   extern __shared__ __align__(128) unsigned char sc_smem[];
   // a group in the ring: records [tokens][NV * DMAX], values [tokens][COLS], scalars [tokens][4]
   constexpr int rec_f = NV * DMAX, group_f = SC_GROUP * (rec_f + COLS + 4);
@@ -164,38 +265,47 @@ state_scan_kernel(const float *__restrict__ rec, const float4 *__restrict__ scal
     return;
   }
 
-  const int sub = tid % LANES, col = tid / LANES, j = slice * COLS + col;
-  const bool live = j < n_cols;
-  float2 S[ROWS / 2];
-  float *sp = state + (((size_t)seq_slot[b] * n_heads + hd) * n_cols + (live ? j : 0)) * d;
+  const int sub = tid % LANES, col = 2 * (tid / LANES), j = slice * COLS + col;
+  float2 S[2][ROWS / 2];
+  float *sp = state + ((size_t)seq_slot[b] * n_heads + hd) * n_cols * (size_t)d;
   auto row_of = [&](int i) { return 4 * (sub + LANES * (i / 4)) + i % 4; };
 #pragma unroll
-  for (int i = 0; i < ROWS; i += 2) {
-    S[i / 2].x = live && row_of(i) < d ? sp[row_of(i)] : 0.f;
-    S[i / 2].y = live && row_of(i + 1) < d ? sp[row_of(i + 1)] : 0.f;
-  }
-  const bool writes = live && sub == 0;
-  float *dst = RULE == RULE_MEMORY && j == dv ? den + (size_t)start * n_heads + hd : out + (size_t)start * ldo + (size_t)hd * dv + j;
-  const long long step = RULE == RULE_MEMORY && j == dv ? n_heads : ldo;
+  for (int c = 0; c < 2; ++c)
+#pragma unroll
+    for (int i = 0; i < ROWS; i += 2) {
+      const float *column = sp + (size_t)(j + c < n_cols ? j + c : 0) * d;
+      S[c][i / 2].x = j + c < n_cols && row_of(i) < d ? column[row_of(i)] : 0.f;
+      S[c][i / 2].y = j + c < n_cols && row_of(i + 1) < d ? column[row_of(i + 1)] : 0.f;
+    }
+  // lane 0 of the columns' lanes writes the first column's results, lane 1 the second's
+  const int jw = j + sub;
+  const bool writes = sub < 2 && jw < n_cols, to_den = RULE == RULE_MEMORY && jw == dv;
+  float *dst = to_den ? den + (size_t)start * n_heads + hd : out + (size_t)start * ldo + (size_t)hd * dv + jw;
+  const long long step = to_den ? n_heads : ldo;
   bool ok = true;
   int slot = 0;
   unsigned phase = 0;
   for (int p = 0; p < n_groups; ++p) {
     ok = __all_sync(0xffffffffu, mbar_wait(bar_full + 8 * slot, phase, abort_flag, status, 72));
     if (!ok) break;
-    const float *g = ring + (size_t)slot * group_f, *gv = g + SC_GROUP * rec_f + col, *gs = g + SC_GROUP * (rec_f + COLS);
-    auto token = [&](int e) {
-      const float *r = g + e * rec_f;
-      const float o = scan_token<RULE, LANES, ROWS>(S, r, r + DMAX, r + 2 * DMAX, ld4(gs + e * 4), gv[e * COLS], sub);
-      if (writes) *dst = o;
-      dst += step;
-    };
+    const unsigned g = smem_u32(ring + (size_t)slot * group_f), gr = g + 16 * sub, gv = g + (SC_GROUP * rec_f + col) * 4,
+                   gs = g + SC_GROUP * (rec_f + COLS) * 4;
     const int nt = n - p * SC_GROUP;
     if (nt >= SC_GROUP) {
+      float o[2][SC_GROUP];
+      scan_group<RULE, LANES, ROWS, rec_f, DMAX, SC_GROUP>(S, gr, gs, gv, COLS * 4, o);
 #pragma unroll
-      for (int e = 0; e < SC_GROUP; ++e) token(e);
+      for (int e = 0; e < SC_GROUP; ++e) {
+        if (writes) *dst = sub ? o[1][e] : o[0][e];
+        dst += step;
+      }
     } else {
-      for (int e = 0; e < nt; ++e) token(e);
+      for (int e = 0; e < nt; ++e) {
+        float o[2][1];
+        scan_group<RULE, LANES, ROWS, rec_f, DMAX, 1>(S, gr + e * rec_f * 4, gs + e * 16, gv + e * COLS * 4, COLS * 4, o);
+        if (writes) *dst = sub ? o[1][0] : o[0][0];
+        dst += step;
+      }
     }
     __syncwarp();
     if ((tid & 31) == 0) mbar_arrive(bar_empty + 8 * slot);
@@ -206,10 +316,11 @@ state_scan_kernel(const float *__restrict__ rec, const float4 *__restrict__ scal
   }
   // only now: this kernel is narrow and runs long, and a dependent let in at its start would sit beside it all that time
   grid_dependents_launch();
-  if (live)
+#pragma unroll
+  for (int c = 0; c < 2; ++c)
 #pragma unroll
     for (int i = 0; i < ROWS; ++i)
-      if (row_of(i) < d) sp[row_of(i)] = i % 2 ? S[i / 2].y : S[i / 2].x;
+      if (j + c < n_cols && row_of(i) < d) sp[(size_t)(j + c) * d + row_of(i)] = i % 2 ? S[c][i / 2].y : S[c][i / 2].x;
 }
 
 // rec [kv_heads, tokens, 2 or 3, llm_scan_padded(d)], scal [heads, tokens, 4], vals [heads, slices, tokens, columns] (llm_scan_columns), state
@@ -255,10 +366,10 @@ LLM_EXPORT int llm_state_scan(int rule, const float *rec, const float *scal, con
 // ---------------------------------------------------------------- what a token brings, packed for the scan
 // where value column j of a head's token t lies in vals
 struct ValuePlace {
-  int cols, slices;
+  int cols, slices, shift;                            // cols = 2^shift
   long long n_tokens;
   __device__ __forceinline__ size_t at(int head, long long t, int j) const {
-    return (((size_t)head * slices + j / cols) * n_tokens + t) * cols + j % cols;
+    return ((((size_t)head * slices + (j >> shift)) * n_tokens + t) << shift) + (j & (cols - 1));
   }
 };
 
@@ -373,11 +484,18 @@ delta_pack_kernel(const float *__restrict__ proj, long long ld, int off_b, int o
         r[dp + c] = y[e] * iq;
       }
     }
-    for (int e = lane; e < group; e += 32) {
-      const int h = head * group + e;
-      const float *row = proj + (size_t)t * ld;
-      const float g = expf(-expf(a_log[h]) * softplus32(row[off_a + h] + dt_bias[h]));
-      scal[(size_t)h * n_tokens + t] = make_float4(g, sigmoid32(row[off_b + h]), kq * iq * ik, 0.f);
+    for (int e = lane; e < group; e += 32) scal[(size_t)(head * group + e) * n_tokens + t].z = kq * iq * ik;
+  };
+  // the gates of the group's heads for n rows from `first` on, a lane each (rows of `rows` only, a bit per row)
+  auto gates = [&](int first, int n, unsigned rows) {
+    if (is_v) return;
+    for (int e = lane; e < n * group; e += 32) {
+      const int i = e / group, h = head * group + e - i * group;
+      if (!((rows >> i) & 1u)) continue;
+      const float *row = proj + (size_t)(first + i) * ld;
+      float4 *dst = scal + (size_t)h * n_tokens + first + i;
+      dst->x = expf(-expf(a_log[h]) * softplus32(row[off_a + h] + dt_bias[h]));
+      dst->y = sigmoid32(row[off_b + h]);
     }
   };
   auto take = [&](int row) {
@@ -394,19 +512,23 @@ delta_pack_kernel(const float *__restrict__ proj, long long ld, int off_b, int o
     // which rows are this CTA's (bit per row); the others belong to their sequence's own CTA
     const int rl = r0 + lane;
     const unsigned mine = __ballot_sync(0xffffffffu, lane < ROWS && rl < r1 && tok_pos[rl < r1 ? rl : r0] - seq_past[tok_seq[rl < r1 ? rl : r0]] >= keep);
+    gates(r0, ROWS, mine);
     if (mine == (1u << ROWS) - 1u) {                   // all of them: the rows' loads do not wait for one another
-      float xa[ROWS][CPL], xb[ROWS][CPL];
+      constexpr int PRE = ROWS < 4 ? ROWS : 4;
       for (int k = keep; k > 0; --k) take(r0 - k);
+      for (int i0 = 0; i0 < ROWS; i0 += PRE) {
+        float xa[PRE][CPL], xb[PRE][CPL];
 #pragma unroll
-      for (int i = 0; i < ROWS; ++i) {
-        A.load(proj + (size_t)(r0 + i) * ld, lane, xa[i]);
-        if (!is_v) B.load(proj + (size_t)(r0 + i) * ld, lane, xb[i]);
-      }
+        for (int i = 0; i < PRE; ++i) {
+          A.load(proj + (size_t)(r0 + i0 + i) * ld, lane, xa[i]);
+          if (!is_v) B.load(proj + (size_t)(r0 + i0 + i) * ld, lane, xb[i]);
+        }
 #pragma unroll
-      for (int i = 0; i < ROWS; ++i) {
-        A.push(xa[i]);
-        if (!is_v) B.push(xb[i]);
-        row_out(r0 + i);
+        for (int i = 0; i < PRE; ++i) {
+          A.push(xa[i]);
+          if (!is_v) B.push(xb[i]);
+          row_out(r0 + i0 + i);
+        }
       }
       return;
     }
@@ -430,6 +552,7 @@ delta_pack_kernel(const float *__restrict__ proj, long long ld, int off_b, int o
       B.push(x);
     }
   }
+  gates(start, min(n, keep), 0xffffffffu);
   for (int i = 0; i < min(n, keep); ++i) {
     take(start + i);
     row_out(start + i);
@@ -450,7 +573,7 @@ LLM_EXPORT int llm_delta_pack(const float *proj, long long ld, int off_b, int of
   LLM_REQUIRE(d <= 256 && dv <= 512, "delta_pack: heads of %d and %d channels are not supported (up to 256 and 512)", d, dv);
   LLM_REQUIRE(taps >= 1 && taps <= DP_MAX_TAPS && conv && (taps == 1 || state), "delta_pack: a convolution of %d taps (1 to %d) needs its weight and state",
               taps, DP_MAX_TAPS);
-  const ValuePlace place{scan_cols(d), scan_slices(d, dv), n_tokens};
+  const ValuePlace place{scan_cols(d), scan_slices(d, dv), scan_shift(d), n_tokens};
   const int widest = scan_dmax(d) > place.cols * place.slices ? scan_dmax(d) : place.cols * place.slices;
   const int n_own = taps > 1 ? n_seqs : 0;
 #define DP_GO(CPL, TAPS, ROWS)                                                                                               \
@@ -554,7 +677,7 @@ LLM_EXPORT int llm_bonus_pack(const float *r, long long ldr, const float *k, lon
   const size_t smem = w2_shared ? with_w2 : (size_t)BP_WARPS * rank * BP_TT * sizeof(float);
   LLM_REQUIRE(smem <= 96 * 1024, "bonus_pack: a decay input of rank %d is not supported", rank);
   LLM_CHECK_CUDA(llm_allow_smem(bonus_pack_kernel, smem), "bonus_pack attribute");
-  const ValuePlace place{scan_cols(d), scan_slices(d, dv), n_tokens};
+  const ValuePlace place{scan_cols(d), scan_slices(d, dv), scan_shift(d), n_tokens};
   llm_launch(bonus_pack_kernel, dim3((unsigned)((n_tokens + BP_WARPS * BP_TT - 1) / (BP_WARPS * BP_TT)), n_heads), dim3(BP_WARPS * 32), smem, stream,
              r, ldr, k, ldk, v, ldv, x1, ldx, rank, w2, w0, u, n_tokens, d, dv, w2_shared, rec, (float4 *)scal, vals, place);
   LLM_CHECK_LAUNCH("bonus_pack");
@@ -666,7 +789,7 @@ LLM_EXPORT int llm_memory_pack(const float *proj, long long ld, int off_q, int o
   llm_launch(memory_gates_kernel, dim3(n_seqs, n_heads), dim3(MG_THREADS), 0, stream, proj, ld, off_i, off_f, bias_i, bias_f, cap, state_m,
              (float4 *)scal, seq_start, seq_slot, n_tokens, n_heads);
   LLM_CHECK_LAUNCH("memory_gates");
-  const ValuePlace place{scan_cols(d), scan_slices(d, dv + 1), n_tokens};
+  const ValuePlace place{scan_cols(d), scan_slices(d, dv + 1), scan_shift(d), n_tokens};
   llm_launch(memory_pack_kernel, dim3((unsigned)((n_tokens + 4 * MP_TT - 1) / (4 * MP_TT)), n_heads), dim3(128), 0, stream, proj, ld, off_q, off_k,
              off_v, q_scale, rec, (float4 *)scal, vals, place, n_tokens, d, dv);
   LLM_CHECK_LAUNCH("memory_pack");
