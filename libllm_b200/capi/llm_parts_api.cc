@@ -73,6 +73,7 @@ Json act_json(const Act &a) {
   j.set("ld", a.ld);
   j.set("parts", a.parts);
   j.set("part_stride", a.part_stride);
+  if (a.col_bias) j.set("col_bias", (int64_t)(uintptr_t)a.col_bias);   // added to the parts' sum by whoever adds the result
   return j;
 }
 

@@ -775,3 +775,41 @@ def moe_route_grouped(logits: torch.Tensor, top: int, correction: Optional[torch
           _ptr(logits), logits.stride(0), T, E, top, {"sigmoid": 0, "softmax": 1}[score], _ptr(correction), n_groups, keep, group_top,
           1 if renormalize else 0, float(norm_eps), float(route_scale), _ptr(chosen), _ptr(weight), _stream())
     return chosen, weight
+
+
+# ---------------------------------------------------------------- attention whose weights stand for themselves
+def sigmoid_attention(form: str, q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, tok_seq: torch.Tensor,
+                      tok_pos: torch.Tensor, seq_start: torch.Tensor, seq_past: torch.Tensor, page_table: torch.Tensor, max_q_len: int,
+                      n_heads: int, n_kv: int, window: Optional[int], scale: float, temp: torch.Tensor, bias: torch.Tensor, cap: float = 0.0,
+                      out_scale: float = 1.0, n_splits: int = 1) -> torch.Tensor:
+    """A visible key's weight is sigmoid(cap tanh(temp[h] s / cap) + bias[h]) (cap 0: no bound), not normalised; the result
+    times ``out_scale``.  ``form``: "generic" (any type), "prompt" (bfloat16, tcgen05) or "single" (bfloat16, one token per
+    sequence, its pages in ``n_splits`` runs)."""
+    _on_gpu(q, out, kcache, vcache, tok_seq, tok_pos, seq_start, seq_past, page_table, temp, bias)
+    T, B = q.shape[0], page_table.shape[0]
+    page_size, d, dv = kcache.shape[2], kcache.shape[3], vcache.shape[3]
+    assert kcache.is_contiguous() and vcache.is_contiguous() and out.shape == (T, n_heads * dv) and q.stride(1) == 1
+    common = [float(scale), _ptr(temp), _ptr(bias), float(cap), float(out_scale)]
+    sizes = [n_heads, n_kv, d, dv, page_size, int(window or 0)]
+    kinds = [c_int] * 6 + [c_float, c_void_p, c_void_p, c_float, c_float]
+    if form == "generic":
+        _call("attention_generic", "llm_attention_generic_sigmoid",
+              [c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int] + kinds + [c_void_p],
+              dtype_code(q.dtype), _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kcache), _ptr(vcache), _ptr(tok_seq), _ptr(tok_pos),
+              _ptr(page_table), page_table.stride(0), T, *sizes, *common, _stream())
+    elif form == "prompt":
+        _call("attention_sigmoid", "llm_sigmoid_prefill",
+              [c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int,
+               c_int] + kinds + [c_void_p, c_void_p],
+              _ptr(q), q.stride(0), T, _ptr(out), out.stride(0), _ptr(kcache), _ptr(vcache), kcache.shape[0], _ptr(seq_start), _ptr(seq_past),
+              _ptr(page_table), page_table.stride(0), B, int(max_q_len), *sizes, *common, _ptr(tc_status(q.device)), _stream())
+    else:
+        ws = torch.empty(B * n_heads * dv * n_splits, dtype=torch.float32, device=q.device)
+        counters = torch.zeros(B * n_kv, dtype=torch.int32, device=q.device)
+        _call("attention_sigmoid", "llm_sigmoid_decode",
+              [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int] + kinds +
+              [c_int, c_void_p, c_void_p, c_void_p],
+              _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kcache), _ptr(vcache), _ptr(tok_pos), _ptr(page_table), page_table.stride(0), B,
+              *sizes, *common, int(n_splits), _ptr(ws), _ptr(counters), _stream())
+        assert int(counters.abs().sum()) == 0, "the counters are left as they were found"
+    return out

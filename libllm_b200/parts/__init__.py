@@ -300,6 +300,8 @@ class PartHandle:
                 shape = (a["parts"], a["rows"], a["cols"]) if a["parts"] > 1 else (a["rows"], a["cols"])
                 strides = (a["part_stride"], a["ld"], 1) if a["parts"] > 1 else (a["ld"], 1)
                 views[key] = DeviceTensor(a["ptr"], a["dtype"], shape, strides)
+                if a.get("col_bias"):          # 32-bit, a value per column: whoever adds the result adds it once
+                    views[key + "_bias"] = DeviceTensor(a["col_bias"], "float32", (a["cols"],))
             else:
                 views[key] = None
         if res.get("table"):
