@@ -66,7 +66,7 @@ template <int TN, int SW, typename TO>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                TO *__restrict__ out, long long ldo, int M, int n_out, int K, int row_tiles, int tok_tiles,
-               int k_parts, int kb_per_part, long long part_stride, int *status) {
+               int k_parts, int kb_per_part, long long part_stride, int group_tiles, int group_rows, int *status) {
   using S = TcShape<TN, SW>;
   constexpr bool SWIGLU = SW == 1;                      // the interleaved tile with the hand-over
   constexpr int STAGES = S::STAGES;
@@ -124,7 +124,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
     const bool leader = elect_one();
     // The walk over this CTA's (tile, k block) pairs, one per stage filled.
     struct Walk {
-      int tile, kb, kb1, tok_tile, row_a, row_b;
+      int tile, kb, kb1, x_row, row_a, row_b;
       bool valid;
     };
     auto start = [&](Walk &w, int tile) {
@@ -132,7 +132,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
       w.valid = tile < n_tiles;
       if (!w.valid) return;
       const int part = tile % k_parts, row_tile = tile / (k_parts * tok_tiles);
-      w.tok_tile = (tile / k_parts) % tok_tiles;
+      w.x_row = (tile / k_parts) % tok_tiles * TN + row_tile / group_tiles * group_rows;
       w.kb = part * kb_per_part;
       w.kb1 = min(n_kblocks_total, w.kb + kb_per_part);
       w.row_a = row_tile * ROWS_OUT;
@@ -157,7 +157,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
     auto load_x = [&](const Walk &w, int stage) {
       if (leader)
         tma_load_2d(smem_u32(smem + (size_t)stage * S::STAGE_BYTES) + S::A_BYTES, &map_x, w.kb * TC_BK,
-                    w.tok_tile * TN, bar_full + 8 * stage);
+                    w.x_row, bar_full + 8 * stage);
     };
     // Weights first: they do not depend on the kernel before this one, so the whole ring
     // is filled with them while that kernel still runs.  Then the wait, then the tokens of
@@ -320,7 +320,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 
 template <int TN, int SW, typename TO>
 int launch_tc(const void *x, long long ldx, const void *W, void *out, long long ldo, int M, int N, int K, int k_parts,
-              long long part_stride, int *status, cudaStream_t stream) {
+              long long part_stride, int *status, cudaStream_t stream, int n_groups = 1, int group_n = 0) {
   using S = TcShape<TN, SW>;
   const int n_out = SW != 0 ? N / 2 : N;
   const int rows_out = SW == 1 ? 64 : 128;
@@ -332,7 +332,7 @@ int launch_tc(const void *x, long long ldx, const void *W, void *out, long long 
   CUtensorMap map_w, map_x;
   int rc = get_map(W, N, K, K, SW == 2 ? 128 : 64, &map_w);
   if (rc != LLM_OK) return rc;
-  rc = get_map(x, M, K, ldx, TN, &map_x);
+  rc = get_map(x, (long long)n_groups * M, K, ldx, TN, &map_x);
   if (rc != LLM_OK) return rc;
   auto kern = gemm_tc_kernel<TN, SW, TO>;
   LLM_CHECK_CUDA(llm_allow_smem(kern, S::SMEM), "gemm_tc attribute");
@@ -340,7 +340,8 @@ int launch_tc(const void *x, long long ldx, const void *W, void *out, long long 
   LLM_REQUIRE(tiles < (1ll << 30), "gemm_tc: too many tiles");
   const int grid = (int)(tiles < sm_count() ? tiles : sm_count());
   LLM_CHECK_CUDA(llm_launch(kern, dim3(grid), dim3(TC_THREADS), S::SMEM, stream, map_w, map_x, (TO *)out, ldo, M, n_out, K,
-                            row_tiles, tok_tiles, k_parts, kb_per_part, part_stride, status),
+                            row_tiles, tok_tiles, k_parts, kb_per_part, part_stride, n_groups > 1 ? group_n / 128 : row_tiles,
+                            n_groups > 1 ? M : 0, status),
                  "gemm_tc launch");
   return LLM_OK;
 }
@@ -408,6 +409,25 @@ LLM_EXPORT int llm_gemm_tc(const void *x, long long ldx, const void *W, void *ou
     if (out_dtype == LLM_F32) return dispatch_tc<false, float>(x, ldx, W, out, ldo, M, N, K, k_parts, part_stride, status, stream);
   }
   LLM_FAIL("gemm_tc: unknown output dtype %d", out_dtype);
+}
+
+// Several products of as many inputs in one launch: x [n_groups * M, K] (input g's rows from g * M on), W the matrices one
+// behind the other, each but the last of group_n rows (a multiple of 128, so that a tile has one input), N rows in all;
+// out [M, N] 32-bit.
+LLM_EXPORT int llm_gemm_tc_grouped(const void *x, long long ldx, const void *W, float *out, long long ldo, int M, int N, int K, int n_groups,
+                                   int group_n, int *status, cudaStream_t stream) {
+  if (M == 0 || N == 0) return LLM_OK;
+  LLM_REQUIRE(M > 0 && N > 0 && K > 0 && n_groups >= 1, "gemm_tc_grouped: bad sizes %d x %d x %d", M, N, K);
+  LLM_REQUIRE(n_groups == 1 || (group_n > 0 && group_n % 128 == 0 && (long long)(n_groups - 1) * group_n < N && (long long)n_groups * group_n >= N),
+              "gemm_tc_grouped: %d matrices of %d rows do not make %d", n_groups, group_n, N);
+  LLM_REQUIRE(K % 8 == 0 && ldx % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)W % 16 == 0, "gemm_tc_grouped: rows must start on 16 bytes");
+#define TC_GROUP(TN) return launch_tc<TN, 0, float>(x, ldx, W, out, ldo, M, N, K, 1, 0, status, stream, n_groups, group_n)
+  if (M <= 16) TC_GROUP(16);
+  if (M <= 32) TC_GROUP(32);
+  if (M <= 64) TC_GROUP(64);
+  if (M <= 128) TC_GROUP(128);
+  TC_GROUP(256);
+#undef TC_GROUP
 }
 
 // ---------------------------------------------------------------- a wait that runs out, for tests

@@ -268,6 +268,14 @@ void gemm_tc(const Act &x, const Weight &w, const Act &out, bool swiglu, int *st
            (long long)(x.rows > 1 ? out.ld : out.cols), code(out.dtype), (int)x.rows, (int)w.rows, (int)x.cols, swiglu ? 1 : 0,
            out.parts, (long long)out.part_stride, status, s);
 }
+LLM_KERNEL("gemm_tc", llm_gemm_tc_grouped, const void *, long long, const void *, float *, long long, int, int, int, int, int, int *,
+           cudaStream_t)
+void gemm_tc_grouped(const Act &x, const Weight &w, const Act &out, int n_groups, int group_n, int *status, cudaStream_t s) {
+  if (x.dtype != DType::BF16 || out.dtype != DType::F32 || x.rows != out.rows * n_groups)
+    LLM_THROW(InvalidArg, "gemm_tc_grouped: bfloat16 inputs stacked one behind the other, 32-bit results");
+  LLM_CALL("gemm_tc", llm_gemm_tc_grouped, x.data, (long long)x.ld, w.data(), (float *)out.data, (long long)out.ld, (int)out.rows, (int)w.rows,
+           (int)x.cols, n_groups, group_n, status, s);
+}
 LLM_KERNEL("gemm_tc", llm_gemm_tc_wait_probe, long long, int *, cudaStream_t)
 void gemm_tc_wait_probe(long long limit_ns, int *status, cudaStream_t s) { LLM_CALL("gemm_tc", llm_gemm_tc_wait_probe, limit_ns, status, s); }
 LLM_KERNEL("gemm_chain", llm_gemm_chain, const ChainJob *, int, int *, int *, cudaStream_t)

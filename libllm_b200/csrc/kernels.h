@@ -63,6 +63,8 @@ void gemm_plain(const Act &x, const Weight &w, const float *bias, const Act &out
 bool gemm_tc_supported(const Act &x, const Weight &w);
 int gemm_tc_suggest_parts(int M, int N, int K);
 void gemm_tc(const Act &x, const Weight &w, const Act &out, bool swiglu, int *status, cudaStream_t s);
+// x [n_groups * rows, K] through the matrices stacked in w, each but the last of group_n rows (a multiple of 128): out [rows, w.rows]
+void gemm_tc_grouped(const Act &x, const Weight &w, const Act &out, int n_groups, int group_n, int *status, cudaStream_t s);
 void gemm_tc_wait_probe(long long limit_ns, int *status, cudaStream_t s);
 // One job of a chain of products and norms run as one launch (csrc/gemm_chain.cu, which has the
 // same structure under the name llm_chain_job).

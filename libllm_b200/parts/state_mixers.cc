@@ -17,6 +17,7 @@
 // rms(o) = sqrt(mean(o^2) + eps) per head.  `out_scale` (1): the mixer's result is multiplied by it (in 32-bit, before the
 // output projection's input is rounded).  A prompt step packs its tokens' vectors, scans them and norms; a step of single
 // tokens is one launch between the products.  The reference has no such mixers.
+#include <algorithm>
 #include <cmath>
 
 #include "config/config.h"
@@ -224,7 +225,21 @@ class TimeMixing : public StateMixer {
     const std::vector<TensorNeed> needs = tensor_needs();
     mu_.buf.allocate((size_t)N_MIX * (size_t)hidden_ * sizeof(float));
     for (int i = 0; i < N_MIX; ++i) l.fetch_into(needs[(size_t)i], DType::F32, mu_.buf.as<float>() + (size_t)i * hidden_);
-    for (int i = 0; i < N_MIX; ++i) stack_rows(l, {needs[(size_t)(R + i)]}, hidden_, &w_[i]);
+    // the five matrices one behind the other, each but the last padded to whole tiles of the grouped product
+    group_n_ = (std::max(q_width_, v_width_) + 127) / 128 * 128;
+    const size_t row = (size_t)hidden_ * dtype_size(l.engine);
+    w_all_.dtype = l.engine;
+    w_all_.rows = (N_MIX - 1) * group_n_ + (rank_ + 7) / 8 * 8;
+    w_all_.cols = hidden_;
+    w_all_.buf.allocate((size_t)w_all_.rows * row, true);
+    for (int i = 0; i < N_MIX; ++i) {
+      const TensorNeed &n = needs[(size_t)(R + i)];
+      w_[i].dtype = l.engine;
+      w_[i].rows = n.shape[0];
+      w_[i].cols = hidden_;
+      w_[i].view = (char *)w_all_.buf.get() + (size_t)(i * group_n_) * row;
+      l.fetch_into(n, l.engine, w_[i].view);
+    }
     w2_ = l.fetch(needs[W2]);
     w0_ = l.fetch(needs[W0]);
     u_ = l.fetch(needs[U]);
@@ -244,11 +259,24 @@ class TimeMixing : public StateMixer {
     kernels::token_shift(x, mu_.buf.as<float>(), N_MIX, mixed, previous, ctx.tok_seq, ctx.tok_pos, ctx.seq_start, ctx.seq_past,
                          ctx.seq_slot, ctx.n_seqs, ctx.decode_only, ctx.stream);
     Act in[N_MIX];
-    for (int i = 0; i < N_MIX; ++i) {
-      Act m = mixed;
-      m.rows = T;
-      m.data = (char *)mixed.data + (size_t)i * (size_t)T * (size_t)hidden_ * dtype_size(ctx.dtype);
-      in[i] = linear(ctx, m, w_[i], nullptr, DType::F32);
+    const FastSwitches &f = fast_switches();
+    if (ctx.dtype == DType::BF16 && f.gemm_tc && T <= f.tc_tokens && group_n_ * (N_MIX - 1) < w_all_.rows && w_all_.rows <= group_n_ * N_MIX &&
+        hidden_ % 8 == 0) {
+      // few tokens: the five products in one launch
+      Act all = ctx.arena->act(DType::F32, T, w_all_.rows);
+      kernels::gemm_tc_grouped(mixed, w_all_, all, N_MIX, (int)group_n_, ctx.tc_status, ctx.stream);
+      for (int i = 0; i < N_MIX; ++i) {
+        in[i] = all;
+        in[i].cols = w_[i].rows;
+        in[i].data = (float *)all.data + (size_t)(i * group_n_);
+      }
+    } else {
+      for (int i = 0; i < N_MIX; ++i) {
+        Act m = mixed;
+        m.rows = T;
+        m.data = (char *)mixed.data + (size_t)i * (size_t)T * (size_t)hidden_ * dtype_size(ctx.dtype);
+        in[i] = linear(ctx, m, w_[i], nullptr, DType::F32);
+      }
     }
     flush_chain(ctx);
     Act y = ctx.arena->act(ctx.dtype, T, v_width_);
@@ -269,9 +297,9 @@ class TimeMixing : public StateMixer {
   }
 
  private:
-  int64_t rank_;
+  int64_t rank_, group_n_ = 0;
   std::vector<std::string> names_;
-  Weight mu_, w_[N_MIX], w2_, w0_, u_, norm_, w_o_;
+  Weight mu_, w_all_, w_[N_MIX], w2_, w0_, u_, norm_, w_o_;
 };
 
 // ---------------------------------------------------------------- matrix memory

@@ -127,12 +127,13 @@ struct Act {
   const float *col_bias = nullptr;
 };
 
-// A weight on the device: [rows, cols] row-major, or a vector (rows = 1).
+// A weight on the device: [rows, cols] row-major, or a vector (rows = 1).  With `view` it is rows of another weight's memory.
 struct Weight {
   DeviceBuffer buf;
   DType dtype = DType::F32;
   int64_t rows = 0, cols = 0;
-  void *data() const { return buf.get(); }
+  void *view = nullptr;
+  void *data() const { return view ? view : buf.get(); }
 };
 
 }  // namespace llm
