@@ -93,10 +93,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   unsigned char *sQ = smem, *sKV = smem + S::Q_BYTES;
   float *xch = reinterpret_cast<float *>(sKV + (size_t)STAGES * 2 * S::KV_BYTES);       // [2][2][128]
   unsigned long long *bars = (unsigned long long *)(xch + 4 * FT_BM);
-  // full[STAGES], empty[STAGES], q_full, s_full[2], p_full[2] (one per score buffer each), o_full, pv_done[2]
+  // full[STAGES], empty[STAGES], q_full, s_full[2], p_full[2] (one per score buffer each), o_full, pv_done[2], last
   const unsigned bar_full = smem_u32(bars), bar_empty = smem_u32(bars + STAGES);
   const unsigned bar_q = smem_u32(bars + 2 * STAGES), bar_sfull = bar_q + 8,
-                 bar_pfull = bar_q + 24, bar_ofull = bar_q + 40, bar_pvdone = bar_q + 48;
+                 bar_pfull = bar_q + 24, bar_ofull = bar_q + 40, bar_pvdone = bar_q + 48, bar_last = bar_q + 64;
   unsigned *tmem_slot = (unsigned *)(bars + 2 * STAGES + 9);
   volatile int *abort_flag = (volatile int *)(tmem_slot + 1);
 
@@ -125,6 +125,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     mbar_init(bar_ofull, 1);
     mbar_init(bar_pvdone, 1);
     mbar_init(bar_pvdone + 8, 1);
+    mbar_init(bar_last, 1);
     *abort_flag = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
@@ -259,6 +260,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           tc_commit(bar_ofull);
           tc_commit(bar_pvdone + 8 * (j & 1));
           tc_commit(bar_empty + 8 * stage);
+          if (j + 1 == n_tiles) tc_commit(bar_last);
         }
         __syncwarp();
       }
@@ -369,10 +371,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       __syncwarp();
       if (lane == 0) mbar_arrive(bar_pfull + 8 * (j & 1));
     }
-    // the last two products one after the other: a parity alone does not tell the last from the last but two
-    if (ok && n_tiles > 1) ok = mbar_wait(bar_ofull, (n_tiles - 2) & 1, abort_flag, status, 20);
-    if (ok) ok = mbar_wait(bar_ofull, (n_tiles - 1) & 1, abort_flag, status, 20);
-    ok = __all_sync(0xffffffffu, ok);
+    // a barrier of its own: the parity of the output's barrier does not tell the last product from the last but two
+    if (ok) ok = __all_sync(0xffffffffu, mbar_wait(bar_last, 0, abort_flag, status, 20));
     // The row's sum is the two threads' sums, first half first.  Every row warp comes here, whatever
     // happened above.
     asm volatile("bar.sync 5, 256;" ::: "memory");          // the last tile's maxima have been read

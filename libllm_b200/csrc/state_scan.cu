@@ -431,7 +431,7 @@ struct ConvLane {
 };
 
 template <int CPL, int TAPS, int ROWS>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, CPL <= 2 && TAPS <= 4 ? 4 : CPL <= 4 && TAPS <= 4 ? 3 : 1)
 delta_pack_kernel(const float *__restrict__ proj, long long ld, int off_b, int off_a, const float *__restrict__ conv, int taps,
                   float *__restrict__ state, const float *__restrict__ dt_bias, const float *__restrict__ a_log, float key_eps, float q_scale,
                   float *__restrict__ rec, float4 *__restrict__ scal, float *__restrict__ vals, ValuePlace place, const int *__restrict__ tok_seq,
@@ -514,8 +514,9 @@ delta_pack_kernel(const float *__restrict__ proj, long long ld, int off_b, int o
     const unsigned mine = __ballot_sync(0xffffffffu, lane < ROWS && rl < r1 && tok_pos[rl < r1 ? rl : r0] - seq_past[tok_seq[rl < r1 ? rl : r0]] >= keep);
     gates(r0, ROWS, mine);
     if (mine == (1u << ROWS) - 1u) {                   // all of them: the rows' loads do not wait for one another
-      constexpr int PRE = ROWS < 4 ? ROWS : 4;
+      constexpr int PRE = CPL <= 2 ? 4 : CPL <= 4 ? 2 : 1;
       for (int k = keep; k > 0; --k) take(r0 - k);
+#pragma unroll 1
       for (int i0 = 0; i0 < ROWS; i0 += PRE) {
         float xa[PRE][CPL], xb[PRE][CPL];
 #pragma unroll
@@ -588,11 +589,11 @@ LLM_EXPORT int llm_delta_pack(const float *proj, long long ld, int off_b, int of
     if (taps <= 4) DP_GO(CPL, 4, ROWS);            \
     else DP_GO(CPL, DP_MAX_TAPS, ROWS);            \
   } while (0)
-  if (widest <= 32) DP_TAPS(1, 8);
-  else if (widest <= 64) DP_TAPS(2, 8);
-  else if (widest <= 128) DP_TAPS(4, 4);
-  else if (widest <= 256) DP_TAPS(8, 2);
-  else DP_TAPS(16, 1);
+  if (widest <= 32) DP_TAPS(1, 16);
+  else if (widest <= 64) DP_TAPS(2, 16);
+  else if (widest <= 128) DP_TAPS(4, 16);
+  else if (widest <= 256) DP_TAPS(8, 8);
+  else DP_TAPS(16, 8);
 #undef DP_TAPS
 #undef DP_GO
   LLM_CHECK_LAUNCH("delta_pack");
