@@ -689,12 +689,13 @@ def rarelorn_config(hidden, runs, heads, kv, dim, ff, vocab, window=1024, expert
 
 
 def rarelorn_numbers(c, batch, rank=16):
-    """(bytes a decode step of `batch` sequences reads apart from cache and state, cache bytes of a sequence as a function of
-    its length, bytes of state a step reads and writes per sequence, prefill flops of T tokens with one wanted row)."""
+    """(bytes a decode step of `batch` sequences reads at least and at most apart from cache and state: the experts that every
+    sequence chooses alike, or that no two share; cache bytes of a sequence as a function of its length, bytes of state a step
+    reads and writes per sequence, prefill flops of T tokens with one wanted row)."""
     H, V = c["width"], c["vocab"]
     loop = c["loop"]
     runs = list(range(loop["start"])) + list(range(loop["start"], loop["stop"])) * loop["times"] + list(range(loop["stop"], len(c["layers"])))
-    used = touched = state = rec = 0
+    used = most = state = rec = 0
     att = []                                          # (window, cache bytes a key, flops a key)
     for i in runs:
         m, kind = c["layers"][i]["mixer"], c["layers"][i]["type"]
@@ -717,14 +718,14 @@ def rarelorn_numbers(c, batch, rank=16):
         f = c["layers"][i]["mlp"]
         r, one = f["router"], 3 * H * f["expert"]["ff"]
         used += mats + r["experts"] * H + r["top"] * one
-        touched += mats + r["experts"] * H + min(r["experts"], batch * r["top"]) * one
+        most += mats + r["experts"] * H + min(r["experts"], batch * r["top"]) * one
 
     def cache_bytes(n):
         return sum(b * min(n, w) for w, b, _ in att)
 
     def prefill_flops(T):
         return 2 * T * used + T * rec + sum(fl * sum(min(p + 1, w) for p in range(T)) for w, _, fl in att) + 2 * V * H
-    return 2 * (touched + V * H), cache_bytes, state, prefill_flops
+    return (2 * (used + V * H), 2 * (most + V * H)), cache_bytes, state, prefill_flops
 
 
 def run_compare_rarelorn(args):
@@ -741,8 +742,8 @@ def run_compare_rarelorn(args):
                 continue
             if label == "sesuzen":
                 cfg = sesuzen_config(hidden, runs, heads, kv, dim, ff, vocab, window, keep)
-                wbytes, kv_tok, state, flops_fn = sesuzen_numbers(cfg, args.batch)
-                cache_fn = lambda n: kv_tok * min(n, window + keep)
+                dense, kv_tok, state, flops_fn = sesuzen_numbers(cfg, args.batch)
+                wbytes, cache_fn = (dense, dense), lambda n: kv_tok * min(n, window + keep)
             else:
                 cfg = rarelorn_config(hidden, runs, heads, kv, dim, ff, vocab, window)
                 wbytes, cache_fn, state, flops_fn = rarelorn_numbers(cfg, args.batch)
@@ -753,15 +754,15 @@ def run_compare_rarelorn(args):
             pre = prefill_rate(model, vocab, lambda T: flops, pk["bf16_tflops"])
             rate, ms, ctx_len, launches = decode_rate(model, args.batch, args.steps, args.warmup, vocab)
             clocks = sampler.stop()
-            step_bytes = wbytes + args.batch * (cache_fn(ctx_len) + state)
+            step_bytes = [b + args.batch * (cache_fn(ctx_len) + state) for b in wbytes]
             print(json.dumps({"compare": name, "model": label, "batch": args.batch, "prompt": PROMPT,
                               "config": {"hidden": hidden, "runs": runs, "heads": heads, "kv_heads": kv, "head_dim": dim, "ff": ff,
                                          "vocab": vocab, "window": window},
                               "prefill": {"ms": round(pre["ms"], 3), "tok_s": round(pre["value"], 1), "tflop": round(flops / 1e12, 3),
                                           "frac_of_gemm_peak": round(pre["frac"], 4)},
                               "decode": {"tok_s": round(rate, 1), "ms_per_step": round(ms, 4), "launches_per_step": launches,
-                                         "step_gb": round(step_bytes / 1e9, 3),
-                                         "hbm_frac": round(step_bytes / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)},
+                                         "step_gb": [round(b / 1e9, 3) for b in step_bytes],      # at least, at most
+                                         "hbm_frac_at_least": round(step_bytes[0] / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)},
                               "clocks": clocks, "peaks": pk["source"]}), flush=True)
             model.engine.close()
             del model
