@@ -16,8 +16,13 @@ Json parse_rot(const Json &raw, const std::string &where, int64_t head_dim) {
     Json sc = Json::object();
     sc.set("factor", s.number("factor"));
     sc.set("original", s.number("original"));
-    sc.set("fast", s.number("fast"));
-    sc.set("slow", s.number("slow"));
+    if (s.present("low") || s.present("high")) {
+      sc.set("low", s.number("low"));
+      sc.set("high", s.number("high"));
+    } else {
+      sc.set("fast", s.number("fast"));
+      sc.set("slow", s.number("slow"));
+    }
     rot.set("scaling", sc);
   } else {
     rot.set("scaling", Json());
@@ -102,6 +107,15 @@ Json rope_description(const Json &rot, int64_t head_dim) {
     p.set("scaling", Json());
   } else {
     Json y = Json::object();
+    if (sc.has("low")) {
+      y.set("rope_type", "llama3");
+      y.set("factor", sc.get("factor"));
+      y.set("original_max_position_embeddings", sc.get("original"));
+      y.set("low_freq_factor", sc.get("low"));
+      y.set("high_freq_factor", sc.get("high"));
+      p.set("scaling", y);
+      return p;
+    }
     y.set("rope_type", "yarn");
     y.set("factor", sc.get("factor"));
     y.set("original_max_position_embeddings", sc.get("original"));

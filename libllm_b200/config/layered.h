@@ -1,11 +1,12 @@
 // Pieces of config.json that designs which list their layers one by one have in common (config/tazizen.cc,
-// config/rarelorn.cc): each checks what it reads and returns it in normal form, every key present.
+// config/rarelorn.cc, config/fomodra.cc): each checks what it reads and returns it in normal form, every key present.
 #pragma once
 #include "config/config.h"
 
 namespace llm {
 
-// {dims, base, scaling {factor, original, fast, slow} or absent}; dims even and at most head_dim
+// {dims, base, scaling {factor, original, fast, slow} (a ramp over the pairs), {factor, original, low, high} (by wavelength) or
+// absent}; dims even and at most head_dim
 Json parse_rot(const Json &raw, const std::string &where, int64_t head_dim);
 // the mixer's `mask` {size}, or no key at all -> {size: number or null}
 Json parse_mask(const ConfigReader &r, const std::string &where);

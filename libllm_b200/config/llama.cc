@@ -195,6 +195,8 @@ void register_builtin_architectures() {
   register_tazizen_architecture();
   extern void register_rarelorn_architecture();    // config/rarelorn.cc
   register_rarelorn_architecture();
+  extern void register_fomodra_architecture();     // config/fomodra.cc
+  register_fomodra_architecture();
 }
 
 }  // namespace llm

@@ -28,9 +28,13 @@
 // second CTA on the same SM fills the rest.  Exponentials are exp2 of scores pre-scaled by
 // log2(e) / sqrt(d).
 //
+// Heads of other sizes, and values of another width than keys: a head's channels are padded to whole blocks of 64 by TMA
+// (channels of K and V beyond the head read as zeros; what the Q tile holds there, the next head's, meets zeros), and the
+// output row is as many columns of tensor memory as the padded value has channels.
+//
 // Semantics as the other attention kernels: token i of a sequence that stands behind `past` cached
 // ones sees keys 0..past+i (src/flint/operators.cc:119-124), head h reads kv head h / (heads /
-// kv_heads) (:43-56), optional window.  Head sizes 64 and 128, pages of 64 tokens.  Every wait has
+// kv_heads) (:43-56), optional window.  Keys of up to 128 channels, values of up to 256, multiples of 8; pages of 64 tokens.  Every wait has
 // a time limit (see tc_common.cuh).  The reference calls FlashAttention-2's sm_80 kernel here
 // (src/flint/cuda/flash_attn.cc:101-186).
 #include "common.cuh"
@@ -45,19 +49,21 @@ constexpr int FT_THREADS = 384;   // warps 0-7: two threads per query row; 8: lo
 constexpr int FT_BM = 128;          // query rows per CTA
 constexpr int FT_BN = 64;           // keys per tile = tokens per page
 
-template <int D>
+template <int KB, int VB>                                   // 64-wide blocks of a key and of a value
 struct FtShape {
-  static constexpr int KB = D / 64;                         // 64-wide blocks of the head size
-  static constexpr int Q_BYTES = FT_BM * D * 2;
-  static constexpr int KV_BYTES = FT_BN * D * 2;            // one of K or V
+  static constexpr int Q_BYTES = FT_BM * KB * 128;
+  static constexpr int K_BYTES = FT_BN * KB * 128, V_BYTES = FT_BN * VB * 128, KV_BYTES = K_BYTES + V_BYTES;
   static constexpr int X_BYTES = 2 * 2 * FT_BM * 4;          // the partners' maxima, two tiles deep
-  static constexpr int STAGES = D == 64 ? 4 : 2;
-  static constexpr int TMEM_COLS = 256;                     // two S buffers (64 columns each) + O (D columns)
-  static constexpr size_t SMEM = Q_BYTES + X_BYTES + (size_t)STAGES * 2 * KV_BYTES + 256;   // two CTAs per SM
+  static constexpr int TMEM_COLS = 2 * FT_BN + 64 * VB <= 256 ? 256 : 512;   // two S buffers (64 columns each) + O
+  static constexpr int CTAS = TMEM_COLS == 256 ? 2 : 1;     // per SM
+  static constexpr int STAGES_FIT = ((CTAS == 2 ? 108 * 1024 : 200 * 1024) - Q_BYTES) / KV_BYTES;
+  static constexpr int STAGES = STAGES_FIT > 4 ? 4 : STAGES_FIT;
+  static_assert(STAGES >= 2, "two tiles in flight");
+  static constexpr size_t SMEM = Q_BYTES + X_BYTES + (size_t)STAGES * KV_BYTES + 256;
   // Registers move from the third warpgroup (loader, issuer) to the row threads.  The CTA is launched
   // with 80 registers a thread (2 CTAs x 384 threads on an SM), and what the row threads take must
   // be what the third warpgroup gives up inside the same CTA: a request beyond that waits for ever.
-  static constexpr int REGS_LAUNCH = 80, REGS_FEW = 48, REGS_MANY = 96;
+  static constexpr int REGS_LAUNCH = CTAS == 2 ? 80 : 168, REGS_FEW = CTAS == 2 ? 48 : 56, REGS_MANY = CTAS == 2 ? 96 : 216;
   static_assert(128 * REGS_FEW + 256 * REGS_MANY <= FT_THREADS * REGS_LAUNCH, "register moves must balance within the CTA");
 };
 
@@ -80,18 +86,19 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
-template <int D>
-__global__ void __launch_bounds__(FT_THREADS, 2)
+template <int KB, int VB>
+__global__ void __launch_bounds__(FT_THREADS, FtShape<KB, VB>::CTAS)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, __nv_bfloat16 *__restrict__ out,
                             long long out_stride, const int *__restrict__ seq_start, const int *__restrict__ seq_past,
-                            const int *__restrict__ page_table, int pt_stride, int n_heads, int n_kv, int window, int block,
-                            int sink, float scale_log2, float null_log2, int *status) {
-  using S = FtShape<D>;
+                            const int *__restrict__ page_table, int pt_stride, int n_heads, int n_kv, int d, int dv, int window,
+                            int block, int sink, float scale_log2, float null_log2, const float *__restrict__ null_scores,
+                            int *status) {
+  using S = FtShape<KB, VB>;
   constexpr int STAGES = S::STAGES;
   extern __shared__ __align__(1024) unsigned char smem[];
   unsigned char *sQ = smem, *sKV = smem + S::Q_BYTES;
-  float *xch = reinterpret_cast<float *>(sKV + (size_t)STAGES * 2 * S::KV_BYTES);       // [2][2][128]
+  float *xch = reinterpret_cast<float *>(sKV + (size_t)STAGES * S::KV_BYTES);       // [2][2][128]
   unsigned long long *bars = (unsigned long long *)(xch + 4 * FT_BM);
   // full[STAGES], empty[STAGES], q_full, s_full[2], p_full[2] (one per score buffer each), o_full, pv_done[2], last
   const unsigned bar_full = smem_u32(bars), bar_empty = smem_u32(bars + STAGES);
@@ -175,9 +182,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     if (n_tiles > 0) {
       if (leader) {
         mbar_expect_tx(bar_q, S::Q_BYTES);
-        for (int kb = 0; kb < S::KB; ++kb) {
-          tma_load_2d(smem_u32(sQ) + kb * (FT_BM * 128), &map_q, h * D + kb * 64, q0 + r0, bar_q);
-          tma_load_2d(smem_u32(sQ) + kb * (FT_BM * 128) + 64 * 128, &map_q, h * D + kb * 64, q0 + r0 + 64, bar_q);
+        for (int kb = 0; kb < KB; ++kb) {
+          tma_load_2d(smem_u32(sQ) + kb * (FT_BM * 128), &map_q, h * d + kb * 64, q0 + r0, bar_q);
+          tma_load_2d(smem_u32(sQ) + kb * (FT_BM * 128) + 64 * 128, &map_q, h * d + kb * 64, q0 + r0 + 64, bar_q);
         }
       }
       int stage = 0;
@@ -187,13 +194,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         ok = __all_sync(0xffffffffu, mbar_wait(bar_empty + 8 * stage, phase ^ 1, abort_flag, status, 11));
         if (!ok) break;
         const int row = (pt[tile_of(j)] * n_kv + kvh) * FT_BN;
-        const unsigned dk = smem_u32(sKV + (size_t)stage * 2 * S::KV_BYTES), dv = dk + S::KV_BYTES;
+        const unsigned tk = smem_u32(sKV + (size_t)stage * S::KV_BYTES), tv = tk + S::K_BYTES;
         if (leader) {
-          mbar_expect_tx(bar_full + 8 * stage, 2 * S::KV_BYTES);
-          for (int kb = 0; kb < S::KB; ++kb) {
-            tma_load_2d(dk + kb * (FT_BN * 128), &map_k, kb * 64, row, bar_full + 8 * stage);
-            tma_load_2d(dv + kb * (FT_BN * 128), &map_v, kb * 64, row, bar_full + 8 * stage);
-          }
+          mbar_expect_tx(bar_full + 8 * stage, S::KV_BYTES);
+          for (int kb = 0; kb < KB; ++kb) tma_load_2d(tk + kb * (FT_BN * 128), &map_k, kb * 64, row, bar_full + 8 * stage);
+          for (int kb = 0; kb < VB; ++kb) tma_load_2d(tv + kb * (FT_BN * 128), &map_v, kb * 64, row, bar_full + 8 * stage);
         }
         if (++stage == STAGES) {
           stage = 0;
@@ -223,10 +228,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
         tc_fence_after();
-        const unsigned ka = smem_u32(sKV + (size_t)stage * 2 * S::KV_BYTES);
+        const unsigned ka = smem_u32(sKV + (size_t)stage * S::KV_BYTES);
         if (leader) {
 #pragma unroll
-          for (int kb = 0; kb < S::KB; ++kb)
+          for (int kb = 0; kb < KB; ++kb)
 #pragma unroll
             for (int kk = 0; kk < 4; ++kk)
               tc_mma(tmem_s + (j & 1) * FT_BN, smem_desc(smem_u32(sQ) + kb * (FT_BM * 128) + kk * 32),
@@ -240,7 +245,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     // ------------------------------------------------------------ tensor-core issue: output
     const bool leader = elect_one();
     if (n_tiles > 0) {
-      constexpr unsigned IDESC_O = instr_desc_mn(FT_BM, D);           // O[128 x D channels], V MN-major
+      constexpr unsigned IDESC_O = instr_desc_mn(FT_BM, 64 * VB);     // O[128 x padded channels], V MN-major
       bool ok = true;
       for (int j = 0; j < n_tiles && ok; ++j) {
         const int stage = j % STAGES;
@@ -249,9 +254,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
         tc_fence_after();
-        const unsigned va = smem_u32(sKV + (size_t)stage * 2 * S::KV_BYTES) + S::KV_BYTES;
+        const unsigned va = smem_u32(sKV + (size_t)stage * S::KV_BYTES) + S::K_BYTES;
         // 16 keys to a product: 8 columns of P (it lies over the scores' first columns), 16 rows of
-        // V; all D channels at once, the second block of 64 channels FT_BN rows further on
+        // V; all channels at once, the next block of 64 channels FT_BN rows further on
         if (leader) {
 #pragma unroll
           for (int kk = 0; kk < FT_BN / 16; ++kk)
@@ -273,7 +278,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int row = quarter * 32 + lane;                       // row of the tile = lane of tensor memory
     const unsigned lane_addr = (unsigned)(quarter * 32) << 16;
     const int pos = past + r0 + row;                           // the row's position in its sequence
-    constexpr int HD = D / 2;                                  // this thread's channels of the output row
+    constexpr int HD = 32 * VB;                                // this thread's channels of the output row
     const unsigned o_addr = tmem_o + lane_addr + half * HD;
     float ref = -INFINITY;            // the exponent's reference, already times log2(e) / sqrt(d)
     float l_run = 0.f;                // sum of this thread's exponentials, relative to ref
@@ -381,8 +386,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const float l_row = xch[row] + xch[FT_BM + row];
     if (ok) {
       tc_fence_after();
-      const float inv = softmax_norm_factor(ref, l_row, null_log2);
-      __nv_bfloat16 *dst = out + (size_t)(q0 + r0 + row) * out_stride + (size_t)h * D + half * HD;
+      const float inv = softmax_norm_factor(ref, l_row, null_scores ? null_scores[h] * 1.4426950408889634f : null_log2);
+      __nv_bfloat16 *dst = out + (size_t)(q0 + r0 + row) * out_stride + (size_t)h * dv + half * HD;
 #pragma unroll
       for (int c0 = 0; c0 < HD; c0 += 32) {
         float t[2][16];
@@ -396,6 +401,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           for (int c = 0; c < 2; ++c)
 #pragma unroll
             for (int h8 = 0; h8 < 2; ++h8) {
+              if (half * HD + c0 + c * 16 + h8 * 8 >= dv) continue;      // channels of the padding
               uint4 v;
               __nv_bfloat162 t0 = __floats2bfloat162_rn(t[c][h8 * 8] * inv, t[c][h8 * 8 + 1] * inv),
                              t1 = __floats2bfloat162_rn(t[c][h8 * 8 + 2] * inv, t[c][h8 * 8 + 3] * inv),
@@ -467,7 +473,7 @@ attention_prefill_wide_kernel(const __grid_constant__ CUtensorMap map_q, const _
                               const __grid_constant__ CUtensorMap map_v, __nv_bfloat16 *__restrict__ out,
                               long long out_stride, const int *__restrict__ seq_start, const int *__restrict__ seq_past,
                               const int *__restrict__ page_table, int pt_stride, int n_heads, int n_kv, int window, int block,
-                              float scale_log2, float null_log2, int *status) {
+                              float scale_log2, float null_log2, const float *__restrict__ null_scores, int *status) {
   using S = FwShape<D>;
   constexpr int STAGES = S::STAGES;
   extern __shared__ __align__(1024) unsigned char smem[];
@@ -783,7 +789,7 @@ attention_prefill_wide_kernel(const __grid_constant__ CUtensorMap map_q, const _
     if (ok && j_hi > j_lo) ok = __all_sync(0xffffffffu, mbar_wait(bar_ofull + 8 * x, (j_hi - j_lo - 1) & 1, abort_flag, status, 38));
     if (ok && j_hi > j_lo) {
       tc_fence_after();
-      const float inv = softmax_norm_factor(ref, l_run, null_log2);
+      const float inv = softmax_norm_factor(ref, l_run, null_scores ? null_scores[h] * 1.4426950408889634f : null_log2);
       __nv_bfloat16 *dst = out + (size_t)(q0 + r0 + x * 128 + row) * out_stride + (size_t)h * D;
 #pragma unroll
       for (int c0 = 0; c0 < D; c0 += 32) {
@@ -825,83 +831,123 @@ attention_prefill_wide_kernel(const __grid_constant__ CUtensorMap map_q, const _
   }
 }
 
-template <int D>
-int launch_prefill_tc(const void *q, long long q_stride, long long n_tokens, void *out, long long out_stride,
-                      const void *kc, const void *vc, long long n_pages, const int *seq_start, const int *seq_past,
-                      const int *page_table, int pt_stride, int n_seqs, int max_q_len, int n_heads, int n_kv, int window,
-                      int block, int sink, float scale, float null_score, int form, int *status, cudaStream_t stream) {
-  using S = FtShape<D>;
-  if (sink > 0) form = 1;                 // kept first positions: the form of 128 rows walks their tiles
+struct PrefillArgs {
+  const void *q;
+  long long q_stride, n_tokens;
+  void *out;
+  long long out_stride;
+  const void *kc, *vc;
+  long long n_pages;
+  const int *seq_start, *seq_past, *page_table;
+  int pt_stride, n_seqs, max_q_len, n_heads, n_kv, d, dv, window, block, sink;
+  float scale, null_score;
+  const float *null_scores;
+  int *status;
+};
+
+int prefill_maps(const PrefillArgs &a, CUtensorMap *map_q, CUtensorMap *map_k, CUtensorMap *map_v) {
+  int rc = get_map(a.q, a.n_tokens, (long long)a.n_heads * a.d, a.q_stride, 64, map_q);
+  if (rc != LLM_OK) return rc;
+  rc = get_map(a.kc, a.n_pages * a.n_kv * FT_BN, a.d, a.d, 64, map_k);
+  if (rc != LLM_OK) return rc;
+  return get_map(a.vc, a.n_pages * a.n_kv * FT_BN, a.dv, a.dv, 64, map_v);
+}
+
+template <int KB, int VB>
+int launch_prefill_tc(const PrefillArgs &a, cudaStream_t stream) {
+  using S = FtShape<KB, VB>;
   CUtensorMap map_q, map_k, map_v;
-  int rc = get_map(q, n_tokens, (long long)n_heads * D, q_stride, 64, &map_q);
+  const int rc = prefill_maps(a, &map_q, &map_k, &map_v);
   if (rc != LLM_OK) return rc;
-  rc = get_map(kc, n_pages * n_kv * FT_BN, D, D, 64, &map_k);
-  if (rc != LLM_OK) return rc;
-  rc = get_map(vc, n_pages * n_kv * FT_BN, D, D, 64, &map_v);
-  if (rc != LLM_OK) return rc;
-  // Measured: at head size 128 the wide form is ahead from 256 rows on (4 prompts of 2,048: 200 against
-  // 206 us, one of 8,192: 539 against 607); at head size 64 only for long prompts (one of 8,192: 430
-  // against 468 us, 8 of 2,048: 278 against 282, 8 of 512: 46 against 44; and inside a whole prompt
-  // step of 2,048 tokens it is 6 us a layer behind, alone on its SM with all of tensor memory).
-  if (form == 2 || (form == 0 && max_q_len > (D == 64 ? 2048 : FT_BM))) {
-    using W = FwShape<D>;
-    auto kern = attention_prefill_wide_kernel<D>;
-    LLM_CHECK_CUDA(llm_allow_smem(kern, W::SMEM), "attention_prefill_tc attribute");
-    dim3 grid(n_heads, n_seqs, (max_q_len + FW_BM - 1) / FW_BM);
-    LLM_CHECK_CUDA(llm_launch(kern, grid, dim3(FW_THREADS), W::SMEM, stream, map_q, map_k, map_v, (__nv_bfloat16 *)out,
-                              out_stride, seq_start, seq_past, page_table, pt_stride, n_heads, n_kv, window, block,
-                              scale * 1.4426950408889634f, null_score * 1.4426950408889634f, status),
-                   "attention_prefill_tc launch");
-    return LLM_OK;
-  }
-  auto kern = attention_prefill_tc_kernel<D>;
+  auto kern = attention_prefill_tc_kernel<KB, VB>;
   LLM_CHECK_CUDA(llm_allow_smem(kern, S::SMEM), "attention_prefill_tc attribute");
-  dim3 grid(n_heads, n_seqs, (max_q_len + FT_BM - 1) / FT_BM);
-  LLM_CHECK_CUDA(llm_launch(kern, grid, dim3(FT_THREADS), S::SMEM, stream, map_q, map_k, map_v, (__nv_bfloat16 *)out,
-                            out_stride, seq_start, seq_past, page_table, pt_stride, n_heads, n_kv, window, block, sink,
-                            scale * 1.4426950408889634f, null_score * 1.4426950408889634f, status),
+  dim3 grid(a.n_heads, a.n_seqs, (a.max_q_len + FT_BM - 1) / FT_BM);
+  LLM_CHECK_CUDA(llm_launch(kern, grid, dim3(FT_THREADS), S::SMEM, stream, map_q, map_k, map_v, (__nv_bfloat16 *)a.out,
+                            a.out_stride, a.seq_start, a.seq_past, a.page_table, a.pt_stride, a.n_heads, a.n_kv, a.d, a.dv, a.window,
+                            a.block, a.sink, a.scale * 1.4426950408889634f, a.null_score * 1.4426950408889634f, a.null_scores, a.status),
+                 "attention_prefill_tc launch");
+  return LLM_OK;
+}
+
+template <int D>
+int launch_prefill_wide(const PrefillArgs &a, cudaStream_t stream) {
+  using W = FwShape<D>;
+  CUtensorMap map_q, map_k, map_v;
+  const int rc = prefill_maps(a, &map_q, &map_k, &map_v);
+  if (rc != LLM_OK) return rc;
+  auto kern = attention_prefill_wide_kernel<D>;
+  LLM_CHECK_CUDA(llm_allow_smem(kern, W::SMEM), "attention_prefill_tc attribute");
+  dim3 grid(a.n_heads, a.n_seqs, (a.max_q_len + FW_BM - 1) / FW_BM);
+  LLM_CHECK_CUDA(llm_launch(kern, grid, dim3(FW_THREADS), W::SMEM, stream, map_q, map_k, map_v, (__nv_bfloat16 *)a.out,
+                            a.out_stride, a.seq_start, a.seq_past, a.page_table, a.pt_stride, a.n_heads, a.n_kv, a.window, a.block,
+                            a.scale * 1.4426950408889634f, a.null_score * 1.4426950408889634f, a.null_scores, a.status),
                  "attention_prefill_tc launch");
   return LLM_OK;
 }
 
 }  // namespace
 
-// 1 if this head size and page size have an instantiation, else 0.
+// 1 if keys of d and values of dv channels over pages of this size have an instantiation, else 0.
+LLM_EXPORT int llm_attention_prefill_tc_takes(int d, int dv, int page_size) {
+  return page_size == FT_BN && d > 0 && d <= 128 && d % 8 == 0 && dv > 0 && dv <= 256 && dv % 8 == 0;
+}
+// The head sizes (values as wide as keys) that fill whole blocks of channels.
 LLM_EXPORT int llm_attention_prefill_tc_supports(int d, int page_size) {
   return page_size == FT_BN && (d == 64 || d == 128);
 }
 
-// q [n_tokens, >= heads*d] bfloat16 (rotated; row stride q_stride elements), out [n_tokens, heads*d],
-// caches [n_pages, kv_heads, 64, d]; sequence b owns rows seq_start[b]..seq_start[b+1]-1, which stand at
+// q [n_tokens, >= heads*d] bfloat16 (rotated; row stride q_stride elements), out [n_tokens, heads*dv],
+// caches [n_pages, kv_heads, 64, d] and [.., dv]; sequence b owns rows seq_start[b]..seq_start[b+1]-1, which stand at
 // positions seq_past[b].. of the sequence; max_q_len bounds the rows of a sequence.  `status` (device
 // int, may be null) receives a non-zero code if a wait inside the kernel ran out of time.  `form`: 0 the
 // library chooses (the wide form when a sequence brings more than 128 rows), 1 CTAs of 128 rows, 2 of 256.
 // `sink` > 0 with a window: the first `sink` positions of a sequence stay visible to all its later queries (form 1).
-// `null_score`: every query also sees one key of that score that has no value (minus infinity: none).
-LLM_EXPORT int llm_attention_prefill_tc_null(const void *q, long long q_stride, long long n_tokens, void *out,
-                                             long long out_stride, const void *kc, const void *vc, long long n_pages,
-                                             const int *seq_start, const int *seq_past, const int *page_table,
-                                             int pt_stride, int n_seqs, int max_q_len, int n_heads, int n_kv, int d,
-                                             int page_size, int window, int block, int sink, float scale, float null_score,
-                                             int form, int *status, cudaStream_t stream) {
+// `null_score`: every query also sees one key of that score that has no value (minus infinity: none);
+// `null_scores` (32-bit, device; may be null): such a score per head instead.
+LLM_EXPORT int llm_attention_prefill_tc_sinks(const void *q, long long q_stride, long long n_tokens, void *out,
+                                              long long out_stride, const void *kc, const void *vc, long long n_pages,
+                                              const int *seq_start, const int *seq_past, const int *page_table,
+                                              int pt_stride, int n_seqs, int max_q_len, int n_heads, int n_kv, int d, int dv,
+                                              int page_size, int window, int block, int sink, float scale, float null_score,
+                                              const float *null_scores, int form, int *status, cudaStream_t stream) {
   if (n_seqs == 0 || max_q_len == 0) return LLM_OK;
   LLM_REQUIRE(sink >= 0 && (sink == 0 || (window > 0 && block == 0)), "attention_prefill_tc: kept first positions go with a window");
   LLM_REQUIRE(form >= 0 && form <= 2, "attention_prefill_tc: form %d is not one of 0, 1, 2", form);
   LLM_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && n_heads > 0 && n_heads <= 65535 && n_kv > 0 && n_heads % n_kv == 0,
               "attention_prefill_tc: bad sizes (%d sequences, %d heads, %d kv heads)", n_seqs, n_heads, n_kv);
   LLM_REQUIRE(max_q_len > 0 && max_q_len <= 65535 * 128, "attention_prefill_tc: %d tokens of one sequence in a step", max_q_len);
-  LLM_REQUIRE(llm_attention_prefill_tc_supports(d, page_size),
-              "attention_prefill_tc: head size %d with pages of %d tokens is not built (64 or 128, pages of 64)", d, page_size);
+  LLM_REQUIRE(llm_attention_prefill_tc_takes(d, dv, page_size),
+              "attention_prefill_tc: head sizes %d / %d with pages of %d tokens are not built (multiples of 8 up to 128 / 256, pages of 64)",
+              d, dv, page_size);
   LLM_REQUIRE(q_stride % 8 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)kc % 16 == 0 && (uintptr_t)vc % 16 == 0 &&
                   out_stride % 8 == 0 && (uintptr_t)out % 16 == 0,
               "attention_prefill_tc: rows must be 16-byte aligned");
   LLM_REQUIRE(window >= 0 && block >= 0 && scale > 0.f, "attention_prefill_tc: bad window, block or scale");
   LLM_REQUIRE(n_pages * n_kv * FT_BN < (1ll << 31), "attention_prefill_tc: the cache has too many rows for one tensor map");
-  if (d == 64)
-    return launch_prefill_tc<64>(q, q_stride, n_tokens, out, out_stride, kc, vc, n_pages, seq_start, seq_past, page_table,
-                                 pt_stride, n_seqs, max_q_len, n_heads, n_kv, window, block, sink, scale, null_score, form, status, stream);
-  return launch_prefill_tc<128>(q, q_stride, n_tokens, out, out_stride, kc, vc, n_pages, seq_start, seq_past, page_table,
-                                pt_stride, n_seqs, max_q_len, n_heads, n_kv, window, block, sink, scale, null_score, form, status, stream);
+  const PrefillArgs a{q, q_stride, n_tokens, out, out_stride, kc, vc, n_pages, seq_start, seq_past, page_table, pt_stride, n_seqs, max_q_len,
+                      n_heads, n_kv, d, dv, window, block, sink, scale, null_score, null_scores, status};
+  const bool exact = d == dv && llm_attention_prefill_tc_supports(d, page_size);
+  if (sink > 0 || !exact) form = 1;       // kept first positions, padded heads: the form of 128 rows
+  // Measured: at head size 128 the wide form is ahead from 256 rows on (4 prompts of 2,048: 200 against
+  // 206 us, one of 8,192: 539 against 607); at head size 64 only for long prompts (one of 8,192: 430
+  // against 468 us, 8 of 2,048: 278 against 282, 8 of 512: 46 against 44; and inside a whole prompt
+  // step of 2,048 tokens it is 6 us a layer behind, alone on its SM with all of tensor memory).
+  if (form == 2 || (form == 0 && max_q_len > (d == 64 ? 2048 : FT_BM)))
+    return d == 64 ? launch_prefill_wide<64>(a, stream) : launch_prefill_wide<128>(a, stream);
+  if (d <= 64) return dv <= 64 ? launch_prefill_tc<1, 1>(a, stream) : dv <= 128 ? launch_prefill_tc<1, 2>(a, stream) : launch_prefill_tc<1, 4>(a, stream);
+  return dv <= 64 ? launch_prefill_tc<2, 1>(a, stream) : dv <= 128 ? launch_prefill_tc<2, 2>(a, stream) : launch_prefill_tc<2, 4>(a, stream);
+}
+
+// Values as wide as keys, one null score for all heads.
+LLM_EXPORT int llm_attention_prefill_tc_null(const void *q, long long q_stride, long long n_tokens, void *out,
+                                             long long out_stride, const void *kc, const void *vc, long long n_pages,
+                                             const int *seq_start, const int *seq_past, const int *page_table,
+                                             int pt_stride, int n_seqs, int max_q_len, int n_heads, int n_kv, int d,
+                                             int page_size, int window, int block, int sink, float scale, float null_score,
+                                             int form, int *status, cudaStream_t stream) {
+  return llm_attention_prefill_tc_sinks(q, q_stride, n_tokens, out, out_stride, kc, vc, n_pages, seq_start, seq_past, page_table, pt_stride,
+                                        n_seqs, max_q_len, n_heads, n_kv, d, d, page_size, window, block, sink, scale, null_score, nullptr,
+                                        form, status, stream);
 }
 
 LLM_EXPORT int llm_attention_prefill_tc(const void *q, long long q_stride, long long n_tokens, void *out,

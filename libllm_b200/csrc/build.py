@@ -50,6 +50,7 @@ FAMILIES: Dict[str, dict] = {
     "rope": dict(sources=["rope.cu"], headers=["common.cuh"]),
     "recurrent": dict(sources=["recurrent.cu"], headers=["common.cuh"]),
     "state_scan": dict(sources=["state_scan.cu"], headers=["common.cuh", "tc_common.cuh"]),
+    "selective_scan": dict(sources=["selective_scan.cu"], headers=["common.cuh"]),
     "attention_generic": dict(sources=["attention_generic.cu"], headers=["common.cuh"]),
     "attention_sigmoid": dict(sources=["attention_sigmoid.cu"], headers=["common.cuh", "mma_tiles.cuh", "tc_common.cuh"]),
     "latent": dict(sources=["latent.cu"], headers=["common.cuh"]),

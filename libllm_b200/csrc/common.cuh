@@ -189,6 +189,17 @@ __device__ __forceinline__ float softmax_norm_factor(float ref, float l, float n
   return a / (l * a + exp2f(null_log2 - top));
 }
 
+// A gated unit of a gate value g and an up value u, both bounded by `limit` (g above, u on both sides; plus infinity: no
+// bounds): g sigmoid(slope g) (u + shift).  {infinity, 1, 0} is silu(g) u, to the bit.
+struct GluShape {
+  float limit, slope, shift;
+};
+__device__ __forceinline__ float glu_value(float g, float u, const GluShape &s) {
+  g = fminf(g, s.limit);
+  u = fminf(fmaxf(u, -s.limit), s.limit);
+  return g / (1.f + expf(-s.slope * g)) * (u + s.shift);
+}
+
 // Sum over a block with a fixed order of additions: warps first, then the warp totals
 // in warp order.  The result does not depend on how many rows the launch has.
 template <int THREADS>

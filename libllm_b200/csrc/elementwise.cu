@@ -11,44 +11,81 @@
 LLM_DEFINE_LAST_ERROR(llm_elementwise_last_error)
 
 // ---------------------------------------------------------------- embedding
+// What a token brings besides its own row.  `ids` (null: not asked for) receives the tokens' numbers as they were
+// resolved, for later kernels of the step.  With `pairs` the row (previous * mul_prev + current * mul_cur) mod buckets of that
+// table [buckets + 1, hidden] is added, for a sequence's first token row `buckets`; the previous token of a step's first
+// token of a sequence is last[slot], which then becomes the sequence's last token of this step.
+struct TokenExtras {
+  int *ids;
+  const void *pairs;
+  long long buckets, mul_prev, mul_cur;
+  int *last;
+  const int *tok_seq, *tok_pos, *seq_start, *seq_slot;
+};
+
 template <typename T>
 __global__ void embedding_kernel(const T *__restrict__ table, const int *__restrict__ tokens,
                                  const int *__restrict__ fed_tokens, const int *__restrict__ fed_rows,
                                  float *__restrict__ out, int hidden, int vocab, const T *__restrict__ pos_table,
-                                 int pos_rows, const int *__restrict__ tok_pos) {
+                                 int pos_rows, const int *__restrict__ tok_pos, TokenExtras ex) {
   grid_dependents_launch();
   grid_dependency_wait();
   const int t = blockIdx.x;
   // A token either comes with the step (tokens[t]) or is the one the previous step sampled for
   // row fed_rows[t] of its batch, still on the device (fed_tokens): the host can then start this
   // step before it has read that token back.
-  int id = tokens[t];
-  if (fed_rows != nullptr && fed_rows[t] >= 0) id = fed_tokens[fed_rows[t]];
   // Token ids are checked on the host before they are uploaded; ids that the sampler
   // wrote on the device are below the vocabulary size by construction.  The clamp keeps
   // the read inside the table whatever happens.
-  id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+  auto resolve = [&](int i) {
+    int id = tokens[i];
+    if (fed_rows != nullptr && fed_rows[i] >= 0) id = fed_tokens[fed_rows[i]];
+    return id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+  };
+  const int id = resolve(t);
+  if (ex.ids && threadIdx.x == 0) ex.ids[t] = id;
   const T *row = table + (size_t)id * hidden;
   float *o = out + (size_t)t * hidden;
+  const T *pair = nullptr;
+  if (ex.pairs) {
+    const int b = ex.tok_seq[t], first = ex.seq_start[b], slot = ex.seq_slot[b];
+    long long r = ex.buckets;
+    if (ex.tok_pos[t] > 0) {
+      const long long prev = t > first ? resolve(t - 1) : ex.last[slot];
+      r = (prev * ex.mul_prev + (long long)id * ex.mul_cur) % ex.buckets;
+      if (r < 0) r += ex.buckets;
+    }
+    pair = (const T *)ex.pairs + (size_t)r * hidden;
+    if (t == first) {                                      // this CTA alone reads the sequence's last token, so it may move it on
+      __syncthreads();
+      if (threadIdx.x == 0) ex.last[slot] = resolve(ex.seq_start[b + 1] - 1);
+    }
+  }
   if (pos_table == nullptr) {
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = to_float(row[i]);
+    if (pair == nullptr) {
+      for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = to_float(row[i]);
+    } else {
+      for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = to_float(row[i]) + to_float(pair[i]);
+    }
     return;
   }
   // a learned vector per position is added to the token's row (32-bit sum of the two stored values)
   int p = tok_pos[t];
   p = p < 0 ? 0 : (p >= pos_rows ? pos_rows - 1 : p);      // the host refuses sequences longer than the table
   const T *prow = pos_table + (size_t)p * hidden;
-  for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = to_float(row[i]) + to_float(prow[i]);
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x)
+    o[i] = to_float(row[i]) + to_float(prow[i]) + (pair ? to_float(pair[i]) : 0.f);
 }
 
-// pos_table [pos_rows, hidden] in the table's type with the tokens' positions tok_pos, or null: no position vectors.
-LLM_EXPORT int llm_embedding_pos(int dtype, const void *table, const int *tokens, const int *fed_tokens,
-                                 const int *fed_rows, float *out, int n_tokens, int hidden, int vocab,
-                                 const void *pos_table, int pos_rows, const int *tok_pos, cudaStream_t stream) {
+static int launch_embedding(int dtype, const void *table, const int *tokens, const int *fed_tokens, const int *fed_rows, float *out,
+                            int n_tokens, int hidden, int vocab, const void *pos_table, int pos_rows, const int *tok_pos,
+                            const TokenExtras &ex, cudaStream_t stream) {
   if (n_tokens == 0) return LLM_OK;
   LLM_REQUIRE(n_tokens > 0 && hidden > 0 && vocab > 0, "embedding: bad sizes");
   LLM_REQUIRE(pos_table == nullptr || (pos_rows > 0 && tok_pos != nullptr), "embedding: position vectors come with the positions");
   LLM_REQUIRE((fed_tokens == nullptr) == (fed_rows == nullptr), "embedding: fed tokens come with their rows");
+  LLM_REQUIRE(ex.pairs == nullptr || (ex.buckets > 0 && ex.last && ex.tok_seq && ex.tok_pos && ex.seq_start && ex.seq_slot),
+              "embedding: rows of token pairs need the buckets, the last tokens and the step's layout");
   int threads = hidden >= 1024 ? 256 : 128;
   // A step's first kernel after its descriptor has arrived, and launched so that it starts only
   // when that is complete: the kernels after it read positions and page tables from the descriptor
@@ -58,14 +95,31 @@ LLM_EXPORT int llm_embedding_pos(int dtype, const void *table, const int *tokens
   // of the step before last.)
   if (dtype == LLM_F32)
     llm_launch_after(embedding_kernel<float>, n_tokens, threads, 0, stream, (const float *)table, tokens, fed_tokens, fed_rows, out, hidden, vocab,
-                     (const float *)pos_table, pos_rows, tok_pos);
+                     (const float *)pos_table, pos_rows, tok_pos, ex);
   else if (dtype == LLM_BF16)
     llm_launch_after(embedding_kernel<__nv_bfloat16>, n_tokens, threads, 0, stream, (const __nv_bfloat16 *)table, tokens, fed_tokens, fed_rows, out, hidden, vocab,
-                     (const __nv_bfloat16 *)pos_table, pos_rows, tok_pos);
+                     (const __nv_bfloat16 *)pos_table, pos_rows, tok_pos, ex);
   else
     LLM_FAIL("embedding: unknown dtype %d", dtype);
   LLM_CHECK_LAUNCH("embedding");
   return LLM_OK;
+}
+
+// pos_table [pos_rows, hidden] in the table's type with the tokens' positions tok_pos, or null: no position vectors.
+LLM_EXPORT int llm_embedding_pos(int dtype, const void *table, const int *tokens, const int *fed_tokens,
+                                 const int *fed_rows, float *out, int n_tokens, int hidden, int vocab,
+                                 const void *pos_table, int pos_rows, const int *tok_pos, cudaStream_t stream) {
+  return launch_embedding(dtype, table, tokens, fed_tokens, fed_rows, out, n_tokens, hidden, vocab, pos_table, pos_rows, tok_pos,
+                          TokenExtras{}, stream);
+}
+
+// The same with the tokens' numbers and the rows of token pairs (TokenExtras); `pairs` is in the table's type.
+LLM_EXPORT int llm_embedding_pairs(int dtype, const void *table, const int *tokens, const int *fed_tokens, const int *fed_rows, float *out,
+                                   int n_tokens, int hidden, int vocab, const void *pos_table, int pos_rows, int *ids, const void *pairs,
+                                   long long buckets, long long mul_prev, long long mul_cur, int *last, const int *tok_seq,
+                                   const int *tok_pos, const int *seq_start, const int *seq_slot, cudaStream_t stream) {
+  const TokenExtras ex{ids, pairs, buckets, mul_prev, mul_cur, last, tok_seq, tok_pos, seq_start, seq_slot};
+  return launch_embedding(dtype, table, tokens, fed_tokens, fed_rows, out, n_tokens, hidden, vocab, pos_table, pos_rows, tok_pos, ex, stream);
 }
 
 LLM_EXPORT int llm_embedding(int dtype, const void *table, const int *tokens, const int *fed_tokens,
@@ -322,6 +376,295 @@ LLM_EXPORT int llm_add_rmsnorm_scaled(float *resid, const void *delta, int delta
   if (delta_dtype == LLM_BF16 && out_dtype == LLM_F32)
     return launch_add_rmsnorm<__nv_bfloat16, float>(resid, delta, n_parts, part_stride, weight, eps, out, rows, n_rows, hidden, stream, col_scale, col_bias);
   LLM_FAIL("add_rmsnorm: unknown dtypes %d, %d", delta_dtype, out_dtype);
+}
+
+// ---------------------------------------------------------------- normed results added to the stream
+// A sublayer's result that is normed before it is added.  Its parts are partial results summed in order:
+//   y = sum of all parts + col_bias, or, with first_parts f > 0 (two results side by side),
+//   y = pair_scale * (unit(sum of parts 0 .. f-1) * w0 + unit(sum of the others) * w1);
+//   v = resid + unit(y) * post   (post null: resid + y),   unit(x) = x / sqrt(mean(x^2) + its eps).
+// The stream receives v (all rows), or with `rows` resid_out receives it for those rows alone (null: nobody does).  `out` (null:
+// none) is the next norm of v, unit(v) * weight, or with a null weight v itself in out's type.  Everything is 32-bit.
+struct ResultNorms {
+  int first_parts;
+  const float *w0, *w1;
+  float pair_eps, pair_scale;
+  const float *post;
+  float post_eps;
+};
+
+// block_sum for several values at once: one pass of barriers
+template <int THREADS, int N>
+__device__ __forceinline__ void block_sums(float (&v)[N], float *scratch /* N * (THREADS / 32 + 1) floats */) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  constexpr int W = THREADS / 32;
+#pragma unroll
+  for (int i = 0; i < N; ++i) v[i] = warp_sum(v[i]);
+  __syncthreads();
+  if (lane == 0)
+#pragma unroll
+    for (int i = 0; i < N; ++i) scratch[i * (W + 1) + warp] = v[i];
+  __syncthreads();
+  if (warp < N) {
+    float t = lane < W ? scratch[warp * (W + 1) + lane] : 0.f;
+    t = warp_sum(t);
+    if (lane == 0) scratch[warp * (W + 1) + W] = t;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < N; ++i) v[i] = scratch[i * (W + 1) + W];
+}
+
+// General form: rows of any width, two rows of `hidden` floats in shared memory.
+template <typename TO, int THREADS>
+__global__ void __launch_bounds__(THREADS)
+stream_norm_kernel(float *__restrict__ resid, const float *__restrict__ delta, int n_parts, size_t part_stride,
+                   const float *__restrict__ col_bias, ResultNorms rn, const float *__restrict__ weight, float eps, TO *__restrict__ out,
+                   const int *__restrict__ rows, float *__restrict__ resid_out, int hidden) {
+  extern __shared__ float norm_rows[];
+  float *ya = norm_rows, *yb = norm_rows + hidden;
+  __shared__ float scratch[2 * (THREADS / 32 + 1)];
+  grid_dependents_launch();
+  grid_dependency_wait();
+  const int i = blockIdx.x;
+  const size_t r = rows ? (size_t)rows[i] : (size_t)i;
+  const int split = rn.first_parts > 0 ? rn.first_parts : n_parts;
+  float ss[2] = {0.f, 0.f};
+  for (int c = threadIdx.x; c < hidden; c += THREADS) {
+    float a = 0.f, b = 0.f;
+    for (int p = 0; p < split; ++p) a += delta[p * part_stride + r * hidden + c];
+    for (int p = split; p < n_parts; ++p) b += delta[p * part_stride + r * hidden + c];
+    if (col_bias) a += col_bias[c];
+    ya[c] = a;
+    yb[c] = b;
+    ss[0] += a * a;
+    ss[1] += b * b;
+  }
+  float sy = 0.f;
+  if (rn.first_parts > 0) {
+    block_sums<THREADS, 2>(ss, scratch);
+    const float ia = rsqrtf(ss[0] / (float)hidden + rn.pair_eps), ib = rsqrtf(ss[1] / (float)hidden + rn.pair_eps);
+    for (int c = threadIdx.x; c < hidden; c += THREADS) {
+      const float y = rn.pair_scale * (ya[c] * ia * rn.w0[c] + yb[c] * ib * rn.w1[c]);
+      ya[c] = y;
+      sy += y * y;
+    }
+  } else {
+    sy = ss[0];
+  }
+  float inv = 1.f;
+  if (rn.post) inv = rsqrtf(block_sum<THREADS>(sy, scratch) / (float)hidden + rn.post_eps);
+  float *x = resid + r * hidden;
+  float sv = 0.f;
+  for (int c = threadIdx.x; c < hidden; c += THREADS) {
+    const float v = x[c] + (rn.post ? ya[c] * inv * rn.post[c] : ya[c]);
+    ya[c] = v;
+    if (!rows) x[c] = v;
+    else if (resid_out) resid_out[(size_t)i * hidden + c] = v;
+    sv += v * v;
+  }
+  if (!out) return;
+  TO *o = out + (size_t)i * hidden;
+  if (!weight) {
+    for (int c = threadIdx.x; c < hidden; c += THREADS) o[c] = from_float<TO>(ya[c]);
+    return;
+  }
+  const float nv = rsqrtf(block_sum<THREADS>(sv, scratch) / (float)hidden + eps);
+  for (int c = threadIdx.x; c < hidden; c += THREADS) o[c] = from_float<TO>(ya[c] * weight[c] * nv);
+}
+
+// Rows of a multiple of 4 channels, at most 4 * VPT * THREADS, in registers (wider rows take the general form); every load of a row (all parts, the stream, the
+// weights) is issued before the first sum.  PAIR: two results side by side.
+template <typename TO, int THREADS, int VPT, int MAXP, bool PAIR>
+__global__ void __launch_bounds__(THREADS)
+stream_norm_vec_kernel(float *__restrict__ resid, const float *__restrict__ delta, int n_parts, size_t part_stride,
+                       const float *__restrict__ col_bias, ResultNorms rn, const float *__restrict__ weight, float eps,
+                       TO *__restrict__ out, const int *__restrict__ rows, float *__restrict__ resid_out, int hidden) {
+  __shared__ float scratch[2 * (THREADS / 32 + 1)];
+  grid_dependents_launch();
+  const int n4 = hidden / 4, i = blockIdx.x;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 w[VPT], pw[VPT], wa[VPT], wb[VPT], cb[VPT], v[VPT], ya[VPT], yb[VPT];
+#pragma unroll
+  for (int j = 0; j < VPT; ++j) {                       // weights: written at load
+    const int c4 = threadIdx.x + j * THREADS;
+    const bool in = c4 < n4;
+    w[j] = in && out && weight ? ld4(weight + 4 * c4) : zero;
+    pw[j] = in && rn.post ? ld4(rn.post + 4 * c4) : zero;
+    if (PAIR) {
+      wa[j] = in ? ld4(rn.w0 + 4 * c4) : zero;
+      wb[j] = in ? ld4(rn.w1 + 4 * c4) : zero;
+    }
+    cb[j] = in && col_bias ? ld4(col_bias + 4 * c4) : zero;
+  }
+  grid_dependency_wait();
+  const size_t r = rows ? (size_t)rows[i] : (size_t)i;
+  float *x = resid + r * hidden;
+  const int split = PAIR ? rn.first_parts : n_parts;
+  float ss[2] = {0.f, 0.f};
+  auto add4 = [](float4 &a, const float4 &b) { a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w; };
+  auto sq4 = [](const float4 &a) { return a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w; };
+#pragma unroll
+  for (int j = 0; j < VPT; ++j) {
+    const int c4 = threadIdx.x + j * THREADS;
+    ya[j] = yb[j] = v[j] = zero;
+    if (c4 < n4) {
+      float4 d[MAXP];
+      v[j] = ld4(x + 4 * c4);
+#pragma unroll
+      for (int p = 0; p < MAXP; ++p)
+        if (p < n_parts) d[p] = ld4(delta + p * part_stride + r * hidden + 4 * c4);
+#pragma unroll
+      for (int p = 0; p < MAXP; ++p)
+        if (p < n_parts) {
+          if (PAIR && p >= split) add4(yb[j], d[p]);
+          else add4(ya[j], d[p]);
+        }
+      add4(ya[j], cb[j]);
+      ss[0] += sq4(ya[j]);
+      if (PAIR) ss[1] += sq4(yb[j]);
+    }
+  }
+  float sy = ss[0];
+  if (PAIR) {
+    block_sums<THREADS, 2>(ss, scratch);
+    const float ia = rsqrtf(ss[0] / (float)hidden + rn.pair_eps), ib = rsqrtf(ss[1] / (float)hidden + rn.pair_eps);
+    sy = 0.f;
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+      ya[j].x = rn.pair_scale * (ya[j].x * ia * wa[j].x + yb[j].x * ib * wb[j].x);
+      ya[j].y = rn.pair_scale * (ya[j].y * ia * wa[j].y + yb[j].y * ib * wb[j].y);
+      ya[j].z = rn.pair_scale * (ya[j].z * ia * wa[j].z + yb[j].z * ib * wb[j].z);
+      ya[j].w = rn.pair_scale * (ya[j].w * ia * wa[j].w + yb[j].w * ib * wb[j].w);
+      sy += sq4(ya[j]);
+    }
+  }
+  if (rn.post) {
+    const float inv = rsqrtf(block_sum<THREADS>(sy, scratch) / (float)hidden + rn.post_eps);
+#pragma unroll
+    for (int j = 0; j < VPT; ++j)
+      ya[j] = make_float4(ya[j].x * inv * pw[j].x, ya[j].y * inv * pw[j].y, ya[j].z * inv * pw[j].z, ya[j].w * inv * pw[j].w);
+  }
+  float sv = 0.f;
+#pragma unroll
+  for (int j = 0; j < VPT; ++j) {
+    const int c4 = threadIdx.x + j * THREADS;
+    add4(v[j], ya[j]);
+    if (c4 < n4) {
+      if (!rows) st4(x + 4 * c4, v[j]);
+      else if (resid_out) st4(resid_out + (size_t)i * hidden + 4 * c4, v[j]);
+      sv += sq4(v[j]);
+    }
+  }
+  if (!out) return;
+  float nv = 1.f;
+  if (weight) nv = rsqrtf(block_sum<THREADS>(sv, scratch) / (float)hidden + eps);
+  TO *o = out + (size_t)i * hidden;
+#pragma unroll
+  for (int j = 0; j < VPT; ++j) {
+    const int c4 = threadIdx.x + j * THREADS;
+    if (c4 < n4)
+      st4(o + 4 * c4, weight ? make_float4(v[j].x * w[j].x * nv, v[j].y * w[j].y * nv, v[j].z * w[j].z * nv, v[j].w * w[j].w * nv) : v[j]);
+  }
+}
+
+template <typename TO>
+static int launch_stream_norm(float *resid, const float *delta, int n_parts, size_t part_stride, const float *col_bias, const ResultNorms &rn,
+                              const float *weight, float eps, TO *out, const int *rows, int n_rows, float *resid_out, int hidden,
+                              cudaStream_t stream) {
+  auto ok16 = [](const void *p) { return (uintptr_t)p % 16 == 0; };
+  const bool aligned = hidden % 4 == 0 && part_stride % 4 == 0 && ok16(resid) && ok16(delta) && ok16(col_bias) && ok16(weight) && ok16(out) &&
+                       ok16(resid_out) && ok16(rn.w0) && ok16(rn.w1) && ok16(rn.post);
+  if (aligned && hidden <= 4096 && n_parts <= 16) {
+#define SN_GO3(T_, V_, MAXP, PAIR)                                                                                                  \
+  llm_launch(stream_norm_vec_kernel<TO, T_, V_, MAXP, PAIR>, n_rows, T_, 0, stream, resid, delta, n_parts, part_stride, col_bias, rn, weight, \
+             eps, out, rows, resid_out, hidden)
+#define SN_GO2(T_, V_, MAXP)                              \
+  do {                                                    \
+    if (rn.first_parts > 0) SN_GO3(T_, V_, MAXP, true);   \
+    else SN_GO3(T_, V_, MAXP, false);                     \
+  } while (0)
+#define SN_GO(MAXP)                                       \
+  do {                                                    \
+    if (hidden <= 2048) SN_GO2(512, 1, MAXP);             \
+    else SN_GO2(512, 2, MAXP);                            \
+  } while (0)
+    if (n_parts <= 2) SN_GO(2);
+    else if (n_parts <= 8) SN_GO(8);
+    else SN_GO(16);
+#undef SN_GO
+#undef SN_GO2
+#undef SN_GO3
+    LLM_CHECK_LAUNCH("stream_norm");
+    return LLM_OK;
+  }
+  constexpr int THREADS = 256;
+  const size_t smem = (size_t)hidden * 2 * sizeof(float);
+  LLM_REQUIRE(smem <= 200 * 1024, "stream_norm: a row of %d values does not fit shared memory", hidden);
+  auto kern = stream_norm_kernel<TO, THREADS>;
+  LLM_CHECK_CUDA(llm_allow_smem(kern, smem), "stream_norm attribute");
+  llm_launch(kern, n_rows, THREADS, smem, stream, resid, delta, n_parts, part_stride, col_bias, rn, weight, eps, out, rows, resid_out, hidden);
+  LLM_CHECK_LAUNCH("stream_norm");
+  return LLM_OK;
+}
+
+LLM_EXPORT int llm_stream_norm(float *resid, const float *delta, int n_parts, long long part_stride, const float *col_bias, int first_parts,
+                               const float *w0, const float *w1, float pair_eps, float pair_scale, const float *post, float post_eps,
+                               const float *weight, float eps, void *out, int out_dtype, const int *rows, int n_rows, float *resid_out,
+                               int hidden, cudaStream_t stream) {
+  if (n_rows == 0) return LLM_OK;
+  LLM_REQUIRE(n_rows > 0 && hidden > 0 && n_parts >= 0 && first_parts >= 0 && first_parts <= n_parts, "stream_norm: bad sizes");
+  LLM_REQUIRE(first_parts == 0 || (first_parts < n_parts && w0 && w1), "stream_norm: two results need their parts and weights");
+  LLM_REQUIRE(n_parts > 0 || !post, "stream_norm: nothing to norm");
+  if (!delta) n_parts = 0;
+  const ResultNorms rn{first_parts, w0, w1, pair_eps, pair_scale, post, post_eps};
+  if (out_dtype == LLM_F32)
+    return launch_stream_norm<float>(resid, delta, n_parts, (size_t)part_stride, col_bias, rn, weight, eps, (float *)out, rows, n_rows,
+                                     resid_out, hidden, stream);
+  if (out_dtype == LLM_BF16)
+    return launch_stream_norm<__nv_bfloat16>(resid, delta, n_parts, (size_t)part_stride, col_bias, rn, weight, eps, (__nv_bfloat16 *)out, rows,
+                                             n_rows, resid_out, hidden, stream);
+  LLM_FAIL("stream_norm: unknown dtype %d", out_dtype);
+}
+
+// ---------------------------------------------------------------- a token's own vector behind a gate
+// out[t, c] = gelu_tanh(z[t, c]) * table[ids[row], offset + c] for c < dim, nought up to out's width; row = rows ? rows[t] : t.
+// z 32-bit, table [vocab, table_width] and out in the engine's type.
+template <typename T>
+__global__ void __launch_bounds__(256)
+token_gate_kernel(const float *__restrict__ z, long long ldz, const T *__restrict__ table, long long table_width, int offset, int dim,
+                  const int *__restrict__ ids, const int *__restrict__ rows, T *__restrict__ out, int ldo, size_t total) {
+  grid_dependents_launch();
+  grid_dependency_wait();
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = idx / ldo;
+    const int c = (int)(idx - t * ldo);
+    float y = 0.f;
+    if (c < dim) {
+      const float g = z[t * ldz + c];
+      const float a = 0.5f * g * (1.f + tanhf(0.79788456080286536f * (g + 0.044715f * g * g * g)));
+      y = a * to_float(table[(size_t)ids[rows ? rows[t] : (int)t] * table_width + offset + c]);
+    }
+    out[idx] = from_float<T>(y);
+  }
+}
+
+LLM_EXPORT int llm_token_gate(int dtype, const float *z, long long ldz, const void *table, long long table_width, int offset, int dim,
+                              const int *ids, const int *rows, void *out, int ldo, int n_rows, cudaStream_t stream) {
+  if (n_rows == 0) return LLM_OK;
+  LLM_REQUIRE(n_rows > 0 && dim > 0 && ldo >= dim && offset >= 0 && offset + (long long)dim <= table_width && ids && table, "token_gate: bad sizes");
+  const size_t total = (size_t)n_rows * ldo;
+  size_t blocks = (total + 255) / 256;
+  if (blocks > (size_t)sm_count() * 16) blocks = (size_t)sm_count() * 16;
+  if (dtype == LLM_F32)
+    llm_launch(token_gate_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, z, ldz, (const float *)table, table_width, offset, dim,
+               ids, rows, (float *)out, ldo, total);
+  else if (dtype == LLM_BF16)
+    llm_launch(token_gate_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(256), 0, stream, z, ldz, (const __nv_bfloat16 *)table, table_width,
+               offset, dim, ids, rows, (__nv_bfloat16 *)out, ldo, total);
+  else LLM_FAIL("token_gate: unknown dtype %d", dtype);
+  LLM_CHECK_LAUNCH("token_gate");
+  return LLM_OK;
 }
 
 // ---------------------------------------------------------------- add + layer norm

@@ -17,7 +17,7 @@
 // 90 KB (few tokens) to 200 KB (prompts) of loads are in flight per SM, which is what a stream from
 // HBM needs.
 //
-// SwiGLU: W is the stacked gate|up matrix [2I, K].  A tile holds gate rows f..f+63 in its lanes
+// SwiGLU, or any gated unit of GluShape: W is the stacked gate|up matrix [2I, K].  A tile holds gate rows f..f+63 in its lanes
 // 0-63 and up rows I+f..I+f+63 in lanes 64-127; the epilogue warps of the upper half hand their
 // values over through shared memory and the lower half stores silu(gate) * up: the stacked
 // product never reaches memory (the reference runs a separate launch, src/flint/cuda/swiglu.cu:29-59,
@@ -66,7 +66,7 @@ template <int TN, int SW, typename TO>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                TO *__restrict__ out, long long ldo, int M, int n_out, int K, int row_tiles, int tok_tiles,
-               int k_parts, int kb_per_part, long long part_stride, int group_tiles, int group_rows, int *status) {
+               int k_parts, int kb_per_part, long long part_stride, int group_tiles, int group_rows, GluShape glu, int *status) {
   using S = TcShape<TN, SW>;
   constexpr bool SWIGLU = SW == 1;                      // the interleaved tile with the hand-over
   constexpr int STAGES = S::STAGES;
@@ -265,7 +265,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
           for (int i = 0; i < 16; ++i) {
             const int tok = tok0 + c0 + i;
             const float g = v[i];
-            if (f < n_out && tok < M) o[(size_t)tok * ldo + f] = from_float<TO>(g / (1.f + expf(-g)) * u[i]);
+            if (f < n_out && tok < M) o[(size_t)tok * ldo + f] = from_float<TO>(glu_value(g, u[i], glu));
           }
         } else if (SWIGLU) {
           // The upper two warps (up rows) hand their values to the lower two (gate rows of the
@@ -286,7 +286,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
               const int tok = tok0 + c0 + i;
               const float up = xch[row_in_tile * 17 + i];
               const float g = v[i];
-              if (f < n_out && tok < M) o[(size_t)tok * ldo + f] = from_float<TO>(g / (1.f + expf(-g)) * up);
+              if (f < n_out && tok < M) o[(size_t)tok * ldo + f] = from_float<TO>(glu_value(g, up, glu));
             }
             __syncwarp();
             if (lane == 0) mbar_arrive(bar_xempty);
@@ -320,7 +320,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 
 template <int TN, int SW, typename TO>
 int launch_tc(const void *x, long long ldx, const void *W, void *out, long long ldo, int M, int N, int K, int k_parts,
-              long long part_stride, int *status, cudaStream_t stream, int n_groups = 1, int group_n = 0) {
+              long long part_stride, const GluShape &glu, int *status, cudaStream_t stream, int n_groups = 1, int group_n = 0) {
   using S = TcShape<TN, SW>;
   const int n_out = SW != 0 ? N / 2 : N;
   const int rows_out = SW == 1 ? 64 : 128;
@@ -341,15 +341,15 @@ int launch_tc(const void *x, long long ldx, const void *W, void *out, long long 
   const int grid = (int)(tiles < sm_count() ? tiles : sm_count());
   LLM_CHECK_CUDA(llm_launch(kern, dim3(grid), dim3(TC_THREADS), S::SMEM, stream, map_w, map_x, (TO *)out, ldo, M, n_out, K,
                             row_tiles, tok_tiles, k_parts, kb_per_part, part_stride, n_groups > 1 ? group_n / 128 : row_tiles,
-                            n_groups > 1 ? M : 0, status),
+                            n_groups > 1 ? M : 0, glu, status),
                  "gemm_tc launch");
   return LLM_OK;
 }
 
 template <bool SWIGLU, typename TO>
 int dispatch_tc(const void *x, long long ldx, const void *W, void *out, long long ldo, int M, int N, int K, int k_parts,
-                long long part_stride, int *status, cudaStream_t stream) {
-#define TC_GO(TN, SW) return launch_tc<TN, SW, TO>(x, ldx, W, out, ldo, M, N, K, k_parts, part_stride, status, stream)
+                long long part_stride, const GluShape &glu, int *status, cudaStream_t stream) {
+#define TC_GO(TN, SW) return launch_tc<TN, SW, TO>(x, ldx, W, out, ldo, M, N, K, k_parts, part_stride, glu, status, stream)
   if (SWIGLU) {
     if (M <= 16) TC_GO(16, 1);
     if (M <= 32) TC_GO(32, 1);
@@ -390,10 +390,11 @@ LLM_EXPORT int llm_gemm_tc_suggest_parts(int M, int N, int K) {
 // x [M, K] bfloat16 (row stride ldx elements), W [N, K] bfloat16 contiguous, out [M, N] of out_dtype,
 // or [M, N/2] with swiglu (W = stacked gate|up).  With k_parts > 1 (plain product, 32-bit out) part p
 // writes its share of K to out + p * part_stride.  `status` (device int, may be null) receives a
-// non-zero code if a wait inside the kernel ran out of time.
-LLM_EXPORT int llm_gemm_tc(const void *x, long long ldx, const void *W, void *out, long long ldo, int out_dtype,
-                           int M, int N, int K, int swiglu, int k_parts, long long part_stride, int *status,
-                           cudaStream_t stream) {
+// non-zero code if a wait inside the kernel ran out of time.  With swiglu the gated unit is (limit, slope, shift)'s (GluShape).
+LLM_EXPORT int llm_gemm_tc_glu(const void *x, long long ldx, const void *W, void *out, long long ldo, int out_dtype,
+                               int M, int N, int K, int swiglu, float limit, float slope, float shift, int k_parts, long long part_stride,
+                               int *status, cudaStream_t stream) {
+  const GluShape glu{limit, slope, shift};
   if (M == 0 || N == 0) return LLM_OK;
   LLM_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_tc: bad sizes %d x %d x %d", M, N, K);
   LLM_REQUIRE(K % 8 == 0 && ldx % 8 == 0, "gemm_tc: K = %d and the row stride %lld must be multiples of 8 (rows start on 16 bytes)", K, ldx);
@@ -402,13 +403,19 @@ LLM_EXPORT int llm_gemm_tc(const void *x, long long ldx, const void *W, void *ou
   LLM_REQUIRE(k_parts >= 1 && k_parts <= 64 && (k_parts == 1 || (!swiglu && out_dtype == LLM_F32)),
               "gemm_tc: parts of K need a plain product with 32-bit output");
   if (swiglu) {
-    if (out_dtype == LLM_BF16) return dispatch_tc<true, __nv_bfloat16>(x, ldx, W, out, ldo, M, N, K, k_parts, part_stride, status, stream);
-    if (out_dtype == LLM_F32) return dispatch_tc<true, float>(x, ldx, W, out, ldo, M, N, K, k_parts, part_stride, status, stream);
+    if (out_dtype == LLM_BF16) return dispatch_tc<true, __nv_bfloat16>(x, ldx, W, out, ldo, M, N, K, k_parts, part_stride, glu, status, stream);
+    if (out_dtype == LLM_F32) return dispatch_tc<true, float>(x, ldx, W, out, ldo, M, N, K, k_parts, part_stride, glu, status, stream);
   } else {
-    if (out_dtype == LLM_BF16) return dispatch_tc<false, __nv_bfloat16>(x, ldx, W, out, ldo, M, N, K, k_parts, part_stride, status, stream);
-    if (out_dtype == LLM_F32) return dispatch_tc<false, float>(x, ldx, W, out, ldo, M, N, K, k_parts, part_stride, status, stream);
+    if (out_dtype == LLM_BF16) return dispatch_tc<false, __nv_bfloat16>(x, ldx, W, out, ldo, M, N, K, k_parts, part_stride, glu, status, stream);
+    if (out_dtype == LLM_F32) return dispatch_tc<false, float>(x, ldx, W, out, ldo, M, N, K, k_parts, part_stride, glu, status, stream);
   }
   LLM_FAIL("gemm_tc: unknown output dtype %d", out_dtype);
+}
+
+LLM_EXPORT int llm_gemm_tc(const void *x, long long ldx, const void *W, void *out, long long ldo, int out_dtype,
+                           int M, int N, int K, int swiglu, int k_parts, long long part_stride, int *status,
+                           cudaStream_t stream) {
+  return llm_gemm_tc_glu(x, ldx, W, out, ldo, out_dtype, M, N, K, swiglu, __builtin_huge_valf(), 1.f, 0.f, k_parts, part_stride, status, stream);
 }
 
 // Several products of as many inputs in one launch: x [n_groups * M, K] (input g's rows from g * M on), W the matrices one
@@ -421,7 +428,7 @@ LLM_EXPORT int llm_gemm_tc_grouped(const void *x, long long ldx, const void *W, 
   LLM_REQUIRE(n_groups == 1 || (group_n > 0 && group_n % 128 == 0 && (long long)(n_groups - 1) * group_n < N && (long long)n_groups * group_n >= N),
               "gemm_tc_grouped: %d matrices of %d rows do not make %d", n_groups, group_n, N);
   LLM_REQUIRE(K % 8 == 0 && ldx % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)W % 16 == 0, "gemm_tc_grouped: rows must start on 16 bytes");
-#define TC_GROUP(TN) return launch_tc<TN, 0, float>(x, ldx, W, out, ldo, M, N, K, 1, 0, status, stream, n_groups, group_n)
+#define TC_GROUP(TN) return launch_tc<TN, 0, float>(x, ldx, W, out, ldo, M, N, K, 1, 0, GluShape{}, status, stream, n_groups, group_n)
   if (M <= 16) TC_GROUP(16);
   if (M <= 32) TC_GROUP(32);
   if (M <= 64) TC_GROUP(64);

@@ -159,8 +159,22 @@ void embedding(DType dt, const void *table, const int *tokens, const int *fed_to
   LLM_CALL("elementwise", llm_embedding_pos, code(dt), table, tokens, fed_rows ? fed_tokens : nullptr, fed_rows, out, n, hidden, vocab,
            pos_table, pos_rows, tok_pos, s);
 }
+LLM_KERNEL("elementwise", llm_embedding_pairs, int, const void *, const int *, const int *, const int *, float *, int, int, int, const void *,
+           int, int *, const void *, long long, long long, long long, int *, const int *, const int *, const int *, const int *, cudaStream_t)
+void embedding_pairs(DType dt, const void *table, const int *tokens, const int *fed_tokens, const int *fed_rows, float *out, int n, int hidden,
+                     int vocab, cudaStream_t s, const void *pos_table, int pos_rows, const int *tok_pos, int *ids, const TokenPairs &p,
+                     const int *tok_seq, const int *seq_start, const int *seq_slot) {
+  LLM_CALL("elementwise", llm_embedding_pairs, code(dt), table, tokens, fed_rows ? fed_tokens : nullptr, fed_rows, out, n, hidden, vocab,
+           pos_table, pos_rows, ids, p.table, p.buckets, p.mul_prev, p.mul_cur, p.last, tok_seq, tok_pos, seq_start, seq_slot, s);
+}
+// passes over the stream that know nothing of results with norms of their own
+static void refuse_normed(const Act *delta, const char *what) {
+  if (delta && delta->data && delta->normed())
+    LLM_THROW(Unsupported, "%s: a pending result with a norm of its own is taken by the RMS norm's pass only", what);
+}
 void add_layernorm(float *resid, const Act *delta, const float *weight, const float *bias, float eps, void *out, DType out_dtype,
                    const int *rows, int n_rows, int hidden, cudaStream_t s) {
+  refuse_normed(delta, "add_layernorm");
   if (delta && (delta->col_scale || delta->col_bias))
     LLM_THROW(Unsupported, "add_layernorm: a pending addition with a scale or a bias over its columns is taken by the RMS norm's pass only");
   const bool has = delta && delta->data;
@@ -180,15 +194,40 @@ void hyper_mix_norm(const float *x_in, long long in_stride, float *x_out, long l
                     const float *mix, const float *outw, const float *inw, const float *norm_w, float eps, void *out, DType out_dtype,
                     const int *rows, int n_rows, int hidden, cudaStream_t s) {
   const bool has = delta && delta->data;
+  refuse_normed(delta, "hyper_mix_norm");
   if (has && delta->dtype != DType::F32) LLM_THROW(InvalidArg, "hyper_mix_norm: a pending result is 32-bit");
   LLM_CALL("elementwise", llm_hyper_mix_norm, x_in, in_stride, x_out, out_stride, n_streams, has ? (const float *)delta->data : nullptr,
            has ? delta->parts : 0, has ? (long long)delta->part_stride : 0, has ? delta->col_scale : nullptr,
            has ? delta->col_bias : nullptr, mix, outw, inw, norm_w, eps, out, code(out_dtype), rows, n_rows, hidden, s);
 }
 void add_scalar(float *x, long long n, float value, cudaStream_t s) { LLM_CALL("elementwise", llm_add_scalar, x, n, value, s); }
+LLM_KERNEL("elementwise", llm_stream_norm, float *, const float *, int, long long, const float *, int, const float *, const float *, float, float,
+           const float *, float, const float *, float, void *, int, const int *, int, float *, int, cudaStream_t)
+static void stream_norm(float *resid, const Act *delta, const float *weight, float eps, void *out, DType out_dtype, const int *rows, int n_rows,
+                        float *resid_out, int hidden, cudaStream_t s) {
+  Act none;
+  const Act &d = delta && delta->data ? *delta : none;
+  if (d.data && (d.dtype != DType::F32 || d.ld != hidden || d.cols != hidden || d.col_scale || (d.col_bias && d.first_parts > 0)))
+    LLM_THROW(Unsupported, "stream_norm: a result with a norm of its own is dense 32-bit rows without a scale (and, of two, without a bias)");
+  LLM_CALL("elementwise", llm_stream_norm, resid, (const float *)d.data, d.data ? d.parts : 0, d.data ? (long long)d.part_stride : 0,
+           d.data ? d.col_bias : nullptr, d.data ? d.first_parts : 0, d.pair_w[0], d.pair_w[1], d.pair_eps, d.pair_scale, d.post, d.post_eps,
+           weight, eps, out, code(out_dtype), rows, n_rows, resid_out, hidden, s);
+}
+void stream_cast(float *resid, const Act *delta, void *out, DType out_dtype, int n_rows, int hidden, cudaStream_t s) {
+  stream_norm(resid, delta, nullptr, 0.f, out, out_dtype, nullptr, n_rows, nullptr, hidden, s);
+}
+LLM_KERNEL("elementwise", llm_token_gate, int, const float *, long long, const void *, long long, int, int, const int *, const int *, void *, int,
+           int, cudaStream_t)
+void token_gate(const Act &z, const void *table, long long table_width, int offset, int dim, const int *ids, const int *rows, const Act &out,
+                cudaStream_t s) {
+  if (z.dtype != DType::F32 || out.ld != out.cols) LLM_THROW(InvalidArg, "token_gate: 32-bit logits, a dense result");
+  LLM_CALL("elementwise", llm_token_gate, code(out.dtype), (const float *)z.data, (long long)z.ld, table, table_width, offset, dim, ids, rows,
+           out.data, (int)out.cols, (int)out.rows, s);
+}
 void add_rmsnorm(float *resid, const Act *delta, const float *weight, float eps, void *out, DType out_dtype, const int *rows,
                  int n_rows, int hidden, cudaStream_t s) {
   const bool has = delta && delta->data;
+  if (has && delta->normed()) return stream_norm(resid, delta, weight, eps, out, out_dtype, rows, n_rows, nullptr, hidden, s);
   LLM_CALL("elementwise", llm_add_rmsnorm_scaled, resid, has ? delta->data : nullptr, has ? code(delta->dtype) : 0,
            has ? delta->parts : 0, has ? (long long)delta->part_stride : 0, weight, eps, out, code(out_dtype), rows, n_rows,
            hidden, has ? delta->col_scale : nullptr, has ? delta->col_bias : nullptr, s);
@@ -197,6 +236,7 @@ LLM_KERNEL("elementwise", llm_add_layernorm_conv, float *, const void *, int, in
            int, int, int, const float *, void *, const int *, int, cudaStream_t)
 void add_layernorm_conv(float *resid, const Act *delta, const float *weight, const float *bias, float eps, void *out, DType out_dtype,
                         int n_rows, int hidden, const float *conv_w, void *state, const int *seq_slot, int taps, cudaStream_t s) {
+  refuse_normed(delta, "add_layernorm_conv");
   if (delta && (delta->col_scale || delta->col_bias))
     LLM_THROW(Unsupported, "add_layernorm_conv: a pending addition with a scale or a bias over its columns is taken by the RMS norm's pass only");
   const bool has = delta && delta->data;
@@ -206,6 +246,8 @@ void add_layernorm_conv(float *resid, const Act *delta, const float *weight, con
 }
 void gather_rows_add(const float *resid, const Act *delta, const int *rows, int n_rows, float *out, int hidden, cudaStream_t s) {
   const bool has = delta && delta->data;
+  if (has && delta->normed())            // the stream itself stays as it is
+    return stream_norm(const_cast<float *>(resid), delta, nullptr, 0.f, nullptr, DType::F32, rows, n_rows, out, hidden, s);
   LLM_CALL("elementwise", llm_gather_rows_add_scaled, resid, has ? delta->data : nullptr, has ? code(delta->dtype) : 0,
            has ? delta->parts : 0, has ? (long long)delta->part_stride : 0, rows, n_rows, out, hidden, has ? delta->col_scale : nullptr,
            has ? delta->col_bias : nullptr, s);
@@ -217,6 +259,7 @@ void clamped_glu(const Act &gu, const float *bias, const Act &out, float limit, 
 LLM_KERNEL("elementwise", llm_concat_stream, const float *, const float *, int, long long, const float *, void *, int, int, int,
            cudaStream_t)
 void concat_stream(const float *resid, const Act *delta, const float *other, const Act &out, int hidden, cudaStream_t s) {
+  refuse_normed(delta, "concat_stream");
   if (delta && (delta->col_scale || delta->col_bias))
     LLM_THROW(Unsupported, "concat_stream: a pending addition with a scale or a bias over its columns is taken by the RMS norm's pass only");
   const bool has = delta && delta->data;
@@ -230,6 +273,7 @@ void swiglu(const Act &gu, void *out, DType out_dtype, cudaStream_t s) {
 LLM_KERNEL("elementwise", llm_stream_add, float *, const float *, int, long long, const float *, const float *, const float *, const float *,
            int, int, cudaStream_t)
 void stream_add(float *resid, const Act *delta, const float *other, const float *vec, int n_rows, int hidden, cudaStream_t s) {
+  refuse_normed(delta, "stream_add");
   if (delta && (delta->dtype != DType::F32 || delta->ld != hidden)) LLM_THROW(InvalidArg, "stream_add: the addition must be dense 32-bit rows");
   LLM_CALL("elementwise", llm_stream_add, resid, delta ? (const float *)delta->data : nullptr, delta ? delta->parts : 0,
            delta ? (long long)delta->part_stride : 0, delta ? delta->col_scale : nullptr, delta ? delta->col_bias : nullptr, other, vec,
@@ -246,8 +290,8 @@ void random_fill(void *out, DType dtype, long long n, unsigned long long seed, i
 // ---------------------------------------------------------------- products
 LLM_KERNEL("gemm_plain", llm_gemm_plain, int, int, const void *, long long, const void *, long long, const float *, void *,
            long long, int, int, int, cudaStream_t)
-LLM_KERNEL("gemm_tc", llm_gemm_tc, const void *, long long, const void *, void *, long long, int, int, int, int, int, int,
-           long long, int *, cudaStream_t)
+LLM_KERNEL("gemm_tc", llm_gemm_tc_glu, const void *, long long, const void *, void *, long long, int, int, int, int, int, float, float, float,
+           int, long long, int *, cudaStream_t)
 LLM_KERNEL("gemv", llm_gemv_bf16, const void *, long long, const void *, void *, long long, int, int, int, int, int, int,
            long long, cudaStream_t)
 
@@ -263,10 +307,10 @@ int gemm_tc_suggest_parts(int M, int N, int K) {
   static auto f = resolve<int (*)(int, int, int)>("gemm_tc", "llm_gemm_tc_suggest_parts");
   return f(M, N, K);
 }
-void gemm_tc(const Act &x, const Weight &w, const Act &out, bool swiglu, int *status, cudaStream_t s) {
-  LLM_CALL("gemm_tc", llm_gemm_tc, x.data, (long long)(x.rows > 1 ? x.ld : x.cols), w.data(), out.data,
+void gemm_tc(const Act &x, const Weight &w, const Act &out, bool swiglu, int *status, cudaStream_t s, const Glu &glu) {
+  LLM_CALL("gemm_tc", llm_gemm_tc_glu, x.data, (long long)(x.rows > 1 ? x.ld : x.cols), w.data(), out.data,
            (long long)(x.rows > 1 ? out.ld : out.cols), code(out.dtype), (int)x.rows, (int)w.rows, (int)x.cols, swiglu ? 1 : 0,
-           out.parts, (long long)out.part_stride, status, s);
+           glu.limit, glu.slope, glu.shift, out.parts, (long long)out.part_stride, status, s);
 }
 LLM_KERNEL("gemm_tc", llm_gemm_tc_grouped, const void *, long long, const void *, float *, long long, int, int, int, int, int, int *,
            cudaStream_t)
@@ -368,32 +412,32 @@ void rope_pairs_place(const Act &qkv, const Act &q_out, int n_heads, int n_kv, i
 }
 
 // ---------------------------------------------------------------- attention
-LLM_KERNEL("attention_generic", llm_attention_generic_ld, int, const void *, long long, void *, long long, const void *, const void *,
+LLM_KERNEL("attention_generic", llm_attention_generic_sinks, int, const void *, long long, void *, long long, const void *, const void *,
            const int *, const int *, const int *, int, int, int, int, int, int, int, int, int, int, int, float, const float *, long long,
-           float, cudaStream_t)
-LLM_KERNEL("attention_decode", llm_attention_decode_null, const void *, long long, void *, long long, const void *, const void *,
+           float, const float *, cudaStream_t)
+LLM_KERNEL("attention_decode", llm_attention_decode_sinks, const void *, long long, void *, long long, const void *, const void *,
            const int *, const int *, int, int, int, int, int, int, int, int, int, int, int, float, float *, float *, const float *,
-           long long, int, float, cudaStream_t)
-LLM_KERNEL("attention_decode_tc", llm_attention_decode_tc, const float *, long long, int, long long, const float *, int, int,
-           const int *, const int *, int, void *, void *, int, int, int, int, int, int, int, int, int, int, int, float, float *,
-           float *, int *, void *, long long, cudaStream_t)
-LLM_KERNEL("attention_prefill", llm_attention_prefill_null, const void *, long long, void *, long long, const void *, const void *,
-           const int *, const int *, const int *, int, int, int, int, int, int, int, int, int, int, float, float, cudaStream_t)
+           long long, int, float, const float *, cudaStream_t)
+LLM_KERNEL("attention_decode_tc", llm_attention_decode_tc_sinks, const float *, long long, int, long long, const float *, int, int,
+           const int *, const int *, int, void *, void *, int, int, int, int, int, int, int, int, int, int, int, int, float, const float *,
+           const float *, float *, float *, int *, void *, long long, cudaStream_t)
+LLM_KERNEL("attention_prefill", llm_attention_prefill_sinks, const void *, long long, void *, long long, const void *, const void *,
+           const int *, const int *, const int *, int, int, int, int, int, int, int, int, int, int, float, float, const float *, cudaStream_t)
 LLM_KERNEL("elementwise", llm_head_gate, void *, int, long long, const float *, long long, int, int, int, cudaStream_t)
 void head_gate(const Act &out, const float *gate, long long gate_stride, int n_heads, int dv, cudaStream_t s) {
   LLM_CALL("elementwise", llm_head_gate, out.data, code(out.dtype), (long long)out.ld, gate, gate_stride, (int)out.rows, n_heads, dv, s);
 }
-LLM_KERNEL("attention_prefill_tc", llm_attention_prefill_tc_null, const void *, long long, long long, void *, long long, const void *,
-           const void *, long long, const int *, const int *, const int *, int, int, int, int, int, int, int, int, int, int, float, float,
-           int, int *, cudaStream_t)
+LLM_KERNEL("attention_prefill_tc", llm_attention_prefill_tc_sinks, const void *, long long, long long, void *, long long, const void *,
+           const void *, long long, const int *, const int *, const int *, int, int, int, int, int, int, int, int, int, int, int, float, float,
+           const float *, int, int *, cudaStream_t)
 
 void attention_generic(const Act &q, const Act &out, const void *kc, const void *vc, const int *tok_seq, const int *tok_pos,
                        const int *page_table, int pt_stride, int n_heads, int n_kv, int d, int dv, int page_size, int window,
                        int block, float scale, const float *gate, long long gate_stride, cudaStream_t s, int sink, int v_ld,
-                       float null_score) {
-  LLM_CALL("attention_generic", llm_attention_generic_ld, code(q.dtype), q.data, (long long)q.ld, out.data, (long long)out.ld, kc, vc,
+                       float null_score, const float *null_scores) {
+  LLM_CALL("attention_generic", llm_attention_generic_sinks, code(q.dtype), q.data, (long long)q.ld, out.data, (long long)out.ld, kc, vc,
            tok_seq, tok_pos, page_table, pt_stride, (int)q.rows, n_heads, n_kv, d, dv, v_ld > 0 ? v_ld : dv, page_size, window, block,
-           sink, scale, gate, gate_stride, null_score, s);
+           sink, scale, gate, gate_stride, null_score, null_scores, s);
 }
 
 // ---------------------------------------------------------------- latent attention
@@ -401,7 +445,8 @@ LLM_KERNEL("latent", llm_latent_place, int, const float *, long long, int, int, 
            const float *, float, const float *, int, int, const int *, const int *, const int *, int, void *, int, cudaStream_t)
 LLM_KERNEL("latent", llm_latent_absorb, int, const float *, long long, const void *, void *, long long, int, int, int, int, int,
            const float *, int, int, const int *, cudaStream_t)
-LLM_KERNEL("latent", llm_latent_expand, int, const void *, long long, const void *, void *, long long, int, int, int, int, cudaStream_t)
+LLM_KERNEL("latent", llm_latent_expand_gated, int, const void *, long long, const void *, void *, long long, int, int, int, int, const float *,
+           long long, cudaStream_t)
 void latent_place(const Act &proj, int off_q, int q_rank, const float *q_weight, const Act &cq_out, int off_kv, int kv_rank, int rot,
                   const float *kv_weight, float eps, const float *table, int table_rows, bool interleaved, const int *tok_seq,
                   const int *tok_pos, const int *page_table, int pt_stride, void *cache, int page_size, cudaStream_t s) {
@@ -416,19 +461,20 @@ void latent_absorb(const Act &q, const void *w_uk, const Act &out, int n_heads, 
   LLM_CALL("latent", llm_latent_absorb, code(out.dtype), (const float *)q.data, (long long)q.ld, w_uk, out.data, (long long)out.ld,
            (int)q.rows, n_heads, d, rot, kv_rank, table, table_rows, interleaved ? 1 : 0, tok_pos, s);
 }
-void latent_expand(const Act &x, const void *w_uv, const Act &out, int n_heads, int kv_rank, int dv, cudaStream_t s) {
+void latent_expand(const Act &x, const void *w_uv, const Act &out, int n_heads, int kv_rank, int dv, cudaStream_t s, const float *gate,
+                   long long gate_stride) {
   if (x.dtype != out.dtype) LLM_THROW(InvalidArg, "latent_expand: input and output have one type");
-  LLM_CALL("latent", llm_latent_expand, code(x.dtype), x.data, (long long)x.ld, w_uv, out.data, (long long)out.ld, (int)x.rows, n_heads,
-           kv_rank, dv, s);
+  LLM_CALL("latent", llm_latent_expand_gated, code(x.dtype), x.data, (long long)x.ld, w_uv, out.data, (long long)out.ld, (int)x.rows, n_heads,
+           kv_rank, dv, gate, gate_stride, s);
 }
 LLM_KERNEL("latent_tc", llm_latent_rows, const void *, int, int, int, const int *, const int *, const int *, int, int, void *, void *,
            cudaStream_t)
 LLM_KERNEL("latent_tc", llm_latent_rotate_q, const float *, long long, void *, long long, int, int, int, int, const float *, int, int,
            const int *, cudaStream_t)
-LLM_KERNEL("latent_tc", llm_latent_prefill, const void *, long long, const void *, long long, const void *, void *, long long, const int *,
-           int, int, int, int, int, int, float, int, cudaStream_t)
-LLM_KERNEL("latent_tc", llm_latent_decode, const void *, long long, const void *, int, const int *, const int *, const int *, int, int,
-           int, int, int, int, float, void *, long long, float *, int, cudaStream_t)
+LLM_KERNEL("latent_tc", llm_latent_prefill_gated, const void *, long long, const void *, long long, const void *, void *, long long, const int *,
+           int, int, int, int, int, int, float, int, const float *, const float *, long long, cudaStream_t)
+LLM_KERNEL("latent_tc", llm_latent_decode_sinks, const void *, long long, const void *, int, const int *, const int *, const int *, int, int,
+           int, int, int, int, float, void *, long long, float *, int, const float *, cudaStream_t)
 void latent_rows(const void *cache, int page_size, int row, int kv_rank, const int *tok_seq, const int *tok_pos, const int *page_table,
                  int pt_stride, int n_tokens, const Act &c_out, const Act &kr_out, cudaStream_t s) {
   if (c_out.dtype != DType::BF16 || c_out.ld != kv_rank || (row > kv_rank && (kr_out.dtype != DType::BF16 || kr_out.ld != row - kv_rank)))
@@ -447,11 +493,12 @@ bool latent_prefill_supported(int d, int rot, int dv) {
   return f(d, rot, dv) != 0;
 }
 void latent_prefill(const Act &q, const Act &kv, const Act &kr, const Act &out, const int *seq_start, int n_seqs, int max_q_len,
-                    int n_heads, int d, int rot, int dv, float scale, cudaStream_t s, int window) {
+                    int n_heads, int d, int rot, int dv, float scale, cudaStream_t s, int window, const float *null_scores,
+                    const float *gate, long long gate_stride) {
   if (q.dtype != DType::BF16 || kv.dtype != DType::BF16 || out.dtype != DType::BF16 || (rot > 0 && (kr.dtype != DType::BF16 || kr.ld != rot)))
     LLM_THROW(InvalidArg, "latent_prefill: bfloat16 operands");
-  LLM_CALL("latent_tc", llm_latent_prefill, q.data, (long long)q.ld, kv.data, (long long)kv.ld, kr.data, out.data, (long long)out.ld,
-           seq_start, n_seqs, max_q_len, n_heads, d, rot, dv, scale, window, s);
+  LLM_CALL("latent_tc", llm_latent_prefill_gated, q.data, (long long)q.ld, kv.data, (long long)kv.ld, kr.data, out.data, (long long)out.ld,
+           seq_start, n_seqs, max_q_len, n_heads, d, rot, dv, scale, window, null_scores, gate, gate_stride, s);
 }
 bool latent_decode_supported(int kv_rank, int rot) {
   static auto f = resolve<int (*)(int, int)>("latent_tc", "llm_latent_decode_supports");
@@ -462,10 +509,10 @@ size_t latent_decode_floats(int n_tokens, int n_heads, int kv_rank, int n_splits
 }
 void latent_decode(const Act &qa, const void *cache, int page_size, const int *tok_seq, const int *tok_pos, const int *page_table,
                    int pt_stride, int n_heads, int kv_rank, int rot, int n_splits, float scale, const Act &out, float *ws, cudaStream_t s,
-                   int window) {
+                   int window, const float *null_scores) {
   if (qa.dtype != DType::BF16 || out.dtype != DType::BF16) LLM_THROW(InvalidArg, "latent_decode: bfloat16 operands");
-  LLM_CALL("latent_tc", llm_latent_decode, qa.data, (long long)qa.ld, cache, page_size, tok_seq, tok_pos, page_table, pt_stride,
-           (int)qa.rows, n_heads, kv_rank, rot, n_splits, scale, out.data, (long long)out.ld, ws, window, s);
+  LLM_CALL("latent_tc", llm_latent_decode_sinks, qa.data, (long long)qa.ld, cache, page_size, tok_seq, tok_pos, page_table, pt_stride,
+           (int)qa.rows, n_heads, kv_rank, rot, n_splits, scale, out.data, (long long)out.ld, ws, window, null_scores, s);
 }
 bool attention_decode_supported(int d, int group) {
   static auto f = resolve<int (*)(int, int)>("attention_decode", "llm_attention_decode_supports");
@@ -474,28 +521,34 @@ bool attention_decode_supported(int d, int group) {
 void attention_decode(const Act &q, const Act &out, const void *kc, const void *vc, const int *tok_pos, const int *page_table,
                       int pt_stride, int n_heads, int n_kv, int d, int page_size, int chunk, int n_splits, int window,
                       int block, float scale, float *ws_o, float *ws_ml, const float *gate, long long gate_stride,
-                      cudaStream_t s, int sink, bool gate_per_channel, float null_score) {
+                      cudaStream_t s, int sink, bool gate_per_channel, float null_score, const float *null_scores) {
   const int B = (int)q.rows;
-  LLM_CALL("attention_decode", llm_attention_decode_null, q.data, (long long)(B > 1 ? q.ld : q.cols), out.data,
+  LLM_CALL("attention_decode", llm_attention_decode_sinks, q.data, (long long)(B > 1 ? q.ld : q.cols), out.data,
            (long long)(B > 1 ? out.ld : out.cols), kc, vc, tok_pos, page_table, pt_stride, B, n_heads, n_kv, d, page_size, chunk,
-           n_splits, window, block, sink, scale, ws_o, ws_ml, gate, gate_stride, gate_per_channel ? 1 : 0, null_score, s);
+           n_splits, window, block, sink, scale, ws_o, ws_ml, gate, gate_stride, gate_per_channel ? 1 : 0, null_score,
+           null_scores, s);
 }
 bool attention_decode_tc_supported(int d, int page_size, int group) {
   static auto f = resolve<int (*)(int, int, int)>("attention_decode_tc", "llm_attention_decode_tc_supports");
   return f(d, page_size, group) != 0;
 }
-int attention_decode_tc_ctas_per_sm(int d) {
-  static auto f = resolve<int (*)(int)>("attention_decode_tc", "llm_attention_decode_tc_ctas_per_sm");
-  return f(d);
+bool attention_decode_tc_takes(int d, int dv, int page_size, int group) {
+  static auto f = resolve<int (*)(int, int, int, int)>("attention_decode_tc", "llm_attention_decode_tc_takes");
+  return f(d, dv, page_size, group) != 0;
+}
+int attention_decode_tc_ctas_per_sm(int d, int dv) {
+  static auto f = resolve<int (*)(int, int)>("attention_decode_tc", "llm_attention_decode_tc_ctas");
+  return f(d, dv);
 }
 void attention_decode_tc(const Act &qkv, const float *table, int table_rows, int rot_dim, const int *tok_pos,
                          const int *page_table, int pt_stride, void *kc, void *vc, bool write_cache, int n_seqs, int n_heads,
                          int n_kv, int d, int page_size, int chunk, int max_len, int n_splits, int window, int block,
-                         float scale, float *ws_o, float *ws_ml, int *counters, const Act &out, cudaStream_t s) {
-  LLM_CALL("attention_decode_tc", llm_attention_decode_tc, (const float *)qkv.data, (long long)(n_seqs > 1 ? qkv.ld : qkv.cols),
+                         float scale, float *ws_o, float *ws_ml, int *counters, const Act &out, cudaStream_t s, int dv, const float *bias,
+                         const float *null_scores) {
+  LLM_CALL("attention_decode_tc", llm_attention_decode_tc_sinks, (const float *)qkv.data, (long long)(n_seqs > 1 ? qkv.ld : qkv.cols),
            qkv.parts, (long long)qkv.part_stride, table, table_rows, rot_dim, tok_pos, page_table, pt_stride, kc, vc,
-           write_cache ? 1 : 0, n_seqs, n_heads, n_kv, d, page_size, chunk, max_len, n_splits, window, block, scale, ws_o, ws_ml,
-           counters, out.data, (long long)(n_seqs > 1 ? out.ld : out.cols), s);
+           write_cache ? 1 : 0, n_seqs, n_heads, n_kv, d, dv > 0 ? dv : d, page_size, chunk, max_len, n_splits, window, block, scale, bias,
+           null_scores, ws_o, ws_ml, counters, out.data, (long long)(n_seqs > 1 ? out.ld : out.cols), s);
 }
 bool attention_prefill_supported(int d, int page_size) {
   static auto f = resolve<int (*)(int, int)>("attention_prefill", "llm_attention_prefill_supports");
@@ -503,21 +556,26 @@ bool attention_prefill_supported(int d, int page_size) {
 }
 void attention_prefill(const Act &q, const Act &out, const void *kc, const void *vc, const int *seq_start, const int *seq_past,
                        const int *page_table, int pt_stride, int n_seqs, int max_q_len, int n_heads, int n_kv, int d,
-                       int page_size, int window, int block, float scale, cudaStream_t s, int sink, float null_score) {
-  LLM_CALL("attention_prefill", llm_attention_prefill_null, q.data, (long long)q.ld, out.data, (long long)out.ld, kc, vc, seq_start,
-           seq_past, page_table, pt_stride, n_seqs, max_q_len, n_heads, n_kv, d, page_size, window, block, sink, scale, null_score, s);
+                       int page_size, int window, int block, float scale, cudaStream_t s, int sink, float null_score, const float *null_scores) {
+  LLM_CALL("attention_prefill", llm_attention_prefill_sinks, q.data, (long long)q.ld, out.data, (long long)out.ld, kc, vc, seq_start,
+           seq_past, page_table, pt_stride, n_seqs, max_q_len, n_heads, n_kv, d, page_size, window, block, sink, scale, null_score,
+           null_scores, s);
 }
 bool attention_prefill_tc_supported(int d, int page_size) {
   static auto f = resolve<int (*)(int, int)>("attention_prefill_tc", "llm_attention_prefill_tc_supports");
   return f(d, page_size) != 0;
 }
+bool attention_prefill_tc_takes(int d, int dv, int page_size) {
+  static auto f = resolve<int (*)(int, int, int)>("attention_prefill_tc", "llm_attention_prefill_tc_takes");
+  return f(d, dv, page_size) != 0;
+}
 void attention_prefill_tc(const Act &q, const Act &out, const void *kc, const void *vc, long long n_pages, const int *seq_start,
                           const int *seq_past, const int *page_table, int pt_stride, int n_seqs, int max_q_len, int n_heads,
                           int n_kv, int d, int page_size, int window, int block, float scale, int *status, cudaStream_t s,
-                          int sink, float null_score) {
-  LLM_CALL("attention_prefill_tc", llm_attention_prefill_tc_null, q.data, (long long)q.ld, (long long)q.rows, out.data,
+                          int sink, float null_score, int dv, const float *null_scores) {
+  LLM_CALL("attention_prefill_tc", llm_attention_prefill_tc_sinks, q.data, (long long)q.ld, (long long)q.rows, out.data,
            (long long)out.ld, kc, vc, n_pages, seq_start, seq_past, page_table, pt_stride, n_seqs, max_q_len, n_heads, n_kv, d,
-           page_size, window, block, sink, scale, null_score, 0, status, s);
+           dv > 0 ? dv : d, page_size, window, block, sink, scale, null_score, null_scores, 0, status, s);
 }
 
 LLM_KERNEL("attention_generic", llm_attention_generic_sigmoid, int, const void *, long long, void *, long long, const void *, const void *,
@@ -591,10 +649,11 @@ void row_gate(const float *x, long long x_stride, float *out, long long out_stri
   LLM_CALL("moe", llm_row_gate, x, x_stride, out, out_stride, n_parts, gate, gate_stride, n_rows, cols, s);
 }
 LLM_KERNEL("moe", llm_moe_sort, const int *, int, int, int, int *, int *, int *, cudaStream_t)
-LLM_KERNEL("moe", llm_moe_rows, int, const void *, long long, const void *, const void *, const int *, const float *, int, int, int,
-           int, int, int, int, float *, cudaStream_t)
-LLM_KERNEL("moe", llm_moe_grouped, const void *, long long, const void *, const void *, const int *, const int *, const int *,
-           const float *, int, int, int, int, int, int, int, int, void *, float *, cudaStream_t)
+LLM_KERNEL("moe", llm_moe_rows_glu, int, const void *, long long, const void *, const void *, const int *, const float *, int, int, int,
+           int, int, int, int, int, float, float, float, float *, cudaStream_t)
+LLM_KERNEL("moe", llm_moe_identity, const void *, long long, const int *, const float *, int, int, int, int, float *, cudaStream_t)
+LLM_KERNEL("moe", llm_moe_grouped_glu, const void *, long long, const void *, const void *, const int *, const int *, const int *,
+           const float *, int, int, int, int, int, int, int, int, float, float, float, void *, float *, cudaStream_t)
 void activation(const Act &in, const Act &out, int act, cudaStream_t s) {
   if (in.ld != in.cols || out.ld != out.cols) LLM_THROW(InvalidArg, "activation: rows must be dense");
   LLM_CALL("moe", llm_activation, code(in.dtype), code(out.dtype), in.data, out.data, (long long)(in.rows * in.cols), act, s);
@@ -610,9 +669,10 @@ int moe_tile_rows() {
 void moe_sort(const int *chosen, int n_rows, int n_experts, int tile_rows, int *offsets, int *perm, int *tiles, cudaStream_t s) {
   LLM_CALL("moe", llm_moe_sort, chosen, n_rows, n_experts, tile_rows, offsets, perm, tiles, s);
 }
-LLM_KERNEL("moe", llm_moe_gather, const void *, long long, const int *, int, int, int, void *, cudaStream_t)
-LLM_KERNEL("moe_tc", llm_moe_tc, const void *, const void *, const void *, const int *, const int *, const int *, const float *, int,
-           int, int, int, int, int, int, int, void *, float *, int *, cudaStream_t)
+LLM_KERNEL("moe", llm_moe_gather_identity, const void *, long long, const int *, int, int, int, void *, const int *, const int *, const float *,
+           int, float *, cudaStream_t)
+LLM_KERNEL("moe_tc", llm_moe_tc_glu, const void *, const void *, const void *, const int *, const int *, const int *, const float *, int,
+           int, int, int, int, int, int, int, float, float, float, void *, float *, int *, cudaStream_t)
 bool moe_tc_supported(int width, int ff) {
   static auto f = resolve<int (*)(int, int)>("moe_tc", "llm_moe_tc_supports");
   return f(width, ff) != 0;
@@ -623,16 +683,16 @@ int moe_tc_tile_rows(int n_rows) {
 }
 void moe_tc(const Act &x, const void *up, const void *down, const int *offsets, const int *perm, const int *tiles,
             const float *weight, int n_experts, int top, int width, int ff, int act, bool weight_on_output, void *xs, void *mid,
-            float *out, int *status, cudaStream_t s, bool gated) {
+            float *out, int *status, cudaStream_t s, bool gated, const Glu &glu, const int *chosen) {
   const int n_rows = (int)x.rows * top;
-  LLM_CALL("moe", llm_moe_gather, x.data, (long long)x.ld, perm, n_rows, top, width, xs, s);
-  LLM_CALL("moe_tc", llm_moe_tc, xs, up, down, offsets, perm, tiles, weight, (int)x.rows, n_experts, top, width, ff, act,
-           weight_on_output ? 1 : 0, gated ? 1 : 0, mid, out, status, s);
+  LLM_CALL("moe", llm_moe_gather_identity, x.data, (long long)x.ld, perm, n_rows, top, width, xs, chosen, offsets, weight, n_experts, out, s);
+  LLM_CALL("moe_tc", llm_moe_tc_glu, xs, up, down, offsets, perm, tiles, weight, (int)x.rows, n_experts, top, width, ff, act,
+           weight_on_output ? 1 : 0, gated ? 1 : 0, glu.limit, glu.slope, glu.shift, mid, out, status, s);
 }
 void moe_rows(const Act &x, const void *up, const void *down, const int *chosen, const float *weight, int top, int width, int ff,
-              int act, bool weight_on_output, float *out, cudaStream_t s, bool gated) {
-  LLM_CALL("moe", llm_moe_rows, code(x.dtype), x.data, (long long)x.ld, up, down, chosen, weight, (int)x.rows, top, width, ff, act,
-           weight_on_output ? 1 : 0, gated ? 1 : 0, out, s);
+              int act, bool weight_on_output, float *out, cudaStream_t s, bool gated, int n_experts, const Glu &glu) {
+  LLM_CALL("moe", llm_moe_rows_glu, code(x.dtype), x.data, (long long)x.ld, up, down, chosen, weight, (int)x.rows, n_experts, top, width, ff,
+           act, weight_on_output ? 1 : 0, gated ? 1 : 0, glu.limit, glu.slope, glu.shift, out, s);
 }
 bool moe_grouped_supported(int width, int ff) {
   static auto f = resolve<int (*)(int, int)>("moe", "llm_moe_grouped_supports");
@@ -640,9 +700,13 @@ bool moe_grouped_supported(int width, int ff) {
 }
 void moe_grouped(const Act &x, const void *up, const void *down, const int *offsets, const int *perm, const int *tiles,
                  const float *weight, int n_experts, int top, int width, int ff, int act, bool weight_on_output, void *mid,
-                 float *out, cudaStream_t s, bool gated) {
-  LLM_CALL("moe", llm_moe_grouped, x.data, (long long)x.ld, up, down, offsets, perm, tiles, weight, (int)x.rows, n_experts, top,
-           width, ff, act, weight_on_output ? 1 : 0, gated ? 1 : 0, mid, out, s);
+                 float *out, cudaStream_t s, bool gated, const Glu &glu) {
+  LLM_CALL("moe", llm_moe_grouped_glu, x.data, (long long)x.ld, up, down, offsets, perm, tiles, weight, (int)x.rows, n_experts, top,
+           width, ff, act, weight_on_output ? 1 : 0, gated ? 1 : 0, glu.limit, glu.slope, glu.shift, mid, out, s);
+}
+void moe_identity(const Act &x, const int *chosen, const float *weight, int n_experts, int top, int width, float *out, cudaStream_t s) {
+  if (x.dtype != DType::BF16) LLM_THROW(InvalidArg, "moe_identity: bfloat16 rows");
+  LLM_CALL("moe", llm_moe_identity, x.data, (long long)x.ld, chosen, weight, (int)x.rows, n_experts, top, width, out, s);
 }
 
 // ---------------------------------------------------------------- state carried from token to token
@@ -803,6 +867,46 @@ void memory_step(const Act &proj, int off_q, int off_k, int off_v, int off_g, in
   LLM_CALL("state_scan", llm_memory_step, (const float *)proj.data, (long long)proj.ld, off_q, off_k, off_v, off_g, off_i, off_f, bias_i,
            bias_f, cap, q_scale, state_m, state, weight, (int)act, eps, out_scale, out.data, code(out.dtype), (long long)out.ld, seq_slot,
            (int)proj.rows, n_heads, d, dv, s);
+}
+
+// ---------------------------------------------------------------- the selective recurrence
+LLM_KERNEL("selective_scan", llm_short_conv_silu, int, const float *, long long, const float *, const float *, int, float *, void *, long long, int,
+           const int *, const int *, const int *, const int *, const int *, int, int, int, cudaStream_t)
+LLM_KERNEL("selective_scan", llm_selective_scan, int, const void *, long long, const float *, long long, const float *, const float *, long long,
+           int, int, const float *, long long, const float *, const float *, float *, void *, long long, const int *, const int *, int, int, int,
+           cudaStream_t)
+LLM_KERNEL("selective_scan", llm_selective_step, int, const void *, long long, const float *, long long, int, const void *, int, const float *, int,
+           int, const float *, long long, const float *, const float *, float *, void *, long long, const int *, int, int, int, cudaStream_t)
+LLM_KERNEL("selective_scan", llm_rows_cast, const float *, long long, int, void *, int, int, cudaStream_t)
+int selective_max_state() { return 256; }
+void rows_cast(const Act &in, int n, const Act &out, cudaStream_t s) {
+  if (in.dtype != DType::F32 || out.dtype != DType::BF16 || out.ld != out.cols) LLM_THROW(InvalidArg, "rows_cast: 32-bit rows to dense bfloat16 rows");
+  LLM_CALL("selective_scan", llm_rows_cast, (const float *)in.data, (long long)in.ld, n, out.data, (int)out.rows, (int)out.cols, s);
+}
+void short_conv_silu(const Act &u, const float *weight, const float *bias, int taps, float *state, const Act &out, const int *tok_seq,
+                     const int *tok_pos, const int *seq_start, const int *seq_past, const int *seq_slot, int n_seqs, bool single_tokens,
+                     cudaStream_t s) {
+  if (u.dtype != DType::F32) LLM_THROW(InvalidArg, "short_conv_silu: 32-bit inputs");
+  LLM_CALL("selective_scan", llm_short_conv_silu, code(out.dtype), (const float *)u.data, (long long)u.ld, weight, bias, taps, state, out.data,
+           (long long)out.ld, (int)out.cols, tok_seq, tok_pos, seq_start, seq_past, seq_slot, n_seqs, (int)out.rows, single_tokens ? 1 : 0, s);
+}
+void selective_scan(const Act &x, const Act &dt_raw, const float *dt_bias, const Act &bc, int off_b, int off_c, const float *z, long long ldz,
+                    const float *a_log, const float *skip, float *state, const Act &out, const int *seq_start, const int *seq_slot, int n_seqs,
+                    int N, cudaStream_t s) {
+  if (dt_raw.dtype != DType::F32 || bc.dtype != DType::F32 || x.dtype != out.dtype)
+    LLM_THROW(InvalidArg, "selective_scan: 32-bit projections, one type for input and result");
+  LLM_CALL("selective_scan", llm_selective_scan, code(x.dtype), x.data, (long long)x.ld, (const float *)dt_raw.data, (long long)dt_raw.ld, dt_bias,
+           (const float *)bc.data, (long long)bc.ld, off_b, off_c, z, ldz, a_log, skip, state, out.data, (long long)out.ld, seq_start, seq_slot,
+           n_seqs, (int)out.cols, N, s);
+}
+void selective_step(const Act &x, const Act &low, int rank, const Weight &w_dt, const float *dt_bias, int off_b, int off_c, const float *z,
+                    long long ldz, const float *a_log, const float *skip, float *state, const Act &out, const int *seq_slot, int N,
+                    cudaStream_t s) {
+  if (low.dtype != DType::F32 || x.dtype != out.dtype || w_dt.dtype != x.dtype)
+    LLM_THROW(InvalidArg, "selective_step: 32-bit projections, one type for input, matrix and result");
+  LLM_CALL("selective_scan", llm_selective_step, code(x.dtype), x.data, (long long)x.ld, (const float *)low.data, (long long)low.ld, rank,
+           w_dt.data(), (int)w_dt.cols, dt_bias, off_b, off_c, z, ldz, a_log, skip, state, out.data, (long long)out.ld, seq_slot, (int)out.rows,
+           (int)out.cols, N, s);
 }
 
 // ---------------------------------------------------------------- sampling

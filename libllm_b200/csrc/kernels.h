@@ -28,8 +28,21 @@ std::vector<std::string> loaded_libraries();
 void embedding(DType table_dtype, const void *table, const int *tokens, const int *fed_tokens, const int *fed_rows,
                float *out, int n_tokens, int hidden, int vocab, cudaStream_t s, const void *pos_table = nullptr, int pos_rows = 0,
                const int *tok_pos = nullptr);   // pos_table [pos_rows, hidden] in the table's type: a learned vector per position, added
+// The same with what a token brings beside its row: `ids` (null: not asked for) receives the tokens' numbers; `pairs`
+// [buckets + 1, hidden] in the table's type (null: none): the row (previous mul_prev + current mul_cur) mod buckets is added, the
+// last row for a sequence's first token; last [slots]: every sequence's last token, read and moved on.
+struct TokenPairs {
+  const void *table = nullptr;
+  long long buckets = 0, mul_prev = 0, mul_cur = 0;
+  int *last = nullptr;
+};
+void embedding_pairs(DType table_dtype, const void *table, const int *tokens, const int *fed_tokens, const int *fed_rows, float *out,
+                     int n_tokens, int hidden, int vocab, cudaStream_t s, const void *pos_table, int pos_rows, const int *tok_pos, int *ids,
+                     const TokenPairs &pairs, const int *tok_seq, const int *seq_start, const int *seq_slot);
 void copy_words(const int *src, int *dst, int n, cudaStream_t s);
 void gather_words(const int *src1, int n1, const int *src2, int n2, int *dst, cudaStream_t s);
+// A pending result with norms of its own (Act::normed()) is taken by this pass and by gather_rows_add.  With a pending result of
+// that kind `weight` may be null: out is then the stream itself in its type.
 void add_rmsnorm(float *resid, const Act *delta, const float *weight, float eps, void *out, DType out_dtype,
                  const int *rows, int n_rows, int hidden, cudaStream_t s);
 // Several residual streams [n_streams][rows][hidden] (in_stride / out_stride floats apart; in_stride 0: all equal to x_in):
@@ -48,6 +61,11 @@ void add_layernorm_conv(float *resid, const Act *delta, const float *weight, con
                         int n_rows, int hidden, const float *conv_w, void *state, const int *seq_slot, int taps, cudaStream_t s);
 // out[i] = resid[rows[i]] + delta's parts at that row (32-bit)
 void gather_rows_add(const float *resid, const Act *delta, const int *rows, int n_rows, float *out, int hidden, cudaStream_t s);
+// The stream with what is pending added (resid moves on; rows null: all of it), in out's type, without a norm.
+void stream_cast(float *resid, const Act *delta, void *out, DType out_dtype, int n_rows, int hidden, cudaStream_t s);
+// out[t, c] = gelu_tanh(z[t, c]) * table[ids[rows ? rows[t] : t], offset + c] for c < dim, nought up to out.cols
+void token_gate(const Act &z, const void *table, long long table_width, int offset, int dim, const int *ids, const int *rows, const Act &out,
+                cudaStream_t s);
 void swiglu(const Act &gu, void *out, DType out_dtype, cudaStream_t s);
 // gu [T, 2 I] (gate | up), bias [2 I] or null; out [T, I] = g * sigmoid(slope g) * (u + up_shift), g and u bounded by limit
 void clamped_glu(const Act &gu, const float *bias, const Act &out, float limit, float slope, float up_shift, cudaStream_t s);
@@ -62,7 +80,12 @@ void random_fill(void *out, DType dtype, long long n, unsigned long long seed, i
 void gemm_plain(const Act &x, const Weight &w, const float *bias, const Act &out, cudaStream_t s);
 bool gemm_tc_supported(const Act &x, const Weight &w);
 int gemm_tc_suggest_parts(int M, int N, int K);
-void gemm_tc(const Act &x, const Weight &w, const Act &out, bool swiglu, int *status, cudaStream_t s);
+// The unit of a gated pair (gate g, up u): g' = min(g, limit), u' = clamp(u, -limit, limit), g' sigmoid(slope g') (u' + shift)
+struct Glu {
+  float limit = __builtin_huge_valf(), slope = 1.f, shift = 0.f;      // silu(g) u
+};
+// swiglu: w is a stacked gate|up matrix and the result the gated unit of the two halves
+void gemm_tc(const Act &x, const Weight &w, const Act &out, bool swiglu, int *status, cudaStream_t s, const Glu &glu = Glu());
 // x [n_groups * rows, K] through the matrices stacked in w, each but the last of group_n rows (a multiple of 128): out [rows, w.rows]
 void gemm_tc_grouped(const Act &x, const Weight &w, const Act &out, int n_groups, int group_n, int *status, cudaStream_t s);
 void gemm_tc_wait_probe(long long limit_ns, int *status, cudaStream_t s);
@@ -134,10 +157,10 @@ constexpr float NO_NULL_KEY = -__builtin_huge_valf();
 void attention_generic(const Act &q, const Act &out, const void *kc, const void *vc, const int *tok_seq, const int *tok_pos,
                        const int *page_table, int pt_stride, int n_heads, int n_kv, int d, int dv, int page_size, int window,
                        int block, float scale, const float *gate, long long gate_stride, cudaStream_t s, int sink = 0, int v_ld = 0,
-                       float null_score = NO_NULL_KEY);
+                       float null_score = NO_NULL_KEY, const float *null_scores = nullptr);
 // v_ld > 0: value rows lie v_ld channels apart (the values are the first dv channels of the key rows when vc is kc).
 // null_score: every query also sees one key of that score that has no value (exp(null_score) joins the softmax's
-// denominator); NO_NULL_KEY: none.
+// denominator); NO_NULL_KEY: none.  null_scores (32-bit per head, device): such a score per head instead.
 // Weights that stand for themselves: sigmoid(cap tanh(temp[h] s / cap) + bias[h]) (cap 0: no bound), not normalised; the result
 // times out_scale.
 void attention_generic_sigmoid(const Act &q, const Act &out, const void *kc, const void *vc, const int *tok_seq, const int *tok_pos,
@@ -165,7 +188,9 @@ void latent_place(const Act &proj, int off_q, int q_rank, const float *q_weight,
 void latent_absorb(const Act &q, const void *w_uk, const Act &out, int n_heads, int d, int rot, int kv_rank, const float *table,
                    int table_rows, bool interleaved, const int *tok_pos, cudaStream_t s);
 // x [T, heads * kv_rank] -> out [T, heads * dv]: out_h = w_uv_h x_h
-void latent_expand(const Act &x, const void *w_uv, const Act &out, int n_heads, int kv_rank, int dv, cudaStream_t s);
+// (times sigmoid(gate[t, h]) with a gate, rows gate_stride apart)
+void latent_expand(const Act &x, const void *w_uv, const Act &out, int n_heads, int kv_rank, int dv, cudaStream_t s, const float *gate = nullptr,
+                   long long gate_stride = 0);
 // ---- latent attention on the tensor cores (csrc/latent_tc.cu), bfloat16
 // The cached rows of the step's tokens, whoever appended them: c_out [T, kv_rank], kr_out [T, row - kv_rank].
 void latent_rows(const void *cache, int page_size, int row, int kv_rank, const int *tok_seq, const int *tok_pos, const int *page_table,
@@ -176,37 +201,44 @@ void latent_rotate_q(const Act &q, const Act &out, int n_heads, int d, int rot, 
 bool latent_prefill_supported(int d, int rot, int dv);
 // Sequences that start at their first token, heads materialised: kv [T, heads * d | heads * dv], kr [T, rot] rotated.
 void latent_prefill(const Act &q, const Act &kv, const Act &kr, const Act &out, const int *seq_start, int n_seqs, int max_q_len,
-                    int n_heads, int d, int rot, int dv, float scale, cudaStream_t s, int window = 0);
+                    int n_heads, int d, int rot, int dv, float scale, cudaStream_t s, int window = 0, const float *null_scores = nullptr,
+                    const float *gate = nullptr, long long gate_stride = 0);
 bool latent_decode_supported(int kv_rank, int rot);
 size_t latent_decode_floats(int n_tokens, int n_heads, int kv_rank, int n_splits);
 // qa [T, heads * (kv_rank + rot)] (latent_absorb) over the cached rows -> out [T, heads * kv_rank]; ws: latent_decode_floats
 void latent_decode(const Act &qa, const void *cache, int page_size, const int *tok_seq, const int *tok_pos, const int *page_table,
                    int pt_stride, int n_heads, int kv_rank, int rot, int n_splits, float scale, const Act &out, float *ws, cudaStream_t s,
-                   int window = 0);
+                   int window = 0, const float *null_scores = nullptr);
 bool attention_decode_supported(int d, int group);
 void attention_decode(const Act &q, const Act &out, const void *kc, const void *vc, const int *tok_pos, const int *page_table,
                       int pt_stride, int n_heads, int n_kv, int d, int page_size, int chunk, int n_splits, int window,
                       int block, float scale, float *ws_o, float *ws_ml, const float *gate, long long gate_stride,
-                      cudaStream_t s, int sink = 0, bool gate_per_channel = false, float null_score = NO_NULL_KEY);
+                      cudaStream_t s, int sink = 0, bool gate_per_channel = false, float null_score = NO_NULL_KEY,
+                      const float *null_scores = nullptr);
 bool attention_decode_tc_supported(int d, int page_size, int group);
-int attention_decode_tc_ctas_per_sm(int d);
+bool attention_decode_tc_takes(int d, int dv, int page_size, int group);
+int attention_decode_tc_ctas_per_sm(int d, int dv);
+// dv 0: values as wide as keys; bias over the stacked row's columns, null_scores per head (32-bit, device; null: none)
 void attention_decode_tc(const Act &qkv, const float *table, int table_rows, int rot_dim, const int *tok_pos,
                          const int *page_table, int pt_stride, void *kc, void *vc, bool write_cache, int n_seqs, int n_heads,
                          int n_kv, int d, int page_size, int chunk, int max_len, int n_splits, int window, int block,
-                         float scale, float *ws_o, float *ws_ml, int *counters, const Act &out, cudaStream_t s);
+                         float scale, float *ws_o, float *ws_ml, int *counters, const Act &out, cudaStream_t s, int dv = 0,
+                         const float *bias = nullptr, const float *null_scores = nullptr);
 bool attention_prefill_supported(int d, int page_size);
 void attention_prefill(const Act &q, const Act &out, const void *kc, const void *vc, const int *seq_start, const int *seq_past,
                        const int *page_table, int pt_stride, int n_seqs, int max_q_len, int n_heads, int n_kv, int d,
-                       int page_size, int window, int block, float scale, cudaStream_t s, int sink = 0, float null_score = NO_NULL_KEY);
+                       int page_size, int window, int block, float scale, cudaStream_t s, int sink = 0, float null_score = NO_NULL_KEY,
+                       const float *null_scores = nullptr);
 bool attention_prefill_tc_supported(int d, int page_size);
+bool attention_prefill_tc_takes(int d, int dv, int page_size);      // padded heads too
 void attention_prefill_tc(const Act &q, const Act &out, const void *kc, const void *vc, long long n_pages, const int *seq_start,
                           const int *seq_past, const int *page_table, int pt_stride, int n_seqs, int max_q_len, int n_heads,
                           int n_kv, int d, int page_size, int window, int block, float scale, int *status, cudaStream_t s,
-                          int sink = 0, float null_score = NO_NULL_KEY);
+                          int sink = 0, float null_score = NO_NULL_KEY, int dv = 0, const float *null_scores = nullptr);
 // out[t, h, :] *= sigmoid(gate[t * gate_stride + h]) for heads of width dv
 void head_gate(const Act &out, const float *gate, long long gate_stride, int n_heads, int dv, cudaStream_t s);
 // ---- routed feed-forward (csrc/moe.cu)
-enum Activation { GeluErf = 0, GeluTanh = 1, Silu = 2, Relu2 = 3 };
+enum Activation { GeluErf = 0, GeluTanh = 1, Silu = 2, Relu2 = 3, BoundedGlu = 4 };   // the last: gated experts alone, its shape a Glu
 void activation(const Act &in, const Act &out, int act, cudaStream_t s);
 // logits [T, E] 32-bit -> chosen [T * top], weight [T * top]; score 0 sigmoid, 1 softmax
 void moe_route(const Act &logits, int n_experts, int top, int score, bool renormalize, int *chosen, float *weight, cudaStream_t s);
@@ -218,22 +250,27 @@ void moe_route_grouped(const Act &logits, int n_experts, int top, int score, con
 void row_gate(const float *x, long long x_stride, float *out, long long out_stride, int n_parts, const float *gate,
               long long gate_stride, int n_rows, int cols, cudaStream_t s);
 int moe_tile_rows();
+// Choices beyond n_experts are identity experts: no place among the sorted rows.
 void moe_sort(const int *chosen, int n_rows, int n_experts, int tile_rows, int *offsets, int *perm, int *tiles, cudaStream_t s);
 // x [T, width]; up [E, ff, width], down [E, width, ff] in x's type; out [top, T, width] 32-bit.  `gated`: up is
 // [E, 2 ff, width], an expert's gate and up rows interleaved, and the expert is down(act(gate x) * up x).
 void moe_rows(const Act &x, const void *up, const void *down, const int *chosen, const float *weight, int top, int width, int ff,
-              int act, bool weight_on_output, float *out, cudaStream_t s, bool gated = false);
+              int act, bool weight_on_output, float *out, cudaStream_t s, bool gated = false, int n_experts = 0x7fffffff,
+              const Glu &glu = Glu());
 bool moe_grouped_supported(int width, int ff);
 void moe_grouped(const Act &x, const void *up, const void *down, const int *offsets, const int *perm, const int *tiles,
                  const float *weight, int n_experts, int top, int width, int ff, int act, bool weight_on_output, void *mid,
-                 float *out, cudaStream_t s, bool gated = false);
+                 float *out, cudaStream_t s, bool gated = false, const Glu &glu = Glu());
+// out[choice, token] = weight * x[token] where the choice is no expert (>= n_experts); moe_rows does this itself.
+void moe_identity(const Act &x, const int *chosen, const float *weight, int n_experts, int top, int width, float *out, cudaStream_t s);
 // The same on tcgen05 (csrc/moe_tc.cu): the table of tiles must have moe_tc_tile_rows(rows) rows to a tile;
 // xs [T * top, width] receives the tokens' rows in sorted order.
 bool moe_tc_supported(int width, int ff);
 int moe_tc_tile_rows(int n_rows);
 void moe_tc(const Act &x, const void *up, const void *down, const int *offsets, const int *perm, const int *tiles,
             const float *weight, int n_experts, int top, int width, int ff, int act, bool weight_on_output, void *xs, void *mid,
-            float *out, int *status, cudaStream_t s, bool gated = false);
+            float *out, int *status, cudaStream_t s, bool gated = false, const Glu &glu = Glu(), const int *chosen = nullptr);
+// (chosen: some choices may be identity experts, whose results are written on the way)
 // ---- state carried from token to token (csrc/recurrent.cu)
 // out = h + conv(h) over time per channel, weight [width, taps] 32-bit; state [slots, taps - 1, width] in h's type.
 // With silu_alone: out = silu(conv(h)), the short convolution of a projection.
@@ -301,6 +338,22 @@ void bonus_step(const Act &r, const Act &k, const Act &v, const Act &g, const Ac
 void memory_step(const Act &proj, int off_q, int off_k, int off_v, int off_g, int off_i, int off_f, const float *bias_i, const float *bias_f,
                  float cap, float q_scale, float *state_m, float *state, const float *weight, GateAct act, float eps, float out_scale,
                  const Act &out, const int *seq_slot, int n_heads, int d, int dv, cudaStream_t s);
+// ---- the selective recurrence (csrc/selective_scan.cu)
+int selective_max_state();
+// out = silu(conv over time of the first out.cols columns of u (32-bit) + bias); weight [taps][channels], state [slots, taps - 1, channels]
+void short_conv_silu(const Act &u, const float *weight, const float *bias, int taps, float *state, const Act &out, const int *tok_seq,
+                     const int *tok_pos, const int *seq_start, const int *seq_past, const int *seq_slot, int n_seqs, bool single_tokens,
+                     cudaStream_t s);
+// x convolved, dt_raw before its bias, B and C at their offsets of the 32-bit rows bc, z 32-bit; state [slots, inner, N]; out = y silu(z)
+void selective_scan(const Act &x, const Act &dt_raw, const float *dt_bias, const Act &bc, int off_b, int off_c, const float *z, long long ldz,
+                    const float *a_log, const float *skip, float *state, const Act &out, const int *seq_start, const int *seq_slot, int n_seqs,
+                    int N, cudaStream_t s);
+// out (bfloat16, dense) = the first n columns of the 32-bit rows `in`, nought beyond them
+void rows_cast(const Act &in, int n, const Act &out, cudaStream_t s);
+// A step of single tokens: low's rows begin with the dt input of `rank` values; w_dt [inner, w_dt.cols], columns beyond the rank nought
+void selective_step(const Act &x, const Act &low, int rank, const Weight &w_dt, const float *dt_bias, int off_b, int off_c, const float *z,
+                    long long ldz, const float *a_log, const float *skip, float *state, const Act &out, const int *seq_slot, int N,
+                    cudaStream_t s);
 // ---- sampling
 void argmax(const float *logits, long long stride, int n_rows, int vocab, int *out, cudaStream_t s);
 void sample(const float *logits, long long stride, int n_rows, int vocab, float temperature, int top_k, float top_p,

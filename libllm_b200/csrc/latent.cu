@@ -32,7 +32,7 @@ __device__ __forceinline__ void rotate_pair(const float *x, const float *cs, int
 }
 
 // ---------------------------------------------------------------- placement
-// proj rows (32-bit): the query latent (q_rank values at off_q) and, when the run has a latent projection of
+// proj rows (32-bit): the query latent (q_rank values at off_q; q_rank 0: none) and, when the run has a latent projection of
 // its own (off_kv >= 0), kv_rank + rot_dim values at off_kv.  cq_out = rms(query latent) * q_weight in the
 // engine's type; cache row of the token = [rms(first kv_rank) * kv_weight | rotated last rot_dim].
 template <typename T, int THREADS>
@@ -47,7 +47,7 @@ latent_place_kernel(const float *__restrict__ proj, long long ld, int off_q, int
   grid_dependency_wait();
   const int t = blockIdx.x;
   const float *row = proj + (size_t)t * ld;
-  {
+  if (q_rank > 0) {
     float ss = 0.f;
     for (int c = threadIdx.x; c < q_rank; c += THREADS) ss = fmaf(row[off_q + c], row[off_q + c], ss);
     const float inv = rsqrtf(block_sum<THREADS>(ss, scratch) / (float)q_rank + eps);
@@ -77,7 +77,7 @@ LLM_EXPORT int llm_latent_place(int dtype, const float *proj, long long ld, int 
                                 const float *table, int table_rows, int interleaved, const int *tok_seq, const int *tok_pos,
                                 const int *page_table, int pt_stride, void *cache, int page_size, cudaStream_t stream) {
   if (n_tokens == 0) return LLM_OK;
-  LLM_REQUIRE(n_tokens > 0 && q_rank > 0 && off_q >= 0 && q_weight && cq_out, "latent_place: bad sizes");
+  LLM_REQUIRE(n_tokens > 0 && q_rank >= 0 && off_q >= 0 && (q_rank == 0 || (q_weight && cq_out)), "latent_place: bad sizes");
   if (off_kv >= 0)
     LLM_REQUIRE(kv_rank > 0 && rot >= 0 && rot % 2 == 0 && kv_weight && cache && page_table && (rot == 0 || (table && table_rows > 0)),
                 "latent_place: bad sizes of the key/value latent");
@@ -173,12 +173,13 @@ LLM_EXPORT int llm_latent_absorb(int dtype, const float *q, long long ldq, const
 // x [tokens, heads, kv_rank] (the weighted sums of cached latents), w_uv [heads * dv, kv_rank]:
 // out[t, h, j] = sum_c x[t, h, c] * w_uv[h * dv + j, c].  A CTA takes one head and TT tokens; a warp owns output
 // channels, its lanes walk a row of w_uv together (in lane order, then the shuffle tree); blockIdx.z shares the
-// output channels out, eight to a CTA.
+// output channels out, eight to a CTA.  `gate` (32-bit, one value per token and head, rows gate_stride apart; null: none): the
+// head's result is multiplied by sigmoid(gate).
 constexpr int LAT_ET = 8;
 template <typename T, int THREADS>
 __global__ void __launch_bounds__(THREADS)
 latent_expand_kernel(const T *__restrict__ x, long long ldx, const T *__restrict__ w_uv, T *__restrict__ out, long long ldo, int n_tokens,
-                     int kv_rank, int dv) {
+                     int kv_rank, int dv, const float *__restrict__ gate, long long gate_stride) {
   extern __shared__ float xs[];                        // [LAT_ET][kv_rank]
   grid_dependents_launch();
   grid_dependency_wait();
@@ -202,14 +203,15 @@ latent_expand_kernel(const T *__restrict__ x, long long ldx, const T *__restrict
     }
 #pragma unroll
     for (int t = 0; t < LAT_ET; ++t) {
-      const float s = warp_sum(acc[t]);
+      float s = warp_sum(acc[t]);
+      if (gate && t < nt) s *= 1.f / (1.f + expf(-gate[(size_t)(t0 + t) * gate_stride + h]));
       if (lane == 0 && t < nt) out[(size_t)(t0 + t) * ldo + (size_t)h * dv + j] = from_float<T>(s);
     }
   }
 }
 
-LLM_EXPORT int llm_latent_expand(int dtype, const void *x, long long ldx, const void *w_uv, void *out, long long ldo, int n_tokens,
-                                 int n_heads, int kv_rank, int dv, cudaStream_t stream) {
+LLM_EXPORT int llm_latent_expand_gated(int dtype, const void *x, long long ldx, const void *w_uv, void *out, long long ldo, int n_tokens,
+                                       int n_heads, int kv_rank, int dv, const float *gate, long long gate_stride, cudaStream_t stream) {
   if (n_tokens == 0) return LLM_OK;
   LLM_REQUIRE(n_tokens > 0 && n_heads > 0 && n_heads <= 65535 && kv_rank > 0 && dv > 0, "latent_expand: bad sizes");
   constexpr int THREADS = 256;
@@ -219,12 +221,17 @@ LLM_EXPORT int llm_latent_expand(int dtype, const void *x, long long ldx, const 
   if (dtype == LLM_F32) {
     LLM_CHECK_CUDA(llm_allow_smem(latent_expand_kernel<float, THREADS>, smem), "latent_expand attribute");
     llm_launch(latent_expand_kernel<float, THREADS>, grid, dim3(THREADS), smem, stream, (const float *)x, ldx, (const float *)w_uv,
-               (float *)out, ldo, n_tokens, kv_rank, dv);
+               (float *)out, ldo, n_tokens, kv_rank, dv, gate, gate_stride);
   } else if (dtype == LLM_BF16) {
     LLM_CHECK_CUDA(llm_allow_smem(latent_expand_kernel<__nv_bfloat16, THREADS>, smem), "latent_expand attribute");
     llm_launch(latent_expand_kernel<__nv_bfloat16, THREADS>, grid, dim3(THREADS), smem, stream, (const __nv_bfloat16 *)x, ldx,
-               (const __nv_bfloat16 *)w_uv, (__nv_bfloat16 *)out, ldo, n_tokens, kv_rank, dv);
+               (const __nv_bfloat16 *)w_uv, (__nv_bfloat16 *)out, ldo, n_tokens, kv_rank, dv, gate, gate_stride);
   } else LLM_FAIL("latent_expand: unknown dtype %d", dtype);
   LLM_CHECK_LAUNCH("latent_expand");
   return LLM_OK;
+}
+
+LLM_EXPORT int llm_latent_expand(int dtype, const void *x, long long ldx, const void *w_uv, void *out, long long ldo, int n_tokens,
+                                 int n_heads, int kv_rank, int dv, cudaStream_t stream) {
+  return llm_latent_expand_gated(dtype, x, ldx, w_uv, out, ldo, n_tokens, n_heads, kv_rank, dv, nullptr, 0, stream);
 }

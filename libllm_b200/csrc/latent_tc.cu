@@ -98,7 +98,9 @@ LLM_EXPORT int llm_latent_rotate_q(const float *q, long long ldq, void *out, lon
 // walked with two tiles in flight, up to the one that holds the CTA's last row; a warp sits out the tiles that lie
 // wholly behind its rows.  q [T, heads * (d + rot)] (rotated), kv [T, heads * d | heads * dv], kr [T, rot]
 // (rotated), out [T, heads * dv]; sequence b owns rows seq_start[b] .. seq_start[b+1]-1 at positions 0 .. ; with
-// `window` > 0 the row at position p sees keys p - window + 1 .. p only.
+// `window` > 0 the row at position p sees keys p - window + 1 .. p only.  null_scores (a score per head; null: none): every row
+// also sees one key of that score that has no value; gate (a value per token and head, rows gate_stride apart; null: none): the
+// head's result is multiplied by its sigmoid.
 // Key rows are d + rot channels rounded up to 16 (the rest zeros), value rows DVP >= dv channels (the rest zeros).
 constexpr int LP_WARPS = 8;
 constexpr int LP_BM = 16 * LP_WARPS;
@@ -107,7 +109,8 @@ template <int DVP>
 __global__ void __launch_bounds__(LP_WARPS * 32)
 latent_prefill_kernel(const __nv_bfloat16 *__restrict__ q, long long ldq, const __nv_bfloat16 *__restrict__ kv, long long ldkv,
                       const __nv_bfloat16 *__restrict__ kr, __nv_bfloat16 *__restrict__ out, long long ldo,
-                      const int *__restrict__ seq_start, int n_heads, int d, int rot, int dv, float scale_log2, int window) {
+                      const int *__restrict__ seq_start, int n_heads, int d, int rot, int dv, float scale_log2, int window,
+                      const float *__restrict__ null_scores, const float *__restrict__ gate, long long gate_stride) {
   constexpr int LDV = DVP + 8;
   constexpr int VCH = DVP / 8;
   constexpr int NT = LT_BN / 8;
@@ -281,7 +284,13 @@ latent_prefill_kernel(const __nv_bfloat16 *__restrict__ q, long long ldq, const 
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
   }
   const int row_a = warp * 16 + g, row_b = row_a + 8;
-  const float inv_a = 1.f / l_run[0], inv_b = 1.f / l_run[1];
+  const float null_log2 = null_scores ? null_scores[h] * 1.4426950408889634f : -INFINITY;
+  float inv_a = softmax_norm_factor(m_run[0] == -INFINITY ? -INFINITY : m_run[0] * scale_log2, l_run[0], null_log2);
+  float inv_b = softmax_norm_factor(m_run[1] == -INFINITY ? -INFINITY : m_run[1] * scale_log2, l_run[1], null_log2);
+  if (gate) {
+    if (row_a < rows) inv_a *= 1.f / (1.f + expf(-gate[(size_t)(q0 + r0 + row_a) * gate_stride + h]));
+    if (row_b < rows) inv_b *= 1.f / (1.f + expf(-gate[(size_t)(q0 + r0 + row_b) * gate_stride + h]));
+  }
   __nv_bfloat16 *oa = out + (size_t)(q0 + r0 + row_a) * ldo + (size_t)h * dv + 2 * t;
   __nv_bfloat16 *ob = out + (size_t)(q0 + r0 + row_b) * ldo + (size_t)h * dv + 2 * t;
 #pragma unroll
@@ -309,20 +318,22 @@ LLM_EXPORT int llm_latent_prefill_supports(int d, int rot, int dv) {
 template <int DVP>
 static int launch_latent_prefill(const void *q, long long ldq, const void *kv, long long ldkv, const void *kr, void *out, long long ldo,
                                  const int *seq_start, int n_seqs, int max_q_len, int n_heads, int d, int rot, int dv, float scale,
-                                 int window, cudaStream_t stream) {
+                                 int window, const float *null_scores, const float *gate, long long gate_stride, cudaStream_t stream) {
   const size_t smem = latent_prefill_smem(d, rot, DVP);
   auto kern = latent_prefill_kernel<DVP>;
   LLM_CHECK_CUDA(llm_allow_smem(kern, smem), "latent_prefill attribute");
   dim3 grid((max_q_len + LP_BM - 1) / LP_BM, n_heads, n_seqs);
   llm_launch(kern, grid, dim3(LP_WARPS * 32), smem, stream, (const __nv_bfloat16 *)q, ldq, (const __nv_bfloat16 *)kv, ldkv,
-             (const __nv_bfloat16 *)kr, (__nv_bfloat16 *)out, ldo, seq_start, n_heads, d, rot, dv, scale * 1.4426950408889634f, window);
+             (const __nv_bfloat16 *)kr, (__nv_bfloat16 *)out, ldo, seq_start, n_heads, d, rot, dv, scale * 1.4426950408889634f, window, null_scores,
+             gate, gate_stride);
   LLM_CHECK_LAUNCH("latent_prefill");
   return LLM_OK;
 }
 
-LLM_EXPORT int llm_latent_prefill(const void *q, long long ldq, const void *kv, long long ldkv, const void *kr, void *out, long long ldo,
-                                  const int *seq_start, int n_seqs, int max_q_len, int n_heads, int d, int rot, int dv, float scale,
-                                  int window, cudaStream_t stream) {
+LLM_EXPORT int llm_latent_prefill_gated(const void *q, long long ldq, const void *kv, long long ldkv, const void *kr, void *out, long long ldo,
+                                        const int *seq_start, int n_seqs, int max_q_len, int n_heads, int d, int rot, int dv, float scale,
+                                        int window, const float *null_scores, const float *gate, long long gate_stride,
+                                        cudaStream_t stream) {
   if (n_seqs == 0 || max_q_len == 0) return LLM_OK;
   LLM_REQUIRE(window >= 0, "latent_prefill: bad window");
   LLM_REQUIRE(llm_latent_prefill_supports(d, rot, dv), "latent_prefill: heads of %d + %d key and %d value channels are not supported", d,
@@ -331,11 +342,18 @@ LLM_EXPORT int llm_latent_prefill(const void *q, long long ldq, const void *kv, 
                   (rot == 0 || kr),
               "latent_prefill: bad sizes");
   switch (latent_dvp(dv)) {
-    case 32: return launch_latent_prefill<32>(q, ldq, kv, ldkv, kr, out, ldo, seq_start, n_seqs, max_q_len, n_heads, d, rot, dv, scale, window, stream);
-    case 64: return launch_latent_prefill<64>(q, ldq, kv, ldkv, kr, out, ldo, seq_start, n_seqs, max_q_len, n_heads, d, rot, dv, scale, window, stream);
-    case 128: return launch_latent_prefill<128>(q, ldq, kv, ldkv, kr, out, ldo, seq_start, n_seqs, max_q_len, n_heads, d, rot, dv, scale, window, stream);
-    default: return launch_latent_prefill<256>(q, ldq, kv, ldkv, kr, out, ldo, seq_start, n_seqs, max_q_len, n_heads, d, rot, dv, scale, window, stream);
+    case 32: return launch_latent_prefill<32>(q, ldq, kv, ldkv, kr, out, ldo, seq_start, n_seqs, max_q_len, n_heads, d, rot, dv, scale, window, null_scores, gate, gate_stride, stream);
+    case 64: return launch_latent_prefill<64>(q, ldq, kv, ldkv, kr, out, ldo, seq_start, n_seqs, max_q_len, n_heads, d, rot, dv, scale, window, null_scores, gate, gate_stride, stream);
+    case 128: return launch_latent_prefill<128>(q, ldq, kv, ldkv, kr, out, ldo, seq_start, n_seqs, max_q_len, n_heads, d, rot, dv, scale, window, null_scores, gate, gate_stride, stream);
+    default: return launch_latent_prefill<256>(q, ldq, kv, ldkv, kr, out, ldo, seq_start, n_seqs, max_q_len, n_heads, d, rot, dv, scale, window, null_scores, gate, gate_stride, stream);
   }
+}
+
+LLM_EXPORT int llm_latent_prefill(const void *q, long long ldq, const void *kv, long long ldkv, const void *kr, void *out, long long ldo,
+                                  const int *seq_start, int n_seqs, int max_q_len, int n_heads, int d, int rot, int dv, float scale,
+                                  int window, cudaStream_t stream) {
+  return llm_latent_prefill_gated(q, ldq, kv, ldkv, kr, out, ldo, seq_start, n_seqs, max_q_len, n_heads, d, rot, dv, scale, window, nullptr,
+                                  nullptr, 0, stream);
 }
 
 // ---------------------------------------------------------------- every other step: all heads over the cached rows
@@ -354,7 +372,7 @@ __global__ void __launch_bounds__(LD_WARPS * 32)
 latent_decode_kernel(const __nv_bfloat16 *__restrict__ qa, long long ldq, const __nv_bfloat16 *__restrict__ cache, int page_size,
                      const int *__restrict__ tok_seq, const int *__restrict__ tok_pos, const int *__restrict__ page_table, int pt_stride,
                      int n_heads, int row, int kv_rank, int n_splits, float scale_log2, __nv_bfloat16 *__restrict__ out, long long ldo,
-                     float *__restrict__ ws_o, float *__restrict__ ws_ml, int window) {
+                     float *__restrict__ ws_o, float *__restrict__ ws_ml, int window, const float *__restrict__ null_scores) {
   constexpr int SL = MAXR / 4;           // value channels of a warp
   constexpr int DT = SL / 8;
   constexpr int NT = LT_BN / 8;
@@ -521,7 +539,11 @@ latent_decode_kernel(const __nv_bfloat16 *__restrict__ qa, long long ldq, const 
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
   }
   if (n_splits == 1) {
-    const float inv_a = 1.f / l_run[0], inv_b = 1.f / l_run[1];
+    auto factor = [&](int head, float m, float l) {
+      return softmax_norm_factor(m == -INFINITY ? -INFINITY : m * scale_log2, l,
+                                 null_scores && head < n_heads ? null_scores[head] * 1.4426950408889634f : -INFINITY);
+    };
+    const float inv_a = factor(head_a, m_run[0], l_run[0]), inv_b = factor(head_b, m_run[1], l_run[1]);
     __nv_bfloat16 *oa = out + (size_t)tok * ldo + (size_t)head_a * kv_rank + 2 * t;
     __nv_bfloat16 *ob = out + (size_t)tok * ldo + (size_t)head_b * kv_rank + 2 * t;
 #pragma unroll
@@ -556,12 +578,13 @@ latent_decode_kernel(const __nv_bfloat16 *__restrict__ qa, long long ldq, const 
   }
 }
 
-// out[t, h, :] = sum_s w_s o_s / sum_s w_s l_s with w_s = 2^(m_s - max m): one CTA per (token, head).  The runs'
+// out[t, h, :] = sum_s w_s o_s / sum_s w_s l_s with w_s = 2^(m_s - max m) (a further key without a value, null_scores, joins the
+// sum of the weights here): one CTA per (token, head).  The runs'
 // weights go through shared memory once, so that the loads of the partial sums are independent of one another.
 constexpr int LJ_MAX = 64;               // runs at most
 __global__ void __launch_bounds__(128)
 latent_join_kernel(const float *__restrict__ ws_o, const float *__restrict__ ws_ml, int n_splits, int kv_rank,
-                   __nv_bfloat16 *__restrict__ out, long long ldo, int n_heads) {
+                   __nv_bfloat16 *__restrict__ out, long long ldo, int n_heads, const float *__restrict__ null_scores) {
   __shared__ float w[LJ_MAX];
   __shared__ float inv_s;
   grid_dependents_launch();
@@ -579,7 +602,7 @@ latent_join_kernel(const float *__restrict__ ws_o, const float *__restrict__ ws_
     if (threadIdx.x == 0) {
       float l = 0.f;
       for (int s = 0; s < n_splits; ++s) l = fmaf(w[s], ml[2 * s + 1], l);       // in the order of the runs
-      inv_s = 1.f / l;
+      inv_s = softmax_norm_factor(m, l, null_scores ? null_scores[h] * 1.4426950408889634f : -INFINITY);
     }
   }
   __syncthreads();
@@ -614,21 +637,23 @@ LLM_EXPORT long long llm_latent_decode_floats_needed(int n_tokens, int n_heads, 
 template <int MAXR>
 static int launch_latent_decode(const void *qa, long long ldq, const void *cache, int page_size, const int *tok_seq, const int *tok_pos,
                                 const int *page_table, int pt_stride, int n_tokens, int n_heads, int row, int kv_rank, int n_splits,
-                                float scale, void *out, long long ldo, float *ws_o, float *ws_ml, int window, cudaStream_t stream) {
+                                float scale, void *out, long long ldo, float *ws_o, float *ws_ml, int window, const float *null_scores,
+                                cudaStream_t stream) {
   const size_t smem = latent_decode_smem(row);
   auto kern = latent_decode_kernel<MAXR>;
   LLM_CHECK_CUDA(llm_allow_smem(kern, smem), "latent_decode attribute");
   dim3 grid(n_splits, (n_heads + LD_HT - 1) / LD_HT, n_tokens);
   llm_launch(kern, grid, dim3(LD_WARPS * 32), smem, stream, (const __nv_bfloat16 *)qa, ldq, (const __nv_bfloat16 *)cache, page_size,
              tok_seq, tok_pos, page_table, pt_stride, n_heads, row, kv_rank, n_splits, scale * 1.4426950408889634f, (__nv_bfloat16 *)out,
-             ldo, ws_o, ws_ml, window);
+             ldo, ws_o, ws_ml, window, null_scores);
   LLM_CHECK_LAUNCH("latent_decode");
   return LLM_OK;
 }
 
-LLM_EXPORT int llm_latent_decode(const void *qa, long long ldq, const void *cache, int page_size, const int *tok_seq, const int *tok_pos,
-                                 const int *page_table, int pt_stride, int n_tokens, int n_heads, int kv_rank, int rot, int n_splits,
-                                 float scale, void *out, long long ldo, float *ws, int window, cudaStream_t stream) {
+LLM_EXPORT int llm_latent_decode_sinks(const void *qa, long long ldq, const void *cache, int page_size, const int *tok_seq, const int *tok_pos,
+                                       const int *page_table, int pt_stride, int n_tokens, int n_heads, int kv_rank, int rot, int n_splits,
+                                       float scale, void *out, long long ldo, float *ws, int window, const float *null_scores,
+                                       cudaStream_t stream) {
   if (n_tokens == 0) return LLM_OK;
   LLM_REQUIRE(window >= 0, "latent_decode: bad window");
   LLM_REQUIRE(llm_latent_decode_supports(kv_rank, rot), "latent_decode: rows of %d + %d channels are not supported", kv_rank, rot);
@@ -639,13 +664,20 @@ LLM_EXPORT int llm_latent_decode(const void *qa, long long ldq, const void *cach
   float *ws_o = ws, *ws_ml = ws ? ws + (size_t)n_tokens * n_heads * n_splits * kv_rank : nullptr;
   int st;
   switch (latent_maxr(kv_rank)) {
-    case 128: st = launch_latent_decode<128>(qa, ldq, cache, page_size, tok_seq, tok_pos, page_table, pt_stride, n_tokens, n_heads, row, kv_rank, n_splits, scale, out, ldo, ws_o, ws_ml, window, stream); break;
-    case 256: st = launch_latent_decode<256>(qa, ldq, cache, page_size, tok_seq, tok_pos, page_table, pt_stride, n_tokens, n_heads, row, kv_rank, n_splits, scale, out, ldo, ws_o, ws_ml, window, stream); break;
-    default: st = launch_latent_decode<512>(qa, ldq, cache, page_size, tok_seq, tok_pos, page_table, pt_stride, n_tokens, n_heads, row, kv_rank, n_splits, scale, out, ldo, ws_o, ws_ml, window, stream); break;
+    case 128: st = launch_latent_decode<128>(qa, ldq, cache, page_size, tok_seq, tok_pos, page_table, pt_stride, n_tokens, n_heads, row, kv_rank, n_splits, scale, out, ldo, ws_o, ws_ml, window, null_scores, stream); break;
+    case 256: st = launch_latent_decode<256>(qa, ldq, cache, page_size, tok_seq, tok_pos, page_table, pt_stride, n_tokens, n_heads, row, kv_rank, n_splits, scale, out, ldo, ws_o, ws_ml, window, null_scores, stream); break;
+    default: st = launch_latent_decode<512>(qa, ldq, cache, page_size, tok_seq, tok_pos, page_table, pt_stride, n_tokens, n_heads, row, kv_rank, n_splits, scale, out, ldo, ws_o, ws_ml, window, null_scores, stream); break;
   }
   if (st != LLM_OK || n_splits == 1) return st;
   llm_launch(latent_join_kernel, dim3(n_heads, n_tokens), dim3(128), 0, stream, (const float *)ws_o, (const float *)ws_ml, n_splits, kv_rank,
-             (__nv_bfloat16 *)out, ldo, n_heads);
+             (__nv_bfloat16 *)out, ldo, n_heads, null_scores);
   LLM_CHECK_LAUNCH("latent_join");
   return LLM_OK;
+}
+
+LLM_EXPORT int llm_latent_decode(const void *qa, long long ldq, const void *cache, int page_size, const int *tok_seq, const int *tok_pos,
+                                 const int *page_table, int pt_stride, int n_tokens, int n_heads, int kv_rank, int rot, int n_splits,
+                                 float scale, void *out, long long ldo, float *ws, int window, cudaStream_t stream) {
+  return llm_latent_decode_sinks(qa, ldq, cache, page_size, tok_seq, tok_pos, page_table, pt_stride, n_tokens, n_heads, kv_rank, rot, n_splits,
+                                 scale, out, ldo, ws, window, nullptr, stream);
 }

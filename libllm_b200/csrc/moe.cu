@@ -11,7 +11,10 @@
 // "output" after it (down is linear too); neither rounds a scaled input to 16 bits.
 // Gated experts, down(act(gate(x)) * up(x)): `up` then holds both matrices of an expert, rows
 // interleaved ([experts, 2 ff, width]: row 2n of gate, row 2n + 1 of up), so that a tile of the first
-// product holds a feature's two halves side by side; the weight goes on the output.
+// product holds a feature's two halves side by side; the weight goes on the output.  Their unit is act(gate) up, or with activation
+// 4 the bounded one of GluShape (common.cuh).
+// Choices beyond the experts (numbers >= n_experts) are identity experts: the row's result is its weight times the token's
+// own row; they have no tensors, are not sorted and take part in neither product.
 //
 // Two forms of the products:
 //  * moe_rows_kernel: one CTA per row, both products on the CUDA cores in 32-bit arithmetic
@@ -30,13 +33,18 @@
 
 LLM_DEFINE_LAST_ERROR(llm_moe_last_error)
 
-enum { ACT_GELU_ERF = 0, ACT_GELU_TANH = 1, ACT_SILU = 2, ACT_RELU2 = 3 };
+enum { ACT_GELU_ERF = 0, ACT_GELU_TANH = 1, ACT_SILU = 2, ACT_RELU2 = 3, ACT_GLU = 4 };
 
 __device__ __forceinline__ float activate(float z, int kind) {
   if (kind == ACT_GELU_ERF) return 0.5f * z * (1.f + erff(z * 0.70710678118654752f));
   if (kind == ACT_GELU_TANH) return 0.5f * z * (1.f + tanhf(0.79788456080286536f * (z + 0.044715f * z * z * z)));
   if (kind == ACT_RELU2) return z > 0.f ? z * z : 0.f;     // the square of max(z, 0)
   return z / (1.f + expf(-z));
+}
+
+// the unit of a gated expert
+__device__ __forceinline__ float gated_unit(float g, float u, int act, const GluShape &glu) {
+  return act == ACT_GLU ? glu_value(g, u, glu) : activate(g, act) * u;
 }
 
 // ---------------------------------------------------------------- choice of experts
@@ -275,7 +283,7 @@ LLM_EXPORT int llm_row_gate(const float *x, long long x_stride, float *out, long
 // One CTA.  offsets[e] .. offsets[e + 1]: the sorted places of expert e's rows; perm[place] = row;
 // tiles[0] = number of row tiles, then (expert, first place) per tile of at most `tile_rows` rows of
 // one expert.  Which place a row gets within its expert depends on the order the threads arrive
-// in; no result depends on it.
+// in; no result depends on it.  Rows of identity experts (chosen >= n_experts) get no place.
 __global__ void __launch_bounds__(1024)
 moe_sort_kernel(const int *__restrict__ chosen, int n_rows, int n_experts, int tile_rows, int *__restrict__ offsets,
                 int *__restrict__ perm, int *__restrict__ tiles) {
@@ -285,7 +293,8 @@ moe_sort_kernel(const int *__restrict__ chosen, int n_rows, int n_experts, int t
   grid_dependency_wait();
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) counts[e] = 0;
   __syncthreads();
-  for (int r = threadIdx.x; r < n_rows; r += blockDim.x) atomicAdd(&counts[chosen[r]], 1);
+  for (int r = threadIdx.x; r < n_rows; r += blockDim.x)
+    if (chosen[r] < n_experts) atomicAdd(&counts[chosen[r]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int o = 0, n_tiles = 0;
@@ -303,7 +312,8 @@ moe_sort_kernel(const int *__restrict__ chosen, int n_rows, int n_experts, int t
     tiles[0] = n_tiles;
   }
   __syncthreads();
-  for (int r = threadIdx.x; r < n_rows; r += blockDim.x) perm[atomicAdd(&cursor[chosen[r]], 1)] = r;
+  for (int r = threadIdx.x; r < n_rows; r += blockDim.x)
+    if (chosen[r] < n_experts) perm[atomicAdd(&cursor[chosen[r]], 1)] = r;
 }
 
 LLM_EXPORT int llm_moe_sort(const int *chosen, int n_rows, int n_experts, int tile_rows, int *offsets, int *perm, int *tiles,
@@ -331,7 +341,7 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 moe_rows_kernel(const T *__restrict__ x, long long ldx, const T *__restrict__ up, const T *__restrict__ down,
                 const int *__restrict__ chosen, const float *__restrict__ weight, int n_tokens, int top, int width, int ff,
-                int act, int weight_on, int gated, float *__restrict__ out) {
+                int act, int weight_on, int gated, int n_experts, GluShape glu, float *__restrict__ out) {
   extern __shared__ float shf[];               // x row [width], hidden [ff]
   float *xs = shf, *hs = shf + width;
   grid_dependents_launch();
@@ -340,6 +350,10 @@ moe_rows_kernel(const T *__restrict__ x, long long ldx, const T *__restrict__ up
   const int e = chosen[r];
   const float w = weight[r];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  if (e >= n_experts) {                        // an identity expert
+    for (int c = threadIdx.x; c < width; c += 256) out[((size_t)j * n_tokens + t) * width + c] = w * to_float(x[(size_t)t * ldx + c]);
+    return;
+  }
   for (int c = threadIdx.x; c < width; c += 256) xs[c] = to_float(x[(size_t)t * ldx + c]);
   __syncthreads();
   const T *wu = up + (size_t)e * ff * width * (gated ? 2 : 1);
@@ -347,7 +361,7 @@ moe_rows_kernel(const T *__restrict__ x, long long ldx, const T *__restrict__ up
     if (gated) {
       const float g = dot_cols(wu + (size_t)(2 * n) * width, xs, width, lane);
       const float u = dot_cols(wu + (size_t)(2 * n + 1) * width, xs, width, lane);
-      if (lane == 0) hs[n] = w * (activate(g, act) * u);
+      if (lane == 0) hs[n] = w * gated_unit(g, u, act, glu);
       continue;
     }
     const float v = dot_cols(wu + (size_t)n * width, xs, width, lane);
@@ -362,9 +376,10 @@ moe_rows_kernel(const T *__restrict__ x, long long ldx, const T *__restrict__ up
   }
 }
 
-LLM_EXPORT int llm_moe_rows(int dtype, const void *x, long long ldx, const void *up, const void *down, const int *chosen,
-                            const float *weight, int n_tokens, int top, int width, int ff, int act, int weight_on, int gated,
-                            float *out, cudaStream_t stream) {
+LLM_EXPORT int llm_moe_rows_glu(int dtype, const void *x, long long ldx, const void *up, const void *down, const int *chosen,
+                                const float *weight, int n_tokens, int n_experts, int top, int width, int ff, int act, int weight_on, int gated,
+                                float limit, float slope, float shift, float *out, cudaStream_t stream) {
+  const GluShape glu{limit, slope, shift};
   if (n_tokens == 0) return LLM_OK;
   LLM_REQUIRE(n_tokens > 0 && top > 0 && width > 0 && ff > 0, "moe_rows: bad sizes");
   LLM_REQUIRE(!gated || weight_on == 1, "moe_rows: gated experts take their weight on the output");
@@ -373,13 +388,47 @@ LLM_EXPORT int llm_moe_rows(int dtype, const void *x, long long ldx, const void 
   if (dtype == LLM_F32) {
     LLM_CHECK_CUDA(llm_allow_smem(moe_rows_kernel<float>, smem), "moe_rows attribute");
     llm_launch(moe_rows_kernel<float>, dim3(n_tokens * top), dim3(256), smem, stream, (const float *)x, ldx, (const float *)up,
-               (const float *)down, chosen, weight, n_tokens, top, width, ff, act, weight_on, gated, out);
+               (const float *)down, chosen, weight, n_tokens, top, width, ff, act, weight_on, gated, n_experts, glu, out);
   } else {
     LLM_CHECK_CUDA(llm_allow_smem(moe_rows_kernel<__nv_bfloat16>, smem), "moe_rows attribute");
     llm_launch(moe_rows_kernel<__nv_bfloat16>, dim3(n_tokens * top), dim3(256), smem, stream, (const __nv_bfloat16 *)x, ldx,
-               (const __nv_bfloat16 *)up, (const __nv_bfloat16 *)down, chosen, weight, n_tokens, top, width, ff, act, weight_on, gated, out);
+               (const __nv_bfloat16 *)up, (const __nv_bfloat16 *)down, chosen, weight, n_tokens, top, width, ff, act, weight_on, gated, n_experts, glu, out);
   }
   LLM_CHECK_LAUNCH("moe_rows");
+  return LLM_OK;
+}
+LLM_EXPORT int llm_moe_rows(int dtype, const void *x, long long ldx, const void *up, const void *down, const int *chosen,
+                            const float *weight, int n_tokens, int top, int width, int ff, int act, int weight_on, int gated,
+                            float *out, cudaStream_t stream) {
+  return llm_moe_rows_glu(dtype, x, ldx, up, down, chosen, weight, n_tokens, 0x7fffffff, top, width, ff, act, weight_on, gated, 0.f, 1.f, 0.f,
+                          out, stream);
+}
+
+// ---------------------------------------------------------------- identity experts alone
+// out[choice, token] = weight * x[token] for every row whose choice is no expert (tokens' rows in eights where they allow it).
+template <typename T>
+__device__ __forceinline__ void identity_row(const T *__restrict__ x, float w, float *__restrict__ o, int c0, int width) {
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+    if (c0 + i < width) o[c0 + i] = w * to_float(x[c0 + i]);
+}
+__global__ void moe_identity_kernel(const __nv_bfloat16 *__restrict__ x, long long ldx, const int *__restrict__ chosen,
+                                    const float *__restrict__ weight, int n_tokens, int n_experts, int top, int width,
+                                    float *__restrict__ out) {
+  grid_dependents_launch();
+  grid_dependency_wait();
+  const int r = blockIdx.x, t = r / top;
+  if (chosen[r] < n_experts) return;
+  for (int c0 = threadIdx.x * 8; c0 < width; c0 += blockDim.x * 8)
+    identity_row(x + (size_t)t * ldx, weight[r], out + ((size_t)(r - t * top) * n_tokens + t) * width, c0, width);
+}
+LLM_EXPORT int llm_moe_identity(const void *x, long long ldx, const int *chosen, const float *weight, int n_tokens, int n_experts, int top,
+                                int width, float *out, cudaStream_t stream) {
+  if (n_tokens == 0) return LLM_OK;
+  LLM_REQUIRE(n_tokens > 0 && top > 0 && width > 0, "moe_identity: bad sizes");
+  llm_launch(moe_identity_kernel, dim3(n_tokens * top), dim3(128), 0, stream, (const __nv_bfloat16 *)x, ldx, chosen, weight, n_tokens, n_experts,
+             top, width, out);
+  LLM_CHECK_LAUNCH("moe_identity");
   return LLM_OK;
 }
 
@@ -393,7 +442,7 @@ constexpr int GLD = GK + GPAD;                 // 40 values = 80 bytes a row: ld
 __global__ void __launch_bounds__(256)
 moe_grouped_kernel(const __nv_bfloat16 *__restrict__ A, long long lda, const __nv_bfloat16 *__restrict__ W, int N, int K,
                    const int *__restrict__ offsets, const int *__restrict__ perm, const int *__restrict__ tiles,
-                   const float *__restrict__ weight, int n_tokens, int top, int act, int weight_on, int second, int gated,
+                   const float *__restrict__ weight, int n_tokens, int top, int act, int weight_on, int second, int gated, GluShape glu,
                    __nv_bfloat16 *__restrict__ mid, float *__restrict__ out) {
   __shared__ __align__(16) __nv_bfloat16 As[GSTAGES][GM][GLD];
   __shared__ __align__(16) __nv_bfloat16 Bs[GSTAGES][GN][GLD];
@@ -484,7 +533,7 @@ moe_grouped_kernel(const __nv_bfloat16 *__restrict__ A, long long lda, const __n
         const float v0 = acc[a][b][half * 2], v1 = acc[a][b][half * 2 + 1];
         if (!second && gated) {
           // columns n (even: the gate's row of feature n / 2) and n + 1 (the up row of the same feature)
-          if (n + 1 < N) mid[(size_t)(place0 + r) * (N / 2) + n / 2] = __float2bfloat16_rn(w * (activate(v0, act) * v1));
+          if (n + 1 < N) mid[(size_t)(place0 + r) * (N / 2) + n / 2] = __float2bfloat16_rn(w * gated_unit(v0, v1, act, glu));
         } else if (!second) {
           __nv_bfloat16 *dst = mid + (size_t)(place0 + r) * N;
           const float y0 = weight_on == 0 ? activate(w * v0, act) : w * activate(v0, act);
@@ -501,9 +550,11 @@ moe_grouped_kernel(const __nv_bfloat16 *__restrict__ A, long long lda, const __n
 }
 
 // x [tokens, width] bfloat16; mid [tokens * top, ff] bfloat16 scratch; out [top, tokens, width] 32-bit.
-LLM_EXPORT int llm_moe_grouped(const void *x, long long ldx, const void *up, const void *down, const int *offsets, const int *perm,
-                               const int *tiles, const float *weight, int n_tokens, int n_experts, int top, int width, int ff,
-                               int act, int weight_on, int gated, void *mid, float *out, cudaStream_t stream) {
+LLM_EXPORT int llm_moe_grouped_glu(const void *x, long long ldx, const void *up, const void *down, const int *offsets, const int *perm,
+                                   const int *tiles, const float *weight, int n_tokens, int n_experts, int top, int width, int ff,
+                                   int act, int weight_on, int gated, float limit, float slope, float shift, void *mid, float *out,
+                                   cudaStream_t stream) {
+  const GluShape glu{limit, slope, shift};
   if (n_tokens == 0) return LLM_OK;
   LLM_REQUIRE(n_tokens > 0 && top > 0 && width > 0 && ff > 0 && n_experts > 0, "moe_grouped: bad sizes");
   LLM_REQUIRE(!gated || weight_on == 1, "moe_grouped: gated experts take their weight on the output");
@@ -514,14 +565,20 @@ LLM_EXPORT int llm_moe_grouped(const void *x, long long ldx, const void *up, con
   const int max_tiles = min(n_experts, n_rows) + n_rows / GM;
   const int n_first = gated ? 2 * ff : ff;
   llm_launch(moe_grouped_kernel, dim3(max_tiles, (n_first + GN - 1) / GN), dim3(256), 0, stream, (const __nv_bfloat16 *)x, ldx,
-             (const __nv_bfloat16 *)up, n_first, width, offsets, perm, tiles, weight, n_tokens, top, act, weight_on, 0, gated,
+             (const __nv_bfloat16 *)up, n_first, width, offsets, perm, tiles, weight, n_tokens, top, act, weight_on, 0, gated, glu,
              (__nv_bfloat16 *)mid, (float *)nullptr);
   LLM_CHECK_LAUNCH("moe_grouped (first product)");
   llm_launch(moe_grouped_kernel, dim3(max_tiles, (width + GN - 1) / GN), dim3(256), 0, stream, (const __nv_bfloat16 *)mid,
-             (long long)ff, (const __nv_bfloat16 *)down, width, ff, offsets, perm, tiles, weight, n_tokens, top, act, weight_on, 1, 0,
+             (long long)ff, (const __nv_bfloat16 *)down, width, ff, offsets, perm, tiles, weight, n_tokens, top, act, weight_on, 1, 0, glu,
              (__nv_bfloat16 *)nullptr, out);
   LLM_CHECK_LAUNCH("moe_grouped (second product)");
   return LLM_OK;
+}
+LLM_EXPORT int llm_moe_grouped(const void *x, long long ldx, const void *up, const void *down, const int *offsets, const int *perm,
+                               const int *tiles, const float *weight, int n_tokens, int n_experts, int top, int width, int ff,
+                               int act, int weight_on, int gated, void *mid, float *out, cudaStream_t stream) {
+  return llm_moe_grouped_glu(x, ldx, up, down, offsets, perm, tiles, weight, n_tokens, n_experts, top, width, ff, act, weight_on, gated, 0.f,
+                             1.f, 0.f, mid, out, stream);
 }
 LLM_EXPORT int llm_moe_grouped_supports(int width, int ff) { return width % 8 == 0 && ff % 8 == 0; }
 
@@ -580,20 +637,31 @@ LLM_EXPORT int llm_activation(int in_dtype, int dtype, const void *in, void *out
 
 // ---------------------------------------------------------------- the tokens' rows in sorted order
 // xs[place] = x[perm[place] / top], 16 bytes to a thread: the operand of the tensor-memory form of the first
-// product (csrc/moe_tc.cu), whose loads want the rows of a tile one behind the other.
+// product (csrc/moe_tc.cu), whose loads want the rows of a tile one behind the other.  With `chosen` (some rows are identity
+// experts') only the first offsets[n_experts] places hold rows, and the identity experts' results go to `out` on the way.
 __global__ void moe_gather_kernel(const uint4 *__restrict__ x, long long ldx16, const int *__restrict__ perm, int top,
-                                  int width16, size_t total, uint4 *__restrict__ xs) {
+                                  int width16, size_t total, uint4 *__restrict__ xs, const int *__restrict__ chosen,
+                                  const int *__restrict__ offsets, const float *__restrict__ weight, int n_experts, int n_tokens,
+                                  float *__restrict__ out) {
   grid_dependents_launch();
   grid_dependency_wait();
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
     const size_t place = idx / width16;
     const int c = (int)(idx - place * width16);
+    if (chosen) {
+      const int r = (int)place, t = r / top;               // the same number as a row
+      if (chosen[r] >= n_experts)
+        identity_row((const __nv_bfloat16 *)(x + (size_t)t * ldx16), weight[r], out + ((size_t)(r - t * top) * n_tokens + t) * width16 * 8, c * 8,
+                     width16 * 8);
+      if (r >= offsets[n_experts]) continue;
+    }
     xs[idx] = x[(size_t)(perm[place] / top) * ldx16 + c];
   }
 }
 
-LLM_EXPORT int llm_moe_gather(const void *x, long long ldx, const int *perm, int n_rows, int top, int width, void *xs,
-                              cudaStream_t stream) {
+LLM_EXPORT int llm_moe_gather_identity(const void *x, long long ldx, const int *perm, int n_rows, int top, int width, void *xs,
+                                       const int *chosen, const int *offsets, const float *weight, int n_experts, float *out,
+                                       cudaStream_t stream) {
   if (n_rows == 0) return LLM_OK;
   LLM_REQUIRE(n_rows > 0 && top > 0 && width % 8 == 0 && ldx % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)xs % 16 == 0,
               "moe_gather: rows of bfloat16 in multiples of 8, 16-byte aligned");
@@ -601,7 +669,11 @@ LLM_EXPORT int llm_moe_gather(const void *x, long long ldx, const int *perm, int
   size_t blocks = (total + 255) / 256;
   if (blocks > (size_t)sm_count() * 32) blocks = (size_t)sm_count() * 32;
   llm_launch_after(moe_gather_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, (const uint4 *)x, ldx / 8, perm, top, width / 8, total,
-             (uint4 *)xs);
+             (uint4 *)xs, chosen, offsets, weight, n_experts, n_rows / top, out);
   LLM_CHECK_LAUNCH("moe_gather");
   return LLM_OK;
+}
+LLM_EXPORT int llm_moe_gather(const void *x, long long ldx, const int *perm, int n_rows, int top, int width, void *xs,
+                              cudaStream_t stream) {
+  return llm_moe_gather_identity(x, ldx, perm, n_rows, top, width, xs, nullptr, nullptr, nullptr, 0, nullptr, stream);
 }

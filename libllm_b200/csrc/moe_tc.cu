@@ -17,7 +17,8 @@
 //                   out[choice][token].
 // Gated experts (csrc/moe.cu has the layout: rows of gate and up interleaved, N = 2 ff): a lane of the first
 // epilogue holds one weight row, so neighbouring lanes hold a feature's gate and up values for the same token;
-// the even lane takes its neighbour's by a shuffle and stores weight * act(gate) * up to mid[place, feature].
+// the even lane takes its neighbour's by a shuffle and stores weight * act(gate) * up (activation 4: weight times the bounded
+// unit of GluShape) to mid[place, feature].
 // A box of sorted rows may reach into the next expert's rows, and a box of weight rows into the next
 // expert's: such products are computed and never stored.  Every wait has a time limit, after which
 // the CTA records a code in `status`, lets its loads land, frees its tensor memory and returns.
@@ -58,7 +59,7 @@ template <int TN, int ACT, bool GATED>
 __global__ void __launch_bounds__(MT_THREADS, 1)
 moe_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, int N, int K,
               const int *__restrict__ offsets, const int *__restrict__ perm, const int *__restrict__ tiles,
-              const float *__restrict__ weight, int n_tokens, int top, int weight_on,
+              const float *__restrict__ weight, int n_tokens, int top, int weight_on, GluShape glu,
               __nv_bfloat16 *__restrict__ mid, float *__restrict__ out, int *status) {
   using S = MtShape<TN>;
   constexpr int STAGES = S::STAGES;
@@ -213,7 +214,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__
             } else if (GATED) {
               const float w = __shfl_sync(0xffffffffu, my_w[c0 >> 5], (c0 & 31) + i);
               const float other = __shfl_xor_sync(0xffffffffu, v[i], 1);     // the odd lane's value: the up row
-              y[i] = w * (mt_activate<SECOND ? 0 : ACT>(v[i]) * other);
+              y[i] = w * (ACT == 4 ? glu_value(v[i], other, glu) : mt_activate<SECOND ? 0 : ACT>(v[i]) * other);
             } else {
               const float w = __shfl_sync(0xffffffffu, my_w[c0 >> 5], (c0 & 31) + i);
               const float a = mt_activate<SECOND ? 0 : ACT>(weight_on == 0 ? w * v[i] : v[i]);
@@ -250,7 +251,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__
 
 template <int TN, int ACT, bool GATED>
 int launch_moe_tc(const void *a, long long n_rows, const void *w, int n_experts, int N, int K, const int *offsets,
-                  const int *perm, const int *tiles, const float *weight, int n_tokens, int top, int weight_on, void *mid,
+                  const int *perm, const int *tiles, const float *weight, int n_tokens, int top, int weight_on, const GluShape &glu, void *mid,
                   float *out, int *status, cudaStream_t stream) {
   using S = MtShape<TN>;
   CUtensorMap map_w, map_x;
@@ -263,7 +264,7 @@ int launch_moe_tc(const void *a, long long n_rows, const void *w, int n_experts,
   const long long most = ((long long)(n_experts < n_rows ? n_experts : n_rows) + n_rows / TN) * ((N + MT_ROWS - 1) / MT_ROWS);
   const int grid = (int)(most < sm_count() ? most : sm_count());
   LLM_CHECK_CUDA(llm_launch_after(kern, dim3(grid), dim3(MT_THREADS), S::SMEM, stream, map_w, map_x, N, K, offsets, perm, tiles, weight,
-                            n_tokens, top, weight_on, (__nv_bfloat16 *)mid, out, status),
+                            n_tokens, top, weight_on, glu, (__nv_bfloat16 *)mid, out, status),
                  "moe_tc launch");
   return LLM_OK;
 }
@@ -277,9 +278,11 @@ LLM_EXPORT int llm_moe_tc_supports(int width, int ff) { return width % 8 == 0 &&
 // xs [tokens * top, width] bfloat16: the tokens' rows in sorted order; up [experts, ff, width], down
 // [experts, width, ff]; mid [tokens * top, ff] bfloat16 scratch; out [top, tokens, width] 32-bit.  The table
 // `tiles` must have been made with tiles of llm_moe_tc_tile_rows(tokens * top) rows.
-LLM_EXPORT int llm_moe_tc(const void *xs, const void *up, const void *down, const int *offsets, const int *perm,
-                          const int *tiles, const float *weight, int n_tokens, int n_experts, int top, int width, int ff,
-                          int act, int weight_on, int gated, void *mid, float *out, int *status, cudaStream_t stream) {
+LLM_EXPORT int llm_moe_tc_glu(const void *xs, const void *up, const void *down, const int *offsets, const int *perm,
+                              const int *tiles, const float *weight, int n_tokens, int n_experts, int top, int width, int ff,
+                              int act, int weight_on, int gated, float limit, float slope, float shift, void *mid, float *out, int *status,
+                              cudaStream_t stream) {
+  const GluShape glu{limit, slope, shift};
   if (n_tokens == 0) return LLM_OK;
   LLM_REQUIRE(!gated || weight_on == 1, "moe_tc: gated experts take their weight on the output");
   LLM_REQUIRE(n_tokens > 0 && top > 0 && width > 0 && ff > 0 && n_experts > 0, "moe_tc: bad sizes");
@@ -287,22 +290,29 @@ LLM_EXPORT int llm_moe_tc(const void *xs, const void *up, const void *down, cons
   LLM_REQUIRE((uintptr_t)xs % 16 == 0 && (uintptr_t)up % 16 == 0 && (uintptr_t)down % 16 == 0 && (uintptr_t)mid % 16 == 0,
               "moe_tc: operands must be 16-byte aligned");
   LLM_REQUIRE((long long)n_experts * (2 * ff > width ? 2 * ff : width) < (1ll << 31), "moe_tc: the stacked weights have too many rows");
-  LLM_REQUIRE(act >= 0 && act <= 3, "moe_tc: unknown activation %d", act);
+  LLM_REQUIRE(act >= 0 && act <= (gated ? 4 : 3), "moe_tc: unknown activation %d", act);
   const long long n_rows = (long long)n_tokens * top;
 #define MT_FIRST(TN, ACT, GATED)                                                                                             \
   launch_moe_tc<TN, ACT, GATED>(xs, n_rows, up, n_experts, GATED ? 2 * ff : ff, width, offsets, perm, tiles, weight, n_tokens, top, \
-                                weight_on, mid, nullptr, status, stream)
-#define MT_ACTS(TN, GATED) (act == 0 ? MT_FIRST(TN, 0, GATED) : act == 1 ? MT_FIRST(TN, 1, GATED) : act == 2 ? MT_FIRST(TN, 2, GATED) : MT_FIRST(TN, 3, GATED))
+                                weight_on, glu, mid, nullptr, status, stream)
+#define MT_ACTS(TN, GATED) (act == 0 ? MT_FIRST(TN, 0, GATED) : act == 1 ? MT_FIRST(TN, 1, GATED) : act == 2 ? MT_FIRST(TN, 2, GATED) : act == 3 ? MT_FIRST(TN, 3, GATED) : MT_FIRST(TN, GATED ? 4 : 0, GATED))
 #define MT_BOTH(TN)                                                                                                          \
   do {                                                                                                                       \
     const int rc = gated ? MT_ACTS(TN, true) : MT_ACTS(TN, false);                                                           \
     if (rc != LLM_OK) return rc;                                                                                             \
     return launch_moe_tc<TN, -1, false>(mid, n_rows, down, n_experts, width, ff, offsets, perm, tiles, weight, n_tokens, top, \
-                                        weight_on, nullptr, out, status, stream);                                            \
+                                        weight_on, glu, nullptr, out, status, stream);                                       \
   } while (0)
   if (llm_moe_tc_tile_rows((int)n_rows) == 32) MT_BOTH(32);
   MT_BOTH(128);
 #undef MT_BOTH
 #undef MT_ACTS
 #undef MT_FIRST
+}
+
+LLM_EXPORT int llm_moe_tc(const void *xs, const void *up, const void *down, const int *offsets, const int *perm,
+                          const int *tiles, const float *weight, int n_tokens, int n_experts, int top, int width, int ff,
+                          int act, int weight_on, int gated, void *mid, float *out, int *status, cudaStream_t stream) {
+  return llm_moe_tc_glu(xs, up, down, offsets, perm, tiles, weight, n_tokens, n_experts, top, width, ff, act, weight_on, gated, 0.f, 1.f, 0.f,
+                        mid, out, status, stream);
 }

@@ -764,7 +764,7 @@ conv_rope_place_kernel(const float *__restrict__ qkv, long long ld, const float 
                        T *__restrict__ vcache, int page_size, int write_cache, int n_tokens, int n_chunks) {
   grid_dependents_launch();
   const int half = rot_dim / 2, rot_units = half / V, head_units = rot_units + (d - rot_dim) / V;
-  const int qk_units = (n_heads + n_kv) * head_units, n_units = qk_units + n_kv * (dv / V);
+  const int qk_units = (n_heads + n_kv) * head_units, n_units = write_cache ? qk_units + n_kv * (dv / V) : n_heads * head_units;   // a run without keys of its own: q alone
   const int unit = blockIdx.y * CP_THREADS + threadIdx.x;
   const int channels = (n_heads + n_kv) * d + n_kv * dv;
   // the unit's channels: c0 and, where it is rotated, c1 = c0 + half
@@ -945,7 +945,8 @@ LLM_EXPORT int llm_conv_rope_place(int dtype, const float *qkv, long long ld, co
   LLM_REQUIRE(rot_dim % 2 == 0 && rot_dim <= d && rot_dim >= 0 && (rot_dim == 0 || (table && table_rows > 0)),
               "conv_rope_place: rotated width %d does not fit head size %d", rot_dim, d);
   const long long channels = (long long)(n_heads + n_kv) * d + (long long)n_kv * dv;
-  LLM_REQUIRE(ld >= channels, "conv_rope_place: the stacked rows are too short");
+  LLM_REQUIRE(write_cache || taps == 1, "conv_rope_place: a run that appends nothing has no convolution over keys and values");
+  LLM_REQUIRE(ld >= (write_cache ? channels : (long long)n_heads * d), "conv_rope_place: the stacked rows are too short");
   const int n_chunks = single_tokens && taps > 1 ? 0 : (n_tokens + CP_ROWS - 1) / CP_ROWS, n_own = taps > 1 ? n_seqs : 0;
   const int esz = dtype == LLM_F32 ? 4 : 2;
   const bool vec = d % 4 == 0 && dv % 4 == 0 && rot_dim % 8 == 0 && ld % 4 == 0 && q_stride % 4 == 0 && (uintptr_t)qkv % 16 == 0 &&
@@ -961,7 +962,8 @@ LLM_EXPORT int llm_conv_rope_place(int dtype, const float *qkv, long long ld, co
              (T *)kcache, (T *)vcache, page_size, write_cache, n_tokens, n_chunks)
 #define CP_TAPS(T, V)                  \
   do {                                 \
-    if (taps <= 4) CP_GO(T, V, 4);     \
+    if (taps == 1) CP_GO(T, V, 1);     \
+    else if (taps <= 4) CP_GO(T, V, 4); \
     else CP_GO(T, V, CP_MAX_TAPS);     \
   } while (0)
   if (dtype == LLM_F32 && vec) CP_TAPS(float, 4);

@@ -97,10 +97,15 @@ TensorNeed Model::added_need(const std::string &name, int64_t rows) const {
   return {name, {rows, spec_.hidden}, TensorRole::Vector, false, 0.1f};
 }
 
+TensorNeed Model::pairs_need() const { return {spec_.token_pairs.table, {spec_.token_pairs.buckets + 1, spec_.hidden}}; }
+TensorNeed Model::token_table_need() const { return {spec_.token_table, {spec_.vocab_size, spec_.token_table_width}}; }
+
 std::vector<TensorNeed> Model::tensor_needs() const {
   std::vector<TensorNeed> needs;
   needs.push_back({spec_.embedding, {spec_.vocab_size, spec_.hidden}});
   if (!spec_.position_table.empty()) needs.push_back({spec_.position_table, {spec_.max_positions, spec_.hidden}});
+  if (!spec_.token_pairs.table.empty()) needs.push_back(pairs_need());
+  if (!spec_.token_table.empty()) needs.push_back(token_table_need());
   for (const auto &l : layers_)
     for (auto &n : l->tensor_needs()) needs.push_back(n);
   for (auto &n : final_norm_->tensor_needs()) needs.push_back(n);
@@ -129,6 +134,8 @@ void Model::load_with(const Loader &loader) {
   const std::vector<TensorNeed> needs = tensor_needs();
   embedding_ = loader.fetch(needs.front());
   if (!spec_.position_table.empty()) positions_ = loader.fetch(needs[1]);
+  if (!spec_.token_pairs.table.empty()) token_pairs_ = loader.fetch(pairs_need());
+  if (!spec_.token_table.empty()) token_table_ = loader.fetch(token_table_need());
   for (auto &l : layers_) l->load(loader);
   final_norm_->load(loader);
   for (auto &kv : input_mixes_) kv.second = loader.fetch({kv.first, {spec_.hidden, 2 * spec_.hidden}});
@@ -171,6 +178,7 @@ void Model::cache_needs(std::vector<CacheNeed> *needs, std::vector<char> *has) c
 std::vector<std::vector<StateNeed>> Model::state_needs() const {
   std::vector<std::vector<StateNeed>> out;
   for (const auto &e : spec_.schedule) out.push_back(layers_[(size_t)e.layer]->state_need());
+  if (!spec_.token_pairs.table.empty()) out.push_back({{"last_token", {1}, DType::I32}});
   return out;
 }
 
@@ -209,8 +217,26 @@ Act Model::forward(StepContext &ctx, KVCache &cache, const std::vector<const int
   const int64_t T = ctx.n_tokens, H = spec_.hidden;
   // several copies of the stream lie one behind the other; the token rows go to the first, the others are equal to it
   float *resid = ctx.arena->alloc_n<float>((size_t)(T * H) * (size_t)spec_.streams);
-  kernels::embedding(embedding_.dtype, embedding_.data(), ctx.tokens, fed_tokens, fed_rows, resid, (int)T, (int)H,
-                     (int)spec_.vocab_size, ctx.stream, positions_.data(), (int)positions_.rows, ctx.tok_pos);
+  if (spec_.token_pairs.table.empty() && spec_.token_table.empty()) {
+    kernels::embedding(embedding_.dtype, embedding_.data(), ctx.tokens, fed_tokens, fed_rows, resid, (int)T, (int)H,
+                       (int)spec_.vocab_size, ctx.stream, positions_.data(), (int)positions_.rows, ctx.tok_pos);
+  } else {
+    kernels::TokenPairs pairs;
+    if (!spec_.token_pairs.table.empty()) {
+      pairs.table = token_pairs_.data();
+      pairs.buckets = spec_.token_pairs.buckets;
+      pairs.mul_prev = spec_.token_pairs.mul_prev;
+      pairs.mul_cur = spec_.token_pairs.mul_cur;
+      pairs.last = (int *)cache.state_view((int)spec_.schedule.size()).at(0).data;
+    }
+    int *ids = spec_.token_table.empty() ? nullptr : ctx.arena->alloc_n<int>((size_t)T);
+    kernels::embedding_pairs(embedding_.dtype, embedding_.data(), ctx.tokens, fed_tokens, fed_rows, resid, (int)T, (int)H,
+                             (int)spec_.vocab_size, ctx.stream, positions_.data(), (int)positions_.rows, ctx.tok_pos, ids, pairs, ctx.tok_seq,
+                             ctx.seq_start, ctx.seq_slot);
+    ctx.token_ids = ids;
+    ctx.token_table = token_table_.data();
+    ctx.token_table_width = spec_.token_table_width;
+  }
   if (spec_.embedding_scale != 1.0) kernels::scale_rows(resid, T * H, (float)spec_.embedding_scale, ctx.stream);
   float *x0 = nullptr;                       // the token rows, kept for the runs that mix them in again
   if (needs_tokens_) {

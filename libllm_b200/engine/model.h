@@ -47,6 +47,7 @@ class Model {
 
   // What the cache must hold, per schedule entry.
   void cache_needs(std::vector<CacheNeed> *needs, std::vector<char> *has) const;
+  // Per schedule entry, then what the model itself keeps (a sequence's last token, where rows of token pairs are added).
   std::vector<std::vector<StateNeed>> state_needs() const;
 
   // Runs the tokens of `ctx` through every scheduled layer and returns 32-bit logits for
@@ -67,12 +68,15 @@ class Model {
   std::vector<std::unique_ptr<Block>> layers_;
   std::unique_ptr<Norm> final_norm_;
   Weight embedding_, head_own_, positions_;        // positions_: ModelSpec::position_table, in the token table's type
+  Weight token_pairs_, token_table_;               // ModelSpec::token_pairs, ModelSpec::token_table
   std::map<std::string, Weight> input_mixes_;      // ScheduleEntry::input_mix -> [hidden, 2 * hidden]
   std::map<std::string, Weight> added_vectors_;    // ScheduleEntry::add_vector -> [rows, hidden], 32-bit
   bool needs_tokens_ = false;                      // some run mixes or adds the token rows in again
   void mix_input(StepContext &ctx, ResidualStream &stream, const float *x0, const Weight &w);
   void add_to_input(StepContext &ctx, ResidualStream &stream, const float *x0, const float *vec);
   TensorNeed added_need(const std::string &name, int64_t rows) const;
+  TensorNeed pairs_need() const;
+  TensorNeed token_table_need() const;
   const Weight *head_ = nullptr;
   bool loaded_ = false;
 };

@@ -162,7 +162,7 @@ std::vector<double> rotary_frequencies(int64_t rotary_dim, double theta, const J
     return freqs;
   }
   if (type != "llama3") LLM_THROW(Config, "rope scaling '%s' is not supported (llama3, yarn)", type.c_str());
-  const double orig = (double)r.integer("original_max_position_embeddings");
+  const double orig = r.number("original_max_position_embeddings");
   const double lo = r.number("low_freq_factor"), hi = r.number("high_freq_factor"), factor = r.number("factor");
   for (auto &f : freqs) {
     const double wavelen = 2.0 * M_PI / f;
@@ -285,9 +285,14 @@ class RotaryEmbedding : public PositionEncoding {
 //                its head_dim channels, sqrt(mean + eps), without a weight (a rotation of pairs (i, i + rotary_dim/2) or none)
 //   null_key     a number s0: every query also sees one key whose score is s0 and which has no value, so that
 //                p_j = exp(s_j) / (exp(s0) + sum exp(s_j)); with 0 the softmax has one added to its denominator
+//   null_scores  a vector [n_heads]: such a score for every head (learned "sinks")
+//   k, v         both left out: the run has no keys and values of its own; the schedule gives it another run's cache
+//                (ScheduleEntry::cache_from), which it reads with its own queries and mask
+//   cache_window with `window`: how many last positions the cache keeps, for later runs that read this run's cache through a wider
+//                window (0: all of them)
 //   q_bias, k_bias, v_bias   names of the biases (default: the matrix's name with "weight" replaced by "bias").
-//                Without a rotation the biases are added where q, k and v are placed (32-bit), so that the
-//                product itself runs on the tensor cores like any other
+//                With the library's own rotation, or none, the biases are added where q, k and v are placed (32-bit), so
+//                that the product itself runs on the tensor cores like any other
 class Attention : public Mixer {
  public:
   Attention(const Json &spec, const BuildEnv &env) : Mixer(spec, env) {
@@ -300,9 +305,13 @@ class Attention : public Mixer {
     bias_ = r.boolean_or("bias", false);
     scale_ = (float)r.number_or("scale", 1.0 / std::sqrt((double)d_), false);
     q_name_ = r.string("q");
-    k_name_ = r.string("k");
     values_from_keys_ = r.string_or("values", "own") == "keys";
-    v_name_ = values_from_keys_ ? std::string() : r.string("v");
+    borrowed_ = !r.present("k") && !r.present("v");
+    k_name_ = borrowed_ ? std::string() : r.string("k");
+    v_name_ = values_from_keys_ || borrowed_ ? std::string() : r.string("v");
+    null_scores_name_ = r.string_or("null_scores", "");
+    cache_window_ = (int)r.integer_or("cache_window", window_, 0);
+    if (cache_window_ > 0 && cache_window_ < window_) r.fail("'cache_window' must not be smaller than 'window'");
     o_name_ = r.string("o");
     if (n_heads_ % n_kv_) LLM_THROW(Config, "attention: %d heads are not a multiple of %d groups", n_heads_, n_kv_);
     dv_ = (int)r.integer_or("v_head_dim", d_);
@@ -330,7 +339,13 @@ class Attention : public Mixer {
     const Json &pos_spec = spec.get("position");
     pairs_place_ = position_ && pos_spec.is_object() && pos_spec.has("pairing") && pos_spec.get("pairing").is_string() &&
                    pos_spec.get("pairing").as_string() == "interleaved" && q_norm_name_.empty();
-    place_adds_bias_ = (!position_ && q_norm_name_.empty()) || pairs_place_;
+    rope_ = position_ && pos_spec.is_object() && pos_spec.get("kind").is_string() && pos_spec.get("kind").as_string() == "rope";
+    // the pass that rotates (pairs i, i + rotary_dim/2, or none) and places can add biases, take values of another width and leave
+    // keys and values out
+    rotate_place_ = (!position_ || rope_) && !pairs_place_ && q_norm_name_.empty() && head_eps_ < 0.f && v_eps_ < 0.f && !values_from_keys_;
+    place_adds_bias_ = (!position_ && q_norm_name_.empty()) || pairs_place_ || rotate_place_;
+    if (borrowed_ && !rotate_place_)
+      LLM_THROW(Unsupported, "attention: a run that reads another run's keys and values goes with a rotation of pairs (i, i + rotary_dim/2) or none, and with no norm");
     if (head_eps_ >= 0.f && (pairs_place_ || !q_norm_name_.empty() || bias_ || v_eps_ >= 0.f || values_from_keys_))
       LLM_THROW(Unsupported, "attention: a norm per head after the rotation goes with a rotation of pairs (i, i + rotary_dim/2) or none, and with no other norm or bias");
     if (head_eps_ >= 0.f) place_adds_bias_ = false;
@@ -342,7 +357,8 @@ class Attention : public Mixer {
     for (const char *key : {"q_bias", "k_bias", "v_bias"}) bias_names_.push_back(r.string_or(key, ""));
     q_width_ = (int64_t)n_heads_ * d_;
     kv_width_ = (int64_t)n_kv_ * d_;
-    v_width_ = values_from_keys_ ? 0 : (int64_t)n_kv_ * dv_;
+    if (borrowed_) kv_width_ = 0;
+    v_width_ = values_from_keys_ || borrowed_ ? 0 : (int64_t)n_kv_ * dv_;
     o_width_ = (int64_t)n_heads_ * dv_;
     gate_offset_ = q_width_ + kv_width_ + v_width_;
     // rows of the stacked matrix: a multiple of 8, so that rows of the 32-bit product start on 32 bytes
@@ -350,16 +366,22 @@ class Attention : public Mixer {
     stacked_rows_ = (gate_offset_ + gate_rows_ + 7) / 8 * 8;
     // the tiled attention kernels take heads whose values are as wide as their keys, in multiples of 16
     plain_ = dv_ == d_ && d_ % 16 == 0 && d_ >= 16 && scale_ > 0.f;
+    // padded heads: the tcgen05 prompt kernel and the fused single-token kernel take multiples of 8, values of their own width
+    padded_ = !plain_ && scale_ > 0.f && d_ % 8 == 0 && d_ <= 128 && dv_ % 8 == 0 && dv_ <= 256;
   }
 
   std::vector<TensorNeed> tensor_needs() const override {
-    std::vector<TensorNeed> needs = {{q_name_, {q_width_, hidden_}}, {k_name_, {kv_width_, hidden_}}};
-    if (!values_from_keys_) needs.push_back({v_name_, {v_width_, hidden_}});
+    std::vector<TensorNeed> needs = {{q_name_, {q_width_, hidden_}}};
+    if (!borrowed_) needs.push_back({k_name_, {kv_width_, hidden_}});
+    if (!values_from_keys_ && !borrowed_) needs.push_back({v_name_, {v_width_, hidden_}});
     needs.push_back({o_name_, {hidden_, o_width_}});
     if (bias_) {
       size_t which = 0;
       for (const auto &p : {std::make_pair(q_name_, q_width_), std::make_pair(k_name_, kv_width_), std::make_pair(v_name_, v_width_)}) {
-        if (p.first.empty()) continue;                 // no value matrix
+        if (p.first.empty()) {                         // no such matrix
+          if (borrowed_) ++which;
+          continue;
+        }
         std::string n = p.first;
         const std::string suffix = "weight";
         if (n.size() >= suffix.size() && n.compare(n.size() - suffix.size(), suffix.size(), suffix) == 0) n.resize(n.size() - suffix.size());
@@ -373,6 +395,7 @@ class Attention : public Mixer {
       needs.push_back({k_norm_name_, {kv_width_}, TensorRole::Vector, false});
     }
     if (!gate_name_.empty()) needs.push_back({gate_name_, {gate_rows_, hidden_}});
+    if (!null_scores_name_.empty()) needs.push_back({null_scores_name_, {(int64_t)n_heads_}, TensorRole::Vector, false});
     if (position_)
       for (auto &n : position_->tensor_needs()) needs.push_back(n);
     return needs;
@@ -387,18 +410,19 @@ class Attention : public Mixer {
     w_qkv_.buf.allocate((size_t)w_qkv_.rows * (size_t)hidden_ * es, true);
     char *p = (char *)w_qkv_.buf.get();
     l.fetch_into(needs[0], l.engine, p);
-    l.fetch_into(needs[1], l.engine, p + (size_t)q_width_ * hidden_ * es);
-    const size_t nv = values_from_keys_ ? 0 : 1;      // matrices and biases of the values
+    const size_t nk = borrowed_ ? 0 : 1, nv = values_from_keys_ || borrowed_ ? 0 : 1;      // matrices and biases of keys and values
+    if (nk) l.fetch_into(needs[1], l.engine, p + (size_t)q_width_ * hidden_ * es);
     if (nv) l.fetch_into(needs[2], l.engine, p + (size_t)(q_width_ + kv_width_) * hidden_ * es);
-    w_o_ = l.fetch(needs[2 + nv]);
-    const size_t first_bias = 3 + nv;
-    size_t next = bias_ ? first_bias + 2 + nv : first_bias;
+    w_o_ = l.fetch(needs[1 + nk + nv]);
+    const size_t first_bias = 2 + nk + nv;
+    size_t next = bias_ ? first_bias + 1 + nk + nv : first_bias;
     if (!q_norm_name_.empty()) {
       q_norm_ = l.fetch(needs[next]);
       k_norm_ = l.fetch(needs[next + 1]);
       next += 2;
     }
-    if (!gate_name_.empty()) l.fetch_into(needs[next], l.engine, p + (size_t)gate_offset_ * hidden_ * es);
+    if (!gate_name_.empty()) l.fetch_into(needs[next++], l.engine, p + (size_t)gate_offset_ * hidden_ * es);
+    if (!null_scores_name_.empty()) null_scores_ = l.fetch(needs[next++]);
     if (bias_) {
       b_qkv_.dtype = DType::F32;
       b_qkv_.rows = 1;
@@ -406,7 +430,7 @@ class Attention : public Mixer {
       b_qkv_.buf.allocate((size_t)w_qkv_.rows * 4, true);
       float *b = b_qkv_.buf.as<float>();
       l.fetch_into(needs[first_bias], DType::F32, b);
-      l.fetch_into(needs[first_bias + 1], DType::F32, b + q_width_);
+      if (nk) l.fetch_into(needs[first_bias + 1], DType::F32, b + q_width_);
       if (nv) l.fetch_into(needs[first_bias + 2], DType::F32, b + q_width_ + kv_width_);
       if (l.engine == DType::BF16 && !place_adds_bias_) {
         static bool said = false;
@@ -427,15 +451,14 @@ class Attention : public Mixer {
     if (env_.dtype != DType::BF16) return fams;
     const FastSwitches &f = fast_switches();
     const int group = n_heads_ / n_kv_;
-    if (!plain_) return fams;
+    if (!plain_ && !padded_) return fams;
     if (!gate_name_.empty()) fams.push_back("elementwise");
-    const bool tiled = env_.page_size == 64 && d_ % 16 == 0 && d_ >= 16 && d_ <= 128;
-    if (f.prefill_attention_tc && env_.page_size == 64 && (d_ == 64 || d_ == 128)) fams.push_back("attention_prefill_tc");
+    const bool tiled = env_.page_size == 64 && d_ % 16 == 0 && d_ >= 16 && d_ <= 128 && plain_;
+    if (f.prefill_attention_tc && env_.page_size == 64 && (d_ == 64 || d_ == 128 || padded_)) fams.push_back("attention_prefill_tc");
     else if (f.prefill_attention && tiled) fams.push_back("attention_prefill");
-    if (f.decode_attention_tc && tiled && group <= 16 && !bias_ && position_ && gate_name_.empty() && q_norm_name_.empty() &&
-        head_eps_ < 0.f && !(null_score_ > kernels::NO_NULL_KEY))
+    if (may_fuse() && env_.page_size == 64 && group <= 16 && d_ <= 128 && dv_ <= 128)
       fams.push_back("attention_decode_tc");
-    else if (f.decode_attention && (d_ == 16 || d_ == 32 || d_ == 64 || d_ == 128) &&
+    else if (plain_ && f.decode_attention && (d_ == 16 || d_ == 32 || d_ == 64 || d_ == 128) &&
              (group == 1 || group == 2 || group == 3 || group == 4 || group == 8))
       fams.push_back("attention_decode");
     return fams;
@@ -449,7 +472,8 @@ class Attention : public Mixer {
     n.n_kv_heads = n_kv_;
     n.k_dim = d_;
     n.v_dim = dv_;
-    n.window = n.kind == "window" ? window_ : 0;
+    if (n.kind == "window" && cache_window_ == 0) n.kind = "full";
+    n.window = n.kind == "window" ? cache_window_ : 0;
     n.block = n.kind == "block" ? block_ : 0;
     n.sink = n.kind == "window" ? sink_ : 0;
     return n;
@@ -457,6 +481,10 @@ class Attention : public Mixer {
 
   Act forward(StepContext &ctx, const Act &x, LayerCache *cache, StateView *) override {
     if (!cache) LLM_THROW(InvalidArg, "attention: the run has no cache to attend over");
+    if (borrowed_ && cache->writes) LLM_THROW(Config, "attention: a run without keys and values of its own needs another run's cache");
+    if (borrowed_ && (cache->need.n_kv_heads != n_kv_ || cache->need.k_dim != d_ || cache->need.v_dim != dv_))
+      LLM_THROW(Config, "attention: the cache holds %d heads of %d / %d channels, this run reads %d of %d / %d", cache->need.n_kv_heads,
+                cache->need.k_dim, cache->need.v_dim, n_kv_, d_, dv_);
     const FastSwitches &f = fast_switches();
     const int group = n_heads_ / n_kv_;
     // The products hand over 32-bit results: q and k are rounded to the engine's type once, after
@@ -465,24 +493,25 @@ class Attention : public Mixer {
     const float *table = position_ ? position_->half_split_table(&table_rows, &rot_dim) : nullptr;
     const bool has_gate = !gate_name_.empty();
     const float *gate = nullptr;
-    const bool has_null = null_score_ > kernels::NO_NULL_KEY;
-    const bool fused = plain_ && !has_gate && q_norm_name_.empty() && head_eps_ < 0.f && !has_null && table && !bias_ && ctx.decode_only && f.decode_attention_tc && ctx.dtype == DType::BF16 &&
-                       kernels::available("attention_decode_tc") && kernels::attention_decode_tc_supported(d_, cache->page_size, group);
+    const float *null_scores = null_scores_name_.empty() ? nullptr : null_scores_.buf.as<float>();
+    const float *bias = bias_ ? b_qkv_.buf.as<float>() : nullptr;
+    const bool fused = may_fuse() && table && ctx.decode_only && ctx.dtype == DType::BF16 && kernels::available("attention_decode_tc") &&
+                       kernels::attention_decode_tc_takes(d_, dv_, cache->page_size, group);
     Act qkv = linear(ctx, x, w_qkv_, bias_ && !place_adds_bias_ ? b_qkv_.buf.as<float>() : nullptr, DType::F32, fused);
     flush_chain(ctx);
     if (fused) {
       const int max_len = std::max(ctx.max_kv_len, 1);
       const int pairs = std::max(1, ctx.n_seqs * n_kv_);
-      const int slots = ctx.sm_count * kernels::attention_decode_tc_ctas_per_sm(d_);
+      const int slots = ctx.sm_count * kernels::attention_decode_tc_ctas_per_sm(d_, dv_);
       // As many key splits as fill the GPU once (all CTAs resident together), each of at least a
       // page at the longest length.  The kernel cuts every sequence's own length into that many
       // runs, so the number depends on the batch and the bound on the length, not on the lengths.
       const int n_splits = std::max(1, std::min(slots / pairs, std::max(1, max_len / cache->page_size)));
-      Act out = ctx.arena->act(DType::BF16, ctx.n_tokens, q_width_);
+      Act out = ctx.arena->act(DType::BF16, ctx.n_tokens, o_width_);
       float *ws_o = nullptr, *ws_ml = nullptr;
       int *counters = nullptr;
       if (n_splits > 1) {
-        ws_o = ctx.arena->alloc_n<float>((size_t)ctx.n_seqs * n_heads_ * n_splits * d_);
+        ws_o = ctx.arena->alloc_n<float>((size_t)ctx.n_seqs * n_heads_ * n_splits * dv_);
         ws_ml = ctx.arena->alloc_n<float>((size_t)ctx.n_seqs * n_heads_ * n_splits * 2);
         if (pairs > ctx.n_zero_counters)
           LLM_THROW(Unsupported, "fused decode attention: %d (sequence, kv head) pairs in one step, %d are provided for", pairs,
@@ -491,7 +520,7 @@ class Attention : public Mixer {
       }
       kernels::attention_decode_tc(qkv, table, table_rows, rot_dim, ctx.tok_pos, cache->page_table, cache->table_width, cache->k,
                                    cache->v, cache->writes, ctx.n_seqs, n_heads_, n_kv_, d_, cache->page_size, 0, max_len, n_splits,
-                                   window_, block_, scale_, ws_o, ws_ml, counters, out, ctx.stream);
+                                   window_, block_, scale_, ws_o, ws_ml, counters, out, ctx.stream, dv_, bias, null_scores);
       return linear(ctx, out, w_o_, nullptr, DType::F32, true);
     }
     Act q = ctx.arena->act(ctx.dtype, ctx.n_tokens, q_width_);
@@ -505,13 +534,17 @@ class Attention : public Mixer {
       kernels::rope_pairs_place(qkv, q, n_heads_, n_kv_, d_, dv_, bias_ ? b_qkv_.buf.as<float>() : nullptr, values_from_keys_, pairs, rows,
                                 rot, ctx.tok_seq, ctx.tok_pos, cache->page_table, cache->table_width, cache->k, cache->v,
                                 cache->page_size, cache->writes, ctx.stream);
-    } else if (place_adds_bias_ && (bias_ || v_eps_ >= 0.f)) {
+    } else if (!position_ && place_adds_bias_ && !borrowed_ && (bias_ || v_eps_ >= 0.f)) {
       kernels::kv_place(qkv, q, n_heads_, n_kv_, d_, dv_, bias_ ? b_qkv_.buf.as<float>() : nullptr, v_eps_, ctx.tok_seq, ctx.tok_pos,
                         cache->page_table, cache->table_width, cache->k, cache->v, cache->page_size, cache->writes, ctx.stream);
     } else if (head_eps_ >= 0.f) {
       if (position_ && !table) LLM_THROW(Unsupported, "attention: a norm per head needs a position part with a half-split table (or none)");
       kernels::rope_headnorm_place(qkv, q, n_heads_, n_kv_, d_, dv_, head_eps_, table, table_rows, rot_dim, ctx.tok_seq, ctx.tok_pos,
                                    cache->page_table, cache->table_width, cache->k, cache->v, cache->page_size, cache->writes, ctx.stream);
+    } else if (rotate_place_ && (!position_ || table) && (bias_ || borrowed_ || dv_ != d_)) {
+      kernels::conv_rope_place(qkv, bias, nullptr, 1, nullptr, q, n_heads_, n_kv_, d_, dv_, table, table_rows, rot_dim, ctx.tok_seq, ctx.tok_pos,
+                               ctx.seq_start, ctx.seq_past, ctx.seq_slot, ctx.n_seqs, cache->page_table, cache->table_width, cache->k, cache->v,
+                               cache->page_size, cache->writes, ctx.decode_only, ctx.stream);
     } else if (!q_norm_name_.empty() || dv_ != d_) {
       if (position_ && !table)
         LLM_THROW(Unsupported, "attention: a q/k norm or values of another width need a position part with a half-split table (or none)");
@@ -529,8 +562,8 @@ class Attention : public Mixer {
     // a gate per channel is applied behind the attention kernel, whichever it is
     const float *channel_gate = gate_per_channel_ ? gate : nullptr;
     if (gate_per_channel_) gate = nullptr;
-    if (ctx.dtype == DType::BF16 && plain_) {
-      if (ctx.decode_only && f.decode_attention && kernels::available("attention_decode") &&
+    if (ctx.dtype == DType::BF16 && (plain_ || padded_)) {
+      if (plain_ && ctx.decode_only && f.decode_attention && kernels::available("attention_decode") &&
           kernels::attention_decode_supported(d_, group)) {
         // enough CTAs to fill the GPU about eight times over at the longest length, runs of at
         // least two pages; the same for every step of a captured graph
@@ -549,21 +582,22 @@ class Attention : public Mixer {
         }
         kernels::attention_decode(q, out, cache->k, cache->v, ctx.tok_pos, cache->page_table, cache->table_width, n_heads_, n_kv_,
                                   d_, cache->page_size, chunk, n_splits, window_, block_, scale_, ws_o, ws_ml,
-                                  channel_gate ? channel_gate : gate, qkv.ld, ctx.stream, sink_, channel_gate != nullptr, null_score_);
+                                  channel_gate ? channel_gate : gate, qkv.ld, ctx.stream, sink_, channel_gate != nullptr, null_score_,
+                                  null_scores);
         gate = nullptr;                 // applied
         channel_gate = nullptr;
         done = true;
-      } else if (f.prefill_attention_tc && (d_ == 64 || d_ == 128) && kernels::available("attention_prefill_tc") &&
-                 kernels::attention_prefill_tc_supported(d_, cache->page_size)) {
+      } else if (f.prefill_attention_tc && (d_ == 64 || d_ == 128 || padded_) && kernels::available("attention_prefill_tc") &&
+                 kernels::attention_prefill_tc_takes(d_, dv_, cache->page_size)) {
         kernels::attention_prefill_tc(q, out, cache->k, cache->v, cache->n_pages, ctx.seq_start, ctx.seq_past, cache->page_table,
                                       cache->table_width, ctx.n_seqs, ctx.max_q_len, n_heads_, n_kv_, d_, cache->page_size, window_,
-                                      block_, scale_, ctx.tc_status, ctx.stream, sink_, null_score_);
+                                      block_, scale_, ctx.tc_status, ctx.stream, sink_, null_score_, dv_, null_scores);
         done = true;
-      } else if (f.prefill_attention && kernels::available("attention_prefill") &&
+      } else if (plain_ && f.prefill_attention && kernels::available("attention_prefill") &&
                  kernels::attention_prefill_supported(d_, cache->page_size)) {
         kernels::attention_prefill(q, out, cache->k, cache->v, ctx.seq_start, ctx.seq_past, cache->page_table, cache->table_width,
                                    ctx.n_seqs, ctx.max_q_len, n_heads_, n_kv_, d_, cache->page_size, window_, block_, scale_, ctx.stream,
-                                   sink_, null_score_);
+                                   sink_, null_score_, null_scores);
         done = true;
       }
       if (done && gate) kernels::head_gate(out, gate, qkv.ld, n_heads_, dv_, ctx.stream);
@@ -571,21 +605,26 @@ class Attention : public Mixer {
     if (!done)
       kernels::attention_generic(q, out, cache->k, cache->v, ctx.tok_seq, ctx.tok_pos, cache->page_table, cache->table_width,
                                  n_heads_, n_kv_, d_, dv_, cache->page_size, window_, block_, scale_, gate, qkv.ld, ctx.stream, sink_, 0,
-                                 null_score_);
+                                 null_score_, null_scores);
     if (channel_gate) kernels::head_gate(out, channel_gate, qkv.ld, n_heads_ * dv_, 1, ctx.stream);
     return linear(ctx, out, w_o_, nullptr, DType::F32, true);
   }
 
  private:
+  // whether a step of single tokens can be one launch behind the product (rotation, append, attention)
+  bool may_fuse() const {
+    return (plain_ || padded_) && gate_name_.empty() && q_norm_name_.empty() && head_eps_ < 0.f && v_eps_ < 0.f && !values_from_keys_ && sink_ == 0 &&
+           !(null_score_ > kernels::NO_NULL_KEY) && position_ && !pairs_place_ && (!bias_ || place_adds_bias_) && fast_switches().decode_attention_tc;
+  }
   int64_t hidden_, q_width_, kv_width_, v_width_, o_width_, gate_offset_, stacked_rows_;
   int64_t gate_rows_ = 0;
-  int n_heads_, n_kv_, d_, dv_, window_, block_, sink_ = 0;
-  bool bias_, plain_, gate_per_channel_ = false, place_adds_bias_ = false, values_from_keys_ = false, pairs_place_ = false;
+  int n_heads_, n_kv_, d_, dv_, window_, block_, sink_ = 0, cache_window_ = 0;
+  bool bias_, plain_, padded_ = false, borrowed_ = false, rope_ = false, rotate_place_ = false, gate_per_channel_ = false, place_adds_bias_ = false, values_from_keys_ = false, pairs_place_ = false;
   float scale_, qk_eps_ = 0.f, v_eps_ = -1.f, head_eps_ = -1.f, null_score_ = kernels::NO_NULL_KEY;
   std::vector<std::string> bias_names_;
-  std::string q_name_, k_name_, v_name_, o_name_, q_norm_name_, k_norm_name_, gate_name_;
+  std::string q_name_, k_name_, v_name_, o_name_, q_norm_name_, k_norm_name_, gate_name_, null_scores_name_;
   std::unique_ptr<PositionEncoding> position_;
-  Weight w_qkv_, w_o_, b_qkv_, q_norm_, k_norm_;
+  Weight w_qkv_, w_o_, b_qkv_, q_norm_, k_norm_, null_scores_;
 };
 
 // ---------------------------------------------------------------- SwiGLU
@@ -622,20 +661,7 @@ class SwiGLU : public FeedForward {
     return fams;
   }
   Act forward(StepContext &ctx, const Act &x) override {
-    const FastSwitches &f = fast_switches();
-    Act m;
-    if (x.dtype == DType::BF16) {
-      m = small_batch_linear(ctx, x, w_gate_up_, ctx.dtype, true, false);
-      // silu(gate) * up of a prompt step in one launch of the tcgen05 product (two accumulators per
-      // tile), where that beats the library product followed by a SwiGLU pass: measured at 2,048
-      // tokens, 129 us against 146 us at K = 2,048, but 403 us against 379 us at K = 4,096.
-      if (!m.data && f.gemm_tc && x.rows >= f.fused_gate_up_tokens && x.cols <= f.fused_gate_up_max_k &&
-          kernels::gemm_tc_supported(x, w_gate_up_)) {
-        m = ctx.arena->act(ctx.dtype, x.rows, inter_);
-        flush_chain(ctx);
-        kernels::gemm_tc(x, w_gate_up_, m, true, ctx.tc_status, ctx.stream);
-      }
-    }
+    Act m = fused_gated_linear(ctx, x, w_gate_up_);
     if (!m.data) {
       Act gu = linear(ctx, x, w_gate_up_, nullptr, DType::F32);
       flush_chain(ctx);
@@ -661,6 +687,11 @@ class SwiGLU : public FeedForward {
 //   ff, ff_norm may be null: the block is the mixer alone
 //   mixer_scale, ff_scale  names of vectors [hidden]: a sublayer's result is multiplied by its vector,
 //               channel by channel, before it is added to the stream (32-bit, in the pass that adds it)
+//   mixer_post, ff_post    {weight, eps}: a sublayer's result y is normed before it is added, y / sqrt(mean(y^2) + eps) * weight
+//               (32-bit, in the pass that adds it and takes the next norm)
+//   side        {dim, offset, gate, proj, norm, eps}: behind the feed-forward the token's own vector e, columns offset ..
+//               offset + dim - 1 of its row of the model's side table (ModelSpec::token_table), is added through the stream itself:
+//               y = proj (gelu_tanh(gate x) * e), x += y / sqrt(mean(y^2) + eps) * norm
 const char *const CONV_STATE = "mixer_conv.inputs";
 class PreNormBlock : public Block {
  public:
@@ -682,6 +713,27 @@ class PreNormBlock : public Block {
     mixer_scale_name_ = r.string_or("mixer_scale", "");
     ff_scale_name_ = ff_ ? r.string_or("ff_scale", "") : "";
     if (!mixer_scale_name_.empty() || !ff_scale_name_.empty()) hidden_ = r.integer("hidden");
+    auto post = [&](const char *key, PostNorm *p) {
+      if (!r.present(key)) return;
+      ConfigReader n(r.object(key), std::string("prenorm block: ") + key);
+      p->name = n.string("weight");
+      p->eps = (float)n.number("eps");
+      hidden_ = r.integer("hidden");
+    };
+    post("mixer_post", &mixer_post_);
+    if (ff_) post("ff_post", &ff_post_);
+    if ((mixer_post_.on() && !mixer_scale_name_.empty()) || (ff_post_.on() && !ff_scale_name_.empty()))
+      r.fail("a sublayer's result has a scale or a norm, not both");
+    if (r.present("side")) {
+      ConfigReader s(r.object("side"), "prenorm block: side");
+      side_dim_ = (int)s.integer("dim");
+      side_offset_ = (int)s.integer("offset", 0);
+      side_gate_name_ = s.string("gate");
+      side_proj_name_ = s.string("proj");
+      side_norm_.name = s.string("norm");
+      side_norm_.eps = (float)s.number("eps");
+      hidden_ = r.integer("hidden");
+    }
   }
   std::vector<Part *> parts() const {
     std::vector<Part *> p = {mixer_norm_.get(), mixer_.get()};
@@ -705,6 +757,13 @@ class PreNormBlock : public Block {
     if (taps_ > 0) out.push_back({conv_name_, {hidden_, (int64_t)taps_}, TensorRole::Vector, false});
     if (!mixer_scale_name_.empty()) out.push_back({mixer_scale_name_, {hidden_}, TensorRole::Vector, false});
     if (!ff_scale_name_.empty()) out.push_back({ff_scale_name_, {hidden_}, TensorRole::Vector, false});
+    for (const PostNorm *p : {&mixer_post_, &ff_post_})
+      if (p->on()) out.push_back(vector_need(p->name));
+    if (side_dim_ > 0) {
+      out.push_back({side_gate_name_, {(int64_t)side_dim_, hidden_}});
+      out.push_back({side_proj_name_, {hidden_, (int64_t)side_dim_}});
+      out.push_back(vector_need(side_norm_.name));
+    }
     return out;
   }
   void load(const Loader &l) override {
@@ -712,12 +771,33 @@ class PreNormBlock : public Block {
     if (taps_ > 0) conv_ = l.fetch({conv_name_, {hidden_, (int64_t)taps_}, TensorRole::Vector, false});
     if (!mixer_scale_name_.empty()) mixer_scale_ = l.fetch({mixer_scale_name_, {hidden_}, TensorRole::Vector, false});
     if (!ff_scale_name_.empty()) ff_scale_ = l.fetch({ff_scale_name_, {hidden_}, TensorRole::Vector, false});
+    for (PostNorm *p : {&mixer_post_, &ff_post_})
+      if (p->on()) p->weight = l.fetch(vector_need(p->name));
+    if (side_dim_ > 0) {
+      // Padded with zeros in bfloat16, so that rows of the products start on 16 bytes: rows of the gate's matrix, columns
+      // of the projection's.
+      const int64_t pad = l.engine == DType::BF16 ? (side_dim_ + 7) / 8 * 8 : side_dim_;
+      const size_t es = dtype_size(l.engine);
+      side_gate_.dtype = side_proj_.dtype = l.engine;
+      side_gate_.rows = side_proj_.cols = pad;
+      side_gate_.cols = side_proj_.rows = hidden_;
+      side_gate_.buf.allocate((size_t)(pad * hidden_) * es, true);
+      side_proj_.buf.allocate((size_t)(pad * hidden_) * es, true);
+      l.fetch_into({side_gate_name_, {(int64_t)side_dim_, hidden_}}, l.engine, side_gate_.buf.get());
+      DeviceBuffer staged((size_t)(hidden_ * side_dim_) * es);
+      l.fetch_into({side_proj_name_, {hidden_, (int64_t)side_dim_}}, l.engine, staged.get());
+      LLM_CUDA(cudaMemcpy2D(side_proj_.buf.get(), (size_t)pad * es, staged.get(), (size_t)side_dim_ * es, (size_t)side_dim_ * es, (size_t)hidden_,
+                            cudaMemcpyDeviceToDevice));
+      side_norm_.weight = l.fetch(vector_need(side_norm_.name));
+    }
   }
   std::vector<std::string> kernel_families() const override {
     std::vector<std::string> out;
     for (Part *p : parts())
       for (auto &f : p->kernel_families()) out.push_back(f);
     if (taps_ > 0) out.push_back("recurrent");
+    if (side_dim_ > 0)
+      for (auto &f : product_families(env_.dtype)) out.push_back(f);
     return out;
   }
   bool capturable() const override {
@@ -763,18 +843,18 @@ class PreNormBlock : public Block {
     // a result that is scaled before it is added cannot be added by the product that makes it
     const float *mixer_scale = mixer_scale_name_.empty() ? nullptr : mixer_scale_.buf.as<float>();
     const float *ff_scale = ff_scale_name_.empty() ? nullptr : ff_scale_.buf.as<float>();
-    sink(mixer_scale == nullptr);
+    sink(mixer_scale == nullptr && !mixer_post_.on());
     Act r = mixer_->forward(ctx, h, cache, state);
     sink(false);
-    stream.pending = r.data == (void *)stream.resid ? Act() : scaled(r, mixer_scale);
+    stream.pending = r.data == (void *)stream.resid ? Act() : mixer_post_.apply(scaled(r, mixer_scale));
     if (ctx.nothing_read_after) {       // no logits wanted from this step: the stream is read by nobody
       flush_chain(ctx);
       stream.pending = Act();
       return;
     }
-    if (!ff_) return;
+    if (!ff_ && side_dim_ == 0) return;
     if (ctx.rows_read_after && ctx.n_rows_read_after < stream.rows && !stream.picked) {
-      // the last layer of a prompt step: the feed-forward of the wanted rows alone
+      // the last layer of a prompt step: what follows the mixer for the wanted rows alone
       flush_chain(ctx);
       const int64_t n = ctx.n_rows_read_after;
       float *few = ctx.arena->alloc_n<float>((size_t)(n * stream.hidden));
@@ -785,14 +865,57 @@ class PreNormBlock : public Block {
       stream.pending = Act();
       stream.picked = true;
     }
-    h = ff_norm_->forward(ctx, stream);
-    sink(ff_scale == nullptr);
-    r = ff_->forward(ctx, h);
-    sink(false);
-    stream.pending = r.data == (void *)stream.resid ? Act() : scaled(r, ff_scale);
+    if (ff_) {
+      h = ff_norm_->forward(ctx, stream);
+      sink(ff_scale == nullptr && !ff_post_.on());
+      r = ff_->forward(ctx, h);
+      sink(false);
+      stream.pending = r.data == (void *)stream.resid ? Act() : ff_post_.apply(scaled(r, ff_scale));
+    }
+    if (side_dim_ > 0) add_side(ctx, stream);
   }
 
  private:
+  // a norm on a sublayer's result before it is added
+  struct PostNorm {
+    std::string name;
+    float eps = 0.f;
+    Weight weight;
+    bool on() const { return !name.empty(); }
+    Act apply(Act r) const {
+      if (!on()) return r;
+      r.post = weight.buf.as<float>();
+      r.post_eps = eps;
+      return r;
+    }
+  };
+  TensorNeed vector_need(const std::string &name) const { return {name, {hidden_}, TensorRole::Vector, false}; }
+  void add_side(StepContext &ctx, ResidualStream &stream) {
+    if (!ctx.token_table || !ctx.token_ids || ctx.token_table_width < side_offset_ + side_dim_)
+      LLM_THROW(InvalidArg, "prenorm block: the model has no side vectors for this layer's tokens");
+    flush_chain(ctx);
+    const int64_t n = stream.rows;
+    Act x;
+    if (ctx.dtype == DType::F32) {         // the stream itself, with everything added
+      if (stream.pending.data)
+        kernels::add_rmsnorm(stream.resid, &stream.pending, nullptr, 0.f, nullptr, ctx.dtype, nullptr, (int)n, (int)hidden_, ctx.stream);
+      x.data = stream.resid;
+      x.dtype = DType::F32;
+      x.rows = n;
+      x.cols = x.ld = hidden_;
+      x.part_stride = n * hidden_;
+    } else {
+      x = ctx.arena->act(ctx.dtype, n, hidden_);
+      kernels::stream_cast(stream.resid, stream.pending.data ? &stream.pending : nullptr, x.data, ctx.dtype, (int)n, (int)hidden_, ctx.stream);
+    }
+    stream.pending = Act();
+    Act z = linear(ctx, x, side_gate_, nullptr, DType::F32);
+    flush_chain(ctx);
+    Act g = ctx.arena->act(ctx.dtype, n, side_proj_.cols);
+    kernels::token_gate(z, ctx.token_table, ctx.token_table_width, side_offset_, side_dim_, ctx.token_ids,
+                        stream.picked ? ctx.rows_read_after : nullptr, g, ctx.stream);
+    stream.pending = side_norm_.apply(linear(ctx, g, side_proj_, nullptr, DType::F32, true));
+  }
   static Act scaled(Act r, const float *scale) {
     if (!scale) return r;
     if (r.col_scale) LLM_THROW(Unsupported, "prenorm block: a sublayer's result carries a scale of its own beside the block's");
@@ -804,8 +927,10 @@ class PreNormBlock : public Block {
   std::unique_ptr<FeedForward> ff_;
   int taps_ = 0;
   int64_t hidden_ = 0;
-  std::string conv_name_, mixer_scale_name_, ff_scale_name_;
-  Weight conv_, mixer_scale_, ff_scale_;
+  std::string conv_name_, mixer_scale_name_, ff_scale_name_, side_gate_name_, side_proj_name_;
+  Weight conv_, mixer_scale_, ff_scale_, side_gate_, side_proj_;
+  PostNorm mixer_post_, ff_post_, side_norm_;
+  int side_dim_ = 0, side_offset_ = 0;
 };
 
 // ---------------------------------------------------------------- pre-norm block over several residual streams
@@ -1101,6 +1226,7 @@ void register_recurrent_parts();      // parts/recurrent.cc
 void register_latent_parts();         // parts/latent.cc
 void register_state_parts();          // parts/state_mixers.cc
 void register_sigmoid_parts();        // parts/sigmoid_attention.cc
+void register_selective_parts();      // parts/selective.cc
 
 void register_builtin_parts() {
   register_part_raw("block", "parallel", factory_of<ParallelBlock>());
@@ -1109,6 +1235,7 @@ void register_builtin_parts() {
   register_latent_parts();
   register_state_parts();
   register_sigmoid_parts();
+  register_selective_parts();
   register_part_raw("norm", "rmsnorm", factory_of<RMSNorm>());
   register_part_raw("norm", "layernorm", factory_of<LayerNorm>());
   register_part_raw("position", "rope", factory_of<RotaryEmbedding>());

@@ -74,7 +74,9 @@ class Mlp : public FeedForward {
 // of neighbours, a group's score is the sum of its `top` (2) largest corrected scores, and only experts of the `keep`
 // best groups can be chosen; `norm_eps`, added to the sum that `renormalize` divides by; `route_scale`, a factor on
 // the weights; `shared_gate`, a matrix [1, hidden]: the shared feed-forward's result is multiplied by sigmoid(gate x),
-// one number per token (its row rides behind the router's rows in one stacked product).
+// one number per token (its row rides behind the router's rows in one stacked product); `identity`, a number of further choices
+// behind the experts (the router and the correction have rows for them too) whose result is the input itself, times the weight;
+// expert.activation "bounded_glu" {limit, slope, up_shift} on gated experts: the unit of "clamped_glu" below.
 class RoutedFeedForward : public FeedForward {
  public:
   RoutedFeedForward(const Json &spec, const BuildEnv &env) : FeedForward(spec, env) {
@@ -82,7 +84,9 @@ class RoutedFeedForward : public FeedForward {
     hidden_ = r.integer("hidden");
     experts_ = (int)r.integer("experts");
     top_ = (int)r.integer("top");
-    if (top_ > experts_) r.fail("'top' exceeds 'experts'");
+    identity_ = (int)r.integer_or("identity", 0, 0);
+    choices_ = experts_ + identity_;
+    if (top_ > choices_) r.fail("'top' exceeds 'experts'");
     const std::string score = r.string_or("score", "softmax");
     if (score != "sigmoid" && score != "softmax") r.fail("'score' must be \"sigmoid\" or \"softmax\"");
     score_ = score == "softmax" ? 1 : 0;
@@ -93,7 +97,17 @@ class RoutedFeedForward : public FeedForward {
     router_ = r.string("router");
     ConfigReader e(r.object("expert"), "moe description: expert");
     inter_ = e.integer("intermediate");
-    act_ = activation_code(e.string_or("activation", "gelu"), e);
+    const std::string act = e.string_or("activation", "gelu");
+    if (act == "bounded_glu") {
+      act_ = kernels::BoundedGlu;
+      const double limit = e.number_or("limit", 0.0, false);
+      if (limit > 0) glu_.limit = (float)limit;
+      glu_.slope = (float)e.number_or("slope", 1.0, false);
+      glu_.shift = (float)e.number_or("up_shift", 0.0, false);
+      if (!e.present("gate")) e.fail("a bounded unit goes with gated experts");
+    } else {
+      act_ = activation_code(act, e);
+    }
     up_ = e.string("up");
     down_ = e.string("down");
     gate_ = e.string_or("gate", "");
@@ -108,16 +122,16 @@ class RoutedFeedForward : public FeedForward {
       groups_ = (int)g.integer("count");
       keep_ = (int)g.integer("keep");
       group_top_ = (int)g.integer_or("top", 2);
-      if (experts_ % groups_) g.fail("'count' must divide the number of experts");
+      if (choices_ % groups_) g.fail("'count' must divide the number of experts");
       if (keep_ > groups_) g.fail("'keep' exceeds 'count'");
-      if ((int64_t)keep_ * (experts_ / groups_) < top_) g.fail("the kept groups hold fewer experts than 'top'");
+      if ((int64_t)keep_ * (choices_ / groups_) < top_) g.fail("the kept groups hold fewer experts than 'top'");
     }
     norm_eps_ = (float)r.number_or("norm_eps", 0.0, false);
     route_scale_ = (float)r.number_or("route_scale", 1.0, false);
     shared_gate_ = r.string_or("shared_gate", "");
     if (!shared_gate_.empty() && !shared_) r.fail("'shared_gate' goes with a 'shared' feed-forward");
     grouped_route_ = !correction_.empty() || groups_ > 1 || norm_eps_ != 0.f || route_scale_ != 1.f;
-    router_rows_ = shared_gate_.empty() ? experts_ : (experts_ + 1 + 7) / 8 * 8;
+    router_rows_ = shared_gate_.empty() ? choices_ : (choices_ + 1 + 7) / 8 * 8;
   }
   static std::string numbered(const std::string &pattern, int e) {
     std::string s = pattern;
@@ -125,7 +139,7 @@ class RoutedFeedForward : public FeedForward {
     return s;
   }
   std::vector<TensorNeed> tensor_needs() const override {
-    std::vector<TensorNeed> needs = {{router_, {(int64_t)experts_, hidden_}}};
+    std::vector<TensorNeed> needs = {{router_, {(int64_t)choices_, hidden_}}};
     for (int e = 0; e < experts_; ++e) {
       needs.push_back({numbered(up_, e), {inter_, hidden_}});
       needs.push_back({numbered(down_, e), {hidden_, inter_}});
@@ -133,7 +147,8 @@ class RoutedFeedForward : public FeedForward {
     }
     if (shared_)
       for (auto &n : shared_->tensor_needs()) needs.push_back(n);
-    if (!correction_.empty()) needs.push_back({correction_, {(int64_t)experts_}, TensorRole::Vector, false});
+    // drawn beside softmax scores: small against a score, so that a drawn model's choices follow its tokens
+    if (!correction_.empty()) needs.push_back({correction_, {(int64_t)choices_}, TensorRole::Vector, false, score_ == 1 ? 0.01f : 1.f});
     if (!shared_gate_.empty()) needs.push_back({shared_gate_, {1, hidden_}});
     return needs;
   }
@@ -149,7 +164,7 @@ class RoutedFeedForward : public FeedForward {
       w_router_.cols = hidden_;
       w_router_.buf.allocate((size_t)router_rows_ * row_bytes, true);
       l.fetch_into(needs[0], l.engine, w_router_.buf.get());
-      l.fetch_into(needs.back(), l.engine, (char *)w_router_.buf.get() + (size_t)experts_ * row_bytes);
+      l.fetch_into(needs.back(), l.engine, (char *)w_router_.buf.get() + (size_t)choices_ * row_bytes);
     }
     if (!correction_.empty()) w_correction_ = l.fetch(needs[needs.size() - (shared_gate_.empty() ? 1 : 2)]);
     const size_t es = dtype_size(l.engine), one = (size_t)(inter_ * hidden_) * es;
@@ -186,11 +201,32 @@ class RoutedFeedForward : public FeedForward {
 
   Act forward(StepContext &ctx, const Act &x) override {
     const int64_t T = x.rows;
-    // the shared expert first: its last product may add to the residual stream as it stores
+    // the shared expert first: its last product may add to the residual stream as it stores, or else put its result (or partial
+    // results) where this part's own parts end
     Act s;
     float *const sink = ctx.residual_sink;
     if (!shared_gate_.empty()) ctx.residual_sink = nullptr;   // a gated result cannot be added by the product that makes it
-    if (shared_) s = shared_->forward(ctx, x);
+    const bool few = x.dtype == DType::BF16 && T <= fast_switches().tc_tokens;
+    const int given = !shared_ ? 0 : few ? 8 : ctx.residual_sink ? 0 : 1;
+    Act out = ctx.arena->act(DType::F32, T, hidden_, top_ + given);
+    float *const after = (float *)out.data + (size_t)top_ * (size_t)(T * hidden_);
+    if (shared_) {
+      // an outer block's room is not for a result that joins this part's
+      float *const outer = ctx.parts_pool;
+      const int cap = ctx.parts_cap, used = ctx.parts_used;
+      const int64_t rows = ctx.parts_rows, cols = ctx.parts_cols;
+      ctx.parts_pool = given > 0 && !ctx.chain ? after : nullptr;
+      ctx.parts_cap = given;
+      ctx.parts_used = 0;
+      ctx.parts_rows = T;
+      ctx.parts_cols = hidden_;
+      s = shared_->forward(ctx, x);
+      ctx.parts_pool = outer;
+      ctx.parts_cap = cap;
+      ctx.parts_used = used;
+      ctx.parts_rows = rows;
+      ctx.parts_cols = cols;
+    }
     const bool s_own = s.data && s.data != (void *)sink;
     ctx.residual_sink = nullptr;                     // what follows returns its own buffers
     Act z = linear(ctx, x, w_router_, nullptr, DType::F32);
@@ -200,11 +236,13 @@ class RoutedFeedForward : public FeedForward {
     int *chosen = ctx.arena->alloc_n<int>((size_t)n_rows);
     float *weight = ctx.arena->alloc_n<float>((size_t)n_rows);
     if (grouped_route_)
-      kernels::moe_route_grouped(z, experts_, top_, score_, correction_.empty() ? nullptr : w_correction_.buf.as<float>(), groups_, keep_,
+      kernels::moe_route_grouped(z, choices_, top_, score_, correction_.empty() ? nullptr : w_correction_.buf.as<float>(), groups_, keep_,
                                  group_top_, renormalize_, norm_eps_, route_scale_, chosen, weight, ctx.stream);
     else
-      kernels::moe_route(z, experts_, top_, score_, renormalize_, chosen, weight, ctx.stream);
-    Act out = ctx.arena->act(DType::F32, T, hidden_, top_ + (s_own ? s.parts : 0));
+      kernels::moe_route(z, choices_, top_, score_, renormalize_, chosen, weight, ctx.stream);
+    const bool in_place = given > 0 && s_own && s.data == (void *)after;
+    if (s_own && !in_place && s.parts > given) out = ctx.arena->act(DType::F32, T, hidden_, top_ + s.parts);
+    out.parts = top_ + (s_own ? s.parts : 0);
     const bool aligned = x.dtype == DType::BF16 && x.ld % 8 == 0 && (uintptr_t)x.data % 16 == 0;
     if (aligned && fast_switches().moe_tc && kernels::available("moe_tc") && kernels::moe_tc_supported((int)hidden_, (int)inter_)) {
       const int tile = kernels::moe_tc_tile_rows(n_rows);
@@ -215,7 +253,8 @@ class RoutedFeedForward : public FeedForward {
       void *mid = ctx.arena->alloc((size_t)n_rows * (size_t)inter_ * 2);
       kernels::moe_sort(chosen, n_rows, experts_, tile, offsets, perm, tiles, ctx.stream);
       kernels::moe_tc(x, w_up_.get(), w_down_.get(), offsets, perm, tiles, weight, experts_, top_, (int)hidden_, (int)inter_, act_,
-                      weight_on_output_, xs, mid, (float *)out.data, ctx.tc_status, ctx.stream, !gate_.empty());
+                      weight_on_output_, xs, mid, (float *)out.data, ctx.tc_status, ctx.stream, !gate_.empty(), glu_,
+                      identity_ > 0 ? chosen : nullptr);
     } else if (aligned && kernels::moe_grouped_supported((int)hidden_, (int)inter_)) {
       const int tile = kernels::moe_tile_rows();
       int *offsets = ctx.arena->alloc_n<int>((size_t)experts_ + 1);
@@ -224,18 +263,19 @@ class RoutedFeedForward : public FeedForward {
       void *mid = ctx.arena->alloc((size_t)n_rows * (size_t)inter_ * 2);
       kernels::moe_sort(chosen, n_rows, experts_, tile, offsets, perm, tiles, ctx.stream);
       kernels::moe_grouped(x, w_up_.get(), w_down_.get(), offsets, perm, tiles, weight, experts_, top_, (int)hidden_, (int)inter_,
-                           act_, weight_on_output_, mid, (float *)out.data, ctx.stream, !gate_.empty());
+                           act_, weight_on_output_, mid, (float *)out.data, ctx.stream, !gate_.empty(), glu_);
+      if (identity_ > 0) kernels::moe_identity(x, chosen, weight, experts_, top_, (int)hidden_, (float *)out.data, ctx.stream);
     } else {
       kernels::moe_rows(x, w_up_.get(), w_down_.get(), chosen, weight, top_, (int)hidden_, (int)inter_, act_, weight_on_output_,
-                        (float *)out.data, ctx.stream, !gate_.empty());
+                        (float *)out.data, ctx.stream, !gate_.empty(), experts_, glu_);
     }
     if (s_own) {
       if (s.dtype != DType::F32 || s.rows != T || s.cols != hidden_ || s.ld != hidden_)
         LLM_THROW(Unsupported, "moe: the shared feed-forward must hand over dense 32-bit rows");
       if (!shared_gate_.empty())
         kernels::row_gate((const float *)s.data, s.part_stride, (float *)out.data + (size_t)top_ * (size_t)out.part_stride,
-                          out.part_stride, s.parts, (const float *)z.data + experts_, z.ld, (int)T, (int)hidden_, ctx.stream);
-      for (int p = 0; p < s.parts && shared_gate_.empty(); ++p)
+                          out.part_stride, s.parts, (const float *)z.data + choices_, z.ld, (int)T, (int)hidden_, ctx.stream);
+      for (int p = 0; p < s.parts && shared_gate_.empty() && !in_place; ++p)
         LLM_CUDA(cudaMemcpyAsync((float *)out.data + (size_t)(top_ + p) * (size_t)out.part_stride,
                                  (const float *)s.data + (size_t)p * (size_t)s.part_stride, sizeof(float) * (size_t)(T * hidden_),
                                  cudaMemcpyDeviceToDevice, ctx.stream));
@@ -245,7 +285,8 @@ class RoutedFeedForward : public FeedForward {
 
  private:
   int64_t hidden_, inter_;
-  int experts_, top_, score_, act_;
+  int experts_, top_, score_, act_, identity_ = 0, choices_ = 0;     // choices: experts and identity experts
+  kernels::Glu glu_;
   bool renormalize_, weight_on_output_, grouped_route_ = false;
   int groups_ = 1, keep_ = 1, group_top_ = 2, router_rows_ = 0;
   float norm_eps_ = 0.f, route_scale_ = 1.f;
@@ -316,10 +357,21 @@ class ClampedGlu : public FeedForward {
     return fams;
   }
   Act forward(StepContext &ctx, const Act &x) override {
-    Act gu = linear(ctx, x, w_gate_up_, nullptr, DType::F32);
-    flush_chain(ctx);
-    Act m = ctx.arena->act(ctx.dtype, x.rows, inter_);
-    kernels::clamped_glu(gu, gate_bias_.empty() ? nullptr : b_gate_up_.buf.as<float>(), m, limit_, slope_, up_shift_, ctx.stream);
+    Act m;
+    if (gate_bias_.empty()) {
+      kernels::Glu glu;
+      if (limit_ > 0.f) glu.limit = limit_;
+      glu.slope = slope_;
+      glu.shift = up_shift_;
+      m = fused_gated_linear(ctx, x, w_gate_up_, &glu);
+      if (m.data) flush_chain(ctx);
+    }
+    if (!m.data) {
+      Act gu = linear(ctx, x, w_gate_up_, nullptr, DType::F32);
+      flush_chain(ctx);
+      m = ctx.arena->act(ctx.dtype, x.rows, inter_);
+      kernels::clamped_glu(gu, gate_bias_.empty() ? nullptr : b_gate_up_.buf.as<float>(), m, limit_, slope_, up_shift_, ctx.stream);
+    }
     if (down_bias_.empty()) return linear(ctx, m, w_down_, nullptr, DType::F32, true);
     // with a bias the product cannot add to the stream as it stores: the bias goes with the result
     float *const sink = ctx.residual_sink;

@@ -9,7 +9,9 @@
 // that width, no value storage).  The products with W_uk and W_uv are moved to the query's side and behind the
 // weighted sum (csrc/latent.cu says how), so a step reads the cached rows once per head and never expands them.
 // A run that the schedule gives another run's cache (ScheduleEntry::cache_from) has no W_dkv of its own: it
-// reads the rows that run appended, with its own W_uk, W_uv and queries.  With `window` w a query at position p sees the
+// reads the rows that run appended, with its own W_uk, W_uv and queries.  Without q_down, q_norm and q_up the queries come from the
+// input directly, q = W_q h (`q`).  `null_scores` (a vector [n_heads]): every query also sees one key of that score that has no
+// value (a learned sink).  `head_gate` (a matrix [n_heads, hidden]): head h's result is multiplied by sigmoid(gate h)_h.  With `window` w a query at position p sees the
 // rows of positions p - w + 1 .. p only, and the cache gives earlier pages back.  The rotation is the position part's
 // (either pairing; its table carries whatever the scaling puts on cosines and sines); `scale` is the
 // description's.  The reference has no such mixer (its attention: src/libllm/llama.cc:178-225).
@@ -36,13 +38,19 @@ class LatentAttention : public Mixer {
     rot_ = (int)r.integer("rot_dim", 0);
     dv_ = (int)r.integer_or("v_head_dim", d_);
     kv_rank_ = (int)r.integer("kv_rank");
-    q_rank_ = (int)r.integer("q_rank");
+    q_rank_ = (int)r.integer_or("q_rank", 0, 0);
     scale_ = (float)r.number_or("scale", 1.0 / std::sqrt((double)(d_ + rot_)), false);
     eps_ = (float)r.number("eps");
     window_ = (int)r.integer_or("window", 0, 0);
-    q_down_ = r.string("q_down");
-    q_norm_ = r.string("q_norm");
-    q_up_ = r.string("q_up");
+    if (q_rank_ > 0) {
+      q_down_ = r.string("q_down");
+      q_norm_ = r.string("q_norm");
+      q_up_ = r.string("q_up");
+    } else {
+      q_ = r.string("q");
+    }
+    null_scores_name_ = r.string_or("null_scores", "");
+    gate_ = r.string_or("head_gate", "");
     kv_down_ = r.string_or("kv_down", "");
     kv_norm_ = r.string_or("kv_norm", "");
     if (kv_down_.empty() != kv_norm_.empty()) r.fail("'kv_down' and 'kv_norm' come together");
@@ -56,40 +64,52 @@ class LatentAttention : public Mixer {
       if (spec.get("position").is_null()) r.fail("rotated channels need a 'position' part");
       position_ = build_as<PositionEncoding>("position", spec.get("position"), env);
     }
-    down_rows_ = ((int64_t)q_rank_ + (own_latent() ? kv_rank_ + rot_ : 0) + 7) / 8 * 8;
+    // the stacked product: [queries, or their latent | latent and rotated key part | gate], each from a multiple of 8 on
+    auto eights = [](int64_t n) { return (n + 7) / 8 * 8; };
+    off_kv_ = q_rank_ > 0 ? q_rank_ : eights((int64_t)n_heads_ * (d_ + rot_));
+    off_gate_ = eights(off_kv_ + (own_latent() ? kv_rank_ + rot_ : 0));
+    down_rows_ = off_gate_ + (gate_.empty() ? 0 : eights(n_heads_));
   }
   bool own_latent() const { return !kv_down_.empty(); }
 
   std::vector<TensorNeed> tensor_needs() const override {
-    std::vector<TensorNeed> needs = {{q_down_, {(int64_t)q_rank_, hidden_}},
-                                     {q_norm_, {(int64_t)q_rank_}, TensorRole::Vector, false},
-                                     {q_up_, {(int64_t)n_heads_ * (d_ + rot_), (int64_t)q_rank_}},
-                                     {k_up_, {(int64_t)n_heads_ * d_, (int64_t)kv_rank_}},
-                                     {v_up_, {(int64_t)n_heads_ * dv_, (int64_t)kv_rank_}},
-                                     {o_, {hidden_, (int64_t)n_heads_ * dv_}}};
+    std::vector<TensorNeed> needs = {k_up_need(), v_up_need(), {o_, {hidden_, (int64_t)n_heads_ * dv_}}};
+    if (q_rank_ > 0) {
+      needs.push_back({q_down_, {(int64_t)q_rank_, hidden_}});
+      needs.push_back({q_norm_, {(int64_t)q_rank_}, TensorRole::Vector, false});
+      needs.push_back({q_up_, {(int64_t)n_heads_ * (d_ + rot_), (int64_t)q_rank_}});
+    } else {
+      needs.push_back({q_, {(int64_t)n_heads_ * (d_ + rot_), hidden_}});
+    }
     if (own_latent()) {
       needs.push_back({kv_down_, {(int64_t)kv_rank_ + rot_, hidden_}});
       needs.push_back({kv_norm_, {(int64_t)kv_rank_}, TensorRole::Vector, false});
     }
+    if (!gate_.empty()) needs.push_back({gate_, {(int64_t)n_heads_, hidden_}});
+    if (!null_scores_name_.empty()) needs.push_back({null_scores_name_, {(int64_t)n_heads_}, TensorRole::Vector, false});
     if (position_)
       for (auto &n : position_->tensor_needs()) needs.push_back(n);
     return needs;
   }
 
   void load(const Loader &l) override {
-    const std::vector<TensorNeed> needs = tensor_needs();
-    const size_t es = dtype_size(l.engine);
-    // both latents' projections are one stacked product [W_dq; W_dkv] with a 32-bit result
+    const size_t es = dtype_size(l.engine), row = (size_t)hidden_ * es;
+    // everything that reads the input is one stacked product with a 32-bit result
     w_down_.dtype = l.engine;
     w_down_.rows = down_rows_;
     w_down_.cols = hidden_;
     w_down_.buf.allocate((size_t)down_rows_ * (size_t)hidden_ * es, true);
-    l.fetch_into(needs[0], l.engine, w_down_.buf.get());
-    w_q_norm_ = l.fetch(needs[1]);
-    w_uq_ = l.fetch(needs[2]);
-    w_uk_ = l.fetch(needs[3]);
-    w_uv_ = l.fetch(needs[4]);
-    w_o_ = l.fetch(needs[5]);
+    char *const stacked = (char *)w_down_.buf.get();
+    if (q_rank_ > 0) {
+      l.fetch_into({q_down_, {(int64_t)q_rank_, hidden_}}, l.engine, stacked);
+      w_q_norm_ = l.fetch({q_norm_, {(int64_t)q_rank_}, TensorRole::Vector, false});
+      w_uq_ = l.fetch({q_up_, {(int64_t)n_heads_ * (d_ + rot_), (int64_t)q_rank_}});
+    } else {
+      l.fetch_into({q_, {(int64_t)n_heads_ * (d_ + rot_), hidden_}}, l.engine, stacked);
+    }
+    w_uk_ = l.fetch(k_up_need());
+    w_uv_ = l.fetch(v_up_need());
+    w_o_ = l.fetch({o_, {hidden_, (int64_t)n_heads_ * dv_}});
     if (l.engine == DType::BF16) {
       // [W_uk; W_uv] stacked, for prompt steps that materialise the heads' keys and values in one product
       const int64_t k_rows = (int64_t)n_heads_ * d_, v_rows = (int64_t)n_heads_ * dv_;
@@ -97,13 +117,15 @@ class LatentAttention : public Mixer {
       w_ukv_.rows = (k_rows + v_rows + 7) / 8 * 8;
       w_ukv_.cols = kv_rank_;
       w_ukv_.buf.allocate((size_t)w_ukv_.rows * (size_t)kv_rank_ * es, true);
-      l.fetch_into(needs[3], l.engine, w_ukv_.buf.get());
-      l.fetch_into(needs[4], l.engine, (char *)w_ukv_.buf.get() + (size_t)k_rows * kv_rank_ * es);
+      l.fetch_into(k_up_need(), l.engine, w_ukv_.buf.get());
+      l.fetch_into(v_up_need(), l.engine, (char *)w_ukv_.buf.get() + (size_t)k_rows * kv_rank_ * es);
     }
     if (own_latent()) {
-      l.fetch_into(needs[6], l.engine, (char *)w_down_.buf.get() + (size_t)q_rank_ * hidden_ * es);
-      w_kv_norm_ = l.fetch(needs[7]);
+      l.fetch_into({kv_down_, {(int64_t)kv_rank_ + rot_, hidden_}}, l.engine, stacked + (size_t)off_kv_ * row);
+      w_kv_norm_ = l.fetch({kv_norm_, {(int64_t)kv_rank_}, TensorRole::Vector, false});
     }
+    if (!gate_.empty()) l.fetch_into({gate_, {(int64_t)n_heads_, hidden_}}, l.engine, stacked + (size_t)off_gate_ * row);
+    if (!null_scores_name_.empty()) null_scores_ = l.fetch({null_scores_name_, {(int64_t)n_heads_}, TensorRole::Vector, false});
     if (position_) position_->load(l);
   }
 
@@ -145,10 +167,22 @@ class LatentAttention : public Mixer {
     const int row = kv_rank_ + rot_;
     Act proj = linear(ctx, x, w_down_, nullptr, DType::F32);
     flush_chain(ctx);
-    Act cq = ctx.arena->act(ctx.dtype, T, q_rank_);
-    kernels::latent_place(proj, 0, q_rank_, w_q_norm_.buf.as<float>(), cq, own_latent() ? q_rank_ : -1, kv_rank_, rot_,
-                          own_latent() ? w_kv_norm_.buf.as<float>() : nullptr, eps_, table, table_rows, interleaved, ctx.tok_seq,
-                          ctx.tok_pos, cache->page_table, cache->table_width, cache->k, cache->page_size, ctx.stream);
+    Act cq;
+    cq.dtype = ctx.dtype;
+    if (q_rank_ > 0) cq = ctx.arena->act(ctx.dtype, T, q_rank_);
+    if (q_rank_ > 0 || own_latent())
+      kernels::latent_place(proj, 0, q_rank_, q_rank_ > 0 ? w_q_norm_.buf.as<float>() : nullptr, cq, own_latent() ? (int)off_kv_ : -1, kv_rank_, rot_,
+                            own_latent() ? w_kv_norm_.buf.as<float>() : nullptr, eps_, table, table_rows, interleaved, ctx.tok_seq,
+                            ctx.tok_pos, cache->page_table, cache->table_width, cache->k, cache->page_size, ctx.stream);
+    const float *gate = gate_.empty() ? nullptr : (const float *)proj.data + off_gate_;
+    const float *null_scores = null_scores_name_.empty() ? nullptr : null_scores_.buf.as<float>();
+    // the queries: a product behind their latent, or the stacked product's first columns
+    auto queries = [&]() {
+      if (q_rank_ > 0) return linear(ctx, cq, w_uq_, nullptr, DType::F32);
+      Act q = proj;
+      q.cols = (int64_t)n_heads_ * (d_ + rot_);
+      return q;
+    };
     const bool tc = ctx.dtype == DType::BF16 && kernels::available("latent_tc");
     bool from_start = !ctx.decode_only && !ctx.captured && (int)ctx.past_lens.size() == ctx.n_seqs;
     for (int past : ctx.past_lens) from_start = from_start && past == 0;
@@ -161,16 +195,16 @@ class LatentAttention : public Mixer {
       kr.cols = kr.ld = rot_;
       kernels::latent_rows(cache->k, cache->page_size, row, kv_rank_, ctx.tok_seq, ctx.tok_pos, cache->page_table, cache->table_width, T,
                            c, kr, ctx.stream);
-      Act q = linear(ctx, cq, w_uq_, nullptr, DType::F32);
+      Act q = queries();
       Act kv = linear(ctx, c, w_ukv_, nullptr, ctx.dtype);
       flush_chain(ctx);
       Act qb = ctx.arena->act(ctx.dtype, T, (int64_t)n_heads_ * (d_ + rot_));
       kernels::latent_rotate_q(q, qb, n_heads_, d_, rot_, table, table_rows, interleaved, ctx.tok_pos, ctx.stream);
       kernels::latent_prefill(qb, kv, kr, heads, ctx.seq_start, ctx.n_seqs, ctx.max_q_len, n_heads_, d_, rot_, dv_, scale_, ctx.stream,
-                              window_);
+                              window_, null_scores, gate, proj.ld);
       return linear(ctx, heads, w_o_, nullptr, DType::F32, true);
     }
-    Act q = linear(ctx, cq, w_uq_, nullptr, DType::F32);
+    Act q = queries();
     flush_chain(ctx);
     Act qa = ctx.arena->act(ctx.dtype, T, (int64_t)n_heads_ * row);
     kernels::latent_absorb(q, w_uk_.buf.get(), qa, n_heads_, d_, rot_, kv_rank_, table, table_rows, interleaved, ctx.tok_pos, ctx.stream);
@@ -187,22 +221,25 @@ class LatentAttention : public Mixer {
       float *ws = nullptr;
       if (n_splits > 1) ws = ctx.arena->alloc_n<float>(kernels::latent_decode_floats(T, n_heads_, kv_rank_, n_splits));
       kernels::latent_decode(qa, cache->k, cache->page_size, ctx.tok_seq, ctx.tok_pos, cache->page_table, cache->table_width, n_heads_,
-                             kv_rank_, rot_, n_splits, scale_, mixed, ws, ctx.stream, window_);
+                             kv_rank_, rot_, n_splits, scale_, mixed, ws, ctx.stream, window_, null_scores);
     } else {
       kernels::attention_generic(qa, mixed, cache->k, cache->k, ctx.tok_seq, ctx.tok_pos, cache->page_table, cache->table_width, n_heads_,
-                                 1, row, kv_rank_, cache->page_size, window_, 0, scale_, nullptr, 0, ctx.stream, 0, row);
+                                 1, row, kv_rank_, cache->page_size, window_, 0, scale_, nullptr, 0, ctx.stream, 0, row, kernels::NO_NULL_KEY,
+                                 null_scores);
     }
-    kernels::latent_expand(mixed, w_uv_.buf.get(), heads, n_heads_, kv_rank_, dv_, ctx.stream);
+    kernels::latent_expand(mixed, w_uv_.buf.get(), heads, n_heads_, kv_rank_, dv_, ctx.stream, gate, proj.ld);
     return linear(ctx, heads, w_o_, nullptr, DType::F32, true);
   }
 
  private:
-  int64_t hidden_, down_rows_;
+  TensorNeed k_up_need() const { return {k_up_, {(int64_t)n_heads_ * d_, (int64_t)kv_rank_}}; }
+  TensorNeed v_up_need() const { return {v_up_, {(int64_t)n_heads_ * dv_, (int64_t)kv_rank_}}; }
+  int64_t hidden_, down_rows_, off_kv_ = 0, off_gate_ = 0;
   int n_heads_, d_, rot_, dv_, kv_rank_, q_rank_, window_ = 0;
   float scale_, eps_;
-  std::string q_down_, q_norm_, q_up_, kv_down_, kv_norm_, k_up_, v_up_, o_;
+  std::string q_, gate_, null_scores_name_, q_down_, q_norm_, q_up_, kv_down_, kv_norm_, k_up_, v_up_, o_;
   std::unique_ptr<PositionEncoding> position_;
-  Weight w_down_, w_q_norm_, w_uq_, w_uk_, w_uv_, w_ukv_, w_o_, w_kv_norm_;
+  Weight w_down_, w_q_norm_, w_uq_, w_uk_, w_uv_, w_ukv_, w_o_, w_kv_norm_, null_scores_;
 };
 
 }  // namespace

@@ -6,6 +6,7 @@
 // (src/flint/cuda/gemm_cublas.cc:160-197) and a kernel of its own when one row is multiplied
 // (src/flint/cuda/matvec.cu:61-87).
 #pragma once
+#include "csrc/kernels.h"
 #include "parts/part.h"
 
 namespace llm {
@@ -31,12 +32,17 @@ std::vector<std::string> product_families(DType dtype);
 // results that go into the residual addition, which adds parts in order) the result may be
 // [parts, T, N] partial products to be summed, or, when the block has named the residual
 // stream's rows (StepContext::residual_sink) and the library product runs, the stream itself with
-// the result already added to it.
+// the result already added to it.  With parts_ok and StepContext::parts_pool the result lies in that room where it fits.
 Act linear(StepContext &ctx, const Act &x, const Weight &w, const float *bias, DType out_dtype, bool parts_ok = false);
 
 // The product for steps of few tokens; data == nullptr when it does not take the case.  With
-// `swiglu`, w is the stacked gate|up matrix [2I, K] and the result is silu(gate) * up, [T, I].
-Act small_batch_linear(StepContext &ctx, const Act &x, const Weight &w, DType out_dtype, bool swiglu, bool parts_ok);
+// `swiglu`, w is the stacked gate|up matrix [2I, K] and the result is silu(gate) * up, [T, I], or with `glu` that gated unit.
+Act small_batch_linear(StepContext &ctx, const Act &x, const Weight &w, DType out_dtype, bool swiglu, bool parts_ok,
+                       const kernels::Glu *glu = nullptr);
+
+// The gated unit of a stacked gate|up product in one launch where the tensor-core product takes it (few tokens, or a prompt
+// step where fusing beats the library product); data == nullptr otherwise.
+Act fused_gated_linear(StepContext &ctx, const Act &x, const Weight &w_gate_up, const kernels::Glu *glu = nullptr);
 
 // out[T, N] = x[T, K] @ w[N, K]^T by cuBLAS (bfloat16 operands, 32-bit accumulation); false when
 // the library is not to be had.

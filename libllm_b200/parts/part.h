@@ -138,6 +138,11 @@ struct StepContext {
   float *parts_pool = nullptr;
   int parts_cap = 0, parts_used = 0;
   int64_t parts_rows = 0, parts_cols = 0;
+  // What a model with a table of side vectors (ModelSpec::token_table) hands its blocks: the tokens' numbers as they were
+  // resolved on the device [T], the table [vocab, token_table_width] in the engine's type.
+  const int *token_ids = nullptr;
+  const void *token_table = nullptr;
+  int64_t token_table_width = 0;
   // Set by the model for the last layer of a step that wants the logits of fewer rows than it has
   // tokens (a prompt whose last token alone is wanted): after that layer's mixer nothing but these
   // rows of the residual stream is read.  A block may then go on with those rows alone

@@ -9,7 +9,8 @@
 // computed (32-bit), so that the products run on the tensor cores; the convolution's last taps - 1 inputs are state of the run.
 //
 // "sum": a list of mixers that all read the same input; the result is the sum of theirs.  At most one keeps keys and values;
-// state of all is kept side by side.
+// state of all is kept side by side.  With `norms` {weights: a name per mixer, eps, scale}, of two mixers, the result is
+// scale * sum_i y_i / sqrt(mean(y_i^2) + eps) * weight_i (32-bit, in the pass that adds it to the stream).
 //
 // Reference counterpart of the attention: src/libllm/llama.cc:178-225 (a softmax, no convolution); none of the sum.
 #include <algorithm>
@@ -215,15 +216,28 @@ class SumMixer : public Mixer {
       caches += mixers_.back()->wants_cache() ? 1 : 0;
     }
     if (caches > 1) LLM_THROW(Unsupported, "sum: %d of the mixers keep keys and values (a run has one cache)", caches);
+    if (!spec.get("norms").is_null()) {
+      ConfigReader r(spec.get("norms"), "sum description: norms");
+      hidden_ = r.integer("hidden");
+      eps_ = (float)r.number("eps");
+      scale_ = (float)r.number_or("scale", 1.0, false);
+      const Json &names = spec.get("norms").get("weights");
+      if (!names.is_array() || names.size() != mixers_.size()) r.fail("'weights' must name a vector per mixer");
+      if (mixers_.size() != 2) LLM_THROW(Unsupported, "sum: results with norms of their own are of two mixers (%zu given)", mixers_.size());
+      for (const auto &n : names.items()) norm_names_.push_back(n.as_string());
+    }
   }
   std::vector<TensorNeed> tensor_needs() const override {
     std::vector<TensorNeed> out;
     for (const auto &m : mixers_)
       for (auto &n : m->tensor_needs()) out.push_back(n);
+    for (const auto &n : norm_names_) out.push_back({n, {hidden_}, TensorRole::Vector, false});
     return out;
   }
   void load(const Loader &l) override {
     for (auto &m : mixers_) m->load(l);
+    norms_.clear();
+    for (const auto &n : norm_names_) norms_.push_back(l.fetch({n, {hidden_}, TensorRole::Vector, false}));
   }
   std::vector<std::string> kernel_families() const override {
     std::vector<std::string> out = {"elementwise"};
@@ -260,16 +274,19 @@ class SumMixer : public Mixer {
     // Steps of few tokens hand back partial products: room where all mixers' parts lie one behind the other, so that the next
     // norm adds them in one pass (an outer block may have given such room already).
     constexpr int POOL_PARTS = 16;
-    const bool own_pool = !ctx.parts_pool && ctx.dtype == DType::BF16 && x.rows <= fast_switches().tc_tokens && !ctx.chain;
+    const bool normed = !norm_names_.empty(), few = ctx.dtype == DType::BF16 && x.rows <= fast_switches().tc_tokens;
+    const bool own_pool = !ctx.parts_pool && (few || normed) && !ctx.chain;
     if (own_pool) {
-      ctx.parts_pool = ctx.arena->alloc_n<float>((size_t)POOL_PARTS * (size_t)(x.rows * x.cols));
-      ctx.parts_cap = POOL_PARTS;
+      ctx.parts_cap = few ? POOL_PARTS : (int)mixers_.size();
+      ctx.parts_pool = ctx.arena->alloc_n<float>((size_t)ctx.parts_cap * (size_t)(x.rows * x.cols));
       ctx.parts_used = 0;
       ctx.parts_rows = x.rows;
       ctx.parts_cols = x.cols;
     }
     Act sum, added;
+    if (normed) ctx.residual_sink = nullptr;             // a normed result cannot be added by the product that makes it
     float *const sink = ctx.residual_sink;
+    int first_parts = 0;
     for (size_t i = 0; i < mixers_.size(); ++i) {
       StateView mine;
       const std::string p = prefix(i);
@@ -284,7 +301,15 @@ class SumMixer : public Mixer {
         added = r;
         continue;
       }
+      if (normed && (r.col_bias || r.normed())) LLM_THROW(Unsupported, "sum: a result that is normed comes without a bias or a norm of its own");
+      if (i == 0) first_parts = r.parts;
       sum = sum.data ? joined(ctx, sum, r) : r;
+    }
+    if (normed) {
+      sum.first_parts = first_parts;
+      for (int i = 0; i < 2; ++i) sum.pair_w[i] = norms_[(size_t)i].buf.as<float>();
+      sum.pair_eps = eps_;
+      sum.pair_scale = scale_;
     }
     if (own_pool) ctx.parts_pool = nullptr;
     return sum.data ? sum : added;
@@ -317,6 +342,10 @@ class SumMixer : public Mixer {
     return s;
   }
   std::vector<std::unique_ptr<Mixer>> mixers_;
+  std::vector<std::string> norm_names_;
+  std::vector<Weight> norms_;
+  int64_t hidden_ = 0;
+  float eps_ = 0.f, scale_ = 1.f;
 };
 
 template <typename T>

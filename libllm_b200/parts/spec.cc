@@ -11,6 +11,18 @@ Json ModelSpec::to_json() const {
   j.set("hidden", hidden);
   j.set("embedding", embedding);
   j.set("position_table", position_table.empty() ? Json() : Json(position_table));
+  if (!token_pairs.table.empty()) {
+    Json tp = Json::object();
+    tp.set("table", token_pairs.table);
+    tp.set("buckets", token_pairs.buckets);
+    tp.set("mul_prev", token_pairs.mul_prev);
+    tp.set("mul_cur", token_pairs.mul_cur);
+    j.set("token_pairs", tp);
+  }
+  if (!token_table.empty()) {
+    j.set("token_table", token_table);
+    j.set("token_table_width", token_table_width);
+  }
   Json ls = Json::array();
   for (const auto &l : layers) ls.push(l);
   j.set("layers", ls);
@@ -49,6 +61,15 @@ ModelSpec ModelSpec::from_json(const Json &j) {
   s.hidden = r.integer("hidden");
   s.embedding = r.string("embedding");
   s.position_table = r.string_or("position_table", "");
+  if (r.present("token_pairs")) {
+    ConfigReader t(r.object("token_pairs"), "model description: token_pairs");
+    s.token_pairs.table = t.string("table");
+    s.token_pairs.buckets = t.integer("buckets");
+    s.token_pairs.mul_prev = t.integer("mul_prev", 0);
+    s.token_pairs.mul_cur = t.integer("mul_cur", 0);
+  }
+  s.token_table = r.string_or("token_table", "");
+  if (!s.token_table.empty()) s.token_table_width = r.integer("token_table_width");
   const Json &ls = j.get("layers");
   if (!ls.is_array()) r.fail("'layers' must be a list of block descriptions");
   for (const auto &l : ls.items()) {

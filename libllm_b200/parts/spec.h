@@ -22,7 +22,9 @@
 //   mixer "attention" also: v_head_dim, qk_norm {q, k, eps}, block (mask), head_gate (parts/builtin.cc)
 //   feed_forward "mlp":    hidden, intermediate, activation (gelu, gelu_tanh, silu), up, down
 //   feed_forward "moe":    hidden, experts, top, score, renormalize, weight_on, router, expert {..}, shared
-//   block "prenorm":       mixer_norm, mixer, ff_norm, ff (descriptions; ff and ff_norm may be null), mixer_conv {taps, weight, hidden}
+//   mixer "selective_scan": a diagonal state per channel (parts/selective.cc)
+//   block "prenorm":       mixer_norm, mixer, ff_norm, ff (descriptions; ff and ff_norm may be null), mixer_conv {taps, weight, hidden},
+//                          mixer_post, ff_post {weight, eps}, side {dim, offset, gate, proj, norm, eps} (parts/builtin.cc)
 //   block "parallel":      norm, mixer, ff (a description or null): x + mixer(norm x) + ff(norm x)
 //   block "hyper":         the pre-norm block over several copies of the residual stream (parts/builtin.cc)
 #pragma once
@@ -50,12 +52,22 @@ struct ScheduleEntry {
   int add_row = 0;
 };
 
+// Rows for pairs of neighbouring tokens, added to the tokens' own: row (previous * mul_prev + current * mul_cur) mod buckets of a
+// table [buckets + 1, hidden], the last row for a sequence's first token.  A sequence's last token is state of the model.
+struct TokenPairSpec {
+  std::string table;                      // empty: none
+  int64_t buckets = 0, mul_prev = 0, mul_cur = 0;
+};
+
 struct ModelSpec {
   std::string name;
   int64_t vocab_size = 0;
   int64_t hidden = 0;
   std::string embedding;                  // tensor name of the token table
   std::string position_table;             // [max_positions, hidden]: a learned vector per position, added to the token's row; empty: none
+  TokenPairSpec token_pairs;
+  std::string token_table;                // [vocab_size, token_table_width]: side vectors of the tokens that blocks read (StepContext::token_table); empty: none
+  int64_t token_table_width = 0;
   std::vector<Json> layers;               // block descriptions
   std::vector<ScheduleEntry> schedule;
   Json final_norm;

@@ -125,6 +125,15 @@ struct Act {
   // memory, either may be null); what is added is (sum of parts + col_bias) * col_scale.
   const float *col_scale = nullptr;
   const float *col_bias = nullptr;
+  // A result that is normed before it is added (32-bit vectors over the columns, device memory), unit(x) = x / sqrt(mean(x^2) +
+  // eps): with first_parts f > 0 it is two results side by side, y = pair_scale * (unit(parts 0 .. f-1) * pair_w[0] +
+  // unit(the other parts) * pair_w[1]), else y is the sum of the parts (+ col_bias); with `post`, unit(y) * post is added.
+  int first_parts = 0;
+  const float *pair_w[2] = {nullptr, nullptr};
+  float pair_eps = 0.f, pair_scale = 1.f;
+  const float *post = nullptr;
+  float post_eps = 0.f;
+  bool normed() const { return post != nullptr || first_parts > 0; }
 };
 
 // A weight on the device: [rows, cols] row-major, or a vector (rows = 1).  With `view` it is rows of another weight's memory.
