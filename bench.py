@@ -673,6 +673,122 @@ def run_compare_tazizen(args):
     return 0
 
 
+# ---------------------------------------------------------------- Fomodra beside Tazizen at equal sizes
+def fomodra_config(hidden, runs, heads, kv, dim, ff, vocab, window=1024, kv_rank=512, experts=32, identity=4, top=4):
+    """A Fomodra model of `runs` layers in the order attention, parallel, latent attention, attention that borrows the first's keys
+    and values, every layer with the routed feed-forward: `experts` experts of ff / 8 and `identity` identity experts, of which
+    `top` (4: half of ff) are chosen, and a shared expert of ff / 2.  Windows and chunks of `window` positions; chunked attention with
+    half the heads and values twice as wide as keys; a scan of 2 * hidden channels with 16 states, a dt input of hidden / 16; latent
+    heads of dim unrotated and dim / 2 rotated channels; side vectors of hidden / 8."""
+    rot, mask = dict(dims=dim, base=2.5e5), dict(size=window)
+    mlp = dict(kind="moe", expert=dict(ff=ff // 8, limit=7.0), shared=dict(ff=ff // 2, limit=7.0),
+               router=dict(experts=experts, identity=identity, top=top))
+    att = dict(heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=dim ** -0.5, rot=rot, mask=mask)
+    left = dict(heads=heads // 2, kv_heads=kv // 2, dim=dim, vdim=2 * dim, scale=dim ** -0.5, mask=mask,
+                rot=dict(dims=dim, base=5e5, scaling=dict(factor=4.0, low=1.0, high=4.0, original=2048)))
+    layers = []
+    for i in range(runs):
+        if i % 4 == 1:
+            L = dict(type="parallel", mixer=dict(left=left, right=dict(inner=2 * hidden, state=16, dt_rank=hidden // 16, conv=4)))
+        elif i % 4 == 2:
+            L = dict(type="latent_attention", mixer=dict(heads=heads, dim=dim, rot_dim=dim // 2, vdim=dim, kv_rank=kv_rank, mask=mask,
+                                                         scale=(dim + dim // 2) ** -0.5, rot=dict(dims=dim // 2, base=1e6)))
+        else:
+            L = dict(type="attention", mixer=dict(att, **({"kv_from": i - 3} if i % 4 == 3 else {})))
+        layers.append(dict(mlp=mlp, **L))
+    return dict(architecture="Fomodra", vocab=vocab, width=hidden, norm=dict(eps=1e-5), layers=layers, token_side=dict(dim=hidden // 8),
+                embedding=dict(bigram=dict(buckets=50021, mul_prev=31337, mul_cur=7)))
+
+
+def fomodra_numbers(c, batch):
+    """(bytes a decode step reads at least and at most apart from cache and state: the experts that every sequence chooses alike, or
+    that no two share; cache bytes of a sequence as a function of its length, bytes of state a step reads and writes per sequence,
+    prefill flops of T tokens with one wanted row)."""
+    H, V = c["width"], c["vocab"]
+    used = most = state = rec = 0
+    att = []                                          # (window or chunk, chunked, cache bytes a key, flops a key)
+    for L in c["layers"]:
+        m = L["mixer"]
+        a = m["left"] if L["type"] == "parallel" else m
+        size = (a.get("mask") or {}).get("size") or (1 << 30)
+        if L["type"] == "latent_attention":
+            row = m["kv_rank"] + m["rot_dim"]
+            mats = H * m["heads"] * (m["dim"] + m["rot_dim"]) + m["heads"] * (m["dim"] + m["vdim"]) * m["kv_rank"] + m["heads"] * m["vdim"] * H
+            mats += H * (row + m["heads"])
+            att.append((size, False, 2 * row, 2 * m["heads"] * (m["dim"] + m["rot_dim"] + m["vdim"])))
+        else:
+            own = "kv_from" not in a
+            mats = H * (a["heads"] * a["dim"] + (a["kv_heads"] * (a["dim"] + a["vdim"]) if own else 0)) + a["heads"] * a["vdim"] * H
+            att.append((size, L["type"] == "parallel", 2 * a["kv_heads"] * (a["dim"] + a["vdim"]), 2 * a["heads"] * (a["dim"] + a["vdim"])))
+        if L["type"] == "parallel":
+            r = m["right"]
+            I, N, R = r["inner"], r["state"], r["dt_rank"]
+            mats += 3 * H * I + I * (R + 2 * N) + I * R
+            state += 2 * 4 * I * (N + r["conv"] - 1)
+            rec += 6 * I * N
+            most += 4 * I * N                         # A_log, 32-bit
+        mats += 2 * H * c["token_side"]["dim"]
+        f = L["mlp"]
+        r, one = f["router"], 3 * H * f["expert"]["ff"]
+        fixed = mats + (r["experts"] + r["identity"]) * H + 3 * H * f["shared"]["ff"]
+        used += fixed + r["top"] * one
+        most += fixed + min(r["experts"], batch * r["top"]) * one
+
+    def seen(p, size, chunked):
+        return p % size + 1 if chunked else min(p + 1, size)
+
+    def cache_bytes(n):
+        return sum(b * seen(n - 1, w, ch) for w, ch, b, _ in att)
+
+    def prefill_flops(T):
+        return 2 * T * used + T * rec + sum(fl * sum(seen(p, w, ch) for p in range(T)) for w, ch, _, fl in att) + 2 * V * H
+    return (2 * (used + V * H), 2 * (most + V * H)), cache_bytes, state, prefill_flops
+
+
+def run_compare_fomodra(args):
+    """Prefill and decode of Fomodra beside Tazizen (the other design with windowed and latent attention, corrected routing and a
+    shared expert), both with random weights, at equal hidden size, number of layers, heads, head size, feed-forward values used per
+    token and vocabulary: one JSON line per size and model."""
+    import torch
+    from libllm_b200 import Model
+    pk = peaks()
+    for name in [n for n in SOBEZEN_SIZES if not args.sizes or n in args.sizes.split(",")]:
+        hidden, runs, heads, kv, dim, ff, vocab = SOBEZEN_SIZES[name]
+        for label in ("tazizen", "fomodra"):
+            if args.model and args.model != label:
+                continue
+            if label == "tazizen":
+                cfg, state = tazizen_config(hidden, runs, heads, kv, dim, ff, vocab), 0
+                most, cache_fn, flops_fn = tazizen_numbers(cfg, args.batch)
+                one = 2 * 3 * hidden * (ff // 8)
+                r = cfg["layers"][0]["mlp"]["router"]
+                wbytes = (most - runs * (min(r["experts"], args.batch * r["top"]) - r["top"]) * one, most)
+            else:
+                cfg = fomodra_config(hidden, runs, heads, kv, dim, ff, vocab)
+                wbytes, cache_fn, state, flops_fn = fomodra_numbers(cfg, args.batch)
+            flops = flops_fn(PROMPT)
+            model = Model.from_random(cfg, seed=0, dtype="bfloat16", max_tokens=args.batch * CONTEXT, max_seq_len=CONTEXT)
+            sampler = ClockSampler()
+            sampler.start()
+            pre = prefill_rate(model, vocab, lambda T: flops, pk["bf16_tflops"])
+            rate, ms, ctx_len, launches = decode_rate(model, args.batch, args.steps, args.warmup, vocab)
+            clocks = sampler.stop()
+            step_bytes = [b + args.batch * (cache_fn(ctx_len) + state) for b in wbytes]
+            print(json.dumps({"compare": name, "model": label, "batch": args.batch, "prompt": PROMPT,
+                              "config": {"hidden": hidden, "layers": runs, "heads": heads, "kv_heads": kv, "head_dim": dim, "ff": ff,
+                                         "vocab": vocab, "order": [L["type"] for L in cfg["layers"]]},
+                              "prefill": {"ms": round(pre["ms"], 3), "tok_s": round(pre["value"], 1), "tflop": round(flops / 1e12, 3),
+                                          "frac_of_gemm_peak": round(pre["frac"], 4)},
+                              "decode": {"tok_s": round(rate, 1), "ms_per_step": round(ms, 4), "launches_per_step": launches,
+                                         "step_gb": [round(b / 1e9, 3) for b in step_bytes],      # at least, at most
+                                         "hbm_frac_at_least": round(step_bytes[0] / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)},
+                              "clocks": clocks, "peaks": pk["source"]}), flush=True)
+            model.engine.close()
+            del model
+            torch.cuda.empty_cache()
+    return 0
+
+
 def rarelorn_config(hidden, runs, heads, kv, dim, ff, vocab, window=1024, experts=32, top=4, taps=4):
     """A Rarelorn model of `runs` layer runs: [parallel, mlstm, delta, delta] as often as the runs ask for (a loop over the
     four layers), every layer with `experts` experts of ff / 4 of which `top` are chosen in the better half of four groups (a
@@ -884,10 +1000,10 @@ def main():
                     help="1b: the benchmark line (default); 3b, 8b: the larger workloads, a line of their own")
     ap.add_argument("--only", choices=["decode", "prefill"], default=None,
                     help="run one part only and print a short line (for profiling; not a bench record)")
-    ap.add_argument("--compare", choices=["sinezen", "sesuzen", "sobezen", "tazizen", "rarelorn"], default=None,
+    ap.add_argument("--compare", choices=["sinezen", "sesuzen", "sobezen", "tazizen", "rarelorn", "fomodra"], default=None,
                     help="Sinezen, Sesuzen, Sobezen or Tazizen beside Llama (Rarelorn beside Sesuzen) at equal sizes: prefill and decode, a line per size and model (not a bench record)")
-    ap.add_argument("--model", choices=["llama", "sesuzen", "sobezen", "tazizen", "rarelorn"], default=None,
-                    help="with --compare sesuzen, sobezen, tazizen or rarelorn: one of the two models only")
+    ap.add_argument("--model", choices=["llama", "sesuzen", "sobezen", "tazizen", "rarelorn", "fomodra"], default=None,
+                    help="with --compare sesuzen, sobezen, tazizen, rarelorn or fomodra: one of the two models only")
     ap.add_argument("--sizes", default=None, help="with --compare: which of the sizes (2k, 4k, 2k-routed), with commas")
     ap.add_argument("--prompt-len", type=int, default=None,
                     help="with --only: prompts of this many tokens instead of 2048 (the context grows to fit)")
@@ -913,6 +1029,8 @@ def main():
         return run_compare_tazizen(args)
     if args.compare == "rarelorn":
         return run_compare_rarelorn(args)
+    if args.compare == "fomodra":
+        return run_compare_fomodra(args)
     if args.compare:
         return run_compare(args)
     if args.workload != "1b":

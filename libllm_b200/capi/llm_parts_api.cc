@@ -60,6 +60,17 @@ Act act_from(const Json &j) {
   a.ld = j.has("ld") ? j.get("ld").as_int() : a.cols;
   a.parts = j.has("parts") ? (int)j.get("parts").as_int() : 1;
   a.part_stride = j.has("part_stride") ? j.get("part_stride").as_int() : a.rows * a.cols;
+  // a result with norms of its own (Act::normed())
+  if (j.has("post")) {
+    a.post = (const float *)ptr_of(j.get("post"));
+    a.post_eps = (float)j.get("post_eps").as_number();
+  }
+  if (j.has("first_parts")) {
+    a.first_parts = (int)j.get("first_parts").as_int();
+    for (size_t i = 0; i < 2; ++i) a.pair_w[i] = (const float *)ptr_of(j.get("pair_w").at(i));
+    a.pair_eps = (float)j.get("pair_eps").as_number();
+    a.pair_scale = (float)j.get("pair_scale").as_number();
+  }
   return a;
 }
 
@@ -74,6 +85,18 @@ Json act_json(const Act &a) {
   j.set("parts", a.parts);
   j.set("part_stride", a.part_stride);
   if (a.col_bias) j.set("col_bias", (int64_t)(uintptr_t)a.col_bias);   // added to the parts' sum by whoever adds the result
+  if (a.post) {                          // and so are its norms
+    j.set("post", (int64_t)(uintptr_t)a.post);
+    j.set("post_eps", (double)a.post_eps);
+  }
+  if (a.first_parts > 0) {
+    j.set("first_parts", a.first_parts);
+    Json w = Json::array();
+    for (const float *p : a.pair_w) w.push((int64_t)(uintptr_t)p);
+    j.set("pair_w", w);
+    j.set("pair_eps", (double)a.pair_eps);
+    j.set("pair_scale", (double)a.pair_scale);
+  }
   return j;
 }
 

@@ -56,7 +56,7 @@ __device__ __forceinline__ float2 ld_l2_pair(const float *p) {
 }
 
 // D, DV: channels of a key and of a value; with EXACT they are the heads' own, else d <= D and dv <= DV are (multiples of 8).
-__host__ __device__ constexpr int decode_tc_ctas(int dmax) { return dmax <= 64 ? 5 : 3; }
+__host__ __device__ constexpr int decode_tc_ctas(int dmax) { return dmax <= 64 ? 5 : dmax <= 128 ? 3 : 2; }
 
 template <int D, int DV, bool EXACT, int DT_WARPS>
 __global__ void __launch_bounds__(DT_WARPS * 32, decode_tc_ctas(D > DV ? D : DV))
@@ -540,7 +540,7 @@ static int launch_decode_tc(const DecodeTcArgs &a, cudaStream_t stream) {
 // how many key splits fill the GPU once.
 LLM_EXPORT int llm_attention_decode_tc_ctas(int d, int dv) {
   const bool exact = d == dv && d % 16 == 0;
-  const int D = exact ? d : d <= 64 ? 64 : 128, DV = exact ? dv : dv <= 64 ? 64 : 128;
+  const int D = exact ? d : d <= 64 ? 64 : 128, DV = exact ? dv : dv <= 64 ? 64 : dv <= 128 ? 128 : 256;
   const size_t smem = decode_tc_tiles(D, DV) + 2048;
   const int by_smem = (int)((227 * 1024) / smem), by_regs = decode_tc_ctas(D > DV ? D : DV);
   return by_smem < by_regs ? (by_smem < 1 ? 1 : by_smem) : by_regs;
@@ -549,7 +549,7 @@ LLM_EXPORT int llm_attention_decode_tc_ctas_per_sm(int d) { return llm_attention
 
 // 1 if these head sizes, page size and group size have an instantiation, else 0.
 LLM_EXPORT int llm_attention_decode_tc_takes(int d, int dv, int page_size, int group) {
-  const bool sizes = d == dv ? d >= 8 && d <= 128 && d % 8 == 0 : d > 0 && d <= 128 && d % 8 == 0 && dv > 0 && dv <= 128 && dv % 8 == 0;
+  const bool sizes = d == dv ? d >= 8 && d <= 128 && d % 8 == 0 : d > 0 && d <= 128 && d % 8 == 0 && dv > 0 && dv <= 256 && dv % 8 == 0;
   return page_size == DT_BN && sizes && group >= 1 && group <= DT_ROWS;
 }
 // The head sizes (values as wide as keys) with an instantiation of exactly their size.
@@ -596,8 +596,11 @@ LLM_EXPORT int llm_attention_decode_tc_sinks(const float *qkv, long long qkv_str
   DT_CASE(16) DT_CASE(32) DT_CASE(48) DT_CASE(64) DT_CASE(80) DT_CASE(96) DT_CASE(112) DT_CASE(128)
 #undef DT_CASE
   if (d == 64 && dv == 128) return launch_decode_tc<64, 128, true>(a, stream);
-  if (d <= 64) return dv <= 64 ? launch_decode_tc<64, 64, false>(a, stream) : launch_decode_tc<64, 128, false>(a, stream);
-  return dv <= 64 ? launch_decode_tc<128, 64, false>(a, stream) : launch_decode_tc<128, 128, false>(a, stream);
+  if (d <= 64)
+    return dv <= 64 ? launch_decode_tc<64, 64, false>(a, stream) : dv <= 128 ? launch_decode_tc<64, 128, false>(a, stream)
+                                                                             : launch_decode_tc<64, 256, false>(a, stream);
+  return dv <= 64 ? launch_decode_tc<128, 64, false>(a, stream) : dv <= 128 ? launch_decode_tc<128, 128, false>(a, stream)
+                                                                            : launch_decode_tc<128, 256, false>(a, stream);
 }
 
 // Values as wide as keys, no bias, no further key.

@@ -683,11 +683,24 @@ int moe_tc_tile_rows(int n_rows) {
 }
 void moe_tc(const Act &x, const void *up, const void *down, const int *offsets, const int *perm, const int *tiles,
             const float *weight, int n_experts, int top, int width, int ff, int act, bool weight_on_output, void *xs, void *mid,
-            float *out, int *status, cudaStream_t s, bool gated, const Glu &glu, const int *chosen) {
+            float *out, int *status, cudaStream_t s, bool gated, const Glu &glu, const int *chosen, bool gathered) {
   const int n_rows = (int)x.rows * top;
-  LLM_CALL("moe", llm_moe_gather_identity, x.data, (long long)x.ld, perm, n_rows, top, width, xs, chosen, offsets, weight, n_experts, out, s);
+  if (!gathered)
+    LLM_CALL("moe", llm_moe_gather_identity, x.data, (long long)x.ld, perm, n_rows, top, width, xs, chosen, offsets, weight, n_experts, out, s);
   LLM_CALL("moe_tc", llm_moe_tc_glu, xs, up, down, offsets, perm, tiles, weight, (int)x.rows, n_experts, top, width, ff, act,
            weight_on_output ? 1 : 0, gated ? 1 : 0, glu.limit, glu.slope, glu.shift, mid, out, status, s);
+}
+LLM_KERNEL("moe", llm_moe_plan, const float *, long long, int, int, int, int, int, const float *, int, int, int, int, float, float, int,
+           const void *, long long, int, int *, float *, int *, int *, int *, void *, float *, cudaStream_t)
+int moe_plan_rows() {
+  static const int n = resolve<int (*)()>("moe", "llm_moe_plan_rows")();
+  return n;
+}
+void moe_plan(const Act &z, const RouteRule &r, int n_experts, int tile_rows, const Act &x, int *chosen, float *weight, int *offsets, int *perm,
+              int *tiles, void *xs, float *out, cudaStream_t s) {
+  LLM_CALL("moe", llm_moe_plan, (const float *)z.data, (long long)z.ld, (int)z.rows, r.choices, n_experts, r.top, r.score, r.correction, r.groups,
+           r.keep, r.group_top, r.renormalize ? 1 : 0, r.norm_eps, r.scale, tile_rows, x.data, (long long)x.ld, (int)x.cols, chosen, weight, offsets,
+           perm, tiles, xs, out, s);
 }
 void moe_rows(const Act &x, const void *up, const void *down, const int *chosen, const float *weight, int top, int width, int ff,
               int act, bool weight_on_output, float *out, cudaStream_t s, bool gated, int n_experts, const Glu &glu) {

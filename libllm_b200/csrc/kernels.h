@@ -254,6 +254,17 @@ int moe_tile_rows();
 void moe_sort(const int *chosen, int n_rows, int n_experts, int tile_rows, int *offsets, int *perm, int *tiles, cudaStream_t s);
 // x [T, width]; up [E, ff, width], down [E, width, ff] in x's type; out [top, T, width] 32-bit.  `gated`: up is
 // [E, 2 ff, width], an expert's gate and up rows interleaved, and the expert is down(act(gate x) * up x).
+// Few tokens (up to moe_plan_rows() rows): moe_route_grouped, moe_sort and the gathering of moe_tc in one launch.
+struct RouteRule {
+  int choices = 0, top = 0, score = 0;             // choices: experts and identity experts
+  const float *correction = nullptr;
+  int groups = 1, keep = 1, group_top = 2;
+  bool renormalize = false;
+  float norm_eps = 0.f, scale = 1.f;
+};
+int moe_plan_rows();
+void moe_plan(const Act &logits, const RouteRule &rule, int n_experts, int tile_rows, const Act &x, int *chosen, float *weight, int *offsets, int *perm,
+              int *tiles, void *xs, float *out, cudaStream_t s);
 void moe_rows(const Act &x, const void *up, const void *down, const int *chosen, const float *weight, int top, int width, int ff,
               int act, bool weight_on_output, float *out, cudaStream_t s, bool gated = false, int n_experts = 0x7fffffff,
               const Glu &glu = Glu());
@@ -269,8 +280,8 @@ bool moe_tc_supported(int width, int ff);
 int moe_tc_tile_rows(int n_rows);
 void moe_tc(const Act &x, const void *up, const void *down, const int *offsets, const int *perm, const int *tiles,
             const float *weight, int n_experts, int top, int width, int ff, int act, bool weight_on_output, void *xs, void *mid,
-            float *out, int *status, cudaStream_t s, bool gated = false, const Glu &glu = Glu(), const int *chosen = nullptr);
-// (chosen: some choices may be identity experts, whose results are written on the way)
+            float *out, int *status, cudaStream_t s, bool gated = false, const Glu &glu = Glu(), const int *chosen = nullptr, bool gathered = false);
+// (gathered: xs holds the rows already, moe_plan; chosen: some choices may be identity experts, whose results are written on the way)
 // ---- state carried from token to token (csrc/recurrent.cu)
 // out = h + conv(h) over time per channel, weight [width, taps] 32-bit; state [slots, taps - 1, width] in h's type.
 // With silu_alone: out = silu(conv(h)), the short convolution of a projection.

@@ -121,36 +121,34 @@ LLM_EXPORT int llm_moe_route(const float *logits, long long ld, int n_tokens, in
 // and only experts of the `keep` best groups can be chosen: the others' c count as minus infinity (c may be
 // negative, so nought would not do).  Weights: s, or with `renormalize` s / (sum of the chosen s + norm_eps), then
 // times route_scale.  Ties go to the lower index.  Everything is 32-bit; a token's result depends on its row alone.
-__global__ void moe_route_grouped_kernel(const float *__restrict__ logits, long long ld, int n_tokens, int n_experts, int top,
-                                         int score_kind, const float *__restrict__ correction, int n_groups, int keep,
-                                         int group_top, int renormalize, float norm_eps, float route_scale,
-                                         int *__restrict__ chosen, float *__restrict__ weight) {
-  extern __shared__ float route_sh[];            // per warp: c [E], group scores [n_groups]
-  grid_dependents_launch();
-  grid_dependency_wait();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int t = blockIdx.x * (blockDim.x >> 5) + warp;
-  if (t >= n_tokens) return;
-  float *c = route_sh + (size_t)warp * (n_experts + n_groups), *gs = c + n_experts;
-  const float *z = logits + (size_t)t * ld;
+struct RouteRule {
+  int n_experts, top, score_kind;                  // n_experts: every choice, identity experts included
+  const float *correction;
+  int n_groups, keep, group_top, renormalize;
+  float norm_eps, route_scale;
+};
+// one token by one warp; c [n_experts] and gs [n_groups] in shared memory are the warp's own
+__device__ __forceinline__ void route_token(const float *__restrict__ z, const RouteRule &R, float *c, float *gs, int lane, int *__restrict__ chosen,
+                                            float *__restrict__ weight) {
+  const int n_experts = R.n_experts, top = R.top;
   float zmax = -INFINITY, denom = 1.f;
-  if (score_kind == 1) {
+  if (R.score_kind == 1) {
     for (int e = lane; e < n_experts; e += 32) zmax = fmaxf(zmax, z[e]);
     zmax = warp_max(zmax);
     float s = 0.f;
     for (int e = lane; e < n_experts; e += 32) s += expf(z[e] - zmax);
     denom = warp_sum(s);
   }
-  auto score_of = [&](int e) { return score_kind == 1 ? expf(z[e] - zmax) / denom : 1.f / (1.f + expf(-z[e])); };
-  for (int e = lane; e < n_experts; e += 32) c[e] = score_of(e) + (correction ? correction[e] : 0.f);
+  auto score_of = [&](int e) { return R.score_kind == 1 ? expf(z[e] - zmax) / denom : 1.f / (1.f + expf(-z[e])); };
+  for (int e = lane; e < n_experts; e += 32) c[e] = score_of(e) + (R.correction ? R.correction[e] : 0.f);
   __syncwarp();
-  if (n_groups > 1) {
-    const int per = n_experts / n_groups;
-    for (int g = lane; g < n_groups; g += 32) {
+  if (R.n_groups > 1) {
+    const int per = n_experts / R.n_groups;
+    for (int g = lane; g < R.n_groups; g += 32) {
       // the sum of the group's group_top largest: each pass takes the largest below (value, index) of the pass before
       float sum = 0.f, last_v = INFINITY;
       int last_e = -1;
-      for (int k = 0; k < group_top && k < per; ++k) {
+      for (int k = 0; k < R.group_top && k < per; ++k) {
         float best = -INFINITY;
         int best_e = -1;
         for (int e = g * per; e < (g + 1) * per; ++e) {
@@ -169,10 +167,10 @@ __global__ void moe_route_grouped_kernel(const float *__restrict__ logits, long 
     }
     __syncwarp();
     // the `keep` best groups, one after another; a kept group's score becomes +infinity as its mark
-    for (int k = 0; k < keep; ++k) {
+    for (int k = 0; k < R.keep; ++k) {
       float best = -INFINITY;
       int best_g = 0x7fffffff;
-      for (int g = lane; g < n_groups; g += 32) {
+      for (int g = lane; g < R.n_groups; g += 32) {
         const float v = gs[g];
         if (v != INFINITY && (best_g == 0x7fffffff || v > best)) {
           best = v;
@@ -222,16 +220,28 @@ __global__ void moe_route_grouped_kernel(const float *__restrict__ logits, long 
     total += s;
     if (lane == 0) {
       c[best_e] = -INFINITY;
-      chosen[(size_t)t * top + j] = best_e;
-      weight[(size_t)t * top + j] = s;
+      chosen[j] = best_e;
+      weight[j] = s;
     }
     __syncwarp();
   }
   for (int j = lane; j < top; j += 32) {
-    float w = weight[(size_t)t * top + j];
-    if (renormalize) w = w / (total + norm_eps);
-    weight[(size_t)t * top + j] = w * route_scale;
+    float w = weight[j];
+    if (R.renormalize) w = w / (total + R.norm_eps);
+    weight[j] = w * R.route_scale;
   }
+}
+
+__global__ void moe_route_grouped_kernel(const float *__restrict__ logits, long long ld, int n_tokens, RouteRule R, int *__restrict__ chosen,
+                                         float *__restrict__ weight) {
+  extern __shared__ float route_sh[];            // per warp: c [E], group scores [n_groups]
+  grid_dependents_launch();
+  grid_dependency_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t = blockIdx.x * (blockDim.x >> 5) + warp;
+  if (t >= n_tokens) return;
+  float *c = route_sh + (size_t)warp * (R.n_experts + R.n_groups);
+  route_token(logits + (size_t)t * ld, R, c, c + R.n_experts, lane, chosen + (size_t)t * R.top, weight + (size_t)t * R.top);
 }
 
 LLM_EXPORT int llm_moe_route_grouped(const float *logits, long long ld, int n_tokens, int n_experts, int top, int score_kind,
@@ -247,8 +257,9 @@ LLM_EXPORT int llm_moe_route_grouped(const float *logits, long long ld, int n_to
               keep, n_experts / n_groups, top);
   const int warps = 4;
   const size_t smem = (size_t)warps * (size_t)(n_experts + n_groups) * sizeof(float);
-  llm_launch(moe_route_grouped_kernel, dim3((n_tokens + warps - 1) / warps), dim3(warps * 32), smem, stream, logits, ld, n_tokens,
-             n_experts, top, score_kind, correction, n_groups, keep, group_top, renormalize, norm_eps, route_scale, chosen, weight);
+  const RouteRule rule{n_experts, top, score_kind, correction, n_groups, keep, group_top, renormalize, norm_eps, route_scale};
+  llm_launch(moe_route_grouped_kernel, dim3((n_tokens + warps - 1) / warps), dim3(warps * 32), smem, stream, logits, ld, n_tokens, rule, chosen,
+             weight);
   LLM_CHECK_LAUNCH("moe_route_grouped");
   return LLM_OK;
 }
@@ -284,36 +295,57 @@ LLM_EXPORT int llm_row_gate(const float *x, long long x_stride, float *out, long
 // tiles[0] = number of row tiles, then (expert, first place) per tile of at most `tile_rows` rows of
 // one expert.  Which place a row gets within its expert depends on the order the threads arrive
 // in; no result depends on it.  Rows of identity experts (chosen >= n_experts) get no place.
-__global__ void __launch_bounds__(1024)
-moe_sort_kernel(const int *__restrict__ chosen, int n_rows, int n_experts, int tile_rows, int *__restrict__ offsets,
-                int *__restrict__ perm, int *__restrict__ tiles) {
-  extern __shared__ int sh[];                  // counts [E], cursor [E]
-  int *counts = sh, *cursor = sh + n_experts;
-  grid_dependents_launch();
-  grid_dependency_wait();
+// By all threads of a block; counts and cursor [E] in shared memory.
+__device__ __forceinline__ void sort_rows(const int *chosen, int n_rows, int n_experts, int tile_rows, int *__restrict__ offsets,
+                                          int *__restrict__ perm, int *__restrict__ tiles, int *counts, int *cursor) {
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) counts[e] = 0;
   __syncthreads();
   for (int r = threadIdx.x; r < n_rows; r += blockDim.x)
     if (chosen[r] < n_experts) atomicAdd(&counts[chosen[r]], 1);
   __syncthreads();
-  if (threadIdx.x == 0) {
-    int o = 0, n_tiles = 0;
-    for (int e = 0; e < n_experts; ++e) {
-      cursor[e] = o;
-      offsets[e] = o;
-      for (int r0 = 0; r0 < counts[e]; r0 += tile_rows) {
-        tiles[1 + 2 * n_tiles] = e;
-        tiles[2 + 2 * n_tiles] = o + r0;
-        ++n_tiles;
+  if (threadIdx.x < 32) {                        // a warp: an expert to a lane, 32 at a time; running sums of rows and of tiles
+    const int lane = threadIdx.x;
+    int rows0 = 0, tiles0 = 0;
+    for (int e0 = 0; e0 < n_experts; e0 += 32) {
+      const int e = e0 + lane, n = e < n_experts ? counts[e] : 0, nt = (n + tile_rows - 1) / tile_rows;
+      int r = n, t = nt;
+#pragma unroll
+      for (int d = 1; d < 32; d <<= 1) {
+        const int a = __shfl_up_sync(0xffffffffu, r, d), b = __shfl_up_sync(0xffffffffu, t, d);
+        if (lane >= d) {
+          r += a;
+          t += b;
+        }
       }
-      o += counts[e];
+      const int o = rows0 + r - n, first = tiles0 + t - nt;
+      if (e < n_experts) {
+        cursor[e] = o;
+        offsets[e] = o;
+        for (int i = 0; i < nt; ++i) {
+          tiles[1 + 2 * (first + i)] = e;
+          tiles[2 + 2 * (first + i)] = o + i * tile_rows;
+        }
+      }
+      rows0 += __shfl_sync(0xffffffffu, r, 31);
+      tiles0 += __shfl_sync(0xffffffffu, t, 31);
     }
-    offsets[n_experts] = o;
-    tiles[0] = n_tiles;
+    if (lane == 0) {
+      offsets[n_experts] = rows0;
+      tiles[0] = tiles0;
+    }
   }
   __syncthreads();
   for (int r = threadIdx.x; r < n_rows; r += blockDim.x)
     if (chosen[r] < n_experts) perm[atomicAdd(&cursor[chosen[r]], 1)] = r;
+}
+
+__global__ void __launch_bounds__(1024)
+moe_sort_kernel(const int *__restrict__ chosen, int n_rows, int n_experts, int tile_rows, int *__restrict__ offsets,
+                int *__restrict__ perm, int *__restrict__ tiles) {
+  extern __shared__ int sh[];                  // counts [E], cursor [E]
+  grid_dependents_launch();
+  grid_dependency_wait();
+  sort_rows(chosen, n_rows, n_experts, tile_rows, offsets, perm, tiles, sh, sh + n_experts);
 }
 
 LLM_EXPORT int llm_moe_sort(const int *chosen, int n_rows, int n_experts, int tile_rows, int *offsets, int *perm, int *tiles,
@@ -673,6 +705,62 @@ LLM_EXPORT int llm_moe_gather_identity(const void *x, long long ldx, const int *
   LLM_CHECK_LAUNCH("moe_gather");
   return LLM_OK;
 }
+// ---------------------------------------------------------------- choice, sorting and gathering of few rows in one launch
+// A step of few tokens (at most MOE_PLAN_ROWS rows): one CTA routes the tokens, a warp each, sorts the rows, brings the tokens' rows
+// into sorted order and writes the identity experts' results: what would be three launches of next to no work each.
+constexpr int MOE_PLAN_ROWS = 64, MOE_PLAN_WARPS = 16;
+__global__ void __launch_bounds__(MOE_PLAN_WARPS * 32)
+moe_plan_kernel(const float *__restrict__ logits, long long ld, int n_tokens, RouteRule R, int n_experts, int tile_rows,
+                const uint4 *__restrict__ x, long long ldx16, int width16, int *chosen, float *weight, int *offsets, int *perm, int *tiles,
+                uint4 *__restrict__ xs, float *__restrict__ out) {
+  extern __shared__ float plan_sh[];             // per warp: c [choices], group scores; then counts [E], cursor [E]
+  const int per = R.n_experts + R.n_groups, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, top = R.top, n_rows = n_tokens * top;
+  int *counts = (int *)(plan_sh + MOE_PLAN_WARPS * per);
+  grid_dependency_wait();
+  for (int t = warp; t < n_tokens; t += MOE_PLAN_WARPS) {
+    float *c = plan_sh + (size_t)warp * per;
+    route_token(logits + (size_t)t * ld, R, c, c + R.n_experts, lane, chosen + (size_t)t * top, weight + (size_t)t * top);
+    __syncwarp();
+  }
+  __syncthreads();
+  sort_rows(chosen, n_rows, n_experts, tile_rows, offsets, perm, tiles, counts, counts + n_experts);
+  __syncthreads();
+  const int placed = offsets[n_experts];
+  for (int idx = threadIdx.x; idx < n_rows * width16; idx += blockDim.x) {
+    const int r = idx / width16, c = idx - r * width16;
+    if (r < placed) xs[idx] = x[(size_t)(perm[r] / top) * ldx16 + c];
+    if (chosen[r] >= n_experts) {
+      const int t = r / top;
+      identity_row((const __nv_bfloat16 *)(x + (size_t)t * ldx16), weight[r], out + ((size_t)(r - t * top) * n_tokens + t) * width16 * 8, c * 8,
+                   width16 * 8);
+    }
+  }
+}
+
+LLM_EXPORT int llm_moe_plan_rows() { return MOE_PLAN_ROWS; }
+// As moe_route_grouped (n_choices: experts and identity experts), moe_sort and moe_gather_identity one behind the other.
+LLM_EXPORT int llm_moe_plan(const float *logits, long long ld, int n_tokens, int n_choices, int n_experts, int top, int score_kind,
+                            const float *correction, int n_groups, int keep, int group_top, int renormalize, float norm_eps, float route_scale,
+                            int tile_rows, const void *x, long long ldx, int width, int *chosen, float *weight, int *offsets, int *perm,
+                            int *tiles, void *xs, float *out, cudaStream_t stream) {
+  if (n_tokens == 0) return LLM_OK;
+  LLM_REQUIRE(n_tokens > 0 && n_experts > 0 && n_choices >= n_experts && top > 0 && top <= n_choices && n_choices <= 512 && tile_rows > 0 &&
+                  n_tokens * top <= MOE_PLAN_ROWS,
+              "moe_plan: %d tokens, %d of %d choices", n_tokens, top, n_choices);
+  LLM_REQUIRE(score_kind == 0 || score_kind == 1, "moe_plan: unknown score %d", score_kind);
+  LLM_REQUIRE(n_groups >= 1 && n_choices % n_groups == 0 && keep >= 1 && keep <= n_groups && group_top >= 1 &&
+                  (n_groups == 1 || (long long)keep * (n_choices / n_groups) >= top),
+              "moe_plan: %d choices in %d groups of which %d are kept", n_choices, n_groups, keep);
+  LLM_REQUIRE(width % 8 == 0 && ldx % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)xs % 16 == 0, "moe_plan: rows of bfloat16 in multiples of 8, 16-byte aligned");
+  const RouteRule rule{n_choices, top, score_kind, correction, n_groups, keep, group_top, renormalize, norm_eps, route_scale};
+  const size_t smem = ((size_t)MOE_PLAN_WARPS * (n_choices + n_groups) + 2 * n_experts) * sizeof(float);
+  LLM_CHECK_CUDA(llm_allow_smem(moe_plan_kernel, smem), "moe_plan attribute");
+  llm_launch(moe_plan_kernel, dim3(1), dim3(MOE_PLAN_WARPS * 32), smem, stream, logits, ld, n_tokens, rule, n_experts, tile_rows,
+             (const uint4 *)x, ldx / 8, width / 8, chosen, weight, offsets, perm, tiles, (uint4 *)xs, out);
+  LLM_CHECK_LAUNCH("moe_plan");
+  return LLM_OK;
+}
+
 LLM_EXPORT int llm_moe_gather(const void *x, long long ldx, const int *perm, int n_rows, int top, int width, void *xs,
                               cudaStream_t stream) {
   return llm_moe_gather_identity(x, ldx, perm, n_rows, top, width, xs, nullptr, nullptr, nullptr, 0, nullptr, stream);

@@ -300,6 +300,7 @@ class PartHandle:
                 shape = (a["parts"], a["rows"], a["cols"]) if a["parts"] > 1 else (a["rows"], a["cols"])
                 strides = (a["part_stride"], a["ld"], 1) if a["parts"] > 1 else (a["ld"], 1)
                 views[key] = DeviceTensor(a["ptr"], a["dtype"], shape, strides)
+                views[key + "_norms"] = {k: a[k] for k in ("post", "post_eps", "first_parts", "pair_w", "pair_eps", "pair_scale") if k in a}
                 if a.get("col_bias"):          # 32-bit, a value per column: whoever adds the result adds it once
                     views[key + "_bias"] = DeviceTensor(a["col_bias"], "float32", (a["cols"],))
             else:

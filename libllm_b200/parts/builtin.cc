@@ -456,7 +456,7 @@ class Attention : public Mixer {
     const bool tiled = env_.page_size == 64 && d_ % 16 == 0 && d_ >= 16 && d_ <= 128 && plain_;
     if (f.prefill_attention_tc && env_.page_size == 64 && (d_ == 64 || d_ == 128 || padded_)) fams.push_back("attention_prefill_tc");
     else if (f.prefill_attention && tiled) fams.push_back("attention_prefill");
-    if (may_fuse() && env_.page_size == 64 && group <= 16 && d_ <= 128 && dv_ <= 128)
+    if (may_fuse() && env_.page_size == 64 && group <= 16 && d_ <= 128 && dv_ <= 256)
       fams.push_back("attention_decode_tc");
     else if (plain_ && f.decode_attention && (d_ == 16 || d_ == 32 || d_ == 64 || d_ == 128) &&
              (group == 1 || group == 2 || group == 3 || group == 4 || group == 8))

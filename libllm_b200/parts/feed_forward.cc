@@ -235,26 +235,34 @@ class RoutedFeedForward : public FeedForward {
     const int n_rows = (int)T * top_;
     int *chosen = ctx.arena->alloc_n<int>((size_t)n_rows);
     float *weight = ctx.arena->alloc_n<float>((size_t)n_rows);
-    if (grouped_route_)
-      kernels::moe_route_grouped(z, choices_, top_, score_, correction_.empty() ? nullptr : w_correction_.buf.as<float>(), groups_, keep_,
-                                 group_top_, renormalize_, norm_eps_, route_scale_, chosen, weight, ctx.stream);
-    else
-      kernels::moe_route(z, choices_, top_, score_, renormalize_, chosen, weight, ctx.stream);
     const bool in_place = given > 0 && s_own && s.data == (void *)after;
     if (s_own && !in_place && s.parts > given) out = ctx.arena->act(DType::F32, T, hidden_, top_ + s.parts);
     out.parts = top_ + (s_own ? s.parts : 0);
     const bool aligned = x.dtype == DType::BF16 && x.ld % 8 == 0 && (uintptr_t)x.data % 16 == 0;
-    if (aligned && fast_switches().moe_tc && kernels::available("moe_tc") && kernels::moe_tc_supported((int)hidden_, (int)inter_)) {
+    const bool tc = aligned && fast_switches().moe_tc && kernels::available("moe_tc") && kernels::moe_tc_supported((int)hidden_, (int)inter_);
+    const kernels::RouteRule rule{choices_, top_, score_, correction_.empty() ? nullptr : w_correction_.buf.as<float>(), groups_, keep_, group_top_,
+                                  renormalize_, norm_eps_, route_scale_};
+    const bool planned = tc && grouped_route_ && n_rows <= kernels::moe_plan_rows() && choices_ <= 512;
+    if (planned) {
+      // with the sorting and the gathering, below
+    } else if (grouped_route_) {
+      kernels::moe_route_grouped(z, choices_, top_, score_, rule.correction, groups_, keep_, group_top_, renormalize_, norm_eps_, route_scale_, chosen,
+                                 weight, ctx.stream);
+    } else {
+      kernels::moe_route(z, choices_, top_, score_, renormalize_, chosen, weight, ctx.stream);
+    }
+    if (tc) {
       const int tile = kernels::moe_tc_tile_rows(n_rows);
       int *offsets = ctx.arena->alloc_n<int>((size_t)experts_ + 1);
       int *perm = ctx.arena->alloc_n<int>((size_t)n_rows);
       int *tiles = ctx.arena->alloc_n<int>(1 + 2 * ((size_t)std::min(experts_, n_rows) + (size_t)(n_rows / tile)));
       void *xs = ctx.arena->alloc((size_t)n_rows * (size_t)hidden_ * 2);
       void *mid = ctx.arena->alloc((size_t)n_rows * (size_t)inter_ * 2);
-      kernels::moe_sort(chosen, n_rows, experts_, tile, offsets, perm, tiles, ctx.stream);
+      if (planned) kernels::moe_plan(z, rule, experts_, tile, x, chosen, weight, offsets, perm, tiles, xs, (float *)out.data, ctx.stream);
+      else kernels::moe_sort(chosen, n_rows, experts_, tile, offsets, perm, tiles, ctx.stream);
       kernels::moe_tc(x, w_up_.get(), w_down_.get(), offsets, perm, tiles, weight, experts_, top_, (int)hidden_, (int)inter_, act_,
                       weight_on_output_, xs, mid, (float *)out.data, ctx.tc_status, ctx.stream, !gate_.empty(), glu_,
-                      identity_ > 0 ? chosen : nullptr);
+                      identity_ > 0 ? chosen : nullptr, planned);
     } else if (aligned && kernels::moe_grouped_supported((int)hidden_, (int)inter_)) {
       const int tile = kernels::moe_tile_rows();
       int *offsets = ctx.arena->alloc_n<int>((size_t)experts_ + 1);

@@ -227,30 +227,28 @@ def token_side(x, tokens, c, w, i) -> torch.Tensor:
     return rms_norm((gelu_tanh(x @ w[p + "gate"].T) * e) @ w[p + "proj"].T, w[p + "norm"], eps)
 
 
-def forward(c: dict, w: Dict[str, torch.Tensor], tokens: List[int], after_runs: Optional[list] = None, margins: Optional[list] = None,
-            rounded=None) -> torch.Tensor:
-    """Logits [n, vocab].  `after_runs` receives the stream after every layer, `margins` the routers' margins.  `rounded`: a
-    function laid on what a library in 16 bits would round (the norms' results and the sublayers' results)."""
+def forward(c: dict, w: Dict[str, torch.Tensor], tokens: List[int], after_runs: Optional[list] = None,
+            margins: Optional[list] = None) -> torch.Tensor:
+    """Logits [n, vocab].  `after_runs` receives the stream after every layer, `margins` the routers' margins."""
     w = {k: v.to(F64) for k, v in w.items()}
     eps = c["norm"]["eps"]
-    keep = rounded or (lambda t: t)
     x = token_rows(c, w, tokens)
     kept: Dict[int, tuple] = {}
     for i, L in enumerate(c["layers"]):
         p, m = f"l{i}.", L["mixer"]
-        h = keep(rms_norm(x, w[p + "norm1"], eps))
+        h = rms_norm(x, w[p + "norm1"], eps)
         if L["type"] == "attention":
             y = windowed_attention(h, w, p + "mix.", m, kept, i)
         elif L["type"] == "latent_attention":
             y = latent_attention(h, w, p + "mix.", m, eps)
         else:
             y = two_mixers(h, w, p + "mix.", m, eps)
-        x = x + rms_norm(keep(y), w[p + "norm1b"], eps)
+        x = x + rms_norm(y, w[p + "norm1b"], eps)
         if L.get("mlp") is not None:
-            h = keep(rms_norm(x, w[p + "norm2"], eps))
-            x = x + rms_norm(keep(experts(h, w, p + "mlp.", L["mlp"], margins)), w[p + "norm2b"], eps)
+            h = rms_norm(x, w[p + "norm2"], eps)
+            x = x + rms_norm(experts(h, w, p + "mlp.", L["mlp"], margins), w[p + "norm2b"], eps)
         if c.get("token_side"):
             x = x + token_side(x, tokens, c, w, i)
         if after_runs is not None:
             after_runs.append(x)
-    return keep(rms_norm(x, w["final.norm"], eps)) @ w["head"].T
+    return rms_norm(x, w["final.norm"], eps) @ w["head"].T
