@@ -100,8 +100,8 @@ def test_windowed_attention_with_sinks_and_a_borrower(sizes, dtype):
     none) and queries of its own."""
     H, G, d, dv, rot, window = sizes
     wide = None if window in (20, 9) else (window or 60) + 37 if H % 2 == 0 else 17
-    layers = [S.layer(S.attn(H, G, d, vdim=dv, rot=rot, mask=window, scale=5.0 / math.sqrt(d)), None),
-              S.layer(S.attn(2 * G, G, d, vdim=dv, rot=rot, mask=wide, scale=5.0 / math.sqrt(d), kv_from=0), None)]
+    layers = [S.layer(S.attn(H, d, kv=G, vdim=dv, rot=rot, mask=window, scale=5.0 / math.sqrt(d)), None),
+              S.layer(S.attn(2 * G, d, kv=G, vdim=dv, rot=rot, mask=wide, scale=5.0 / math.sqrt(d), kv_from=0), None)]
     (m, b), w, spec = mixers_of(layers, dtype, 21)
     assert spec[0]["mixer"]["null_scores"] == "l0.mix.sink" and "k" not in spec[1]["mixer"]
     x = inputs(9)
@@ -188,7 +188,7 @@ def test_a_planted_key_is_seen_up_to_the_edge(sizes, kind, dtype):
 def test_a_sink_takes_its_share(sizes, dtype):
     """Sinks far above every score (next to nothing is left), far below (they count for nothing) and beside them, head by head."""
     H, G, d, dv = sizes
-    layers = [S.layer(S.attn(H, G, d, vdim=dv, mask=90, scale=0.5 / math.sqrt(d)), None)]
+    layers = [S.layer(S.attn(H, d, kv=G, vdim=dv, mask=90, scale=0.5 / math.sqrt(d)), None)]
 
     def sharpen(w):
         w["l0.mix.sink"] = torch.tensor([20.0, -60.0, 3.0, 0.0])[:H].clone()
@@ -307,8 +307,8 @@ def test_experts_among_identity_experts(sizes, T, dtype):
     got = summed(m.forward(dict(step=Step([T], [0]).json, x=act(xs)))["out"]).cpu()
     margins = []
     ref = P.experts(x.double(), w, "l0.mlp.", f, margins)
-    sure = margins[0] > (1e-5 if dtype == "float32" else 0.01)           # a closer call is no test of the products
-    assert int(sure.sum()) >= 0.8 * T
+    sure = margins[0] > 1e-5           # a closer call is no test (the input is exact in both types, and so is the router's product)
+    assert int(sure.sum()) >= 0.9 * T
     close(got[sure], ref[sure], dtype, f"experts {sizes}, {T} tokens", roundings=1.0 if dtype == "bfloat16" else 2.0)
 
 
@@ -327,7 +327,7 @@ def test_all_choices_are_identity_or_none_is(identity_alone, dtype):
         assert float((ref - x.double()).abs().max()) < 1e-12              # the weights add up to one
         close(got, ref, "float32", "identity experts alone")             # no product, no rounding
     else:
-        sure = margins[0] > 0.01
+        sure = margins[0] > 1e-5
         close(got[sure], ref[sure], dtype, "experts alone")
 
 
