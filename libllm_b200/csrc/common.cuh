@@ -151,6 +151,20 @@ __device__ __forceinline__ __nv_bfloat16 from_float<__nv_bfloat16>(float v) {
 }
 
 // Four consecutive values as 32-bit floats, from or to either element type.
+// the sum of the `parts` partial results p[0], p[stride], .., in that order, eight on their way at once
+__device__ __forceinline__ float sum_parts(const float *__restrict__ p, int parts, long long stride) {
+  if (parts == 1) return p[0];
+  float sum = 0.f;
+  for (int p0 = 0; p0 < parts; p0 += 8) {
+    float v[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = p0 + i < parts ? p[(p0 + i) * stride] : 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) sum += v[i];
+  }
+  return sum;
+}
+
 __device__ __forceinline__ float4 ld4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
 __device__ __forceinline__ float4 ld4(const __nv_bfloat16 *p) {
   const uint2 raw = *reinterpret_cast<const uint2 *>(p);

@@ -629,10 +629,10 @@ LLM_EXPORT int llm_stream_norm(float *resid, const float *delta, int n_parts, lo
 
 // ---------------------------------------------------------------- a token's own vector behind a gate
 // out[t, c] = gelu_tanh(z[t, c]) * table[ids[row], offset + c] for c < dim, nought up to out's width; row = rows ? rows[t] : t.
-// z 32-bit, table [vocab, table_width] and out in the engine's type.
+// z 32-bit (the sum of z_parts partial products), table [vocab, table_width] and out in the engine's type.
 template <typename T>
 __global__ void __launch_bounds__(256)
-token_gate_kernel(const float *__restrict__ z, long long ldz, const T *__restrict__ table, long long table_width, int offset, int dim,
+token_gate_kernel(const float *__restrict__ z, long long ldz, int z_parts, long long z_stride, const T *__restrict__ table, long long table_width, int offset, int dim,
                   const int *__restrict__ ids, const int *__restrict__ rows, T *__restrict__ out, int ldo, size_t total) {
   grid_dependents_launch();
   grid_dependency_wait();
@@ -641,7 +641,7 @@ token_gate_kernel(const float *__restrict__ z, long long ldz, const T *__restric
     const int c = (int)(idx - t * ldo);
     float y = 0.f;
     if (c < dim) {
-      const float g = z[t * ldz + c];
+      const float g = sum_parts(z + t * ldz + c, z_parts, z_stride);
       const float a = 0.5f * g * (1.f + tanhf(0.79788456080286536f * (g + 0.044715f * g * g * g)));
       y = a * to_float(table[(size_t)ids[rows ? rows[t] : (int)t] * table_width + offset + c]);
     }
@@ -649,7 +649,7 @@ token_gate_kernel(const float *__restrict__ z, long long ldz, const T *__restric
   }
 }
 
-LLM_EXPORT int llm_token_gate(int dtype, const float *z, long long ldz, const void *table, long long table_width, int offset, int dim,
+LLM_EXPORT int llm_token_gate(int dtype, const float *z, long long ldz, int z_parts, long long z_stride, const void *table, long long table_width, int offset, int dim,
                               const int *ids, const int *rows, void *out, int ldo, int n_rows, cudaStream_t stream) {
   if (n_rows == 0) return LLM_OK;
   LLM_REQUIRE(n_rows > 0 && dim > 0 && ldo >= dim && offset >= 0 && offset + (long long)dim <= table_width && ids && table, "token_gate: bad sizes");
@@ -657,10 +657,10 @@ LLM_EXPORT int llm_token_gate(int dtype, const float *z, long long ldz, const vo
   size_t blocks = (total + 255) / 256;
   if (blocks > (size_t)sm_count() * 16) blocks = (size_t)sm_count() * 16;
   if (dtype == LLM_F32)
-    llm_launch(token_gate_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, z, ldz, (const float *)table, table_width, offset, dim,
+    llm_launch(token_gate_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, z, ldz, z_parts, z_stride, (const float *)table, table_width, offset, dim,
                ids, rows, (float *)out, ldo, total);
   else if (dtype == LLM_BF16)
-    llm_launch(token_gate_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(256), 0, stream, z, ldz, (const __nv_bfloat16 *)table, table_width,
+    llm_launch(token_gate_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(256), 0, stream, z, ldz, z_parts, z_stride, (const __nv_bfloat16 *)table, table_width,
                offset, dim, ids, rows, (__nv_bfloat16 *)out, ldo, total);
   else LLM_FAIL("token_gate: unknown dtype %d", dtype);
   LLM_CHECK_LAUNCH("token_gate");

@@ -216,12 +216,12 @@ static void stream_norm(float *resid, const Act *delta, const float *weight, flo
 void stream_cast(float *resid, const Act *delta, void *out, DType out_dtype, int n_rows, int hidden, cudaStream_t s) {
   stream_norm(resid, delta, nullptr, 0.f, out, out_dtype, nullptr, n_rows, nullptr, hidden, s);
 }
-LLM_KERNEL("elementwise", llm_token_gate, int, const float *, long long, const void *, long long, int, int, const int *, const int *, void *, int,
+LLM_KERNEL("elementwise", llm_token_gate, int, const float *, long long, int, long long, const void *, long long, int, int, const int *, const int *, void *, int,
            int, cudaStream_t)
 void token_gate(const Act &z, const void *table, long long table_width, int offset, int dim, const int *ids, const int *rows, const Act &out,
                 cudaStream_t s) {
   if (z.dtype != DType::F32 || out.ld != out.cols) LLM_THROW(InvalidArg, "token_gate: 32-bit logits, a dense result");
-  LLM_CALL("elementwise", llm_token_gate, code(out.dtype), (const float *)z.data, (long long)z.ld, table, table_width, offset, dim, ids, rows,
+  LLM_CALL("elementwise", llm_token_gate, code(out.dtype), (const float *)z.data, (long long)z.ld, z.parts, (long long)z.part_stride, table, table_width, offset, dim, ids, rows,
            out.data, (int)out.cols, (int)out.rows, s);
 }
 void add_rmsnorm(float *resid, const Act *delta, const float *weight, float eps, void *out, DType out_dtype, const int *rows,
@@ -690,7 +690,7 @@ void moe_tc(const Act &x, const void *up, const void *down, const int *offsets, 
   LLM_CALL("moe_tc", llm_moe_tc_glu, xs, up, down, offsets, perm, tiles, weight, (int)x.rows, n_experts, top, width, ff, act,
            weight_on_output ? 1 : 0, gated ? 1 : 0, glu.limit, glu.slope, glu.shift, mid, out, status, s);
 }
-LLM_KERNEL("moe", llm_moe_plan, const float *, long long, int, int, int, int, int, const float *, int, int, int, int, float, float, int,
+LLM_KERNEL("moe", llm_moe_plan, const float *, long long, int, long long, int, int, int, int, int, const float *, int, int, int, int, float, float, int,
            const void *, long long, int, int *, float *, int *, int *, int *, void *, float *, cudaStream_t)
 int moe_plan_rows() {
   static const int n = resolve<int (*)()>("moe", "llm_moe_plan_rows")();
@@ -698,7 +698,7 @@ int moe_plan_rows() {
 }
 void moe_plan(const Act &z, const RouteRule &r, int n_experts, int tile_rows, const Act &x, int *chosen, float *weight, int *offsets, int *perm,
               int *tiles, void *xs, float *out, cudaStream_t s) {
-  LLM_CALL("moe", llm_moe_plan, (const float *)z.data, (long long)z.ld, (int)z.rows, r.choices, n_experts, r.top, r.score, r.correction, r.groups,
+  LLM_CALL("moe", llm_moe_plan, (const float *)z.data, (long long)z.ld, z.parts, (long long)z.part_stride, (int)z.rows, r.choices, n_experts, r.top, r.score, r.correction, r.groups,
            r.keep, r.group_top, r.renormalize ? 1 : 0, r.norm_eps, r.scale, tile_rows, x.data, (long long)x.ld, (int)x.cols, chosen, weight, offsets,
            perm, tiles, xs, out, s);
 }
@@ -888,7 +888,7 @@ LLM_KERNEL("selective_scan", llm_short_conv_silu, int, const float *, long long,
 LLM_KERNEL("selective_scan", llm_selective_scan, int, const void *, long long, const float *, long long, const float *, const float *, long long,
            int, int, const float *, long long, const float *, const float *, float *, void *, long long, const int *, const int *, int, int, int,
            cudaStream_t)
-LLM_KERNEL("selective_scan", llm_selective_step, int, const void *, long long, const float *, long long, int, const void *, int, const float *, int,
+LLM_KERNEL("selective_scan", llm_selective_step, int, const void *, long long, const float *, long long, int, long long, int, const void *, int, const float *, int,
            int, const float *, long long, const float *, const float *, float *, void *, long long, const int *, int, int, int, cudaStream_t)
 LLM_KERNEL("selective_scan", llm_rows_cast, const float *, long long, int, void *, int, int, cudaStream_t)
 int selective_max_state() { return 256; }
@@ -917,7 +917,8 @@ void selective_step(const Act &x, const Act &low, int rank, const Weight &w_dt, 
                     cudaStream_t s) {
   if (low.dtype != DType::F32 || x.dtype != out.dtype || w_dt.dtype != x.dtype)
     LLM_THROW(InvalidArg, "selective_step: 32-bit projections, one type for input, matrix and result");
-  LLM_CALL("selective_scan", llm_selective_step, code(x.dtype), x.data, (long long)x.ld, (const float *)low.data, (long long)low.ld, rank,
+  LLM_CALL("selective_scan", llm_selective_step, code(x.dtype), x.data, (long long)x.ld, (const float *)low.data, (long long)low.ld, low.parts,
+           (long long)low.part_stride, rank,
            w_dt.data(), (int)w_dt.cols, dt_bias, off_b, off_c, z, ldz, a_log, skip, state, out.data, (long long)out.ld, seq_slot, (int)out.rows,
            (int)out.cols, N, s);
 }

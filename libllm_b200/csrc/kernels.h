@@ -63,7 +63,7 @@ void add_layernorm_conv(float *resid, const Act *delta, const float *weight, con
 void gather_rows_add(const float *resid, const Act *delta, const int *rows, int n_rows, float *out, int hidden, cudaStream_t s);
 // The stream with what is pending added (resid moves on; rows null: all of it), in out's type, without a norm.
 void stream_cast(float *resid, const Act *delta, void *out, DType out_dtype, int n_rows, int hidden, cudaStream_t s);
-// out[t, c] = gelu_tanh(z[t, c]) * table[ids[rows ? rows[t] : t], offset + c] for c < dim, nought up to out.cols
+// out[t, c] = gelu_tanh(z[t, c]) (partial products are added) * table[ids[rows ? rows[t] : t], offset + c] for c < dim, nought up to out.cols
 void token_gate(const Act &z, const void *table, long long table_width, int offset, int dim, const int *ids, const int *rows, const Act &out,
                 cudaStream_t s);
 void swiglu(const Act &gu, void *out, DType out_dtype, cudaStream_t s);
@@ -254,7 +254,7 @@ int moe_tile_rows();
 void moe_sort(const int *chosen, int n_rows, int n_experts, int tile_rows, int *offsets, int *perm, int *tiles, cudaStream_t s);
 // x [T, width]; up [E, ff, width], down [E, width, ff] in x's type; out [top, T, width] 32-bit.  `gated`: up is
 // [E, 2 ff, width], an expert's gate and up rows interleaved, and the expert is down(act(gate x) * up x).
-// Few tokens (up to moe_plan_rows() rows): moe_route_grouped, moe_sort and the gathering of moe_tc in one launch.
+// Few tokens (up to moe_plan_rows() rows): the logits' partial products added, moe_route_grouped, moe_sort and the gathering of moe_tc in one launch.
 struct RouteRule {
   int choices = 0, top = 0, score = 0;             // choices: experts and identity experts
   const float *correction = nullptr;
@@ -361,7 +361,7 @@ void selective_scan(const Act &x, const Act &dt_raw, const float *dt_bias, const
                     int N, cudaStream_t s);
 // out (bfloat16, dense) = the first n columns of the 32-bit rows `in`, nought beyond them
 void rows_cast(const Act &in, int n, const Act &out, cudaStream_t s);
-// A step of single tokens: low's rows begin with the dt input of `rank` values; w_dt [inner, w_dt.cols], columns beyond the rank nought
+// A step of single tokens: low's rows (partial products are added) begin with the dt input of `rank` values; w_dt [inner, w_dt.cols], columns beyond the rank nought
 void selective_step(const Act &x, const Act &low, int rank, const Weight &w_dt, const float *dt_bias, int off_b, int off_c, const float *z,
                     long long ldz, const float *a_log, const float *skip, float *state, const Act &out, const int *seq_slot, int N,
                     cudaStream_t s);

@@ -296,6 +296,7 @@ LLM_EXPORT int llm_row_gate(const float *x, long long x_stride, float *out, long
 // one expert.  Which place a row gets within its expert depends on the order the threads arrive
 // in; no result depends on it.  Rows of identity experts (chosen >= n_experts) get no place.
 // By all threads of a block; counts and cursor [E] in shared memory.
+template <bool STABLE = false>
 __device__ __forceinline__ void sort_rows(const int *chosen, int n_rows, int n_experts, int tile_rows, int *__restrict__ offsets,
                                           int *__restrict__ perm, int *__restrict__ tiles, int *counts, int *cursor) {
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) counts[e] = 0;
@@ -336,7 +337,15 @@ __device__ __forceinline__ void sort_rows(const int *chosen, int n_rows, int n_e
   }
   __syncthreads();
   for (int r = threadIdx.x; r < n_rows; r += blockDim.x)
-    if (chosen[r] < n_experts) perm[atomicAdd(&cursor[chosen[r]], 1)] = r;
+    if (chosen[r] < n_experts) {
+      if (STABLE) {
+        int before = 0;
+        for (int q = 0; q < r; ++q) before += chosen[q] == chosen[r];
+        perm[cursor[chosen[r]] + before] = r;
+      } else {
+        perm[atomicAdd(&cursor[chosen[r]], 1)] = r;
+      }
+    }
 }
 
 __global__ void __launch_bounds__(1024)
@@ -706,40 +715,63 @@ LLM_EXPORT int llm_moe_gather_identity(const void *x, long long ldx, const int *
   return LLM_OK;
 }
 // ---------------------------------------------------------------- choice, sorting and gathering of few rows in one launch
-// A step of few tokens (at most MOE_PLAN_ROWS rows): one CTA routes the tokens, a warp each, sorts the rows, brings the tokens' rows
-// into sorted order and writes the identity experts' results: what would be three launches of next to no work each.
-constexpr int MOE_PLAN_ROWS = 64, MOE_PLAN_WARPS = 16;
+// A step of few tokens (at most MOE_PLAN_ROWS rows): every CTA routes the tokens, a warp each, and sorts the rows (an expert's in
+// their order, so that all CTAs have the same), then brings its columns of the tokens' rows into sorted order and writes those of the
+// identity experts' results: what would be three launches of next to no work each.  The logits may come as partial products, which
+// are added here.
+constexpr int MOE_PLAN_ROWS = 64, MOE_PLAN_WARPS = 32;
 __global__ void __launch_bounds__(MOE_PLAN_WARPS * 32)
-moe_plan_kernel(const float *__restrict__ logits, long long ld, int n_tokens, RouteRule R, int n_experts, int tile_rows,
+moe_plan_kernel(const float *__restrict__ logits, long long ld, int z_parts, long long z_stride, int n_tokens, RouteRule R, int n_experts, int tile_rows,
                 const uint4 *__restrict__ x, long long ldx16, int width16, int *chosen, float *weight, int *offsets, int *perm, int *tiles,
                 uint4 *__restrict__ xs, float *__restrict__ out) {
-  extern __shared__ float plan_sh[];             // per warp: c [choices], group scores; then counts [E], cursor [E]
-  const int per = R.n_experts + R.n_groups, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, top = R.top, n_rows = n_tokens * top;
+  extern __shared__ float plan_sh[];             // per warp: z and c [choices], group scores; then counts [E], cursor [E], correction
+  __shared__ int chosen_s[MOE_PLAN_ROWS], perm_s[MOE_PLAN_ROWS];
+  __shared__ float weight_s[MOE_PLAN_ROWS];
+  const int per = 2 * R.n_experts + R.n_groups, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, top = R.top, n_rows = n_tokens * top;
   int *counts = (int *)(plan_sh + MOE_PLAN_WARPS * per);
+  if (R.correction) {
+    float *corr = (float *)(counts + 2 * n_experts);
+    for (int e = threadIdx.x; e < R.n_experts; e += blockDim.x) corr[e] = R.correction[e];
+    R.correction = corr;
+  }
+  __syncthreads();
   grid_dependency_wait();
   for (int t = warp; t < n_tokens; t += MOE_PLAN_WARPS) {
-    float *c = plan_sh + (size_t)warp * per;
-    route_token(logits + (size_t)t * ld, R, c, c + R.n_experts, lane, chosen + (size_t)t * top, weight + (size_t)t * top);
+    float *z = plan_sh + (size_t)warp * per, *c = z + R.n_experts;
+    for (int e = lane; e < R.n_experts; e += 32) z[e] = sum_parts(logits + (size_t)t * ld + e, z_parts, z_stride);
+    __syncwarp();
+    route_token(z, R, c, c + R.n_experts, lane, chosen_s + t * top, weight_s + t * top);
     __syncwarp();
   }
   __syncthreads();
-  sort_rows(chosen, n_rows, n_experts, tile_rows, offsets, perm, tiles, counts, counts + n_experts);
+  const bool first = blockIdx.x == 0;
+  if (first)
+    for (int r = threadIdx.x; r < n_rows; r += blockDim.x) {
+      chosen[r] = chosen_s[r];
+      weight[r] = weight_s[r];
+    }
+  // offsets and tiles: every CTA writes the same numbers
+  if (threadIdx.x < MOE_PLAN_ROWS) perm_s[threadIdx.x] = -1;
+  sort_rows<true>(chosen_s, n_rows, n_experts, tile_rows, offsets, perm_s, tiles, counts, counts + n_experts);
   __syncthreads();
-  const int placed = offsets[n_experts];
-  for (int idx = threadIdx.x; idx < n_rows * width16; idx += blockDim.x) {
-    const int r = idx / width16, c = idx - r * width16;
-    if (r < placed) xs[idx] = x[(size_t)(perm[r] / top) * ldx16 + c];
-    if (chosen[r] >= n_experts) {
+  // a warp a row; this CTA's columns
+  const int c = blockIdx.x * 32 + lane;
+  for (int r = warp; r < n_rows; r += MOE_PLAN_WARPS) {
+    const int from = perm_s[r];                  // < 0: beyond the placed rows
+    if (first && lane == 0 && from >= 0) perm[r] = from;
+    if (from >= 0 && c < width16) xs[(size_t)r * width16 + c] = x[(size_t)(from / top) * ldx16 + c];
+    if (chosen_s[r] >= n_experts) {
       const int t = r / top;
-      identity_row((const __nv_bfloat16 *)(x + (size_t)t * ldx16), weight[r], out + ((size_t)(r - t * top) * n_tokens + t) * width16 * 8, c * 8,
-                   width16 * 8);
+      if (c < width16)
+        identity_row((const __nv_bfloat16 *)(x + (size_t)t * ldx16), weight_s[r], out + ((size_t)(r - t * top) * n_tokens + t) * width16 * 8, c * 8,
+                     width16 * 8);
     }
   }
 }
 
 LLM_EXPORT int llm_moe_plan_rows() { return MOE_PLAN_ROWS; }
 // As moe_route_grouped (n_choices: experts and identity experts), moe_sort and moe_gather_identity one behind the other.
-LLM_EXPORT int llm_moe_plan(const float *logits, long long ld, int n_tokens, int n_choices, int n_experts, int top, int score_kind,
+LLM_EXPORT int llm_moe_plan(const float *logits, long long ld, int z_parts, long long z_stride, int n_tokens, int n_choices, int n_experts, int top, int score_kind,
                             const float *correction, int n_groups, int keep, int group_top, int renormalize, float norm_eps, float route_scale,
                             int tile_rows, const void *x, long long ldx, int width, int *chosen, float *weight, int *offsets, int *perm,
                             int *tiles, void *xs, float *out, cudaStream_t stream) {
@@ -753,9 +785,9 @@ LLM_EXPORT int llm_moe_plan(const float *logits, long long ld, int n_tokens, int
               "moe_plan: %d choices in %d groups of which %d are kept", n_choices, n_groups, keep);
   LLM_REQUIRE(width % 8 == 0 && ldx % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)xs % 16 == 0, "moe_plan: rows of bfloat16 in multiples of 8, 16-byte aligned");
   const RouteRule rule{n_choices, top, score_kind, correction, n_groups, keep, group_top, renormalize, norm_eps, route_scale};
-  const size_t smem = ((size_t)MOE_PLAN_WARPS * (n_choices + n_groups) + 2 * n_experts) * sizeof(float);
+  const size_t smem = ((size_t)MOE_PLAN_WARPS * (2 * n_choices + n_groups) + 2 * n_experts + n_choices) * sizeof(float);
   LLM_CHECK_CUDA(llm_allow_smem(moe_plan_kernel, smem), "moe_plan attribute");
-  llm_launch(moe_plan_kernel, dim3(1), dim3(MOE_PLAN_WARPS * 32), smem, stream, logits, ld, n_tokens, rule, n_experts, tile_rows,
+  llm_launch(moe_plan_kernel, dim3((width / 8 + 31) / 32), dim3(MOE_PLAN_WARPS * 32), smem, stream, logits, ld, z_parts, z_stride, n_tokens, rule, n_experts, tile_rows,
              (const uint4 *)x, ldx / 8, width / 8, chosen, weight, offsets, perm, tiles, (uint4 *)xs, out);
   LLM_CHECK_LAUNCH("moe_plan");
   return LLM_OK;

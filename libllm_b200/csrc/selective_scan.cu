@@ -11,10 +11,12 @@
 //
 //  * short_conv_silu: the convolution, a thread four channels and a run of rows, the last taps values in registers.
 //  * selective_scan: a step of any tokens.  A CTA takes 128 / L channels of one sequence, L lanes to a channel, each with NS of its
-//    N states in registers, and walks the tokens in groups of 16 (8 with many states).  While a group is worked on, the next one's values are on
+//    N states in registers (few: what bounds it is how many warps there are to hide one another's latency), and walks the tokens in
+//    groups of 32 (8 with many states).  While a group is worked on, the next one's values are on
 //    their way into registers; behind it they go, with everything that needs no state already computed (softplus, dt x, D x,
 //    silu z), into the other of two buffers in shared memory: one barrier a group.  The only dependence between tokens is the
-//    state's fused multiply-add; the sums over n are joined by shuffles off that chain.
+//    state's fused multiply-add; sixteen tokens' sums over n are joined together, off that chain, by shuffles that leave each lane
+//    one token's.  Tokens beyond the sequence's last have dt = 0 and leave the state as it is: no branch in the loop.
 //  * selective_step: a step of single tokens, with the product that makes dt (a row of dt_rank values per channel) in the same
 //    launch.
 // A channel's arithmetic is the same function wherever it is computed and depends on its own sequence alone.
@@ -29,9 +31,26 @@ namespace {
 
 constexpr float LOG2E = 1.4426950408889634f;
 
-__device__ __forceinline__ float silu_of(float v) { return v / (1.f + expf(-v)); }
-// log(1 + e^v) without overflow: max(v, 0) + log1p(e^-|v|)
-__device__ __forceinline__ float softplus_of(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+// FAST: for results that are rounded to 16 bits; a few 1e-7 of the value
+template <bool FAST = false>
+__device__ __forceinline__ float silu_of(float v) {
+  return FAST ? __fdividef(v, 1.f + __expf(-v)) : v / (1.f + expf(-v));
+}
+// log(1 + e^v) without overflow: max(v, 0) + log1p(e^-|v|); FAST: log1p(e) = 2 artanh(e / (2 + e)) by its Taylor series, whose
+// argument is a third at most
+template <bool FAST = false>
+__device__ __forceinline__ float softplus_of(float v) {
+  if (!FAST) return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v)));
+  const float e = __expf(-fabsf(v)), s = __fdividef(e, 2.f + e), s2 = s * s;
+  float p = 1.f / 13.f;
+  p = fmaf(p, s2, 1.f / 11.f);
+  p = fmaf(p, s2, 1.f / 9.f);
+  p = fmaf(p, s2, 1.f / 7.f);
+  p = fmaf(p, s2, 1.f / 5.f);
+  p = fmaf(p, s2, 1.f / 3.f);
+  p = fmaf(p, s2, 1.f);
+  return fmaf(2.f * s, p, fmaxf(v, 0.f));
+}
 
 // ---------------------------------------------------------------- the short convolution
 // u [tokens, ld] 32-bit, weight [taps][channels] 32-bit, bias [channels]; out [tokens, channels].  Rows whose window lies inside
@@ -107,12 +126,27 @@ short_conv_silu_kernel(const float *__restrict__ u, long long ld, const float *_
 #pragma unroll
       for (int j = 0; j < TAPS; ++j)
         if (j < taps) y[e] = fmaf(w[j][e], win[j][e], y[e]);
-      y[e] = silu_of(y[e] + bs[e]);
+      y[e] = silu_of<sizeof(T) == 2>(y[e] + bs[e]);
     }
     sc_store<T, V>(out + (size_t)row * ldo + c0, y);
   };
   if ((int)blockIdx.x < n_chunks) {
     const int r0 = blockIdx.x * SC_ROWS, r1 = min(n_tokens, r0 + SC_ROWS);
+    if (TAPS <= 4 && mine == (1u << SC_ROWS) - 1u) {       // all of them: every row's loads on their way at once
+      float in[SC_ROWS + TAPS - 1][V];
+#pragma unroll
+      for (int i = 0; i < SC_ROWS + TAPS - 1; ++i)
+        if (i < SC_ROWS + keep) sc_load<V>(u + (size_t)(r0 - keep + i) * ld + c0, in[i]);
+#pragma unroll
+      for (int i = 0; i < SC_ROWS + TAPS - 1; ++i)
+        if (i < SC_ROWS + keep) {
+#pragma unroll
+          for (int e = 0; e < V; ++e) x[e] = in[i][e];
+          shift();
+          if (i >= keep) place(r0 - keep + i);
+        }
+      return;
+    }
     for (int row = r0; row < r1; ++row) {
       if (!((mine >> (row - r0)) & 1u)) continue;
       if (row == r0 || !((mine >> (row - r0 - 1)) & 1u))
@@ -140,24 +174,19 @@ short_conv_silu_kernel(const float *__restrict__ u, long long ld, const float *_
 }
 
 // ---------------------------------------------------------------- the recurrence over a step's tokens
-constexpr int SS_THREADS = 128;
+constexpr int SCAN_THREADS = 128, SCAN_GROUP = 32;
+constexpr int SS_THREADS = 128;                          // of a step of single tokens
 
-// One token of one lane's states: a = exp2(dt A log2 e), S <- a S + dx B, sum += S C.  al2: A log2 e.
-template <int NS>
-__device__ __forceinline__ float scan_token(float (&S)[NS], const float (&al2)[NS], float dt, float dx, const float *__restrict__ B,
-                                            const float *__restrict__ C) {
-  float acc = 0.f;
-#pragma unroll
-  for (int i = 0; i < NS; i += 4) {
-    const float4 b = ld4(B + i), c = ld4(C + i);
-    const float bb[4] = {b.x, b.y, b.z, b.w}, cc[4] = {c.x, c.y, c.z, c.w};
-#pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      S[i + k] = fmaf(exp2f(dt * al2[i + k]), S[i + k], dx * bb[k]);
-      acc = fmaf(S[i + k], cc[k], acc);
-    }
-  }
-  return acc;
+// 2^x of a number that is never above nought, in one instruction
+__device__ __forceinline__ float decay_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// One token of one state: a = exp2(dt A log2 e), S <- a S + dx B, y += S C.  al2: A log2 e.
+__device__ __forceinline__ void scan_state(float &S, float al2, float dt, float dx, float B, float C, float &y) {
+  S = fmaf(decay_exp2(dt * al2), S, dx * B);
+  y = fmaf(S, C, y);
 }
 template <int L>
 __device__ __forceinline__ float lanes_sum(float v) {
@@ -166,136 +195,184 @@ __device__ __forceinline__ float lanes_sum(float v) {
   return v;
 }
 
-// a lane's states' decays (al2) and, if wanted, the states themselves; states beyond N are nought and stay so
-template <int NS>
-__device__ __forceinline__ void lane_states(const float *__restrict__ a_log, const float *__restrict__ st, int c, int n0, int N, bool in,
+// NT values' sums over L lanes at once, by halving: lane bit k picks the half of what is left after k exchanges, so that a lane ends
+// with the sums of NT / L values (of one, where L > NT) from first_of<L, NT>(lane) on, in v[0], v[1], ..
+template <int L, int NT>
+__device__ __forceinline__ void lanes_sums(float (&v)[NT], int lane) {
+#pragma unroll
+  for (int o = 1, half = NT / 2; o < L; o <<= 1, half >>= 1) {
+    if (half > 0) {
+      const bool upper = lane & o;
+#pragma unroll
+      for (int i = 0; i < NT / 2; ++i)
+        if (i < half) {
+          const float other = __shfl_xor_sync(0xffffffffu, upper ? v[i] : v[i + half], o);
+          v[i] = (upper ? v[i + half] : v[i]) + other;
+        }
+    } else {
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+    }
+  }
+}
+template <int L, int NT>
+__device__ __forceinline__ int first_of(int lane) {
+  int at = 0;
+#pragma unroll
+  for (int o = 1, half = NT / 2; o < L && half > 0; o <<= 1, half >>= 1)
+    if (lane & o) at += half;
+  return at;
+}
+
+// the decays (al2) and values of a lane's states, lane + i L; states beyond N are nought and stay so
+template <int L, int NS>
+__device__ __forceinline__ void lane_states(const float *__restrict__ a_log, const float *__restrict__ st, int c, int lane, int N, bool in,
                                             float (&al2)[NS], float (&S)[NS]) {
 #pragma unroll
   for (int i = 0; i < NS; ++i) {
-    const bool has = in && n0 + i < N;
-    al2[i] = has ? -expf(a_log[(size_t)c * N + n0 + i]) * LOG2E : 0.f;
-    S[i] = has ? st[(size_t)c * N + n0 + i] : 0.f;
+    const bool has = in && lane + i * L < N;
+    al2[i] = has ? fmaxf(-expf(a_log[(size_t)c * N + lane + i * L]) * LOG2E, -3e38f) : 0.f;   // finite: 0 times it is 0
+    S[i] = has ? st[(size_t)c * N + lane + i * L] : 0.f;
   }
 }
 
 template <typename T, int L, int NS>
-__global__ void __launch_bounds__(SS_THREADS)
+__global__ void __launch_bounds__(SCAN_THREADS)
 selective_scan_kernel(const T *__restrict__ x, long long ldx, const float *__restrict__ dt_raw, long long ld_dt,
                       const float *__restrict__ dt_bias, const float *__restrict__ bc, long long ld_bc, int off_b, int off_c,
                       const float *__restrict__ z, long long ldz, const float *__restrict__ a_log, const float *__restrict__ skip,
                       float *__restrict__ state, T *__restrict__ out, long long ldo, const int *__restrict__ seq_start,
                       const int *__restrict__ seq_slot, int inner, int N) {
-  constexpr int CH = SS_THREADS / L, NP = L * NS;        // channels of the CTA, padded states
-  constexpr int SS_TG = NP <= 128 ? 16 : 8;              // tokens of a group
-  constexpr int PER = SS_TG * CH / SS_THREADS;           // (token, channel) pairs a thread brings in (none: some threads bring one)
-  constexpr int PAIRS = PER > 0 ? PER : 1;
-  constexpr int NB = (2 * SS_TG * NP + SS_THREADS - 1) / SS_THREADS;
-  __shared__ __align__(16) float4 tok[2][SS_TG][CH];     // dt, dt x, D x, silu(z)
-  __shared__ __align__(16) float bcs[2][SS_TG][2][NP];
-  __shared__ float ys[2][SS_TG][CH];
+  constexpr int CH = SCAN_THREADS / L, NP = L * NS;      // channels of the CTA, padded states
+  constexpr int TG = NP <= 64 ? SCAN_GROUP : 8;          // tokens of a group
+  constexpr int PAIRS = (TG * CH + SCAN_THREADS - 1) / SCAN_THREADS, ROWS = SCAN_THREADS / CH;   // (token, channel) pairs a thread brings in
+  constexpr int NB = (2 * TG * NP + SCAN_THREADS - 1) / SCAN_THREADS;
+  constexpr int NT = TG < 16 ? TG : 16;                  // tokens whose sums over the lanes are made together
+  __shared__ __align__(16) float dts[2][CH][TG + 4], dxs[2][CH][TG + 4];   // dt, dt x
+  __shared__ __align__(16) float bcs[2][2][TG / 4][NP][4];                 // B, C: four tokens' beside one another
+  __shared__ float ys[2][TG][CH];
   grid_dependents_launch();
-  const int tid = threadIdx.x, lane = tid % L, ch = tid / L, c = blockIdx.x * CH + ch, n0 = lane * NS;
+  const int tid = threadIdx.x, lane = tid % L, ch = tid / L, c = blockIdx.x * CH + ch;
   const int b = blockIdx.y;
-  // the pairs this thread brings in: channel lc of tokens lt + i * (SS_THREADS / CH)
-  const int lc = tid % CH, lt = tid / CH, gc = blockIdx.x * CH + lc;
-  const bool l_in = gc < inner;
-  const float bias = l_in ? dt_bias[gc] : 0.f, dsk = l_in ? skip[gc] : 0.f;
+  const int lc = tid % CH, lt = tid / CH, gc = blockIdx.x * CH + lc;       // the pairs this thread brings in and stores: tokens lt + i ROWS
+  const bool mine = gc < inner;
+  const float bias = mine ? dt_bias[gc] : 0.f, dsk = mine ? skip[gc] : 0.f;
   grid_dependency_wait();
   const int start = seq_start[b], n = seq_start[b + 1] - start;
   if (n <= 0) return;
   float *st = state + (size_t)seq_slot[b] * inner * N;
   float al2[NS], S[NS];
-  lane_states<NS>(a_log, st, c, n0, N, c < inner, al2, S);
+  lane_states<L, NS>(a_log, st, c, lane, N, c < inner, al2, S);
 
-  float rx[PAIRS], rd[PAIRS], rz[PAIRS], rb[NB];
+  float rx[PAIRS], rd[PAIRS], rz[PAIRS], rb[NB], add[PAIRS], gate[PAIRS];  // on their way; of the group in the works: D x and silu(z)
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int i = 0; i < PAIRS; ++i) {
-      const int t = t0 + lt + i * (SS_THREADS / CH);
-      const bool in = l_in && t < n && lt + i * (SS_THREADS / CH) < SS_TG;
-      const size_t row = (size_t)(start + (in ? t : 0));
+      const int t = lt + i * ROWS;
+      const bool in = mine && t < TG && t0 + t < n;
+      const size_t row = (size_t)(start + (in ? t0 + t : 0));
       rx[i] = in ? to_float(x[row * ldx + gc]) : 0.f;
       rd[i] = in ? dt_raw[row * ld_dt + gc] : 0.f;
       rz[i] = in ? z[row * ldz + gc] : 0.f;
     }
 #pragma unroll
     for (int i = 0; i < NB; ++i) {
-      const int k = tid + i * SS_THREADS, t = k / (2 * NP), m = k - t * 2 * NP, which = m / NP, s = m - which * NP;
-      const bool in = t < SS_TG && t0 + t < n && s < N;
-      rb[i] = in ? bc[(size_t)(start + t0 + t) * ld_bc + (which ? off_c : off_b) + s] : 0.f;
+      const int k = tid + i * SCAN_THREADS, t = k / (2 * NP), m = k - t * 2 * NP, which = m / NP, s = m - which * NP;
+      const bool has = t < TG && t0 + t < n && s < N;
+      rb[i] = has ? bc[(size_t)(start + t0 + t) * ld_bc + (which ? off_c : off_b) + s] : 0.f;
     }
   };
-  auto leave = [&](int buf) {
+  auto leave = [&](int buf, int t0) {
 #pragma unroll
     for (int i = 0; i < PAIRS; ++i) {
-      const int t = lt + i * (SS_THREADS / CH);
-      if (t >= SS_TG) continue;
-      const float dt = softplus_of(rd[i] + bias);
-      tok[buf][t][lc] = make_float4(dt, dt * rx[i], dsk * rx[i], silu_of(rz[i]));
+      const int t = lt + i * ROWS;
+      if (t >= TG) continue;
+      const float dt = t0 + t < n ? softplus_of<sizeof(T) == 2>(rd[i] + bias) : 0.f;
+      dts[buf][lc][t] = dt;
+      dxs[buf][lc][t] = dt * rx[i];
     }
 #pragma unroll
     for (int i = 0; i < NB; ++i) {
-      const int k = tid + i * SS_THREADS;
-      if (k < 2 * SS_TG * NP) (&bcs[buf][0][0][0])[k] = rb[i];
+      const int k = tid + i * SCAN_THREADS, t = k / (2 * NP), m = k - t * 2 * NP, which = m / NP, s = m - which * NP;
+      if (t < TG) bcs[buf][which][t / 4][s][t % 4] = rb[i];
     }
   };
-  auto store = [&](int t0, int buf) {                    // a finished group's rows
+  auto keep = [&]() {
 #pragma unroll
     for (int i = 0; i < PAIRS; ++i) {
-      const int t = lt + i * (SS_THREADS / CH);
-      if (t < SS_TG && t0 + t < n && l_in) out[(size_t)(start + t0 + t) * ldo + gc] = from_float<T>(ys[buf][t][lc]);
+      add[i] = dsk * rx[i];
+      gate[i] = silu_of<sizeof(T) == 2>(rz[i]);
     }
   };
   fetch(0);
-  leave(0);
+  leave(0, 0);
+  keep();
   __syncthreads();
-  for (int t0 = 0, g = 0; t0 < n; t0 += SS_TG, ++g) {
+  for (int t0 = 0, g = 0; t0 < n; t0 += TG, ++g) {
     const int buf = g & 1;
-    const bool more = t0 + SS_TG < n;
-    if (more) fetch(t0 + SS_TG);
-    const int nt = min(SS_TG, n - t0);
-    auto one = [&](int t) {
-      const float4 v = tok[buf][t][ch];
-      const float y = lanes_sum<L>(scan_token<NS>(S, al2, v.x, v.y, &bcs[buf][t][0][n0], &bcs[buf][t][1][n0]));
-      if (lane == 0) ys[buf][t][ch] = (y + v.z) * v.w;
-    };
-    if (nt == SS_TG) {
-#pragma unroll 4
-      for (int t = 0; t < SS_TG; ++t) one(t);
-    } else {
-      for (int t = 0; t < nt; ++t) one(t);
+    const bool more = t0 + TG < n;
+    if (more) fetch(t0 + TG);
+#pragma unroll
+    for (int q0 = 0; q0 < TG / 4; q0 += NT / 4) {
+      float y[NT];
+#pragma unroll
+      for (int q = 0; q < NT / 4; ++q) {
+        const float4 dt = ld4(&dts[buf][ch][4 * (q0 + q)]), dx = ld4(&dxs[buf][ch][4 * (q0 + q)]);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) y[4 * q + k] = 0.f;
+#pragma unroll
+        for (int i = 0; i < NS; ++i) {
+          const float4 B = ld4(bcs[buf][0][q0 + q][lane + i * L]), C = ld4(bcs[buf][1][q0 + q][lane + i * L]);
+          scan_state(S[i], al2[i], dt.x, dx.x, B.x, C.x, y[4 * q]);
+          scan_state(S[i], al2[i], dt.y, dx.y, B.y, C.y, y[4 * q + 1]);
+          scan_state(S[i], al2[i], dt.z, dx.z, B.z, C.z, y[4 * q + 2]);
+          scan_state(S[i], al2[i], dt.w, dx.w, B.w, C.w, y[4 * q + 3]);
+        }
+      }
+      lanes_sums<L, NT>(y, lane);
+#pragma unroll
+      for (int i = 0; i < (NT > L ? NT / L : 1); ++i)
+        if (lane < NT) ys[buf][4 * q0 + first_of<L, NT>(lane) + i][ch] = y[i];
     }
-    if (more) leave(buf ^ 1);
+    if (more) leave(buf ^ 1, t0 + TG);
     __syncthreads();
-    store(t0, buf);
+#pragma unroll
+    for (int i = 0; i < PAIRS; ++i) {
+      const int t = lt + i * ROWS;
+      if (mine && t < TG && t0 + t < n)
+        out[(size_t)(start + t0 + t) * ldo + gc] = from_float<T>((ys[buf][t][lc] + add[i]) * gate[i]);
+    }
+    if (more) keep();
   }
 #pragma unroll
   for (int i = 0; i < NS; ++i)
-    if (c < inner && n0 + i < N) st[(size_t)c * N + n0 + i] = S[i];
+    if (c < inner && lane + i * L < N) st[(size_t)c * N + lane + i * L] = S[i];
 }
 
 // ---------------------------------------------------------------- a step of single tokens
-// Row b is sequence b's token.  low [rows, ..] 32-bit holds dt_rank values, then B and C at their offsets; w_dt [inner, ldw] in the
-// engine's type.
+// Row b is sequence b's token.  low [rows, ..] 32-bit (the sum of low_parts partial products, low_stride floats apart) holds dt_rank
+// values, then B and C at their offsets; w_dt [inner, ldw] in the engine's type.
 template <typename T, int L, int NS>
 __global__ void __launch_bounds__(SS_THREADS)
-selective_step_kernel(const T *__restrict__ x, long long ldx, const float *__restrict__ low, long long ld_low, int rank,
+selective_step_kernel(const T *__restrict__ x, long long ldx, const float *__restrict__ low, long long ld_low, int low_parts,
+                      long long low_stride, int rank,
                       const T *__restrict__ w_dt, int ldw, const float *__restrict__ dt_bias, int off_b, int off_c,
                       const float *__restrict__ z, long long ldz, const float *__restrict__ a_log, const float *__restrict__ skip,
                       float *__restrict__ state, T *__restrict__ out, long long ldo, const int *__restrict__ seq_slot, int inner, int N) {
   constexpr int CH = SS_THREADS / L, NP = L * NS;
-  extern __shared__ float low_s[];                       // B [NP], C [NP], then the dt input [rank]
+  extern __shared__ __align__(16) float low_s[];         // B [NP], C [NP], then the dt input [rank]
   grid_dependents_launch();
-  const int tid = threadIdx.x, lane = tid % L, c = blockIdx.x * CH + tid / L, n0 = lane * NS, b = blockIdx.y;
+  const int tid = threadIdx.x, lane = tid % L, c = blockIdx.x * CH + tid / L, b = blockIdx.y;
   const bool in = c < inner;
   const float bias = in ? dt_bias[c] : 0.f, dsk = in ? skip[c] : 0.f;
   float al2[NS], S[NS];
   float *st = state + (size_t)seq_slot[b] * inner * N;
   grid_dependency_wait();
-  lane_states<NS>(a_log, st, c, n0, N, in, al2, S);
+  lane_states<L, NS>(a_log, st, c, lane, N, in, al2, S);
   const float *lr = low + (size_t)b * ld_low;
-  for (int i = tid; i < 2 * NP + rank; i += SS_THREADS)
-    low_s[i] = i >= 2 * NP ? lr[i - 2 * NP] : i >= NP ? (i - NP < N ? lr[off_c + i - NP] : 0.f) : (i < N ? lr[off_b + i] : 0.f);
+  for (int i = tid; i < 2 * NP + rank; i += SS_THREADS) {
+    const int at = i >= 2 * NP ? i - 2 * NP : i >= NP ? (i - NP < N ? off_c + i - NP : -1) : (i < N ? off_b + i : -1);
+    low_s[i] = at >= 0 ? sum_parts(lr + at, low_parts, low_stride) : 0.f;
+  }
   const float xv = in ? to_float(x[(size_t)b * ldx + c]) : 0.f, zv = in ? z[(size_t)b * ldz + c] : 0.f;
   __syncthreads();
   float raw = 0.f;
@@ -314,10 +391,13 @@ selective_step_kernel(const T *__restrict__ x, long long ldx, const float *__res
     }
   }
   const float dt = softplus_of(lanes_sum<L>(raw) + bias);
-  const float y = lanes_sum<L>(scan_token<NS>(S, al2, dt, dt * xv, low_s + n0, low_s + NP + n0));
+  float y = 0.f;
+#pragma unroll
+  for (int i = 0; i < NS; ++i) scan_state(S[i], al2[i], dt, dt * xv, low_s[lane + i * L], low_s[NP + lane + i * L], y);
+  y = lanes_sum<L>(y);
 #pragma unroll
   for (int i = 0; i < NS; ++i)
-    if (in && n0 + i < N) st[(size_t)c * N + n0 + i] = S[i];
+    if (in && lane + i * L < N) st[(size_t)c * N + lane + i * L] = S[i];
   if (in && lane == 0) out[(size_t)b * ldo + c] = from_float<T>((y + dsk * xv) * silu_of(zv));
 }
 
@@ -359,8 +439,17 @@ LLM_EXPORT int llm_short_conv_silu(int dtype, const float *u, long long ld, cons
 
 LLM_EXPORT int llm_selective_max_state() { return 256; }
 
-// lanes of a channel and states of a lane for N states per channel
-#define SS_SHAPES(GO)                     \
+// lanes of a channel and states of a lane for N states per channel: few states a lane over a step's tokens, where the tokens come one
+// after another; few lanes in a step of single tokens, whose channels fill the machine
+#define SCAN_SHAPES(GO)                   \
+  do {                                    \
+    if (N <= 16) GO(16, 1);               \
+    else if (N <= 32) GO(16, 2);          \
+    else if (N <= 64) GO(32, 2);          \
+    else if (N <= 128) GO(32, 4);         \
+    else GO(32, 8);                       \
+  } while (0)
+#define STEP_SHAPES(GO)                   \
   do {                                    \
     if (N <= 16) GO(4, 4);                \
     else if (N <= 32) GO(4, 8);           \
@@ -380,13 +469,13 @@ LLM_EXPORT int llm_selective_scan(int dtype, const void *x, long long ldx, const
   LLM_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && inner > 0 && N > 0 && state && a_log && skip && dt_bias, "selective_scan: bad sizes");
   LLM_REQUIRE(N <= llm_selective_max_state(), "selective_scan: %d states a channel are not supported (up to %d)", N, llm_selective_max_state());
 #define SS_GO2(T, L, NS)                                                                                                              \
-  llm_launch(selective_scan_kernel<T, L, NS>, dim3((inner + SS_THREADS / L - 1) / (SS_THREADS / L), n_seqs), dim3(SS_THREADS), 0, stream,       \
+  llm_launch(selective_scan_kernel<T, L, NS>, dim3((inner + SCAN_THREADS / L - 1) / (SCAN_THREADS / L), n_seqs), dim3(SCAN_THREADS), 0, stream,   \
              (const T *)x, ldx, dt_raw, ld_dt, dt_bias, bc, ld_bc, off_b, off_c, z, ldz, a_log, skip, state, (T *)out, ldo, seq_start, seq_slot, \
              inner, N)
 #define SS_F32(L, NS) SS_GO2(float, L, NS)
 #define SS_BF16(L, NS) SS_GO2(__nv_bfloat16, L, NS)
-  if (dtype == LLM_F32) SS_SHAPES(SS_F32);
-  else if (dtype == LLM_BF16) SS_SHAPES(SS_BF16);
+  if (dtype == LLM_F32) SCAN_SHAPES(SS_F32);
+  else if (dtype == LLM_BF16) SCAN_SHAPES(SS_BF16);
   else LLM_FAIL("selective_scan: unsupported dtype %d", dtype);
 #undef SS_F32
 #undef SS_BF16
@@ -397,7 +486,8 @@ LLM_EXPORT int llm_selective_scan(int dtype, const void *x, long long ldx, const
 
 // Single tokens: low [n_seqs, ..] 32-bit rows = the dt input (rank values), B and C at their offsets; w_dt [inner, ldw] in the
 // engine's type, columns beyond the rank nought.
-LLM_EXPORT int llm_selective_step(int dtype, const void *x, long long ldx, const float *low, long long ld_low, int rank, const void *w_dt,
+LLM_EXPORT int llm_selective_step(int dtype, const void *x, long long ldx, const float *low, long long ld_low, int low_parts,
+                                  long long low_stride, int rank, const void *w_dt,
                                   int ldw, const float *dt_bias, int off_b, int off_c, const float *z, long long ldz, const float *a_log,
                                   const float *skip, float *state, void *out, long long ldo, const int *seq_slot, int n_seqs, int inner,
                                   int N, cudaStream_t stream) {
@@ -405,16 +495,17 @@ LLM_EXPORT int llm_selective_step(int dtype, const void *x, long long ldx, const
   LLM_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && inner > 0 && N > 0 && rank > 0 && ldw >= rank && state && a_log && skip && dt_bias && w_dt,
               "selective_step: bad sizes");
   LLM_REQUIRE(N <= llm_selective_max_state(), "selective_step: %d states a channel are not supported (up to %d)", N, llm_selective_max_state());
+  LLM_REQUIRE(low_parts >= 1 && low_parts <= 64, "selective_step: %d partial products", low_parts);
   LLM_REQUIRE(rank <= 8192, "selective_step: a dt input of %d values is not supported", rank);
   LLM_REQUIRE(ldw % 4 != 0 || (uintptr_t)w_dt % 16 == 0, "selective_step: the dt matrix must start on 16 bytes");
 #define SS_GO2(T, L, NS)                                                                                                              \
   llm_launch(selective_step_kernel<T, L, NS>, dim3((inner + SS_THREADS / L - 1) / (SS_THREADS / L), n_seqs), dim3(SS_THREADS),         \
-             (size_t)(2 * L * NS + rank) * sizeof(float), stream, (const T *)x, ldx, low, ld_low, rank, (const T *)w_dt, ldw, dt_bias,  \
+             (size_t)(2 * L * NS + rank) * sizeof(float), stream, (const T *)x, ldx, low, ld_low, low_parts, low_stride, rank, (const T *)w_dt, ldw, dt_bias,  \
              off_b, off_c, z, ldz, a_log, skip, state, (T *)out, ldo, seq_slot, inner, N)
 #define SS_F32(L, NS) SS_GO2(float, L, NS)
 #define SS_BF16(L, NS) SS_GO2(__nv_bfloat16, L, NS)
-  if (dtype == LLM_F32) SS_SHAPES(SS_F32);
-  else if (dtype == LLM_BF16) SS_SHAPES(SS_BF16);
+  if (dtype == LLM_F32) STEP_SHAPES(SS_F32);
+  else if (dtype == LLM_BF16) STEP_SHAPES(SS_BF16);
   else LLM_FAIL("selective_step: unsupported dtype %d", dtype);
 #undef SS_F32
 #undef SS_BF16

@@ -909,7 +909,11 @@ class PreNormBlock : public Block {
       kernels::stream_cast(stream.resid, stream.pending.data ? &stream.pending : nullptr, x.data, ctx.dtype, (int)n, (int)hidden_, ctx.stream);
     }
     stream.pending = Act();
-    Act z = linear(ctx, x, side_gate_, nullptr, DType::F32);
+    float *const pool = ctx.parts_pool, *const sink = ctx.residual_sink;
+    ctx.parts_pool = ctx.residual_sink = nullptr;        // few tokens' partial products are added behind; the gate is no result of the block's
+    Act z = linear(ctx, x, side_gate_, nullptr, DType::F32, true);
+    ctx.parts_pool = pool;
+    ctx.residual_sink = sink;
     flush_chain(ctx);
     Act g = ctx.arena->act(ctx.dtype, n, side_proj_.cols);
     kernels::token_gate(z, ctx.token_table, ctx.token_table_width, side_offset_, side_dim_, ctx.token_ids,

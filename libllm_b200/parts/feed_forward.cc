@@ -131,7 +131,7 @@ class RoutedFeedForward : public FeedForward {
     shared_gate_ = r.string_or("shared_gate", "");
     if (!shared_gate_.empty() && !shared_) r.fail("'shared_gate' goes with a 'shared' feed-forward");
     grouped_route_ = !correction_.empty() || groups_ > 1 || norm_eps_ != 0.f || route_scale_ != 1.f;
-    router_rows_ = shared_gate_.empty() ? choices_ : (choices_ + 1 + 7) / 8 * 8;
+    router_rows_ = (choices_ + (shared_gate_.empty() ? 0 : 1) + 7) / 8 * 8;
   }
   static std::string numbered(const std::string &pattern, int e) {
     std::string s = pattern;
@@ -154,9 +154,7 @@ class RoutedFeedForward : public FeedForward {
   }
   void load(const Loader &l) override {
     const auto needs = tensor_needs();
-    if (shared_gate_.empty()) {
-      w_router_ = l.fetch(needs[0]);
-    } else {
+    {
       // [router; the shared feed-forward's gate; zeros up to a multiple of 8 rows]
       const size_t row_bytes = (size_t)hidden_ * dtype_size(l.engine);
       w_router_.dtype = l.engine;
@@ -164,7 +162,7 @@ class RoutedFeedForward : public FeedForward {
       w_router_.cols = hidden_;
       w_router_.buf.allocate((size_t)router_rows_ * row_bytes, true);
       l.fetch_into(needs[0], l.engine, w_router_.buf.get());
-      l.fetch_into(needs.back(), l.engine, (char *)w_router_.buf.get() + (size_t)choices_ * row_bytes);
+      if (!shared_gate_.empty()) l.fetch_into(needs.back(), l.engine, (char *)w_router_.buf.get() + (size_t)choices_ * row_bytes);
     }
     if (!correction_.empty()) w_correction_ = l.fetch(needs[needs.size() - (shared_gate_.empty() ? 1 : 2)]);
     const size_t es = dtype_size(l.engine), one = (size_t)(inter_ * hidden_) * es;
@@ -229,20 +227,24 @@ class RoutedFeedForward : public FeedForward {
     }
     const bool s_own = s.data && s.data != (void *)sink;
     ctx.residual_sink = nullptr;                     // what follows returns its own buffers
-    Act z = linear(ctx, x, w_router_, nullptr, DType::F32);
+    const int n_rows = (int)T * top_;
+    const bool aligned = x.dtype == DType::BF16 && x.ld % 8 == 0 && (uintptr_t)x.data % 16 == 0;
+    const bool tc = aligned && fast_switches().moe_tc && kernels::available("moe_tc") && kernels::moe_tc_supported((int)hidden_, (int)inter_);
+    const bool planned = tc && grouped_route_ && n_rows <= kernels::moe_plan_rows() && choices_ <= 512;
+    // the logits of few tokens as partial products, where whoever reads them adds them
+    float *const outer_pool = ctx.parts_pool;
+    ctx.parts_pool = nullptr;
+    Act z = linear(ctx, x, w_router_, nullptr, DType::F32, planned && shared_gate_.empty());
+    ctx.parts_pool = outer_pool;
     ctx.residual_sink = sink;
     flush_chain(ctx);
-    const int n_rows = (int)T * top_;
     int *chosen = ctx.arena->alloc_n<int>((size_t)n_rows);
     float *weight = ctx.arena->alloc_n<float>((size_t)n_rows);
     const bool in_place = given > 0 && s_own && s.data == (void *)after;
     if (s_own && !in_place && s.parts > given) out = ctx.arena->act(DType::F32, T, hidden_, top_ + s.parts);
     out.parts = top_ + (s_own ? s.parts : 0);
-    const bool aligned = x.dtype == DType::BF16 && x.ld % 8 == 0 && (uintptr_t)x.data % 16 == 0;
-    const bool tc = aligned && fast_switches().moe_tc && kernels::available("moe_tc") && kernels::moe_tc_supported((int)hidden_, (int)inter_);
     const kernels::RouteRule rule{choices_, top_, score_, correction_.empty() ? nullptr : w_correction_.buf.as<float>(), groups_, keep_, group_top_,
                                   renormalize_, norm_eps_, route_scale_};
-    const bool planned = tc && grouped_route_ && n_rows <= kernels::moe_plan_rows() && choices_ <= 512;
     if (planned) {
       // with the sorting and the gathering, below
     } else if (grouped_route_) {

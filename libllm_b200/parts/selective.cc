@@ -109,11 +109,17 @@ class SelectiveScan : public Mixer {
     Act xc = ctx.arena->act(ctx.dtype, T, inner_);
     kernels::short_conv_silu(proj, conv_.buf.as<float>(), conv_bias_.buf.as<float>(), taps_, inputs, xc, ctx.tok_seq, ctx.tok_pos, ctx.seq_start,
                              ctx.seq_past, ctx.seq_slot, ctx.n_seqs, ctx.decode_only, ctx.stream);
-    Act low = linear(ctx, xc, w_x_, nullptr, DType::F32);
+    const bool single = ctx.decode_only && T == ctx.n_seqs;
+    // partial products where the kernel behind adds them; not the room or the stream of the block's own result
+    float *const pool = ctx.parts_pool, *const sink = ctx.residual_sink;
+    ctx.parts_pool = ctx.residual_sink = nullptr;
+    Act low = linear(ctx, xc, w_x_, nullptr, DType::F32, single);
+    ctx.parts_pool = pool;
+    ctx.residual_sink = sink;
     flush_chain(ctx);
     const int off_b = rank_, off_c = rank_ + state_;
     Act y = ctx.arena->act(ctx.dtype, T, inner_);
-    if (ctx.decode_only && T == ctx.n_seqs) {
+    if (single) {
       kernels::selective_step(xc, low, rank_, w_dt_, dt_bias_.buf.as<float>(), off_b, off_c, z, proj.ld, a_log_.buf.as<float>(),
                               skip_.buf.as<float>(), S, y, ctx.seq_slot, state_, ctx.stream);
     } else {

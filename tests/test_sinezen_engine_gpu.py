@@ -98,8 +98,18 @@ def test_unequal_batches_against_each_request_alone(name, dtype):
             total = p + n_dec - (j if b % 2 == 0 else 3 - j)
             reqs.append((f"b{b}r{j}", Z.tokens(c, total, 100 * b + j), p))
         got = replay_batch(engine, reqs)
+        # a choice turned by rounding changes the positions behind it too, as far as a mask reaches: most of a short request.  So
+        # the count is over the batch, and the median over each request.
+        routed = dtype == "bfloat16" and Z.is_routed(c)
+        refs = {rid: plain(name, c, w, toks) for rid, toks, p in reqs}
+        if routed:
+            pair = [torch.cat([rows[rid].cpu().double() / refs[rid].double().square().mean().sqrt() for rid, _, _ in reqs]) for rows in (got, refs)]
+            Z.check_rows(pair[0], pair[1], dtype, f"{name} batch {b}")
         for rid, toks, p in reqs:
-            Z.check_rows(got[rid], plain(name, c, w, toks), dtype, f"{name} batch {b} {rid}", routed=Z.is_routed(c))
+            if routed:
+                assert float(Z.row_errors(got[rid], refs[rid]).median()) < Z.TOL[dtype] / 3, f"{name} batch {b} {rid}"
+            else:
+                Z.check_rows(got[rid], refs[rid], dtype, f"{name} batch {b} {rid}", routed=Z.is_routed(c))
             if dtype == "float32" and b == 0:
                 single = replay_batch(alone, [(rid, toks, p)])[rid]
                 assert float(Z.row_errors(got[rid], single).max()) < Z.TOL[dtype], f"{name} {rid}: the batch changes the result"
