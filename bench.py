@@ -1001,7 +1001,7 @@ def main():
     ap.add_argument("--only", choices=["decode", "prefill"], default=None,
                     help="run one part only and print a short line (for profiling; not a bench record)")
     ap.add_argument("--compare", choices=["sinezen", "sesuzen", "sobezen", "tazizen", "rarelorn", "fomodra"], default=None,
-                    help="Sinezen, Sesuzen, Sobezen or Tazizen beside Llama (Rarelorn beside Sesuzen) at equal sizes: prefill and decode, a line per size and model (not a bench record)")
+                    help="Sinezen, Sesuzen, Sobezen or Tazizen beside Llama (Rarelorn beside Sesuzen, Fomodra beside Tazizen) at equal sizes: prefill and decode, a line per size and model (not a bench record)")
     ap.add_argument("--model", choices=["llama", "sesuzen", "sobezen", "tazizen", "rarelorn", "fomodra"], default=None,
                     help="with --compare sesuzen, sobezen, tazizen, rarelorn or fomodra: one of the two models only")
     ap.add_argument("--sizes", default=None, help="with --compare: which of the sizes (2k, 4k, 2k-routed), with commas")
